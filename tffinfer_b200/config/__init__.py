@@ -4,4 +4,5 @@ from .tipezen_config import TipezenConfig, TipezenLayer, RotaryConfig
 from .dominex_config import DominexConfig, DominexLayer, DominexExperts
 from .sadupel_config import SadupelConfig, SadupelLayer, SadupelExperts
 from .nugosun_config import NugosunConfig, NugosunLayer, NugosunMlp
+from .kadodra_config import KadodraConfig, KadodraLayer, KadodraMlp
 from .engine_config import EngineConfig

@@ -10,6 +10,9 @@
 // * score(p, n) = (q . k_n) * scale * temp[h]  -  r1[h] * ln(1 + r2[h] * (p - n)), with per-head float32 arrays temp
 //   (null: 1) and r1, r2 (null: no distance term); with ``softcap`` > 0 the scaled product is first squashed to
 //   softcap * tanh(. / softcap);
+// * ``sink`` (per-head float32, null: none): one more term exp(sink[h]) in the softmax's denominator, a key without a
+//   value that is neither scaled, capped nor masked; a row's running maximum and sum start from it (in the first share
+//   when the key range is cut);
 // * the output is multiplied by out_scale and may go to a column block of a wider row (out_ld, out_off).
 //
 // A tile is ROWS packed rows of one request and one key/value head: row r of the request is (token r / G, query head
@@ -33,6 +36,7 @@ struct TileArgs {
     float scale; int window, chunk;
     float softcap;                                  // > 0: a scaled score s becomes softcap * tanh(s / softcap)
     const float* temp; const float* r1; const float* r2;
+    const float* sink;
     float out_scale; int q_ld, out_ld, out_off;
     int splits; float* part_o; float* part_ml;     // splits > 1: shares of the key range, merged by a second kernel
     // Keys and values of THIS step's tokens in plain rows instead of the cache (tensor-core form only; every request of the
@@ -100,7 +104,10 @@ attention_tile_kernel(const TQ* __restrict__ q, const TC* __restrict__ cache, TQ
     // softmax phase: warp w owns rows 4w .. 4w+3, lane = key of the block
     float m_run[4], l_run[4];
 #pragma unroll
-    for (int i = 0; i < 4; ++i) { m_run[i] = -INFINITY; l_run[i] = 0.f; }
+    for (int i = 0; i < 4; ++i) {
+        m_run[i] = -INFINITY; l_run[i] = 0.f;
+        if (a.sink && split == 0) { m_run[i] = a.sink[kvh * G + (r0 + warp * 4 + i) % G]; l_run[i] = 1.f; }
+    }
     const int* table = a.block_table + (size_t)b * a.table_width;
 
     // the tile's key blocks, in equal contiguous shares when the key range is cut (a share may be empty)
@@ -377,7 +384,10 @@ attention_tile_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict__ c
         for (int e = 0; e < 4; ++e) o[j][e] = 0.f;
     float m_run[4], l_run[4];                                   // softmax phase: warp w owns rows 4w .. 4w+3
 #pragma unroll
-    for (int i = 0; i < 4; ++i) { m_run[i] = -INFINITY; l_run[i] = 0.f; }
+    for (int i = 0; i < 4; ++i) {
+        m_run[i] = -INFINITY; l_run[i] = 0.f;
+        if (a.sink && split == 0) { m_run[i] = a.sink[kvh * G + (r0 + warp * 4 + i) % G]; l_run[i] = 1.f; }
+    }
     const int* table = a.block_table + (size_t)b * a.table_width;
     const int vch = own_v ? (vst - 8) / 8 : 0;
 
@@ -596,7 +606,7 @@ TFF_API int tff_attention_tile(
     void* out, int out_ld, int out_off, int num_requests, int max_q_len, int nq, int nkv, int d, int dv, float scale,
     int window, int chunk, const float* temp, const float* r1, const float* r2, float out_scale,
     int num_tokens, int splits, float* part_o, float* part_ml,
-    const void* k_dense, const void* v_dense, int k_ld, int v_ld, float softcap, cudaStream_t stream) {
+    const void* k_dense, const void* v_dense, int k_ld, int v_ld, float softcap, const float* sink, cudaStream_t stream) {
     if (num_requests <= 0 || max_q_len <= 0) return TFF_OK;
     if ((k_dense == nullptr) != (v_dense == nullptr)) return TFF_ERR_BAD_ARGUMENT;
     if (k_dense) { planes = 2; slot = d > dv ? d : dv; page_size = 1; }      // no cache is read: any consistent geometry
@@ -609,6 +619,7 @@ TFF_API int tff_attention_tile(
     a.v_offset = planes == 2 ? (long long)nkv * page_size * slot : 0;
     a.slot = slot; a.page_size = page_size; a.nq = nq; a.nkv = nkv; a.d = d; a.dv = dv; a.scale = scale;
     a.softcap = softcap > 0.f ? softcap : 0.f;
+    a.sink = sink;
     a.window = window; a.chunk = chunk; a.temp = temp; a.r1 = r1; a.r2 = r2; a.out_scale = out_scale;
     a.q_ld = q_ld; a.out_ld = out_ld; a.out_off = out_off;
     if (splits < 1 || (splits > 1 && (!part_o || !part_ml))) return TFF_ERR_BAD_ARGUMENT;

@@ -12,8 +12,11 @@ namespace tc5 {
 // EPI_GEGLU: as EPI_SWIGLU with the tanh form of gelu on the gate, 0.5 g (1 + tanh(sqrt(2/pi) (g + 0.044715 g^3))),
 // which is g / (1 + exp(-2 sqrt(2/pi) (g + 0.044715 g^3))): the same exponential and division as silu
 // EPI_RELU2: a plain product stored as bfloat16 with the square of relu applied, relu(x)^2 (a feed-forward without a gate).
-enum Epilogue : int { EPI_STORE = 0, EPI_ADD = 1, EPI_SWIGLU = 2, EPI_QKV = 3, EPI_GEGLU = 4, EPI_RELU2 = 5 };
-__host__ __device__ constexpr bool epi_gated(int e) { return e == EPI_SWIGLU || e == EPI_GEGLU; }
+// EPI_CLIP: gated, g' sigmoid(slope g') (u' + 1) with g' = min(g, limit) and u' = u held within -limit .. limit.
+enum Epilogue : int { EPI_STORE = 0, EPI_ADD = 1, EPI_SWIGLU = 2, EPI_QKV = 3, EPI_GEGLU = 4, EPI_RELU2 = 5, EPI_CLIP = 6 };
+__host__ __device__ constexpr bool epi_gated(int e) { return e == EPI_SWIGLU || e == EPI_GEGLU || e == EPI_CLIP; }
+
+struct GateConstants { float limit, slope; };     // EPI_CLIP's
 
 // act(g) of the gated epilogues with the fast exponential and division (the result is rounded to bfloat16)
 template <int EPI>
@@ -22,13 +25,24 @@ __device__ __forceinline__ float gate_act_fast(float g) {
     else return __fdividef(g, 1.0f + __expf(-g));
 }
 
+template <int EPI>
+__device__ __forceinline__ float gated_fast(float g, float u, GateConstants gc) {
+    if constexpr (EPI == EPI_CLIP) {
+        g = fminf(g, gc.limit);
+        u = fminf(fmaxf(u, -gc.limit), gc.limit);
+        return __fdividef(g, 1.0f + __expf(-gc.slope * g)) * (u + 1.0f);
+    }
+    return gate_act_fast<EPI>(g) * u;
+}
+
 // One warp's quarter (32 rows) of the tile: TMEM -> registers -> two alternating 4 KB boxes of swizzled
 // shared memory (``my_stage``) -> TMA stores, or float32 add-reductions when the product is added to what
 // ``out`` holds or the tile is a share of its K range (``partial``).  ``t_addr``: TMEM address of the warp's
 // lane quarter and the tile's first column; ``chunk_no`` counts the warp's boxes over the whole kernel.
 template <int BN, int EPI, typename TC>
 __device__ __forceinline__ void epilogue_quarter_tma(uint32_t t_addr, uint32_t my_stage, uint32_t& chunk_no, int lane, int q,
-                                                     int lane_row0, int col_row0, bool partial, const CUtensorMap* tm_out) {
+                                                     int lane_row0, int col_row0, bool partial, const CUtensorMap* tm_out,
+                                                     GateConstants gc = GateConstants{0.f, 0.f}) {
     // 128-byte-wide column chunks: 32 float32 or 64 bfloat16 per row
     constexpr int CW = 128 / (int)sizeof(TC);      // output columns per chunk
     constexpr int AW = epi_gated(EPI) ? 128 : CW;   // accumulator columns per chunk
@@ -54,8 +68,8 @@ __device__ __forceinline__ void epilogue_quarter_tma(uint32_t t_addr, uint32_t m
 #pragma unroll
                 for (int j = 0; j < 8; ++j) {
                     const float g0 = __uint_as_float(g[2 * j]), g1 = __uint_as_float(g[2 * j + 1]);
-                    const float a0 = gate_act_fast<EPI>(g0) * __uint_as_float(u[2 * j]);
-                    const float a1 = gate_act_fast<EPI>(g1) * __uint_as_float(u[2 * j + 1]);
+                    const float a0 = gated_fast<EPI>(g0, __uint_as_float(u[2 * j]), gc);
+                    const float a1 = gated_fast<EPI>(g1, __uint_as_float(u[2 * j + 1]), gc);
                     __nv_bfloat162 b2 = __floats2bfloat162_rn(a0, a1);
                     packed[h * 8 + j] = *reinterpret_cast<uint32_t*>(&b2);
                 }

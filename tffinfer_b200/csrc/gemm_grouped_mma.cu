@@ -32,10 +32,16 @@ __device__ __forceinline__ void mma16816(float (&c)[4], const uint32_t (&a)[4], 
                  : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
                  : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
-__device__ __forceinline__ float act_of(float g, int act) {
-    if (act == 0) return g / (1.0f + expf(-g));
+// act(g) u; act 3 is g' sigmoid(slope g') (u' + 1), g' = min(g, limit), u' = u held within -limit .. limit
+__device__ __forceinline__ float gate_of(float g, float u, int act, float limit, float slope) {
+    if (act == 0) return g / (1.0f + expf(-g)) * u;
+    if (act == 3) {
+        g = fminf(g, limit);
+        u = fminf(fmaxf(u, -limit), limit);
+        return g / (1.0f + expf(-slope * g)) * (u + 1.0f);
+    }
     const float c = 0.7978845608028654f * (g + 0.044715f * g * g * g);
-    return 0.5f * g * (1.0f + tanhf(c));
+    return 0.5f * g * (1.0f + tanhf(c)) * u;
 }
 
 template <typename TCc, bool GATED>
@@ -45,7 +51,8 @@ gemm_grouped_mma_kernel(const bf16* __restrict__ A, long long lda, long long a_g
                         TCc* __restrict__ C, long long ldc, long long c_gs,
                         const int* __restrict__ tile_group, const int* __restrict__ tile_row0,
                         const int* __restrict__ tile_row_end, const int* __restrict__ num_tiles,
-                        const int* __restrict__ row_map, int M, int N, int K, int act) {
+                        const int* __restrict__ row_map, const int* __restrict__ a_rows, int M, int N, int K, int act,
+                        float limit, float slope) {
     extern __shared__ __align__(16) unsigned char smem_raw[];
     bf16* As = (bf16*)smem_raw;                               // [STAGES][MBM][LDS]
     bf16* Bs = As + STAGES * MBM * LDS;                       // [STAGES][MBN][LDS]
@@ -53,8 +60,8 @@ gemm_grouped_mma_kernel(const bf16* __restrict__ A, long long lda, long long a_g
     pdl_wait();
     int g, m0, m_end;
     if (tile_group != nullptr) {
-        if ((int)blockIdx.y >= *num_tiles) return;
-        g = tile_group[blockIdx.y]; m0 = tile_row0[blockIdx.y]; m_end = tile_row_end[blockIdx.y];
+        if ((int)blockIdx.y >= __ldcg(num_tiles)) return;        // the tables are a kernel's ahead: past the first-level cache
+        g = __ldcg(tile_group + blockIdx.y); m0 = __ldcg(tile_row0 + blockIdx.y); m_end = __ldcg(tile_row_end + blockIdx.y);
     } else {
         g = blockIdx.z; m0 = blockIdx.y * MBM; m_end = M;
     }
@@ -64,6 +71,13 @@ gemm_grouped_mma_kernel(const bf16* __restrict__ A, long long lda, long long a_g
     const bf16* Ag = A + (size_t)g * a_gs;
     const bf16* Bg = B + (size_t)g * b_gs;
     const int kt = (K + MBK - 1) / MBK;
+    // where this thread's rows of A lie (row r of the sorted order is row a_rows[r] of A when there is such a table)
+    long long a_off[MBM * CHUNKS / THREADS];
+#pragma unroll
+    for (int i = 0; i < MBM * CHUNKS / THREADS; ++i) {
+        const int r = m0 + (tid + i * THREADS) / CHUNKS;
+        a_off[i] = r < m_end ? (long long)(a_rows ? __ldcg(a_rows + r) : r) * lda : 0;
+    }
 
     auto load_stage = [&](int s, int k0) {
 #pragma unroll
@@ -72,7 +86,7 @@ gemm_grouped_mma_kernel(const bf16* __restrict__ A, long long lda, long long a_g
             const bool ka = k0 + kc < K;
             const bool oka = ka && (m0 + r < m_end);
             cp_async16(smem_addr(As + ((size_t)s * MBM + r) * LDS + kc),
-                       oka ? (const void*)(Ag + (size_t)(m0 + r) * lda + k0 + kc) : (const void*)Ag, oka ? 16 : 0);
+                       oka ? (const void*)(Ag + a_off[i] + k0 + kc) : (const void*)Ag, oka ? 16 : 0);
             const bool okb = ka && (n0 + r < N);
             cp_async16(smem_addr(Bs + ((size_t)s * MBN + r) * LDS + kc),
                        okb ? (const void*)(Bg + (size_t)(n0 + r) * ldb + k0 + kc) : (const void*)Bg, okb ? 16 : 0);
@@ -129,7 +143,7 @@ gemm_grouped_mma_kernel(const bf16* __restrict__ A, long long lda, long long a_g
         for (int half = 0; half < 2; ++half) {
             const int m = m0 + wm * 32 + mi * 16 + (lane >> 2) + half * 8;
             if (m >= m_end) continue;
-            const long long row = row_map ? row_map[m] : m;
+            const long long row = row_map ? __ldcg(row_map + m) : m;
             TCc* crow = C + (size_t)g * c_gs + (size_t)row * ldc;
             if constexpr (GATED) {
 #pragma unroll
@@ -138,7 +152,7 @@ gemm_grouped_mma_kernel(const bf16* __restrict__ A, long long lda, long long a_g
 #pragma unroll
                     for (int e = 0; e < 2; ++e)
                         if (f + e < N / 2)
-                            crow[f + e] = from_f32<TCc>(act_of(acc[mi][t][half * 2 + e], act) * acc[mi][t + 4][half * 2 + e]);
+                            crow[f + e] = from_f32<TCc>(gate_of(acc[mi][t][half * 2 + e], acc[mi][t + 4][half * 2 + e], act, limit, slope));
                 }
             } else {
 #pragma unroll
@@ -159,12 +173,14 @@ gemm_grouped_mma_kernel(const bf16* __restrict__ A, long long lda, long long a_g
 }  // namespace
 
 // A and B bfloat16.  gated != 0: B's N rows are gate and up rows alternating in blocks of 64 and C has N / 2 columns.
-// c_dt 0 = float32, 1 = bfloat16.  The ragged form's tiles must have been planned with tff_gemm_grouped_mma_tile_rows().
+// c_dt 0 = float32, 1 = bfloat16.  ``a_rows`` (ragged form; null: A is in the sorted order), ``act``, ``limit`` and ``slope``
+// as for tff_gemm_grouped.  The ragged form's tiles must have been planned with tff_gemm_grouped_mma_tile_rows().
 TFF_API int tff_gemm_grouped_mma(
     const void* A, long long lda, long long a_gs, const void* B, long long ldb, long long b_gs,
     void* C, int c_dt, long long ldc, long long c_gs,
     const int* tile_group, const int* tile_row0, const int* tile_row_end, const int* num_tiles, int max_tiles,
-    const int* row_map, int groups, int M, int N, int K, int gated, int act, cudaStream_t stream) {
+    const int* row_map, const int* a_rows, int groups, int M, int N, int K, int gated, int act, float limit, float slope,
+    cudaStream_t stream) {
     if (N <= 0 || K <= 0 || !A || !B || !C) return TFF_ERR_BAD_ARGUMENT;
     if ((K & 7) || (lda & 7) || (ldb & 7) || (a_gs & 7) || (b_gs & 7) || ((uintptr_t)A & 15) || ((uintptr_t)B & 15) ||
         (gated && (N & 127)))
@@ -185,7 +201,7 @@ TFF_API int tff_gemm_grouped_mma(
         cudaFuncSetAttribute(gemm_grouped_mma_kernel<TCc, G>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_BYTES); \
         return tff_launch_pdl(gemm_grouped_mma_kernel<TCc, G>, grid, dim3(THREADS), (size_t)SMEM_BYTES, stream,     \
                               (const bf16*)A, lda, a_gs, (const bf16*)B, ldb, b_gs, (TCc*)C, ldc, c_gs, tile_group, \
-                              tile_row0, tile_row_end, num_tiles, row_map, M, N, K, act);                           \
+                              tile_row0, tile_row_end, num_tiles, row_map, a_rows, M, N, K, act, limit, slope);                           \
     } while (0)
     if (c_dt == 0 && gated) TFF_GM(float, true);
     if (c_dt == 0) TFF_GM(float, false);

@@ -62,7 +62,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_lane,   // operand whose r
                const __grid_constant__ CUtensorMap tm_col,    // operand whose rows land on TMEM columns (box 64 x BN)
                const __grid_constant__ CUtensorMap tm_out,    // output, boxes of 128 bytes x 32 rows (TMA_OUT only)
                TC* __restrict__ out, int rows_lane, int rows_col, int K, int ldo, int stream_k, int* error_flag,
-               const int* __restrict__ lane_group, int group_rows) {
+               const int* __restrict__ lane_group, int group_rows, GateConstants gc) {
     // lane_group (normal orientation only; null: one product): the 128-row tile t of the lane operand belongs to group
     // lane_group[t] and is multiplied with rows [g * group_rows, (g + 1) * group_rows) of the column operand; a tile of
     // group -1 is skipped by all three roles.  The table is written by a kernel ahead: read it behind pdl_wait.
@@ -239,7 +239,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_lane,   // operand whose r
                 }
             } else if constexpr (TMA_OUT) {
                 epilogue_quarter_tma<BN, EPI, TC>(t_addr, staging + (uint32_t)((warp - 2) * 2) * 4096u, chunk_no, lane, q,
-                                                  lane_row0, col_row0, partial, &tm_out);
+                                                  lane_row0, col_row0, partial, &tm_out, gc);
             } else {
                 const int lr = lane_row0 + q * 32 + lane;          // row of the lane operand
 #pragma unroll 1
@@ -293,7 +293,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_lane,   // operand whose r
 template <int BN, bool SWAP, int EPI, typename TC, bool TMA_OUT>
 int launch_tc(const CUtensorMap& tl, const CUtensorMap& tc, const CUtensorMap& to, void* out,
               int rows_lane, int rows_col, int K, int ldo, int stream_k, cudaStream_t stream,
-              const int* lane_group = nullptr, int group_rows = 0) {
+              const int* lane_group = nullptr, int group_rows = 0, GateConstants gc = GateConstants{0.f, 0.f}) {
     using Cfg = TileCfg<BN, TMA_OUT, SWAP>;
     auto kern = gemm_tc_kernel<BN, SWAP, EPI, TC, TMA_OUT>;
     static bool configured = false;
@@ -318,7 +318,7 @@ int launch_tc(const CUtensorMap& tl, const CUtensorMap& tc, const CUtensorMap& t
     if (ctas <= 0) return TFF_ERR_LAUNCH;
     if (ctas > units) ctas = units;
     return tff_launch_pdl(kern, dim3((unsigned)ctas), dim3(NUM_THREADS), (size_t)Cfg::kSmemBytes, stream, tl, tc, to,
-                          (TC*)out, rows_lane, rows_col, K, ldo, stream_k, tff_device_error_flag(), lane_group, group_rows);
+                          (TC*)out, rows_lane, rows_col, K, ldo, stream_k, tff_device_error_flag(), lane_group, group_rows, gc);
 }
 
 template <int BN, bool SWAP, bool TMA_OUT>
@@ -451,12 +451,12 @@ TFF_API int tff_gemm_tc_act(const void* A, const void* W, void* out, int M, int 
 // and tile t is multiplied with its group's rows of W:  out[rows, group_rows] = A W_g^T (act 2, not gated: the square of
 // relu of it, bfloat16), or, gated, out[rows,
 // group_rows / 2] = act(A Wg_g^T) * (A Wu_g^T) with every group's gate and up rows alternating in blocks of 64 as
-// above.  The rows of a routed feed-forward's tokens, sorted by expert with every expert's share padded to 128.
+// above (act 3: the clipped form with ``limit`` and ``slope``).  The rows of a routed feed-forward's tokens, sorted by expert with every expert's share padded to 128.
 TFF_API int tff_gemm_tc_grouped(const void* A, const void* W, void* out, int out_is_bf16, int rows, int groups,
-                                int group_rows, int K, int bn, int gated, int act, const int* lane_group,
-                                cudaStream_t stream) {
+                                int group_rows, int K, int bn, int gated, int act, float limit, float slope,
+                                const int* lane_group, cudaStream_t stream) {
     if (rows <= 0 || groups <= 0 || group_rows <= 0) return TFF_OK;
-    if (K <= 0 || !lane_group || (act != 0 && act != 1 && !(act == 2 && !gated))) return TFF_ERR_BAD_ARGUMENT;
+    if (K <= 0 || !lane_group || (act != 0 && act != 1 && !(act == 2 && !gated) && !(act == 3 && gated))) return TFF_ERR_BAD_ARGUMENT;
     if (K % 8 != 0 || rows % BM != 0 || (bn != 128 && bn != 256)) return TFF_ERR_UNSUPPORTED;
     if (((uintptr_t)A & 15) || ((uintptr_t)W & 15) || ((uintptr_t)out & 15)) return TFF_ERR_UNSUPPORTED;
     if (tff_device_error_flag() == nullptr) return TFF_ERR_LAUNCH;
@@ -467,6 +467,11 @@ TFF_API int tff_gemm_tc_grouped(const void* A, const void* W, void* out, int out
         const int I = group_rows / 2;
         if (group_rows % 128 != 0 || !out_is_bf16) return TFF_ERR_UNSUPPORTED;
         if (!tff_tensor_map_2d(out, rows, I, 32, 64, 2, &to)) return TFF_ERR_DRIVER;
+        if (act == 3) {
+            const GateConstants gc{limit, slope};
+            if (bn == 256) return launch_tc<256, false, EPI_CLIP, bf16, true>(tl, tc, to, out, rows, group_rows, K, I, 0, stream, lane_group, group_rows, gc);
+            return launch_tc<128, false, EPI_CLIP, bf16, true>(tl, tc, to, out, rows, group_rows, K, I, 0, stream, lane_group, group_rows, gc);
+        }
         if (act) {
             if (bn == 256) return launch_tc<256, false, EPI_GEGLU, bf16, true>(tl, tc, to, out, rows, group_rows, K, I, 0, stream, lane_group, group_rows);
             return launch_tc<128, false, EPI_GEGLU, bf16, true>(tl, tc, to, out, rows, group_rows, K, I, 0, stream, lane_group, group_rows);

@@ -10,6 +10,9 @@
 //            and the combine kernel adds them from the input rows
 //   plan     one block: the experts' row ranges in the sorted order, the tile table of the grouped product (tiles of
 //            ``tile_rows`` rows that never span two experts), and the counters back to zero for the next call
+//   table    instead of route and plan where a table gives every token id its experts (no router): one block counts the
+//            experts' pairs in shared memory, lays out their rows and tiles as plan does, and gives every pair its place
+//            (an atomic cursor in shared memory, as gather's), its weight 1/top, and every place its token row
 //   gather   per pair: its place among its expert's rows (an atomic cursor: the order within an expert is not fixed,
 //            but a row's result does not depend on its place), row_map[place] = pair, and the expert's input row
 //            x[place] = w * h[token] (weight on the input) or h[token]
@@ -217,6 +220,92 @@ __global__ void moe_plan_kernel(int* __restrict__ counts, int E, int tile_rows, 
     *num_tiles = n;
 }
 
+constexpr int TABLE_THREADS = 1024;
+
+__global__ void __launch_bounds__(TABLE_THREADS)
+moe_table_kernel(const int* __restrict__ tokens, const int* __restrict__ table, int table_rows, int P, int top, int E,
+                 int tile_rows, int pad_rows, int* __restrict__ pair_expert, float* __restrict__ pair_weight,
+                 int* __restrict__ row_map, int* __restrict__ token_of_row, int* __restrict__ place_of_pair,
+                 int* __restrict__ tile_group, int* __restrict__ tile_row0, int* __restrict__ tile_row_end,
+                 int* __restrict__ num_tiles, int* __restrict__ lane_group, int lane_tiles) {
+    extern __shared__ int smi[];
+    int* count = smi;                          // [E] pairs of the expert, later its cursor
+    int* first = smi + E;                      // [E] its first row
+    int* tile0 = first + E;                    // [E] its first tile
+    pdl_launch_dependents();
+    const int tid = threadIdx.x;
+    for (int e = tid; e < E; e += TABLE_THREADS) count[e] = 0;
+    __syncthreads();
+    pdl_wait();
+    if (lane_group)
+        for (int i = tid; i < lane_tiles; i += TABLE_THREADS) lane_group[i] = -1;
+    const float w = 1.0f / (float)top;
+    for (int i = tid; i < P; i += TABLE_THREADS) {
+        const int tok = tokens[i / top];
+        int e = (tok >= 0 && tok < table_rows) ? table[(size_t)tok * top + i % top] : -1;
+        if (e < 0 || e >= E) e = -1;           // the host refuses such ids and tables; never a wrong row
+        pair_expert[i] = e;
+        pair_weight[i] = w;
+        if (e >= 0) atomicAdd(&count[e], 1);
+    }
+    __syncthreads();
+    if (tid < 32) {                            // rows and tiles of the experts ahead, 32 experts at a time
+        int rows = 0, tiles = 0;
+        for (int e0 = 0; e0 < E; e0 += 32) {
+            const int e = e0 + tid;
+            const int c = e < E ? count[e] : 0;
+            int r = pad_rows > 0 ? (c + pad_rows - 1) / pad_rows * pad_rows : c, n = (c + tile_rows - 1) / tile_rows;
+            const int own_r = r, own_n = n;
+#pragma unroll
+            for (int o = 1; o < 32; o <<= 1) {
+                const int a = __shfl_up_sync(0xffffffffu, r, o), b = __shfl_up_sync(0xffffffffu, n, o);
+                if (tid >= o) { r += a; n += b; }
+            }
+            if (e < E) { first[e] = rows + r - own_r; tile0[e] = tiles + n - own_n; }
+            rows += __shfl_sync(0xffffffffu, r, 31);
+            tiles += __shfl_sync(0xffffffffu, n, 31);
+        }
+        if (tid == 0) *num_tiles = tiles;
+    }
+    __syncthreads();
+    for (int e = tid; e < E; e += TABLE_THREADS) {
+        const int c = count[e], r0 = first[e];
+        int n = tile0[e];
+        for (int r = r0; r < r0 + c; r += tile_rows, ++n) {
+            tile_group[n] = e; tile_row0[n] = r; tile_row_end[n] = r0 + c;
+            if (lane_group) lane_group[r / pad_rows] = e;
+        }
+        count[e] = r0;                         // from here on the cursor
+    }
+    __syncthreads();
+    for (int i = tid; i < P; i += TABLE_THREADS) {
+        const int e = pair_expert[i];          // this thread wrote it
+        const int place = e >= 0 ? atomicAdd(&count[e], 1) : -1;
+        if (place >= 0) { row_map[place] = i; token_of_row[place] = i / top; }
+        if (place_of_pair) place_of_pair[i] = place;
+    }
+}
+
+// x[place_of_pair[pair]] = h[pair / top]; rows of whole tiles beyond an expert's own are left as they are (their products
+// are never read).
+template <typename TH>
+__global__ void __launch_bounds__(128)
+moe_spread_kernel(const TH* __restrict__ h, int W, int top, const int* __restrict__ place_of_pair, TH* __restrict__ x) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int place = __ldcg(place_of_pair + blockIdx.x);
+    if (place < 0) return;
+    const TH* src = h + (size_t)(blockIdx.x / top) * W;
+    TH* dst = x + (size_t)place * W;
+    constexpr int N = 16 / sizeof(TH);
+    if (W % N == 0 && (((uintptr_t)h | (uintptr_t)x) & 15) == 0) {
+        for (int i = threadIdx.x; i < W / N; i += 128)
+            reinterpret_cast<uint4*>(dst)[i] = __ldcg(reinterpret_cast<const uint4*>(src) + i);
+    } else {
+        for (int i = threadIdx.x; i < W; i += 128) dst[i] = src[i];
+    }
+}
+
 template <typename TH>
 __global__ void __launch_bounds__(128)
 moe_gather_kernel(const TH* __restrict__ h, int W, int top, const int* __restrict__ pair_expert,
@@ -257,12 +346,12 @@ moe_combine_kernel(const float* __restrict__ y, int W, int top, const float* __r
     float acc = 0.f;
     for (int k = 0; k < top; ++k) {
         const size_t pair = (size_t)t * top + k;              // y in (token, rank) order, or in the sorted order
-        if (pair_expert && pair_expert[pair] < 0) {           // an identity expert: the weight times the input itself
+        if (pair_expert && __ldcg(pair_expert + pair) < 0) {           // an identity expert: the weight times the input itself
             acc = fmaf(pair_weight[pair], to_f32<TH>(h[(size_t)t * W + i]), acc);
             continue;
         }
-        const float w = weight_on_output ? pair_weight[pair] : 1.f;
-        acc = fmaf(w, y[(place_of_pair ? (size_t)place_of_pair[pair] : pair) * W + i], acc);
+        const float w = weight_on_output ? __ldcg(pair_weight + pair) : 1.f;
+        acc = fmaf(w, __ldcg(y + (place_of_pair ? (size_t)__ldcg(place_of_pair + pair) : pair) * W + i), acc);
     }
     const size_t at = (size_t)t * W + i;
     out[at] = residual ? residual[at] + acc : acc;
@@ -307,6 +396,33 @@ TFF_API int tff_moe_plan(int* counts, int E, int tile_rows, int* cursor, int* ti
         return TFF_ERR_BAD_ARGUMENT;
     return tff_launch_pdl(moe_plan_kernel, dim3(1), dim3(128), 0, stream, counts, E, tile_rows, cursor, tile_group,
                           tile_row0, tile_row_end, num_tiles, pad_rows, lane_group, lane_tiles);
+}
+
+// tokens [P / top] int32, table [table_rows, top] int32.  Outputs as tff_moe_route, tff_moe_plan and tff_moe_gather leave
+// them (place_of_pair and lane_group may be null), and token_of_row: sorted place -> row of the step's tokens.
+TFF_API int tff_moe_table(const int* tokens, const int* table, int table_rows, int P, int top, int E, int tile_rows,
+                          int pad_rows, int* pair_expert, float* pair_weight, int* row_map, int* token_of_row,
+                          int* place_of_pair, int* tile_group, int* tile_row0, int* tile_row_end, int* num_tiles,
+                          int* lane_group, int lane_tiles, cudaStream_t stream) {
+    if (P <= 0) return TFF_OK;
+    if (!tokens || !table || table_rows <= 0 || top <= 0 || P % top || E <= 0 || tile_rows <= 0 || pad_rows < 0 ||
+        (pad_rows > 0 && pad_rows != tile_rows) || (lane_group && pad_rows <= 0) || !pair_expert || !pair_weight || !row_map ||
+        !token_of_row || !tile_group || !tile_row0 || !tile_row_end || !num_tiles)
+        return TFF_ERR_BAD_ARGUMENT;
+    const size_t smem = (size_t)3 * E * sizeof(int);
+    if (smem > 48 * 1024) return TFF_ERR_UNSUPPORTED;
+    return tff_launch_pdl(moe_table_kernel, dim3(1), dim3(TABLE_THREADS), smem, stream, tokens, table, table_rows, P, top, E,
+                          tile_rows, pad_rows, pair_expert, pair_weight, row_map, token_of_row, place_of_pair, tile_group,
+                          tile_row0, tile_row_end, num_tiles, lane_group, lane_tiles);
+}
+
+TFF_API int tff_moe_spread(const void* h, int h_dt, int pairs, int W, int top, const int* place_of_pair, void* x,
+                           cudaStream_t stream) {
+    if (pairs <= 0) return TFF_OK;
+    if (!h || !x || !place_of_pair || top <= 0 || W <= 0) return TFF_ERR_BAD_ARGUMENT;
+    if (h_dt == 0)
+        return tff_launch_pdl(moe_spread_kernel<float>, dim3(pairs), dim3(128), 0, stream, (const float*)h, W, top, place_of_pair, (float*)x);
+    return tff_launch_pdl(moe_spread_kernel<bf16>, dim3(pairs), dim3(128), 0, stream, (const bf16*)h, W, top, place_of_pair, (bf16*)x);
 }
 
 TFF_API int tff_moe_gather(const void* h, int h_dt, int pairs, int W, int top, const int* pair_expert,

@@ -17,6 +17,11 @@
 // element walks the chunks in order.  Chunks are aligned to absolute positions of the request, so that the order of
 // the additions that make a token's output depends on its position (and on where a portion was cut), not on what
 // else is in the batch.
+//
+// The raw form (tff_retention_raw) is the recurrence alone: q, k and v are column blocks of float32 rows, optionally
+// with a silu applied where they are read, and the output is o itself in float32 (norms and gates are another kernel's
+// business).  Its decode kernel (steps of one token a request) streams the state through registers: a CTA per 32 value
+// columns of a (head, request), four columns a thread, all rows of a thread asked for ahead of the arithmetic.
 #include "common.cuh"
 #include <type_traits>
 
@@ -38,13 +43,19 @@ template <> __device__ __forceinline__ void store4<bf16>(bf16* p, float a, float
 }
 
 struct RetParams {
-    const float* q; const float* k; float* vg; int ld, v_off, g_off;
+    const float* q; const float* k; int q_ld, k_ld; float* vg; int ld, v_off, g_off;
+    int silu;                          // q, k and v pass through a silu where they are read
     int clear;                         // v and g are set to zero behind the read (the rows are an accumulator buffer)
     float* state; int num_slots;
     const int* q_start; const int* pos_start; const int* slots;
     const float* decay;                // [H] on the device
     void* out; int H, d, dv; float eps;
 };
+
+__device__ __forceinline__ float ret_in(float x, int silu) { return silu ? x / (1.0f + expf(-x)) : x; }
+__device__ __forceinline__ float4 ret_in4(float4 x, int silu) {
+    return make_float4(ret_in(x.x, silu), ret_in(x.y, silu), ret_in(x.z, silu), ret_in(x.w, silu));
+}
 
 // ------------------------------------------------------------------ token by token
 // IN_SMEM: the head's state fits shared memory beside the rest (else it is worked on where it lies)
@@ -77,8 +88,8 @@ retention_step_kernel(RetParams p) {
     for (int t = t0; t < t1; ++t) {
         __syncthreads();
         for (int i = threadIdx.x; i < d; i += NT) {
-            sq[i] = p.q[(size_t)t * p.H * d + (size_t)h * d + i];
-            sk[i] = p.k[(size_t)t * p.H * d + (size_t)h * d + i];
+            sq[i] = p.q[(size_t)t * p.q_ld + (size_t)h * d + i];
+            sk[i] = p.k[(size_t)t * p.k_ld + (size_t)h * d + i];
         }
         for (int i = threadIdx.x; i < dv; i += NT) {
             sv[i] = p.vg[(size_t)t * p.ld + p.v_off + h * dv + i];
@@ -115,6 +126,81 @@ retention_step_kernel(RetParams p) {
     }
     __syncthreads();
     if (IN_SMEM) for (int e = threadIdx.x; e < d * dv; e += NT) gs[e] = S[e];
+}
+
+// The raw form: VEC value columns a thread (4: 16-byte accesses), 32 columns a CTA.
+constexpr int DT = 128;
+
+template <int VEC>
+__global__ void __launch_bounds__(DT)
+retention_decode_kernel(RetParams p) {
+    extern __shared__ __align__(16) float sm[];
+    constexpr int LX = 32 / VEC, NY = DT / LX, UNROLL = 8;
+    typedef typename std::conditional<VEC == 4, float4, float>::type V;
+    pdl_launch_dependents();
+    const int h = blockIdx.y, b = blockIdx.z, d = p.d, dv = p.dv;
+    float* sq = sm;                     // [d]
+    float* sk = sq + d;                 // [d]
+    float* part = sk + d;               // [NY][33]
+    const int lx = threadIdx.x % LX, ty = threadIdx.x / LX;
+    const int j = blockIdx.x * 32 + lx * VEC;
+    const bool active = j < dv;
+    const int t0 = p.q_start[b], t1 = p.q_start[b + 1];
+    const int slot = p.slots[b];
+    const float decay = p.decay[h];
+    const bool ok = t1 > t0 && slot >= 0 && slot < p.num_slots;
+    float* S = p.state + ((size_t)(ok ? slot : 0) * p.H + h) * d * dv + j;
+    bool fresh = p.pos_start[b] == 0;
+    if (ok && !fresh && active && lx == 0)        // into the second-level cache while the kernels ahead are still at work
+        for (int i = ty; i < d; i += NY) asm volatile("prefetch.global.L2 [%0];" ::"l"(S + (size_t)i * dv));
+    pdl_wait();
+    if (!ok) return;
+    for (int t = t0; t < t1; ++t, fresh = false) {
+        __syncthreads();
+        for (int i = threadIdx.x; i < d; i += DT) {
+            sq[i] = ret_in(__ldcg(p.q + (size_t)t * p.q_ld + (size_t)h * d + i), p.silu);
+            sk[i] = ret_in(__ldcg(p.k + (size_t)t * p.k_ld + (size_t)h * d + i), p.silu);
+        }
+        float v[VEC], acc[VEC];
+#pragma unroll
+        for (int c = 0; c < VEC; ++c) {
+            v[c] = active ? ret_in(__ldcg(p.vg + (size_t)t * p.ld + p.v_off + (size_t)h * dv + j + c), p.silu) : 0.f;
+            acc[c] = 0.f;
+        }
+        __syncthreads();
+        if (active) {
+            for (int i0 = ty; i0 < d; i0 += NY * UNROLL) {
+                V s[UNROLL];
+#pragma unroll
+                for (int u = 0; u < UNROLL; ++u) {
+                    const int i = i0 + u * NY;
+                    if constexpr (VEC == 4) s[u] = make_float4(0.f, 0.f, 0.f, 0.f); else s[u] = 0.f;
+                    if (i < d && !fresh) s[u] = __ldcg(reinterpret_cast<const V*>(S + (size_t)i * dv));
+                }
+#pragma unroll
+                for (int u = 0; u < UNROLL; ++u) {
+                    const int i = i0 + u * NY;
+                    if (i >= d) continue;
+                    const float ki = sk[i], qi = sq[i];
+                    float* e = reinterpret_cast<float*>(&s[u]);
+#pragma unroll
+                    for (int c = 0; c < VEC; ++c) {
+                        e[c] = fmaf(decay, e[c], ki * v[c]);
+                        acc[c] = fmaf(e[c], qi, acc[c]);
+                    }
+                    *reinterpret_cast<V*>(S + (size_t)i * dv) = s[u];
+                }
+            }
+        }
+#pragma unroll
+        for (int c = 0; c < VEC; ++c) part[ty * 33 + lx * VEC + c] = acc[c];
+        __syncthreads();
+        if (threadIdx.x < 32 && blockIdx.x * 32 + threadIdx.x < dv) {
+            float o = 0.f;
+            for (int y = 0; y < NY; ++y) o += part[y * 33 + threadIdx.x];
+            ((float*)p.out)[(size_t)t * p.H * dv + (size_t)h * dv + blockIdx.x * 32 + threadIdx.x] = o;
+        }
+    }
 }
 
 // ------------------------------------------------------------------ chunk by chunk
@@ -216,12 +302,12 @@ retention_local_kernel(RetParams p, int num_requests, float* __restrict__ acc, f
     __syncthreads();
     for (int e = threadIdx.x; e < n * d; e += NT) {
         const int i = e / d, r = e % d;
-        sq[i * dP + r] = p.q[(size_t)(c.t + i) * p.H * d + (size_t)h * d + r];
-        skT[r * C + i] = p.k[(size_t)(c.t + i) * p.H * d + (size_t)h * d + r];
+        sq[i * dP + r] = ret_in(__ldcg(p.q + (size_t)(c.t + i) * p.q_ld + (size_t)h * d + r), p.silu);
+        skT[r * C + i] = ret_in(__ldcg(p.k + (size_t)(c.t + i) * p.k_ld + (size_t)h * d + r), p.silu);
     }
     for (int e = threadIdx.x; e < n * dv; e += NT) {
         const int i = e / dv, r = e % dv;
-        sv[i * vP + r] = p.vg[(size_t)(c.t + i) * p.ld + p.v_off + h * dv + r];
+        sv[i * vP + r] = ret_in(__ldcg(p.vg + (size_t)(c.t + i) * p.ld + p.v_off + h * dv + r), p.silu);
         if (p.clear) p.vg[(size_t)(c.t + i) * p.ld + p.v_off + h * dv + r] = 0.f;
     }
     __syncthreads();
@@ -259,7 +345,9 @@ retention_scan_kernel(RetParams p, int num_requests, float* __restrict__ U) {
     const int count = (pos0 + len - 1) / C - pos0 / C + 1;
     typedef typename std::conditional<VEC == 4, float4, float>::type V;
     V* gs = reinterpret_cast<V*>(p.state + ((size_t)slot * p.H + h) * p.d * p.dv + e);
-    V S = *gs;
+    V S;
+    if (pos0 == 0) { if constexpr (VEC == 4) S = make_float4(0.f, 0.f, 0.f, 0.f); else S = 0.f; }
+    else S = __ldcg(gs);
     const size_t stride = (size_t)p.H * p.d * p.dv / VEC;             // V's between a chunk's U and the next one's
     V* u0 = reinterpret_cast<V*>(U + ((size_t)first_chunk * p.H + h) * p.d * p.dv + e);
     float g_full = 1.f;
@@ -269,7 +357,7 @@ retention_scan_kernel(RetParams p, int num_requests, float* __restrict__ U) {
     for (int c0 = 0; c0 < count; c0 += 8) {
         V add[8];
 #pragma unroll
-        for (int j = 0; j < 8; ++j) if (c0 + j < count) add[j] = u0[(size_t)(c0 + j) * stride];
+        for (int j = 0; j < 8; ++j) if (c0 + j < count) add[j] = __ldcg(u0 + (size_t)(c0 + j) * stride);
 #pragma unroll
         for (int j = 0; j < 8; ++j) {
             const int c = c0 + j;
@@ -294,7 +382,8 @@ retention_scan_kernel(RetParams p, int num_requests, float* __restrict__ U) {
 // at 128 x 128: two CTAs an SM, one loading while the other multiplies).
 constexpr int NB = 64;
 
-template <typename TO>
+// RAW: the outputs themselves go to ``out`` (float32): no norm, no gate
+template <typename TO, bool RAW>
 __global__ void __launch_bounds__(NT)
 retention_finish_kernel(RetParams p, int num_requests, const float* __restrict__ acc, const float* __restrict__ U) {
     extern __shared__ __align__(16) float sm[];
@@ -312,20 +401,21 @@ retention_finish_kernel(RetParams p, int num_requests, const float* __restrict__
     if (!have) return;
     const int n = c.n;
     const float* Sc = U + ((size_t)blockIdx.x * p.H + h) * d * dv;
-    const float* qg = p.q + (size_t)c.t * p.H * d + (size_t)h * d;
+    const float* qg = p.q + (size_t)c.t * p.q_ld + (size_t)h * d;
     // rows of four: 16-byte loads when every row starts on such a boundary
-    const bool vec = (d & 3) == 0 && (dv & 3) == 0 && (((uintptr_t)p.q | (uintptr_t)U) & 15) == 0;
+    const bool vec = (d & 3) == 0 && (dv & 3) == 0 && (p.q_ld & 3) == 0 && (((uintptr_t)p.q | (uintptr_t)U) & 15) == 0;
     if (vec) {
         const int d4 = d >> 2;
         for (int e = threadIdx.x; e < pad4(n) * d4; e += NT) {
             const int i = e / d4, r = e % d4;
             reinterpret_cast<float4*>(sq + i * dP)[r] =
-                i < n ? reinterpret_cast<const float4*>(qg + (size_t)i * p.H * d)[r] : make_float4(0.f, 0.f, 0.f, 0.f);
+                i < n ? ret_in4(__ldcg(reinterpret_cast<const float4*>(qg + (size_t)i * p.q_ld) + r), p.silu)
+                      : make_float4(0.f, 0.f, 0.f, 0.f);
         }
     } else {
         for (int e = threadIdx.x; e < C * dP; e += NT) sq[e] = 0.f;
         __syncthreads();
-        for (int e = threadIdx.x; e < n * d; e += NT) sq[(e / d) * dP + e % d] = qg[(size_t)(e / d) * p.H * d + e % d];
+        for (int e = threadIdx.x; e < n * d; e += NT) sq[(e / d) * dP + e % d] = ret_in(__ldcg(qg + (size_t)(e / d) * p.q_ld + e % d), p.silu);
     }
     // the chunk's local part goes into the output tile first (the product below adds to it): loads asked for together
     // here, not one by one between the product's stores
@@ -333,9 +423,9 @@ retention_finish_kernel(RetParams p, int num_requests, const float* __restrict__
     if (vec && (((uintptr_t)acc) & 15) == 0) {
         const int v4 = dv >> 2;
         for (int e = threadIdx.x; e < n * v4; e += NT)
-            reinterpret_cast<float4*>(so + (e / v4) * vP)[e % v4] = reinterpret_cast<const float4*>(ag + (size_t)(e / v4) * p.H * dv)[e % v4];
+            reinterpret_cast<float4*>(so + (e / v4) * vP)[e % v4] = __ldcg(reinterpret_cast<const float4*>(ag + (size_t)(e / v4) * p.H * dv) + e % v4);
     } else {
-        for (int e = threadIdx.x; e < n * dv; e += NT) so[(e / dv) * vP + e % dv] = ag[(size_t)(e / dv) * p.H * dv + e % dv];
+        for (int e = threadIdx.x; e < n * dv; e += NT) so[(e / dv) * vP + e % dv] = __ldcg(ag + (size_t)(e / dv) * p.H * dv + e % dv);
     }
     for (int n0 = 0; n0 < dv; n0 += NB) {
         const int nb = min(NB, dv - n0);
@@ -344,12 +434,12 @@ retention_finish_kernel(RetParams p, int num_requests, const float* __restrict__
             const int b4 = nb >> 2;
             for (int e = threadIdx.x; e < d * b4; e += NT) {
                 const int r = e / b4, cc = e % b4;
-                reinterpret_cast<float4*>(sS + r * NB)[cc] = reinterpret_cast<const float4*>(Sc + (size_t)r * dv + n0)[cc];
+                reinterpret_cast<float4*>(sS + r * NB)[cc] = __ldcg(reinterpret_cast<const float4*>(Sc + (size_t)r * dv + n0) + cc);
             }
         } else {
             for (int e = threadIdx.x; e < dP * NB; e += NT) {
                 const int r = e / NB, cc = e % NB;
-                sS[e] = (r < d && cc < nb) ? Sc[(size_t)r * dv + n0 + cc] : 0.f;
+                sS[e] = (r < d && cc < nb) ? __ldcg(Sc + (size_t)r * dv + n0 + cc) : 0.f;
             }
         }
         __syncthreads();
@@ -358,6 +448,17 @@ retention_finish_kernel(RetParams p, int num_requests, const float* __restrict__
         });
     }
     __syncthreads();
+    if constexpr (RAW) {
+        float* og = (float*)p.out + (size_t)c.t * p.H * dv + (size_t)h * dv;
+        if (vec && ((uintptr_t)p.out & 15) == 0) {
+            const int v4 = dv >> 2;
+            for (int e = threadIdx.x; e < n * v4; e += NT)
+                reinterpret_cast<float4*>(og + (size_t)(e / v4) * p.H * dv)[e % v4] = reinterpret_cast<const float4*>(so + (e / v4) * vP)[e % v4];
+        } else {
+            for (int e = threadIdx.x; e < n * dv; e += NT) og[(size_t)(e / dv) * p.H * dv + e % dv] = so[(e / dv) * vP + e % dv];
+        }
+        return;
+    }
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     float* gg = p.vg + (size_t)c.t * p.ld + p.g_off + h * dv;         // the chunk's gates, rows ld apart
     if (vec && (p.ld & 3) == 0 && (((uintptr_t)gg | (uintptr_t)p.out) & 15) == 0) {
@@ -416,6 +517,38 @@ TFF_API long long tff_retention_workspace(int num_tokens, int num_requests, int 
     return (long long)num_tokens * H * dv + chunks * H * d * dv;
 }
 
+namespace {
+
+constexpr size_t MOST = 224 * 1024;        // dynamic shared memory a CTA may ask for here (the kernels have a little static on top)
+
+// The three kernels of the chunked form; FIN the finish kernel of the form asked for.
+template <typename Fin>
+int launch_chunked(const RetParams& p, int num_requests, float* workspace, int num_tokens, Fin finish, cudaStream_t stream) {
+    if (!workspace || num_tokens <= 0) return TFF_ERR_BAD_ARGUMENT;
+    const int H = p.H, d = p.d, dv = p.dv, dP = pad4(d), vP = pad4(dv);
+    const size_t smem1 = sizeof(float) * ((size_t)C * dP + (size_t)dP * C + (size_t)C * vP + (size_t)C * C);
+    const size_t smem3 = sizeof(float) * ((size_t)C * dP + (size_t)dP * NB + (size_t)C * vP);
+    if (smem1 > MOST || smem3 > MOST) return TFF_ERR_UNSUPPORTED;
+    const int chunks = num_tokens / C + 2 * num_requests;
+    float* acc = workspace;
+    float* U = workspace + (size_t)num_tokens * H * dv;
+    if (cudaFuncSetAttribute(retention_local_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)MOST) != cudaSuccess ||
+        cudaFuncSetAttribute(finish, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)MOST) != cudaSuccess)
+        return TFF_ERR_LAUNCH;
+    int st = tff_launch_pdl(retention_local_kernel, dim3(chunks, H), dim3(NT), smem1, stream, p, num_requests, acc, U);
+    if (st != TFF_OK) return st;
+    if ((d * dv) % 4 == 0 && ((uintptr_t)p.state & 15) == 0 && ((uintptr_t)U & 15) == 0)
+        st = tff_launch_pdl(retention_scan_kernel<4>, dim3((d * dv / 4 + NT - 1) / NT, H, num_requests), dim3(NT), (size_t)0,
+                            stream, p, num_requests, U);
+    else
+        st = tff_launch_pdl(retention_scan_kernel<1>, dim3((d * dv + NT - 1) / NT, H, num_requests), dim3(NT), (size_t)0,
+                            stream, p, num_requests, U);
+    if (st != TFF_OK) return st;
+    return tff_launch_pdl(finish, dim3(chunks, H), dim3(NT), smem3, stream, p, num_requests, (const float*)acc, (const float*)U);
+}
+
+}  // namespace
+
 // clear_vg != 0: the v and g columns of ``vg`` are set to zero once read.
 // chunked != 0: chunk by chunk (portions of prompts; ``workspace`` of tff_retention_workspace floats, ``num_tokens``
 // the step's tokens); else token by token (decoded tokens).  TFF_ERR_UNSUPPORTED when a head does not fit the
@@ -430,41 +563,13 @@ TFF_API int tff_retention(
         return TFF_ERR_BAD_ARGUMENT;
     if (num_requests > 65535 || H > 65535) return TFF_ERR_UNSUPPORTED;
     RetParams p;
-    p.q = q; p.k = k; p.vg = vg; p.clear = clear_vg; p.ld = ld; p.v_off = v_off; p.g_off = g_off;
+    p.q = q; p.k = k; p.q_ld = p.k_ld = H * d; p.vg = vg; p.clear = clear_vg; p.ld = ld; p.v_off = v_off; p.g_off = g_off;
+    p.silu = 0;
     p.state = state; p.num_slots = num_slots; p.q_start = q_start; p.pos_start = pos_start; p.slots = slots;
     p.decay = decay; p.out = out; p.H = H; p.d = d; p.dv = dv; p.eps = eps;
-    constexpr size_t MOST = 224 * 1024;        // dynamic shared memory a CTA may ask for here (the kernels have a little static on top)
     if (chunked) {
-        if (!workspace || num_tokens <= 0) return TFF_ERR_BAD_ARGUMENT;
-        const int dP = pad4(d), vP = pad4(dv);
-        const size_t smem1 = sizeof(float) * ((size_t)C * dP + (size_t)dP * C + (size_t)C * vP + (size_t)C * C);
-        const size_t smem3 = sizeof(float) * ((size_t)C * dP + (size_t)dP * NB + (size_t)C * vP);
-        if (smem1 > MOST || smem3 > MOST) return TFF_ERR_UNSUPPORTED;
-        const int chunks = num_tokens / C + 2 * num_requests;
-        float* acc = workspace;
-        float* U = workspace + (size_t)num_tokens * H * dv;
-        static bool configured = false;
-        if (!configured) {
-            if (cudaFuncSetAttribute(retention_local_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)MOST) != cudaSuccess ||
-                cudaFuncSetAttribute(retention_finish_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)MOST) != cudaSuccess ||
-                cudaFuncSetAttribute(retention_finish_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)MOST) != cudaSuccess)
-                return TFF_ERR_LAUNCH;
-            configured = true;
-        }
-        int st = tff_launch_pdl(retention_local_kernel, dim3(chunks, H), dim3(NT), smem1, stream, p, num_requests, acc, U);
-        if (st != TFF_OK) return st;
-        if ((d * dv) % 4 == 0 && ((uintptr_t)state & 15) == 0 && ((uintptr_t)U & 15) == 0)
-            st = tff_launch_pdl(retention_scan_kernel<4>, dim3((d * dv / 4 + NT - 1) / NT, H, num_requests), dim3(NT), (size_t)0,
-                                stream, p, num_requests, U);
-        else
-            st = tff_launch_pdl(retention_scan_kernel<1>, dim3((d * dv + NT - 1) / NT, H, num_requests), dim3(NT), (size_t)0,
-                                stream, p, num_requests, U);
-        if (st != TFF_OK) return st;
-        if (out_is_bf16)
-            return tff_launch_pdl(retention_finish_kernel<bf16>, dim3(chunks, H), dim3(NT), smem3, stream, p, num_requests,
-                                  (const float*)acc, (const float*)U);
-        return tff_launch_pdl(retention_finish_kernel<float>, dim3(chunks, H), dim3(NT), smem3, stream, p, num_requests,
-                              (const float*)acc, (const float*)U);
+        if (out_is_bf16) return launch_chunked(p, num_requests, workspace, num_tokens, retention_finish_kernel<bf16, false>, stream);
+        return launch_chunked(p, num_requests, workspace, num_tokens, retention_finish_kernel<float, false>, stream);
     }
     const size_t rest = sizeof(float) * ((size_t)2 * d + dv + (size_t)(NT / (dv < NT ? dv : NT)) * dv + 32);
     const int in_smem = sizeof(float) * (size_t)d * dv + rest <= MOST ? 1 : 0;
@@ -486,4 +591,30 @@ TFF_API int tff_retention(
     }
     if (out_is_bf16) return tff_launch_pdl(retention_step_kernel<bf16, false>, grid, dim3(NT), smem, stream, p);
     return tff_launch_pdl(retention_step_kernel<float, false>, grid, dim3(NT), smem, stream, p);
+}
+
+// The recurrence alone: q, k, v are column blocks of the float32 rows ``proj`` (leading dimension ld, first columns q_off,
+// k_off, v_off), passed through a silu when ``silu`` is set; out float32 [T, H*dv].  A request that brings position 0
+// starts from a zero state whatever its slot holds.  chunked as above.
+TFF_API int tff_retention_raw(
+    const float* proj, int ld, int q_off, int k_off, int v_off, int silu, float* state, int num_slots, const int* q_start,
+    const int* pos_start, const int* slots, const float* decay, float* out, int num_requests, int H, int d, int dv,
+    int chunked, float* workspace, int num_tokens, cudaStream_t stream) {
+    if (num_requests <= 0) return TFF_OK;
+    if (!proj || !state || !q_start || !pos_start || !slots || !decay || !out || H <= 0 || d <= 0 || dv <= 0 || q_off < 0 ||
+        k_off < 0 || v_off < 0 || q_off + H * d > ld || k_off + H * d > ld || v_off + H * dv > ld)
+        return TFF_ERR_BAD_ARGUMENT;
+    if (num_requests > 65535 || H > 65535) return TFF_ERR_UNSUPPORTED;
+    RetParams p;
+    p.q = proj + q_off; p.k = proj + k_off; p.q_ld = p.k_ld = ld; p.vg = const_cast<float*>(proj); p.clear = 0; p.ld = ld;
+    p.v_off = v_off; p.g_off = 0; p.silu = silu;
+    p.state = state; p.num_slots = num_slots; p.q_start = q_start; p.pos_start = pos_start; p.slots = slots;
+    p.decay = decay; p.out = out; p.H = H; p.d = d; p.dv = dv; p.eps = 0.f;
+    if (chunked) return launch_chunked(p, num_requests, workspace, num_tokens, retention_finish_kernel<float, true>, stream);
+    const bool vec = dv % 4 == 0 && ((uintptr_t)state & 15) == 0;
+    const size_t smem = sizeof(float) * ((size_t)2 * d + 32 * 33);
+    if (smem > 48 * 1024) return TFF_ERR_UNSUPPORTED;
+    const dim3 grid((dv + 31) / 32, H, num_requests);
+    if (vec) return tff_launch_pdl(retention_decode_kernel<4>, grid, dim3(DT), smem, stream, p);
+    return tff_launch_pdl(retention_decode_kernel<1>, grid, dim3(DT), smem, stream, p);
 }

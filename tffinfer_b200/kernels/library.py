@@ -422,7 +422,9 @@ class CudaKernels:
     def _foldable_weight(self, w) -> bool:
         return w.dtype == torch.bfloat16 and w.is_contiguous() and w.data_ptr() % 16 == 0 and w.shape[1] % 8 == 0
 
-    ACTIVATION_CODES = {"silu": 0, "gelu_tanh": 1, "relu2": 2}    # relu2: the square of relu, of one product (not gated)
+    ACTIVATION_CODES = {"silu": 0, "gelu_tanh": 1, "relu2": 2,     # relu2: the square of relu, of one product (not gated)
+                        "clipped_swish": 3}    # gated: g sigmoid(1.702 g) (u + 1), g and u clipped at a limit (experts only)
+    CLIPPED_SLOPE = 1.702
 
     def gated_mlp(self, h, w_gate_up, w_down, residual, inter: int, activation: str = "silu", out=None) -> None:
         """residual += down(act(gate(h)) * up(h)); ``h`` the activation rows or a DeferredNorm of them.  With
@@ -699,6 +701,51 @@ class CudaKernels:
             self._acc_zero[vg.data_ptr()] = True
         self.launches += kernels
 
+    def lightning(self, h, w_in, batch, state, decay, norm_w, eps: float, out, H, d, dv) -> None:
+        """The whole of a lightning attention between its input rows and its output projection -> out [T, H*dv]: one
+        product for q, k, v and the gate (``w_in`` rows [q | k | v | gate | padding]) into float32; the recurrence over
+        ``state`` [slots, H, d, dv] with ``decay`` [H], a silu on q, k and v where its kernels read them; the RMS norm over
+        all heads with ``norm_w`` [H*dv] and the sigmoid gate."""
+        T = h.shape[0]
+        if isinstance(h, DeferredNorm):
+            h = h.materialize()
+        proj = self.projection_buffer(T, w_in.shape[0], h.device, h.dtype)
+        self.gemm(h, w_in, proj)
+        o = torch.empty((T, H * dv), dtype=torch.float32, device=h.device)
+        self.retention_raw(proj, 0, H * d, 2 * H * d, True, state, batch, decay, o, H, d, dv)
+        self.gated_norm(o, H * dv, proj, 2 * H * d + H * dv, norm_w, eps, False, out, clear_cols=(0, proj.shape[1]),
+                        last_reader=True, gate_act="sigmoid")
+
+    def retention_raw(self, proj, q_off: int, k_off: int, v_off: int, silu: bool, state, batch, decay, out, H, d, dv,
+                      chunked: Optional[bool] = None) -> None:
+        """The recurrence S <- decay S + k v^T, o = S^T q per head over ``state`` [slots, H, d, dv] (float32) -> out
+        float32 [T, H*dv]; q, k and v are columns q_off.., k_off.., v_off.. of the float32 rows ``proj``, passed through a
+        silu when ``silu``.  ``chunked`` as for ``retention``.  ``proj`` is left as it is."""
+        self._need_cuda(proj, state, decay, out)
+        T, ld = proj.shape
+        assert proj.dtype == state.dtype == decay.dtype == out.dtype == torch.float32 and tuple(out.shape) == (T, H * dv)
+        assert tuple(state.shape[1:]) == (H, d, dv) and decay.numel() == H
+        if chunked is None:
+            chunked = batch.max_q_len > 1
+
+        def run(ch: bool):
+            ws = None
+            if ch:
+                self.lib.tff_retention_workspace.restype = ctypes.c_longlong
+                need = int(self.lib.tff_retention_workspace(_c_int(T), _c_int(batch.num_requests), _c_int(H), _c_int(d), _c_int(dv)))
+                ws = torch.empty(need, dtype=torch.float32, device=proj.device)
+            return self.lib.tff_retention_raw(
+                _ptr(proj), _c_int(ld), _c_int(q_off), _c_int(k_off), _c_int(v_off), _c_int(1 if silu else 0), _ptr(state),
+                _c_int(state.shape[0]), _ptr(batch.q_start), _ptr(batch.pos_start), _ptr(batch.slots), _ptr(decay), _ptr(out),
+                _c_int(batch.num_requests), _c_int(H), _c_int(d), _c_int(dv), _c_int(1 if ch else 0), _ptr(ws), _c_int(T),
+                self._stream())
+        status = run(chunked)
+        if status == -2 and chunked:
+            chunked = False
+            status = run(False)                            # a head too large for the chunked form's shared memory
+        self._check(status, "retention_raw")
+        self.launches += 3 if chunked else 1
+
     # ------------------------------------------------------- attention in float32 tiles (any sizes, latent caches, biases)
     @staticmethod
     def _layer_cache(kv_cache, kv_layer: int):
@@ -715,19 +762,21 @@ class CudaKernels:
 
     def attention_tile(self, q, batch, block_table, kv_cache, kv_layer, page_size, out, nq, nkv, d, dv, scale,
                        window: int = 0, chunk: int = 0, temp=None, r1=None, r2=None, out_scale: float = 1.0,
-                       out_off: int = 0, num_splits=None, dense=None, softcap: float = 0.0) -> None:
+                       out_off: int = 0, num_splits=None, dense=None, softcap: float = 0.0, sink=None) -> None:
         """q [T, nq*d] against the paged cache -> columns out_off .. out_off + nq*dv of ``out`` (times out_scale), in
         float32 arithmetic whatever the storage type.  The cache has two planes (keys, values) or one (the value
         of a token is the first dv elements of its key).  Visibility: causal, within ``window`` keys, within the
         query's block of ``chunk`` positions.  Scores: (q . k) * scale * temp[h] - r1[h] * ln(1 + r2[h] * distance)
         (temp, r1, r2 float32 [nq] or None); with ``softcap`` > 0 the scaled product is squashed to softcap * tanh(. / softcap)
-        ahead of the distance term.  ``dense`` = (keys [T, nkv*d], values [T, nkv*dv]) of this step's own tokens
+        ahead of the distance term.  ``sink`` (float32 [nq] or None): a score per head that joins the softmax's denominator.
+        ``dense`` = (keys [T, nkv*d], values [T, nkv*dv]) of this step's own tokens
         instead of the cache: for steps whose requests all start at position 0 (bfloat16, tensor-core form only)."""
         self._need_cuda(q, block_table, out, temp, r1, r2)
         T = q.shape[0]
         assert q.dtype == out.dtype and q.shape[1] == nq * d and out.shape[0] == T and out.shape[1] >= out_off + nq * dv
-        for v in (temp, r1, r2):
+        for v in (temp, r1, r2, sink):
             assert v is None or (v.dtype == torch.float32 and v.numel() == nq)
+        self._need_cuda(sink)
         kd = vd = None
         if dense is not None:
             kd, vd = dense
@@ -750,7 +799,7 @@ class CudaKernels:
             _c_int(batch.max_q_len), _c_int(nq), _c_int(nkv), _c_int(d), _c_int(dv), _c_float(scale), _c_int(window),
             _c_int(chunk), _ptr(temp), _ptr(r1), _ptr(r2), _c_float(out_scale), _c_int(T), _c_int(splits), _ptr(part_o),
             _ptr(part_ml), _ptr(kd), _ptr(vd), _c_int(kd.shape[1] if kd is not None else 0),
-            _c_int(vd.shape[1] if vd is not None else 0), _c_float(softcap), self._stream()), "attention_tile")
+            _c_int(vd.shape[1] if vd is not None else 0), _c_float(softcap), _ptr(sink), self._stream()), "attention_tile")
         self.launches += 2 if splits > 1 else 1
 
     def tile_splits(self, batch, nq: int, nkv: int, window: int = 0, chunk: int = 0) -> int:
@@ -769,30 +818,33 @@ class CudaKernels:
 
     # ------------------------------------------------------- many small products in one launch
     def gemm_grouped(self, a, b, c, groups: int, M: int, N: int, K: int, lda: int, a_gs: int, ldb: int, b_gs: int,
-                     ldc: int, c_gs: int, gated: str = "", activation: str = "silu", tiles=None, row_map=None) -> None:
+                     ldc: int, c_gs: int, gated: str = "", activation: str = "silu", tiles=None, row_map=None,
+                     a_rows=None, limit: float = 0.0) -> None:
         """c_g = a_g @ b_g^T ([M, K] x [N, K]^T) for ``groups`` groups whose operands lie a_gs, b_gs, c_gs elements apart
         (rows lda, ldb, ldc elements apart), float32 accumulation with a fixed order of additions.  ``gated``: b_g holds
         2N rows, gate and up, "blocked" ([N gate | N up]) or "interleaved" (alternating in blocks of 64: stack_gate_up), and
         c_g = act(a gate^T) * (a up^T).  ``tiles`` = (tile_group, tile_row0, tile_row_end, num_tiles, max_tiles, tile rows)
         is the ragged form (rows of ``a`` sorted by group, the table on the device); ``row_map`` sends product row r to
-        row row_map[r] of ``c``.  bfloat16 operands of aligned sizes run on the tensor cores (csrc/gemm_grouped_mma.cu),
+        row row_map[r] of ``c``, ``a_rows`` (int32) says that sorted row r is row a_rows[r] of ``a``.  ``limit`` is
+        "clipped_swish"'s.  bfloat16 operands of aligned sizes run on the tensor cores (csrc/gemm_grouped_mma.cu),
         everything else as float32 FMAs (csrc/gemm_grouped.cu)."""
-        self._need_cuda(a, b, c, row_map)
+        self._need_cuda(a, b, c, row_map, a_rows)
         assert gated in ("", "blocked", "interleaved")
         tg = tr0 = tre = nt = None
         max_tiles, tile_rows = 0, 0
         if tiles is not None:
             tg, tr0, tre, nt, max_tiles, tile_rows = tiles
         code = self.ACTIVATION_CODES[activation]
-        if not gated and code < 2:
+        if not gated and code != 2:
             code = 0                      # a plain product: only a function of one product ("relu2") is applied to it
         act = _c_int(code)
+        clip = (_c_float(limit), _c_float(self.CLIPPED_SLOPE))
         ll = ctypes.c_longlong
         if self.grouped_on_tensor_cores(a, b, K, lda, a_gs, ldb, b_gs, gated, N) and tile_rows in (0, self.grouped_tile_rows(True)):
             status = self.lib.tff_gemm_grouped_mma(
                 _ptr(a), ll(lda), ll(a_gs), _ptr(b), ll(ldb), ll(b_gs), _ptr(c), _c_int(_dt(c)), ll(ldc), ll(c_gs),
-                _ptr(tg), _ptr(tr0), _ptr(tre), _ptr(nt), _c_int(max_tiles), _ptr(row_map), _c_int(groups), _c_int(M),
-                _c_int(2 * N if gated else N), _c_int(K), _c_int(1 if gated else 0), act, self._stream())
+                _ptr(tg), _ptr(tr0), _ptr(tre), _ptr(nt), _c_int(max_tiles), _ptr(row_map), _ptr(a_rows), _c_int(groups), _c_int(M),
+                _c_int(2 * N if gated else N), _c_int(K), _c_int(1 if gated else 0), act, *clip, self._stream())
             self._check(status, "gemm_grouped_mma")
             self.launches += 1
             return
@@ -803,7 +855,7 @@ class CudaKernels:
         self._check(self.lib.tff_gemm_grouped(
             _ptr(a), _c_int(_dt(a)), ll(lda), ll(a_gs), _ptr(b), b2, _c_int(_dt(b)), ll(ldb), ll(b_gs),
             _ptr(c), _c_int(_dt(c)), ll(ldc), ll(c_gs), _ptr(tg), _ptr(tr0), _ptr(tre), _ptr(nt), _c_int(max_tiles),
-            _ptr(row_map), _c_int(groups), _c_int(M), _c_int(N), _c_int(K), act,
+            _ptr(row_map), _ptr(a_rows), _c_int(groups), _c_int(M), _c_int(N), _c_int(K), act, *clip,
             _c_int(self.GATE_UP_BLOCK if gated == "interleaved" else 0), self._stream()), "gemm_grouped")
         self.launches += 1
 
@@ -975,14 +1027,16 @@ class CudaKernels:
 
     # ------------------------------------------------------- routed feed-forward (mixture of experts)
     def routed_mlp(self, h, w_router, w_gate_up, layout: str, w_down, residual, top: int, renormalize: bool = False,
-                   weight_on: str = "output", activation: str = "silu", out=None, router=None) -> None:
+                   weight_on: str = "output", activation: str = "silu", out=None, router=None, limit: float = 0.0) -> None:
         """residual += sum over a token's ``top`` experts of down_e(act(gate_e(x)) * up_e(x)), the experts chosen by
         the largest sigmoid(W_r h) (computed in float32), weights the scores themselves or renormalised to sum 1;
         ``weight_on`` "input": x = w h and the outputs are summed as they are; "output": x = h and the outputs are
         summed with the weights.  (w_gate_up, layout) = stack_gate_up(...) [E, 2*ff, W], w_down [E, W, ff].  With
         ``layout`` "plain" the experts are not gated: w_gate_up is [E, ff, W] and an expert is down_e(act(up_e(x))) with
         ``activation`` a function of one product ("relu2").  ``router`` (see moe_dispatch): softmax scores, a correction of
-        the choice, groups of experts, identity experts (router outputs beyond the E experts: weight times the input).
+        the choice, groups of experts, identity experts (router outputs beyond the E experts: weight times the input);
+        with score "table" there is no router (``w_router`` None): an integer table gives every token id its experts, each
+        with weight 1/top (moe_table).  ``limit``: the clipping of the activation "clipped_swish".
         With ``residual`` None the sum goes to ``out``.  Six launches, no host synchronisation: route, plan, gather, two
         grouped products over the tokens sorted by expert, combine (a token's experts are added in the order of their
         rank)."""
@@ -994,13 +1048,17 @@ class CudaKernels:
         E, ff = w_gate_up.shape[0], (w_gate_up.shape[1] if plain else w_gate_up.shape[1] // 2)
         up_rows = ff if plain else 2 * ff
         identity = int((router or {}).get("identity", 0))
-        assert tuple(w_router.shape) == (E + identity, W) and tuple(w_gate_up.shape) == (E, up_rows, W)
+        by_table = (router or {}).get("score") == "table"
+        assert by_table or tuple(w_router.shape) == (E + identity, W)
+        assert tuple(w_gate_up.shape) == (E, up_rows, W)
         assert tuple(w_down.shape) == (E, W, ff)
         assert weight_on in ("input", "output") and 0 < top <= E + identity
         if plain and activation not in ("relu2",):
             raise KernelError(f"experts that are not gated take the activation 'relu2', got '{activation}'")
-        if not plain and activation not in ("silu", "gelu_tanh"):
-            raise KernelError(f"gated experts take the activations 'silu' and 'gelu_tanh', got '{activation}'")
+        if not plain and activation not in ("silu", "gelu_tanh", "clipped_swish"):
+            raise KernelError(f"gated experts take the activations 'silu', 'gelu_tanh' and 'clipped_swish', got '{activation}'")
+        if activation == "clipped_swish" and not limit > 0:
+            raise KernelError("clipped_swish needs a positive limit")
         target = residual if residual is not None else out
         assert target.dtype == torch.float32 and tuple(target.shape) == (T, W)
         P = T * top
@@ -1011,20 +1069,32 @@ class CudaKernels:
             # Prompt-sized: the tcgen05 product in its grouped form.  Every expert's rows are padded to whole tiles of 128
             # in the sorted order, both products write in that order, and the sum gathers a token's rows from it.
             rows = -(-(P + E * 127) // 128) * 128
-            pair_weight, row_map, tiles, x, lane_group, place, *pe = self.moe_dispatch(
-                h, w_router, top, renormalize, weight_on == "input", 128, padded_rows=rows, router=router)
+            if by_table:
+                pe = []
+                pair_weight, row_map, tiles, _, lane_group, place = self.moe_table(router, T, top, E, 128, padded_rows=rows)
+                x = torch.empty((rows, W), dtype=h.dtype, device=h.device)
+                self.moe_spread(h, place, top, x)
+            else:
+                pair_weight, row_map, tiles, x, lane_group, place, *pe = self.moe_dispatch(
+                    h, w_router, top, renormalize, weight_on == "input", 128, padded_rows=rows, router=router)
             act = torch.empty((rows, ff), dtype=h.dtype, device=h.device)
-            self.gemm_tc_grouped(x, w_gate_up, act, E, up_rows, W, lane_group, gated=not plain, activation=activation)
+            self.gemm_tc_grouped(x, w_gate_up, act, E, up_rows, W, lane_group, gated=not plain, activation=activation,
+                                 limit=limit)
             y = torch.empty((rows, W), dtype=torch.float32, device=h.device)
             self.gemm_tc_grouped(act, w_down, y, E, W, ff, lane_group)
             self.moe_combine(y, pair_weight if weight_on == "output" else None, top, residual, target, place,
                              identity=(pe[0], pair_weight, h) if pe else None)
             return
-        pair_weight, row_map, tiles, x, *pe = self.moe_dispatch(h, w_router, top, renormalize, weight_on == "input",
-                                                                self.grouped_tile_rows(tc), router=router)
+        a_rows = None
+        if by_table:             # the product reads the tokens' rows where they are
+            pair_weight, row_map, tiles, a_rows = self.moe_table(router, T, top, E, self.grouped_tile_rows(tc))
+            x, pe = h, []
+        else:
+            pair_weight, row_map, tiles, x, *pe = self.moe_dispatch(h, w_router, top, renormalize, weight_on == "input",
+                                                                    self.grouped_tile_rows(tc), router=router)
         act = torch.empty((P, ff), dtype=h.dtype, device=h.device)
         self.gemm_grouped(x, w_gate_up, act, E, 0, ff, W, W, 0, W, up_rows * W, ff, 0, gated="" if plain else layout,
-                          activation=activation, tiles=tiles)
+                          activation=activation, tiles=tiles, a_rows=a_rows, limit=limit)
         y = torch.empty((P, W), dtype=torch.float32, device=h.device)
         self.gemm_grouped(act, w_down, y, E, 0, W, ff, ff, 0, ff, W * ff, W, 0, tiles=tiles, row_map=row_map)
         self.moe_combine(y, pair_weight if weight_on == "output" else None, top, residual, target,
@@ -1034,7 +1104,7 @@ class CudaKernels:
     GROUPED_TCGEN05_FROM = 1024      # (token, expert) pairs of a step from which the experts run on the tcgen05 product
 
     def gemm_tc_grouped(self, a, w, out, groups: int, group_rows: int, K: int, lane_group, gated: bool = False,
-                        activation: str = "silu") -> None:
+                        activation: str = "silu", limit: float = 0.0) -> None:
         """out = a @ w_g^T tile by tile of 128 rows of ``a``, tile t with group lane_group[t] (int32 on the device, -1: no
         such tile) of ``w`` [groups, group_rows, K]; gated: w_g holds gate and up rows alternating in blocks of 64 and
         out has group_rows / 2 columns.  The tcgen05 product of csrc/gemm_tc.cu in its grouped form."""
@@ -1045,11 +1115,12 @@ class CudaKernels:
         assert out.shape[1] == (group_rows // 2 if gated else group_rows)
         bn = 256 if (group_rows % 256 == 0 and rows >= 2048) else 128
         code = self.ACTIVATION_CODES[activation]
-        if not gated and code < 2:
+        if not gated and code != 2:
             code = 0                      # a plain product: only a function of one product ("relu2") is applied to it
         self._check(self.lib.tff_gemm_tc_grouped(_ptr(a), _ptr(w), _ptr(out), _c_int(_dt(out)), _c_int(rows), _c_int(groups),
                                                  _c_int(group_rows), _c_int(K), _c_int(bn), _c_int(1 if gated else 0),
-                                                 _c_int(code), _ptr(lane_group), self._stream()), "gemm_tc_grouped")
+                                                 _c_int(code), _c_float(limit), _c_float(self.CLIPPED_SLOPE),
+                                                 _ptr(lane_group), self._stream()), "gemm_tc_grouped")
         self.launches += 1
 
     def moe_dispatch(self, h, w_router, top: int, renormalize: bool, scale_rows: bool, tile_rows: int = 0,
@@ -1109,6 +1180,39 @@ class CudaKernels:
         if padded_rows:
             return (pair_weight, row_map, tiles, x, lane_group, place) + extra
         return (pair_weight, row_map, tiles, x) + extra
+
+    def moe_table(self, router, T: int, top: int, E: int, tile_rows: int, padded_rows: int = 0):
+        """The choice and sorting of a routed feed-forward whose experts a table gives: ``router`` = dict(table=int32
+        [rows, top], tokens=int32 [T]).  Returns (pair_weight (1/top), row_map, the tile table, a_rows int32: sorted place ->
+        token row) and, with ``padded_rows``, lane_group and place_of_pair, as moe_dispatch does.  One launch."""
+        table, tokens = router["table"], router["tokens"]
+        self._need_cuda(table, tokens)
+        assert table.dtype == tokens.dtype == torch.int32 and table.shape[1] == top and tokens.numel() == T
+        dev, P, bm = table.device, T * top, tile_rows
+        max_tiles = -(-P // bm) + E
+        R = max(P, padded_rows)
+        lane_tiles = padded_rows // bm if padded_rows else 0
+        sizes = [P, R, R, max_tiles, max_tiles, max_tiles, 1, lane_tiles, P if padded_rows else 0]
+        ints = torch.empty(sum(sizes), dtype=torch.int32, device=dev)
+        pair_expert, row_map, a_rows, tg, tr0, tre, nt, lane_group, place = ints.split(sizes)
+        pair_weight = torch.empty(P, dtype=torch.float32, device=dev)
+        if not padded_rows:
+            lane_group = place = None
+        self._check(self.lib.tff_moe_table(
+            _ptr(tokens), _ptr(table), _c_int(table.shape[0]), _c_int(P), _c_int(top), _c_int(E), _c_int(bm),
+            _c_int(bm if padded_rows else 0), _ptr(pair_expert), _ptr(pair_weight), _ptr(row_map), _ptr(a_rows), _ptr(place),
+            _ptr(tg), _ptr(tr0), _ptr(tre), _ptr(nt), _ptr(lane_group), _c_int(lane_tiles), self._stream()), "moe_table")
+        self.launches += 1
+        tiles = (tg, tr0, tre, nt, max_tiles, bm)
+        return (pair_weight, row_map, tiles, a_rows) + ((lane_group, place) if padded_rows else ())
+
+    def moe_spread(self, h, place_of_pair, top: int, x) -> None:
+        """x[place_of_pair[t*top + k]] = h[t]: the tokens' rows in the padded sorted order of the tcgen05 product."""
+        self._need_cuda(h, place_of_pair, x)
+        assert h.dtype == x.dtype and h.shape[1] == x.shape[1] and place_of_pair.numel() == h.shape[0] * top
+        self._check(self.lib.tff_moe_spread(_ptr(h), _c_int(_dt(h)), _c_int(place_of_pair.numel()), _c_int(h.shape[1]),
+                                            _c_int(top), _ptr(place_of_pair), _ptr(x), self._stream()), "moe_spread")
+        self.launches += 1
 
     def moe_combine(self, y, pair_weight, top: int, residual, out, place_of_pair=None, identity=None) -> None:
         """out[t] = residual[t] + sum_k w[t, k] * y[t*top + k] in the order of k (pair_weight None: plain sum); with
@@ -1201,9 +1305,9 @@ class CudaKernels:
     RECURRENCE_SEGMENT = 256      # portions longer than this run as segments side by side, joined by a scan (the kernel's constant)
 
     def gated_norm(self, o, group: int, gate, gate_off: int, weight, eps: float, gate_first: bool, out, out_off: int = 0,
-                   out_scale: float = 1.0, clear_cols=None, last_reader: bool = False) -> None:
+                   out_scale: float = 1.0, clear_cols=None, last_reader: bool = False, gate_act: str = "silu") -> None:
         """o float32 [T, width] in groups of ``group`` columns: RMS norm of every group times weight[c mod len(weight)]
-        and the silu of columns gate_off .. of the float32 rows ``gate``, the gate ahead of the norm (``gate_first``) or
+        and the silu (``gate_act`` "sigmoid": the sigmoid) of columns gate_off .. of the float32 rows ``gate``, the gate ahead of the norm (``gate_first``) or
         behind it -> columns out_off .. of ``out`` times out_scale.  ``clear_cols`` = (lo, hi): when ``gate`` is one of
         the accumulator buffers kept at zero between uses, those columns of it are set back to zero; ``last_reader``
         says that nothing else of its rows is left unread, so that the buffer counts as clean again."""
@@ -1215,12 +1319,13 @@ class CudaKernels:
         lo, hi = clear_cols if clear_cols is not None else (0, 0)
         self._check(self.lib.tff_gated_norm(
             _ptr(o), _c_int(width), _c_int(group), _ptr(gate), _c_int(gate.shape[1]), _c_int(gate_off), _ptr(weight),
-            _c_int(weight.numel()), _c_float(eps), _c_int(1 if gate_first else 0), _ptr(out), _c_int(_dt(out)),
+            _c_int(weight.numel()), _c_float(eps), _c_int(1 if gate_first else 0),
+            _c_int({"silu": 0, "sigmoid": 1}[gate_act]), _ptr(out), _c_int(_dt(out)),
             _c_int(out.shape[1]), _c_int(out_off), _c_float(out_scale), _c_int(clear), _c_int(lo), _c_int(hi), _c_int(T),
             self._stream()), "gated_norm")
         if clear and last_reader:
             self._acc_zero[gate.data_ptr()] = True
-        self.launches += 2 if clear and hi > lo else 1
+        self.launches += 1
 
     def causal_conv(self, proj, col0: int, channels: int, weight, bias, activation: str, state, state_off: int, batch,
                     out, update_state: bool = False) -> bool:
@@ -1262,7 +1367,8 @@ class CudaKernels:
 
     def latent_attend(self, h, w_down, q_norm_w, kv_norm_w, eps: float, w_uq, w_uk_t, w_uv, freq, batch, block_table,
                       kv_cache, kv_layer, page_size, out, heads: int, dim: int, rot_dim: int, vdim: int, q_rank: int,
-                      kv_rank: int, scale: float, write_cache: bool, w_uk=None, shared=None) -> None:
+                      kv_rank: int, scale: float, write_cache: bool, w_uk=None, shared=None, window: int = 0,
+                      sink=None) -> None:
         """The whole of a latent attention between its input rows and its output projection -> out [T, heads*vdim].
         ``w_down`` rows [query latent (q_rank) | kv latent (kv_rank) | shared rotated key part (rot_dim)], the last two
         absent when the layer reads another layer's cache (``write_cache`` False).  The cache has one plane with a slot
@@ -1270,6 +1376,9 @@ class CudaKernels:
         part goes through W_uk^T instead (``w_uk_t`` [heads, kv_rank, dim]), attention then runs with one shared
         key/value head over the slots (keys the whole slot, values its first kv_rank elements), and W_uv [heads*vdim,
         kv_rank] takes every head's mixed latent to its value size.
+
+        With ``q_rank`` 0 there is no query latent: the first heads * (dim + rot_dim) rows of ``w_down`` make the query heads
+        themselves.  ``window`` and ``sink`` (float32 [heads] or None) as for attention_tile.
 
         A step of whole prompts (every request starts at position 0, bfloat16, aligned sizes) takes the other form: the
         step's latents are also kept in plain rows (``shared``, a dict that lives for the step, hands them to the layers
@@ -1287,25 +1396,37 @@ class CudaKernels:
                  and slot % 8 == 0 and kv_rank % 8 == 0)
         key = ("latent rows", kv_cache.data_ptr(), kv_layer)
         assert kv_cache is not None and kv_cache.shape[2] == 1 and kv_cache.shape[3] == 1 and kv_cache.shape[-1] == slot
-        assert w_down.shape[0] >= (q_rank + slot if write_cache else q_rank)      # rows beyond are padding
+        q_cols = q_rank if q_rank else heads * (dim + rot_dim)
+        assert w_down.shape[0] >= (q_cols + slot if write_cache else q_cols)      # rows beyond are padding
         f, rot_dims, mag, inter = freq if freq is not None else (None, 0, 1.0, True)
-        if rot_dims and (not inter or mag != 1.0):
-            raise KernelError("latent attention turns interleaved pairs by plain angles")
+        turn = (rot_dims, not inter, mag)
         proj = self.projection_buffer(T, w_down.shape[0], dev, dt)
         self.gemm(h, w_down, proj)
-        cq = torch.empty((T, q_rank), dtype=dt, device=dev)
+        cq = torch.empty((T, q_rank), dtype=dt, device=dev) if q_rank else None
         rows = None
         if whole and write_cache:
             rows = shared[key] = torch.empty((T, slot), dtype=dt, device=dev)
         elif whole:
             rows = shared.get(key)
-        self.latent_finish(proj, cq, q_norm_w, kv_norm_w, eps, f, rot_dim, rot_dims, batch, block_table, kv_cache, kv_layer,
-                           page_size, q_rank, kv_rank if write_cache else 0, dense_out=rows if write_cache else None)
-        q = torch.empty((T, heads * (dim + rot_dim)), dtype=dt, device=dev)
-        self.gemm(cq, w_uq, q)
-        if (rows is not None and w_uk is not None and (dim + rot_dim) % 8 == 0 and vdim % 8 == 0
-                and tuple(rows.shape) == (T, slot)):
-            self.latent_q_rot(q, q, f, batch, heads, dim, rot_dim, rot_dims, dim)          # in place: the head's own row
+        per_head = (rows is not None and w_uk is not None and (dim + rot_dim) % 8 == 0 and vdim % 8 == 0
+                    and tuple(rows.shape) == (T, slot))
+        q_lat = None if per_head else torch.empty((T, heads * slot), dtype=dt, device=dev)
+        if q_rank:
+            q_ld = dim + rot_dim                                 # elements between the heads of ``q``
+            q = torch.empty((T, heads * q_ld), dtype=dt, device=dev)
+            q_heads = None
+        else:
+            q_ld = dim + rot_dim if per_head else dim
+            q = torch.empty((T, heads * q_ld), dtype=dt, device=dev)
+            q_heads = (heads, dim, q, 0, q, dim) if per_head else (heads, dim, q, 0, q_lat, kv_rank)
+        self.latent_finish(proj, cq, q_norm_w, kv_norm_w, eps, f, rot_dim, turn, batch, block_table, kv_cache, kv_layer,
+                           page_size, q_rank, kv_rank if write_cache else 0, dense_out=rows if write_cache else None,
+                           q_heads=q_heads)
+        if q_rank:
+            self.gemm(cq, w_uq, q)
+        if per_head:
+            if q_rank:
+                self.latent_q_rot(q, q, f, batch, heads, dim, rot_dim, turn, dim)          # in place: the head's own row
             keys = torch.empty((T, heads * (dim + rot_dim)), dtype=dt, device=dev)
             self.gemm_grouped(rows, w_uk, keys, heads, T, dim, kv_rank, slot, 0, kv_rank, dim * kv_rank,
                               heads * (dim + rot_dim), dim + rot_dim)
@@ -1317,41 +1438,59 @@ class CudaKernels:
             self.gemm_grouped(rows, w_uv, values, heads, T, vdim, kv_rank, slot, 0, kv_rank, vdim * kv_rank,
                               heads * vdim, vdim)
             self.attention_tile(q, batch, block_table, kv_cache, kv_layer, page_size, out, heads, heads, dim + rot_dim,
-                                vdim, scale, dense=(keys, values))
+                                vdim, scale, window=window, sink=sink, dense=(keys, values))
             return
-        q_lat = torch.empty((T, heads * slot), dtype=dt, device=dev)
-        self.gemm_grouped(q, w_uk_t, q_lat, heads, T, kv_rank, dim, heads * (dim + rot_dim), dim + rot_dim,
+        self.gemm_grouped(q, w_uk_t, q_lat, heads, T, kv_rank, dim, heads * q_ld, q_ld,
                           dim, kv_rank * dim, heads * slot, slot)
-        self.latent_q_rot(q, q_lat, f, batch, heads, dim, rot_dim, rot_dims, kv_rank)
+        if q_rank:
+            self.latent_q_rot(q, q_lat, f, batch, heads, dim, rot_dim, turn, kv_rank)
         o_lat = torch.empty((T, heads * kv_rank), dtype=dt, device=dev)
-        self.attention_tile(q_lat, batch, block_table, kv_cache, kv_layer, page_size, o_lat, heads, 1, slot, kv_rank, scale)
+        self.attention_tile(q_lat, batch, block_table, kv_cache, kv_layer, page_size, o_lat, heads, 1, slot, kv_rank, scale,
+                            window=window, sink=sink)
         self.gemm_grouped(o_lat, w_uv, out, heads, T, vdim, kv_rank, heads * kv_rank, kv_rank, kv_rank, vdim * kv_rank,
                           heads * vdim, vdim)
 
-    def latent_finish(self, proj, cq, q_norm_w, kv_norm_w, eps, freq, rot_dim, rot_dims, batch, block_table, kv_cache,
-                      kv_layer, page_size, q_rank, kv_rank, dense_out=None) -> None:
+    def latent_finish(self, proj, cq, q_norm_w, kv_norm_w, eps, freq, rot_dim, turn, batch, block_table, kv_cache,
+                      kv_layer, page_size, q_rank, kv_rank, dense_out=None, q_heads=None) -> None:
         """csrc/latent.cu: the float32 rows [q latent | kv latent | rotated key part] -> normed query latents ``cq`` and,
         with kv_rank > 0, the token's cache slot [normed kv latent | rotated key part] (and the same vector into row t of
-        ``dense_out`` [T, slot], when given)."""
+        ``dense_out`` [T, slot], when given).  ``turn`` = (rotated dimensions, pairs as halves?, magnitude).  ``q_heads`` =
+        (heads, dim, u, u_col, r, r_col) with q_rank 0: the rows start with the query heads themselves, whose unrotated
+        parts go to columns u_col .. of every head's row of ``u`` [T, heads * row] and turned parts to columns r_col .. of
+        ``r``'s."""
         self._need_cuda(proj, cq, q_norm_w, kv_norm_w, freq, block_table)
         T = proj.shape[0]
+        rot_dims, halves, mag = turn
+        act = cq if q_heads is None else q_heads[2]
+        qh = (_c_int(0), _c_int(0), _vp(0), _c_int(0), _c_int(0), _vp(0), _c_int(0), _c_int(0))
+        if q_heads is not None:
+            heads, dim, u, u_col, r, r_col = q_heads
+            self._need_cuda(u, r)
+            assert u.dtype == r.dtype and u.shape[0] == r.shape[0] == T and u.shape[1] % heads == 0 and r.shape[1] % heads == 0
+            u_hs, r_hs = u.shape[1] // heads, r.shape[1] // heads
+            assert q_rank == 0 and u_col + dim <= u_hs and r_col + rot_dim <= r_hs
+            qh = (_c_int(heads), _c_int(dim), _vp(u.data_ptr() + u_col * u.element_size()), _c_int(u.shape[1]), _c_int(u_hs),
+                  _vp(r.data_ptr() + r_col * r.element_size()), _c_int(r.shape[1]), _c_int(r_hs))
         c_ptr, page_stride = self._layer_cache(kv_cache, kv_layer)
         clear = 1 if proj.data_ptr() in self._acc_zero else 0
         self._check(self.lib.tff_latent_finish(
             _ptr(proj), _c_int(proj.shape[1]), _c_int(clear), _c_int(q_rank), _c_int(kv_rank), _c_int(rot_dim),
-            _c_int(rot_dims), _ptr(q_norm_w), _ptr(kv_norm_w), _c_float(eps), _ptr(freq), _ptr(batch.positions),
+            _c_int(rot_dims), _c_int(1 if halves else 0), _c_float(mag), *qh, _ptr(q_norm_w), _ptr(kv_norm_w), _c_float(eps),
+            _ptr(freq), _ptr(batch.positions),
             _ptr(batch.tok_req), _ptr(block_table), _c_int(block_table.shape[1]), c_ptr if kv_rank > 0 else _vp(0),
-            ctypes.c_longlong(page_stride), _c_int(page_size), _c_int(kv_cache.shape[-1]), _ptr(cq), _c_int(_dt(cq)),
+            ctypes.c_longlong(page_stride), _c_int(page_size), _c_int(kv_cache.shape[-1]), _ptr(cq), _c_int(_dt(act)),
             _ptr(dense_out), _c_int(T), self._stream()), "latent_finish")
         if clear:
             self._acc_zero[proj.data_ptr()] = True
         self.launches += 1
 
-    def latent_q_rot(self, q, q_lat, freq, batch, heads, dim, rot_dim, rot_dims, kv_rank) -> None:
+    def latent_q_rot(self, q, q_lat, freq, batch, heads, dim, rot_dim, turn, kv_rank) -> None:
         """The rotated part of every query head of the rows ``q`` into its place in ``q_lat`` (same type; a head's row
         of ``q_lat`` has kv_rank + rot_dim elements, so with kv_rank = dim and q_lat = q the rotation is in place)."""
         assert q.dtype == q_lat.dtype
-        self._check(self.lib.tff_latent_q_rot(_ptr(q), _c_int(dim), _c_int(rot_dim), _c_int(rot_dims), _ptr(freq),
+        rot_dims, halves, mag = turn
+        self._check(self.lib.tff_latent_q_rot(_ptr(q), _c_int(dim), _c_int(rot_dim), _c_int(rot_dims),
+                                              _c_int(1 if halves else 0), _c_float(mag), _ptr(freq),
                                               _ptr(batch.positions), _ptr(q_lat), _c_int(_dt(q_lat)), _c_int(kv_rank),
                                               _c_int(heads), _c_int(q.shape[0]), self._stream()), "latent_q_rot")
         self.launches += 1

@@ -4,3 +4,4 @@ from . import tipezen  # noqa: F401  (registration)
 from . import dominex  # noqa: F401  (registration)
 from . import sadupel  # noqa: F401  (registration)
 from . import nugosun  # noqa: F401  (registration)
+from . import kadodra  # noqa: F401  (registration)

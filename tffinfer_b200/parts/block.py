@@ -37,6 +37,24 @@ class PreNormBlock(Block):
         return x
 
 
+@register_part("block", "parallel_shared_norm")
+class ParallelSharedNormBlock(Block):
+    """The mixer and the feed-forward side by side on ONE norm's output: ``h = norm(x)``, ``x <- x + (mixer(h) + ffn(h))``,
+    both adding into the stream; a layer without a feed-forward is the mixer alone."""
+
+    def __init__(self, mixer, feed_forward, mixer_norm=None, ffn_norm=None, extra_norms=None):
+        super().__init__(mixer, feed_forward, mixer_norm, ffn_norm, extra_norms)
+        if mixer_norm is None or ffn_norm is not None:
+            raise ValueError("the parallel_shared_norm arrangement has one norm, mixer_norm: both sublayers read its output")
+
+    def forward(self, x, ctx: LayerContext, act_dtype):
+        h = self.mixer_norm.forward(x, ctx.ops, act_dtype)
+        x = self.mixer.forward(h, ctx, residual=x)
+        if self.feed_forward is not None:
+            x = self.feed_forward.forward(h, ctx, residual=x)
+        return x
+
+
 @register_part("block", "parallel_pre_norm")
 class ParallelPreNormBlock(Block):
     """The mixer and the feed-forward side by side, each behind a norm of its own, both norms reading the same

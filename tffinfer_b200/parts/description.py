@@ -47,10 +47,12 @@ class ScheduleEntry:
     ``cache_of`` names an EARLIER schedule entry whose cache this run reads instead of
     keeping one (it then writes nothing).  ``add_vector`` = (tensor name, row): that row of a
     [rows, hidden] tensor of the model (``ModelDescription.vector_tables``) is added to the
-    residual right before this run."""
+    residual right before this run.  ``add_embedding``: the embedding output (the residual as it was ahead of
+    the first run) is added to the residual right before this run."""
     layer: int
     cache_of: Optional[int] = None
     add_vector: Optional[tuple] = None
+    add_embedding: bool = False
 
 
 @dataclass

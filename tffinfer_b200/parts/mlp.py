@@ -60,3 +60,34 @@ class SwiGLU(FeedForward):
             ctx.ops.gated_mlp(h, self.w_gate_up, self.w_down, residual, self.intermediate_size,
                               activation=self.activation)
         return residual
+
+
+@register_part("feed_forward", "plain_mlp")
+class PlainMLP(FeedForward):
+    """Dense feed-forward without a gate and without biases: ``down(act(up h))``, ``activation`` "relu2" (the square of
+    relu)."""
+    ACTIVATIONS = ("relu2",)
+
+    def __init__(self, hidden_size: int, intermediate_size: int, activation: str = "relu2", names=None, prefix: str = ""):
+        super().__init__(prefix)
+        self.hidden_size, self.intermediate_size = int(hidden_size), int(intermediate_size)
+        if activation not in self.ACTIVATIONS:
+            raise ValueError(f"activation must be one of {self.ACTIVATIONS}, got '{activation}'")
+        self.activation = activation
+        self.names = {"up": "up", "down": "down"}
+        self.names.update(names or {})
+        self.w_up = self.w_down = None
+
+    def weight_specs(self) -> Dict[str, WeightSpec]:
+        return {self.names["up"]: WeightSpec((self.intermediate_size, self.hidden_size), MATRIX),
+                self.names["down"]: WeightSpec((self.hidden_size, self.intermediate_size), MATRIX)}
+
+    def load(self, tensors, ops, act_dtype) -> None:
+        self.w_up, self.w_down = tensors[self.names["up"]], tensors[self.names["down"]]
+
+    def forward(self, h, ctx, residual):
+        out = None
+        if residual is None:
+            out = ctx.ops.sublayer_output(h.shape[0], self.hidden_size, h.device, h.dtype)
+        ctx.ops.plain_mlp(h, self.w_up, self.w_down, residual, self.activation, out=out)
+        return residual if residual is not None else out

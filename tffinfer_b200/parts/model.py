@@ -121,6 +121,9 @@ class Model:
             p.forward(x.x if d.streams > 0 else x, batch, ops, states[si] if si is not None else None, copies=d.streams)
         for pos in self.positions.values():
             x = pos.embed(x, batch, ops)
+        x0 = None                  # the embedding output, kept where a later run wants it again
+        if any(entry.add_embedding for entry in d.schedule):
+            x0 = (x.x[:, 0] if d.streams > 0 else x).clone()
         shared: Dict[str, torch.Tensor] = {}
         for e, entry in enumerate(d.schedule):
             b = bindings[e]
@@ -138,6 +141,11 @@ class Model:
                     x.add_vector(vec)              # runs with the layer's read of the residual
                 else:
                     ops.stream_step(x.view(T, 1, d.hidden_size), bias=vec)
+            if entry.add_embedding:
+                if d.streams > 0:
+                    x.write(x0, None, None, None)  # runs with the layer's read of the residual
+                else:
+                    ops.stream_step(x.view(T, 1, d.hidden_size), y=x0)
             x = self.blocks[entry.layer].forward(x, ctx, act_dtype)
             if self.layer_hook is not None:
                 self.layer_hook(e, x.total() if d.streams > 0 else x)

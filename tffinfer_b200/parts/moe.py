@@ -9,8 +9,12 @@ token uses ``top``.
         largest c, and only members of the ``keep`` best groups can be chosen
     chosen = the ``top`` outputs of largest c (the lower index wins a tie)
     w_e = s_e, or s_e / sum over the chosen when ``renormalize``
+    ``router_score`` "table": no router; an integer table (tensor "table" [table_rows, top], the entries of a row differ)
+        gives every token id its experts, each with weight 1/top
     weight_on "input":   out = sum_e f_e(w_e h)          weight_on "output":  out = sum_e w_e f_e(h)
     f_e(x) = down_e( act(gate_e(x)) * up_e(x) )          ``gated`` (activation "silu" or "gelu_tanh")
+    f_e(x) = down_e( g sigmoid(1.702 g) (u + 1) ), g = min(gate_e(x), limit), u = clamp(up_e(x), -limit, limit)
+                                                         ``gated``, activation "clipped_swish" with ``activation_limit``
     f_e(x) = down_e( act(up_e(x)) )                      not gated (activation "relu2", the square of relu)
 
 The last ``identity_experts`` router outputs have no tensors: f_e(x) = x.  ``shared_intermediate`` > 0 adds one more
@@ -27,18 +31,18 @@ from typing import Dict
 import torch
 
 from ..registry import register_part
-from .base import FeedForward, WeightSpec, MATRIX, VECTOR
+from .base import FeedForward, WeightSpec, MATRIX, VECTOR, INT_TABLE
 
 
 @register_part("feed_forward", "routed_experts")
 class RoutedExperts(FeedForward):
-    ACTIVATIONS = ("silu", "gelu_tanh")
+    ACTIVATIONS = ("silu", "gelu_tanh", "clipped_swish")
     PLAIN_ACTIVATIONS = ("relu2",)
 
     def __init__(self, hidden_size: int, intermediate_size: int, num_experts: int, top: int, activation: str = "silu",
                  renormalize: bool = False, weight_on: str = "output", gated: bool = True, router_score: str = "sigmoid",
                  correction: bool = False, groups=None, identity_experts: int = 0, shared_intermediate: int = 0,
-                 router_bias: bool = False, names=None, prefix: str = ""):
+                 router_bias: bool = False, activation_limit: float = 0.0, table_rows: int = 0, names=None, prefix: str = ""):
         super().__init__(prefix)
         self.hidden_size, self.intermediate_size = int(hidden_size), int(intermediate_size)
         self.num_experts, self.top = int(num_experts), int(top)
@@ -54,8 +58,16 @@ class RoutedExperts(FeedForward):
             raise ValueError(f"activation of {'gated' if self.gated else 'plain'} experts must be one of {allowed}, got '{activation}'")
         if weight_on not in ("input", "output"):
             raise ValueError(f"weight_on must be 'input' or 'output', got '{weight_on}'")
-        if router_score not in ("sigmoid", "softmax", "softmax_chosen"):
-            raise ValueError(f"router_score must be 'sigmoid', 'softmax' or 'softmax_chosen', got '{router_score}'")
+        if router_score not in ("sigmoid", "softmax", "softmax_chosen", "table"):
+            raise ValueError(f"router_score must be 'sigmoid', 'softmax', 'softmax_chosen' or 'table', got '{router_score}'")
+        self.table_rows = int(table_rows)
+        if router_score == "table" and (self.table_rows <= 0 or correction or groups is not None or identity_experts
+                                        or router_bias or renormalize or weight_on != "output"):
+            raise ValueError("experts chosen by a table need table_rows; they have no router scores to correct, group, "
+                             "bias or renormalise, no identity experts, and their weight is on the output")
+        self.activation_limit = float(activation_limit)
+        if activation == "clipped_swish" and (not self.activation_limit > 0 or shared_intermediate):
+            raise ValueError("clipped_swish needs activation_limit > 0 (and is not built for a shared expert)")
         self.router_bias = bool(router_bias)
         self.activation, self.renormalize, self.weight_on = activation, bool(renormalize), weight_on
         self.router_score, self.correction = router_score, bool(correction)
@@ -66,10 +78,10 @@ class RoutedExperts(FeedForward):
         self.groups = (count, keep)
         self.shared_intermediate = int(shared_intermediate)
         self.names = {"router": "router", "router_bias": "router.b", "expert": "e{}", "gate": "gate", "up": "up", "down": "down",
-                      "correction": "correction", "shared": "shared"}
+                      "correction": "correction", "shared": "shared", "table": "table"}
         self.names.update(names or {})
         self.w_router = self.w_gate_up = self.w_down = self.correction_w = self.router_bias_w = None
-        self.shared_up = self.shared_down = None
+        self.shared_up = self.shared_down = self.table = None
         self.gate_up_layout = "blocked"
 
     def _expert(self, e: int, which: str) -> str:
@@ -79,7 +91,10 @@ class RoutedExperts(FeedForward):
         return f"{self.names['shared']}.{self.names[which]}"
 
     def weight_specs(self) -> Dict[str, WeightSpec]:
-        s = {self.names["router"]: WeightSpec((self.outputs, self.hidden_size), MATRIX)}
+        if self.router_score == "table":
+            s = {self.names["table"]: WeightSpec((self.table_rows, self.top), INT_TABLE, below=self.num_experts)}
+        else:
+            s = {self.names["router"]: WeightSpec((self.outputs, self.hidden_size), MATRIX)}
         if self.correction:
             s[self.names["correction"]] = WeightSpec((self.outputs,), VECTOR, init="normal", init_scale=0.05)
         if self.router_bias:
@@ -101,7 +116,12 @@ class RoutedExperts(FeedForward):
             ts = [[tensors[self._expert(e, w)] for e in range(self.num_experts)] for w in which]
             same = all(t.dtype == ts[0][0].dtype for l in ts for t in l)
             return [[t if same else t.to(torch.float32) for t in l] for l in ts]
-        self.w_router = tensors[self.names["router"]]
+        if self.router_score == "table":
+            self.table = tensors[self.names["table"]].contiguous()
+            if int(self.table.min()) < 0 or int(self.table.max()) >= self.num_experts:
+                raise ValueError(f"'{self.full_name(self.names['table'])}' names experts outside 0 .. {self.num_experts - 1}")
+        else:
+            self.w_router = tensors[self.names["router"]]
         if self.correction:
             self.correction_w = tensors[self.names["correction"]].to(torch.float32).contiguous()
         if self.router_bias:
@@ -122,7 +142,9 @@ class RoutedExperts(FeedForward):
                 self.shared_up = tensors[self._shared("up")]
             self.shared_down = tensors[self._shared("down")]
 
-    def _router(self):
+    def _router(self, ctx):
+        if self.router_score == "table":
+            return dict(score="table", table=self.table, tokens=ctx.batch.token_ids)
         if (self.router_score, self.correction_w, self.groups, self.identity_experts, self.router_bias_w) == \
                 ("sigmoid", None, (1, 1), 0, None):
             return None
@@ -136,7 +158,7 @@ class RoutedExperts(FeedForward):
             target = torch.empty((h.shape[0], self.hidden_size), dtype=torch.float32, device=h.device)
         ops.routed_mlp(h, self.w_router, self.w_gate_up, self.gate_up_layout, self.w_down, residual, self.top,
                        self.renormalize, self.weight_on, self.activation, out=None if residual is not None else target,
-                       router=self._router())
+                       router=self._router(ctx), limit=self.activation_limit)
         if self.shared_intermediate > 0:              # one more expert that every token uses, added to the sum
             if self.gated:
                 ops.gated_mlp(h, self.shared_up, self.shared_down, target, self.shared_intermediate,

@@ -28,6 +28,14 @@ def _stream(seed: int, name: str) -> torch.Generator:
     return g
 
 
+def random_choices(spec: WeightSpec, gen: torch.Generator, device="cpu") -> torch.Tensor:
+    """An integer table: every row holds different values below ``spec.below`` in a random order (zeros when it is 0)."""
+    if spec.below <= 0:
+        return torch.zeros(spec.shape, dtype=torch.int32, device=device)
+    order = torch.rand((spec.shape[0], spec.below), generator=gen, device=device).argsort(dim=1)
+    return order[:, :spec.shape[1]].to(torch.int32).contiguous()
+
+
 def random_tensor(seed: int, name: str, spec: WeightSpec, init_std: float, norm_noise: float,
                   store_dtype: torch.dtype) -> torch.Tensor:
     g = _stream(seed, name)
@@ -35,7 +43,7 @@ def random_tensor(seed: int, name: str, spec: WeightSpec, init_std: float, norm_
         raise ValueError(f"tensor '{name}' has a size that only a file gives ({list(spec.shape)}): the configuration must "
                          f"state it where weights are made at random")
     if spec.role == INT_TABLE:
-        return torch.zeros(spec.shape, dtype=torch.int32)
+        return random_choices(spec, g)
     if spec.init == "zeros":
         t = torch.zeros(spec.shape, dtype=torch.float32)
     elif spec.init == "one_plus_normal":
@@ -86,7 +94,7 @@ def random_tensors_on_device(cfg: ModelConfig, seed: int, device, store_dtype: s
         if spec.optional:
             continue
         if spec.role == INT_TABLE:
-            out[name] = torch.zeros(spec.shape, dtype=torch.int32, device=device)
+            out[name] = random_choices(spec, gen, device)
         elif spec.init == "one_plus_normal":
             s = norm_noise if spec.init_scale is None else spec.init_scale
             t = torch.ones(spec.shape, dtype=torch.float32, device=device)
