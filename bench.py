@@ -861,19 +861,133 @@ def run_nugosun(steps: int, warmup: int, sizes=None) -> int:
     return 0
 
 
+# The Kadodra design beside Nugosun (the closest of the other models: latent attention and linear attention over matrix
+# states, two sublayers side by side, dense and routed feed-forwards) at the same width: (width, latent heads, dim, rot_dim,
+# vdim, kv_rank, window, lightning heads, key size, value size, experts, chosen, expert ff, dense ff).  Six layers, lightning
+# and latent in turn, of which layers 2 and 3 run twice (eight layer runs, as many as the twin has layers); the dense
+# feed-forward has no gate, so its ff is 1.5 times the twin's for the same arithmetic.
+KADODRA_SIZES = {"2k": (2048, 16, 128, 64, 128, 512, 1024, 16, 128, 128, 16, 2, 3072, 9216),
+                 "4k": (4096, 32, 128, 64, 128, 512, 1024, 32, 128, 128, 16, 2, 6144, 18432)}
+KADODRA_LOOP = (2, 4, 2)
+
+
+def kadodra_engine(size: str, max_live: int, cache_tokens: int, graphs: bool, step_tokens: int):
+    import torch
+    import tffinfer_b200 as tff
+    from tffinfer_b200.config.kadodra_config import KadodraConfig, KadodraLayer, KadodraMlp, KadodraLatent, KadodraLightning
+    from tffinfer_b200.config.tipezen_config import RotaryConfig
+    from tffinfer_b200.weights import random_tensors_on_device
+    W, H, D, R, VD, KR, WIN, LH, LD, LV, E, TOP, F, DF = KADODRA_SIZES[size]
+    light = KadodraLayer("lightning", mlp=KadodraMlp("dense", DF), lightning=KadodraLightning(
+        LH, LD, LV, tuple(1.0 - 2.0 ** -(3 + 6.0 * i / LH) for i in range(LH))))
+    latent = KadodraLayer("latent_attention", mlp=KadodraMlp("moe", F, E, TOP, 7.0), latent=KadodraLatent(
+        H, D, R, VD, KR, (D + R) ** -0.5, RotaryConfig(5e5, R, (4.0, 4096.0, 16.0, 2.0)), WIN))
+    cfg = KadodraConfig("Kadodra", vocab_size=TIPEZEN_VOCAB, hidden_size=W, norm_eps=1e-6, logit_scale=0.25, loop=KADODRA_LOOP,
+                        layers=(light, latent) * 3)
+    tensors = random_tensors_on_device(cfg, 0, "cuda", "bfloat16")
+    ecfg = tff.EngineConfig(dtype="bfloat16", page_size=PAGE_SIZE, max_cache_tokens=cache_tokens, max_live_requests=max_live,
+                            max_tokens_per_step=step_tokens, max_model_len=8192, use_cuda_graphs=graphs)
+    runner = tff.ModelRunner(config=cfg, tensors=tensors, engine_config=ecfg)
+    del tensors
+    torch.cuda.empty_cache()
+    return tff.Engine(runner=runner), cfg
+
+
+def run_kadodra(steps: int, warmup: int, sizes=None) -> int:
+    """Prefill and decode throughput of the Kadodra design beside Nugosun at the same layer sizes, one JSON line a point,
+    and for each model the device time of a step by kind of kernel call; for Kadodra also what its own kernels reach: the
+    recurrence in TFLOP/s of its chunk form (prompt step) and as a fraction of the measured copy rate for the states it
+    reads and writes (decode step), the norm over all heads, the kernel between the latent projections and the attention,
+    the sorting by the table and the sum of experts as fractions of the copy rate, the windowed attention and the experts'
+    products in TFLOP/s."""
+    import torch
+    peaks = load_peaks()
+    steps = min(steps, 32)
+    P = PROMPT_LEN
+    clocks = ClockSampler()
+    clocks.start()
+    for size in (sizes or KADODRA_SIZES):
+        W, H, D, R, VD, KR, WIN, LH, LD, LV, E, TOP, F, DF = KADODRA_SIZES[size]
+        for model, make in (("kadodra", kadodra_engine), ("nugosun", nugosun_engine)):
+            need = 64 * (P + warmup + steps + 64 + 72)
+            engine, cfg = make(size, 64, need, True, P)
+            pms = prefill_run(engine, iters=3, warmup=2, seed=1, prompt_len=P)
+            print(json.dumps({"point": "prefill", "model": model, "size": size, "layers": TIPEZEN_LAYERS, "tokens": P,
+                              "ms": round(pms, 3), "tok_s": round(P / (pms / 1e3), 1)}), flush=True)
+            for b in (8, 64):
+                run = decode_run(engine, b, steps, warmup, seed=b, prompt_len=P)
+                print(json.dumps({"point": "decode", "model": model, "size": size, "layers": TIPEZEN_LAYERS, "batch": b,
+                                  "context": round(run["mean_context"]), "tok_s": round(run["tok_s"], 1),
+                                  "ms_per_step": round(run["ms_per_step"], 4), "launches_per_step": run["launches"] // steps}),
+                      flush=True)
+            del engine
+            torch.cuda.empty_cache()
+            engine, cfg = make(size, 8, 8 * (P + 64), False, P)
+            kinds = traced_kinds(engine, P, 8)
+            line = {"point": "kernels", "model": model, "size": size, "prefill_tokens": P, "decode_batch": 8,
+                    "prefill_ms_by_kind": kinds.get("prefill"), "decode_ms_by_kind": kinds.get("decode"), "peaks": peaks["source"]}
+            if model == "kadodra":
+                nl = TIPEZEN_LAYERS // 2                        # runs of either kind of layer
+                gnorm_b = lambda T: nl * T * LH * LV * (4 + 4 + 2)
+                finish_b = lambda T: nl * T * ((H * (D + R) + KR + R) * 4 + H * (D + R) * 2 + (KR + R) * 2 * (2 if T == P else 1))
+                combine_b = lambda T: nl * T * W * (TOP * 4 + 4 + 4)
+                spread_b = lambda T: nl * T * TOP * W * (2 + 2)
+                norm_b = lambda T: (2 * nl * T + 1) * W * (4 + 2)
+                fr = {}
+                for step, T in (("prefill", P), ("decode", 8)):
+                    k = kinds.get(step) or {}
+                    for kind, nbytes in (("gated_norm", gnorm_b(T)), ("latent_finish", finish_b(T)), ("moe_combine", combine_b(T)),
+                                         ("moe_spread", spread_b(T)), ("rmsnorm", norm_b(T))):
+                        if kind in k:
+                            fr[f"{step}_{kind}_hbm_frac"] = round(nbytes / (k[kind][1] / 1e3) / 1e9 / peaks["hbm_gbs"], 4)
+                k = kinds.get("prefill") or {}
+                if "retention_raw" in k:          # chunks of 64 tokens: A = Q K^T and A V, U = K^T V and Q S
+                    flops = nl * LH * (P / 64.0) * 2.0 * 64 * (64 * LD + 64 * LV + 2 * LD * LV)
+                    fr["prefill_retention_raw_fp32_tflops"] = round(flops / (k["retention_raw"][1] / 1e3) / 1e12, 2)
+                if "attention_tile" in k:
+                    span = min(WIN, P)
+                    pairs = span * (span + 1) / 2.0 + (P - span) * span
+                    fr["prefill_attention_tile_tflops"] = round(nl * H * pairs * 2.0 * (D + R + VD) / (k["attention_tile"][1] / 1e3) / 1e12, 2)
+                if "gemm_tc_grouped" in k:
+                    fr["prefill_experts_tcgen05_tflops"] = round(nl * P * TOP * 3 * 2.0 * W * F / (k["gemm_tc_grouped"][1] / 1e3) / 1e12, 2)
+                    fr["prefill_experts_tcgen05_frac"] = round(fr["prefill_experts_tcgen05_tflops"] / peaks["bf16_tflops"], 4)
+                if "gemm_tc" in k:                # lightning in and out, latent down and out, dense down; the up product is gemm_act
+                    flops = nl * P * 2.0 * W * (2 * LH * LD + 3 * LH * LV + H * (D + R) + KR + R + H * VD + DF)
+                    fr["prefill_dense_products_frac"] = round(flops / (k["gemm_tc"][1] / 1e3) / 1e12 / peaks["bf16_tflops"], 4)
+                if "gemm_act" in k:
+                    fr["prefill_gemm_act_frac"] = round(nl * P * 2.0 * W * DF / (k["gemm_act"][1] / 1e3) / 1e12 / peaks["bf16_tflops"], 4)
+                kd = kinds.get("decode") or {}
+                if "retention_raw" in kd:
+                    fr["decode_retention_raw_hbm_frac"] = round(nl * 8 * LH * LD * LV * 4 * 2 / (kd["retention_raw"][1] / 1e3) / 1e9 / peaks["hbm_gbs"], 4)
+                if "attention_tile" in kd:
+                    fr["decode_attention_tile_hbm_frac"] = round(nl * 8 * min(WIN, P) * (KR + R) * 2 / (kd["attention_tile"][1] / 1e3) / 1e9 / peaks["hbm_gbs"], 4)
+                if "gemm_grouped" in kd:          # the experts that 8 tokens of random ids touch, and the heads' projections
+                    touched = E * (1.0 - (1.0 - TOP / float(E)) ** 8)
+                    w_b = nl * (touched * 3 * W * F * 2 + H * KR * (D + VD) * 2)
+                    fr["decode_experts_touched"] = round(touched, 1)
+                    fr["decode_gemm_grouped_hbm_frac"] = round(w_b / (kd["gemm_grouped"][1] / 1e3) / 1e9 / peaks["hbm_gbs"], 4)
+                line["fractions"] = fr
+            print(json.dumps(line), flush=True)
+            del engine
+            torch.cuda.empty_cache()
+    clocks.stop()
+    print(json.dumps({"point": "clocks", "clocks": clocks.summary()}), flush=True)
+    return 0
+
+
 def main() -> int:
     ap = argparse.ArgumentParser()
-    ap.add_argument("--workload", default="headline", choices=["headline", "sweep", "attn_decode", "shapes", "tipezen", "dominex", "sadupel", "nugosun"] + sorted(WORKLOADS),
+    ap.add_argument("--workload", default="headline", choices=["headline", "sweep", "attn_decode", "shapes", "tipezen", "dominex", "sadupel", "nugosun", "kadodra"] + sorted(WORKLOADS),
                     help="headline: the decode/prefill benchmark; sweep: the same shape at further batch sizes and "
                          "context lengths; attn_decode: the decode attention alone; shapes: the layer sizes of the other "
-                         "models of the family; tipezen: the Tipezen design beside Qwen3 at equal layer sizes; dominex: the Dominex design beside Tipezen at equal layer sizes; sadupel: the Sadupel design beside Dominex at equal layer sizes; nugosun: the Nugosun design beside Dominex at equal layer sizes; else a whole workload through "
+                         "models of the family; tipezen: the Tipezen design beside Qwen3 at equal layer sizes; dominex: the Dominex design beside Tipezen at equal layer sizes; sadupel: the Sadupel design beside Dominex at equal layer sizes; nugosun: the Nugosun design beside Dominex at equal layer sizes; kadodra: the Kadodra design beside Nugosun at equal layer sizes; else a whole workload through "
                          "the scheduler")
     ap.add_argument("--gpus", type=int, default=1)
     ap.add_argument("--steps", type=int, default=64)
     ap.add_argument("--warmup", type=int, default=4)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--batch", type=int, default=8)
-    ap.add_argument("--size", default="", help="with --workload dominex, sadupel or nugosun: one of its layer sizes (2k, 4k) instead of all")
+    ap.add_argument("--size", default="", help="with --workload dominex, sadupel, nugosun or kadodra: one of its layer sizes (2k, 4k) instead of all")
     ap.add_argument("--layers", type=int, default=SHAPE["num_layers"],
                     help="fewer layers than the shape has (both numbers are reported)")
     ap.add_argument("--skip-points", action="store_true", help="only the headline batch (no batch 1 / 64, no prefill)")
@@ -904,6 +1018,8 @@ def main() -> int:
         return run_sadupel(args.steps, warmup, [args.size] if args.size else None)
     if args.workload == "nugosun":
         return run_nugosun(args.steps, warmup, [args.size] if args.size else None)
+    if args.workload == "kadodra":
+        return run_kadodra(args.steps, warmup, [args.size] if args.size else None)
     if args.workload != "headline":
         return run_workload(args.workload, 0 if args.layers == SHAPE["num_layers"] else args.layers)
 
