@@ -34,11 +34,12 @@ class RequestError(ValueError):
     """A request the engine cannot run (unknown id, token out of range, too long)."""
 
 
-def _make_ops(device: str):
+def _make_ops(device: str, model: Model):
+    """The kernel library with the kernels that the model's parts name."""
     from ..kernels.library import CudaKernels
     if not str(device).startswith("cuda"):
         raise RuntimeError(f"tffinfer_b200 runs on CUDA devices only (sm_100a); got device '{device}'")
-    return CudaKernels()
+    return CudaKernels(files=model.kernel_files())
 
 
 class ModelRunner:
@@ -53,7 +54,6 @@ class ModelRunner:
         import tffinfer_b200.models  # noqa: F401  registers the architectures
         self.ecfg = (engine_config or EngineConfig()).normalized()
         self.device = torch.device(self.ecfg.device)
-        self.ops = ops if ops is not None else _make_ops(self.ecfg.device)
         self.act_dtype = _TORCH_DTYPES[self.ecfg.dtype]
         if model_dir is not None:
             cj = read_config_json(model_dir)
@@ -67,6 +67,7 @@ class ModelRunner:
             arch = get_architecture(config.architecture)
         self.desc = arch.describe(self.config)
         self.model = Model(self.desc)
+        self.ops = ops if ops is not None else _make_ops(self.ecfg.device, self.model)
         expected = self.model.expected_tensors()
         if model_dir is not None:
             held = load_model_weights(model_dir, expected, self.act_dtype, self.device)

@@ -89,10 +89,12 @@ class DeferredNorm:
 class CudaKernels:
     """Loads (building first if needed) the sm_100a kernel library."""
 
-    def __init__(self, verbose_build: bool = True):
+    def __init__(self, verbose_build: bool = True, files=None):
+        """``files``: names of the CUDA sources that are needed beside the core ones (None: all); a method whose kernel
+        was not asked for fails when it is called."""
         if not torch.cuda.is_available():
             raise KernelError("tffinfer_b200 needs a CUDA device (sm_100a): torch.cuda.is_available() is False")
-        path = _build.library_path(build=True, verbose=verbose_build)
+        path = _build.library_path(build=True, verbose=verbose_build, files=files)
         try:
             self.lib = ctypes.CDLL(path)
         except OSError as e:

@@ -44,6 +44,9 @@ class GQAttention(Mixer):
         self.kv_width = self.num_kv_heads * self.head_dim
         self.w_qkv = self.w_o = self.q_norm_w = self.k_norm_w = None
 
+    def kernel_files(self):
+        return ("attention_bf16", "attention_decode", "attention_prefill", "attention_generic")
+
     def cache_need(self):
         return KVNeed(self.num_kv_heads, self.head_dim, self.window)
 
@@ -146,6 +149,10 @@ class GatedSinkAttention(Mixer):
         self.cache_dim = max(self.head_dim, self.v_head_dim)     # a cache slot holds a key or a value
         self.w_in = self.w_o = self.lam = self.sink_w = None
         self.conv_w = self.conv_wt = self.norm_w = None
+
+    def kernel_files(self):
+        return ("attention_bf16", "attention_decode", "attention_prefill", "attention_generic",
+                "qkv_finish", "short_conv")
 
     def cache_need(self):
         kv = KVNeed(self.num_kv_heads, self.cache_dim, self.window)
@@ -272,6 +279,9 @@ class BiasedChunkAttention(SplitMixer):
         self.v_width = self.num_kv_heads * self.v_head_dim
         self.cache_dim = max(self.head_dim, self.v_head_dim)     # a cache slot holds a key or a value
         self.w_in = self.w_o = self.temp = self.r1 = self.r2 = self.bias = None
+
+    def kernel_files(self):
+        return ("attention_tile", "qkv_finish")
 
     def cache_need(self):
         spans = [s for s in (self.chunk, self.window) if s > 0]

@@ -93,6 +93,11 @@ class Part:
     def full_name(self, rel: str) -> str:
         return f"{self.prefix}.{rel}" if self.prefix else rel
 
+    def kernel_files(self) -> Tuple[str, ...]:
+        """Names of the CUDA sources (csrc/<name>.cu) whose kernels this part calls beside the core ones
+        (csrc/build.py): a fresh checkout compiles what its model needs."""
+        return ()
+
     def load(self, tensors: Dict[str, torch.Tensor], ops, act_dtype: torch.dtype) -> None:
         """Receive the tensors named by weight_specs() (relative names), already on the
         device and in the dtype their role asks for.  Merging happens here."""

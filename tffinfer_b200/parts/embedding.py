@@ -27,6 +27,9 @@ class HashedPairEmbedding(EmbeddingExtra):
         self.name = name
         self.table = None
 
+    def kernel_files(self):
+        return ("short_conv",)
+
     def state_need(self):
         return StateNeed((1,), "int32")
 

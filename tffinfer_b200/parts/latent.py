@@ -47,6 +47,9 @@ class LatentAttention(Mixer):
         self.w_down = self.w_uq = self.w_uk_t = self.w_uk = self.w_uv = self.w_o = self.q_norm_w = self.kv_norm_w = None
         self.sink_w = None
 
+    def kernel_files(self):
+        return ("latent", "attention_tile", "gemm_grouped", "gemm_grouped_mma")
+
     def cache_need(self):
         return KVNeed(1, self.kv_rank + self.rot_dim, self.window, planes=1)
 

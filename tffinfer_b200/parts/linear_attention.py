@@ -41,6 +41,9 @@ class GatedLinearAttention(Mixer):
         self.v_width = self.num_heads * self.v_head_dim
         self.w_in = self.w_o = self.w_a1 = self.w_a2 = self.decay_bias = self.norm_w = None
 
+    def kernel_files(self):
+        return ("linear_recurrence", "gated_norm")
+
     def cache_need(self):
         return StateNeed((self.num_heads * self.head_dim * self.v_head_dim,), "float32")
 

@@ -33,6 +33,9 @@ class SwiGLU(FeedForward):
         self.names.update(names or {})
         self.w_gate_up = self.w_down = None
 
+    def kernel_files(self):
+        return ("gemm_tc_cluster",)
+
     def weight_specs(self) -> Dict[str, WeightSpec]:
         n = self.names
         return {

@@ -79,6 +79,13 @@ class Model:
                 out[name] = spec
         return out
 
+    def kernel_files(self) -> List[str]:
+        """The CUDA sources that the model's parts need beside the core ones."""
+        files = {f for p in self.all_parts() for f in p.kernel_files()}
+        if self.desc.streams > 0 or any(e.add_vector or e.add_embedding for e in self.desc.schedule):
+            files.add("streams")
+        return sorted(files)
+
     def load(self, tensors: Dict[str, torch.Tensor], ops, act_dtype: torch.dtype, device) -> None:
         d = self.desc
         self.embed = tensors[d.embed_name]

@@ -90,6 +90,10 @@ class RoutedExperts(FeedForward):
     def _shared(self, which: str) -> str:
         return f"{self.names['shared']}.{self.names[which]}"
 
+    def kernel_files(self):
+        return ("moe", "gemm_grouped", "gemm_grouped_mma") + (
+            ("gemm_tc_cluster",) if self.gated and self.shared_intermediate > 0 else ())
+
     def weight_specs(self) -> Dict[str, WeightSpec]:
         if self.router_score == "table":
             s = {self.names["table"]: WeightSpec((self.table_rows, self.top), INT_TABLE, below=self.num_experts)}

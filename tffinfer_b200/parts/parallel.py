@@ -40,6 +40,9 @@ class ParallelMixers(Mixer):
         self._needs = tuple(n for n in needs if n is not None)
         self.w_in = self.w_out = None
 
+    def kernel_files(self):
+        return tuple(f for m in self.branches for f in m.kernel_files())
+
     def cache_need(self):
         if not self._needs:
             return None

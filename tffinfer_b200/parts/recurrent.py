@@ -30,6 +30,9 @@ class MinGRU(SplitMixer):
         self.names.update(names or {})
         self.w_in = self.w_o = self.bz = self.bx = None
 
+    def kernel_files(self):
+        return ("mingru",)
+
     def cache_need(self):
         return StateNeed((self.width,), "float32")
 

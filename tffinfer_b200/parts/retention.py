@@ -40,6 +40,9 @@ class Retention(Mixer):
         self.v_width = self.num_heads * self.v_head_dim
         self.w_in = self.w_o = self.decay_dev = None
 
+    def kernel_files(self):
+        return ("retention", "qkv_finish")
+
     def cache_need(self):
         return StateNeed((self.num_heads, self.head_dim, self.v_head_dim), "float32")
 
@@ -104,6 +107,9 @@ class LightningAttention(Mixer):
         self.names.update(names or {})
         self.qk_width, self.v_width = self.num_heads * self.head_dim, self.num_heads * self.v_head_dim
         self.w_in = self.w_o = self.norm_w = self.decay_dev = None
+
+    def kernel_files(self):
+        return ("retention", "gated_norm")
 
     def cache_need(self):
         return StateNeed((self.num_heads, self.head_dim, self.v_head_dim), "float32")

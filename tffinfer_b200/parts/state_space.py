@@ -52,6 +52,9 @@ class SelectiveStateSpace(SplitMixer):
         self.names.update(names or {})
         self.w_in = self.w_o = self.conv_w = self.conv_b = self.dt_bias = self.rate_log = self.skip = self.norm_w = None
 
+    def kernel_files(self):
+        return ("causal_conv", "linear_recurrence", "gated_norm")
+
     def cache_need(self):
         return StateNeed((self.conv_state + self.num_heads * self.state_size * self.head_dim,), "float32")
 
