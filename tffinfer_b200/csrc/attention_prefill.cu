@@ -42,7 +42,14 @@
 // A cubic on the FMA pipe for part of the exponentials made it slower at every share tried.
 // CTAs are handed out longest walk first over all kv heads.
 // Same contract as the rows mode of attention_bf16.cu, which it replaces when the page size
-// is 8/16/32/64.  Every mbarrier wait is bounded; a timeout raises the library's error word.
+// is 8/16/32/64.
+// The dense form (tff_attention_dense) takes the keys and values of the step's own tokens from plain rows instead of the
+// cache, for steps whose requests all start at position 0 (a latent attention that has made per-head keys and values of
+// a whole prompt): keys of up to 192 elements, values of up to 128, one box of 64 rows per 64 columns.  A key may lie in
+// two tensors: columns of its own head, and a part that all heads share (the rotated part of a latent attention), which is
+// then read where it is.  Tensor memory has room for 128 elements of a query row of either tile; what goes beyond
+// (columns 128 to 191) lies in shared memory, and its products take A from there.
+//  Every mbarrier wait is bounded; a timeout raises the library's error word.
 // Every wait lets the hardware suspend the warp: the waiting warps share their schedulers with the softmax warps
 // of the other tile, and polled they took issue slots from those (5 % of the kernel's time).
 #define TFF_SUSPENDED_WAITS
@@ -72,7 +79,6 @@ using tc5::tmem_ld_wait;
 
 constexpr int BLOCK_M = 128;
 constexpr int BLOCK_N = 64;
-constexpr int NSTAGES = 5;
 #ifndef TURN_AFTER
 #define TURN_AFTER 8          // of the 8 chunks of a block's exponentials, after which the other tile may begin its own
 #endif
@@ -168,25 +174,47 @@ struct PrefillParams {
     int nq, nkv; float scale_log2; int window;
     float scale_over_cap, cap_log2; int sink; const float* gate; const float* sink_val;   // AttnExtra, ready for the kernel
     int* error_flag;
+    int d, dv;                           // elements of a query row and of an output row (DENSE; at most DK and DV)
+    int k_halves, k_head;                // DENSE: 64-column halves of a key that come from tm_k, columns between its heads
+    int r_col;                           // DENSE: first column of the shared part in tm_r
+};
+
+template <int DK, int DV, int QT>
+struct PrefillCfg {
+    static constexpr int kStageBytes = BLOCK_N * (DK + DV) * 2;     // K then V, each [64-column half][64 keys][128 B]
+    static constexpr int kQExtra = DK > 128 ? (DK - 128) / 64 * BLOCK_M * 128 : 0;     // a tile's query columns beyond 128
+    static constexpr int kStages = DK > 128 ? (QT == 2 ? 3 : 4) : 5;
+    static constexpr int kBars = 2 * kStages + BARS_PER_TILE * QT + 8;
+    static constexpr int kSmem = kStages * kStageBytes + QT * (2 * BLOCK_M * BLOCK_N * 2 + kQExtra) + 8 * kBars + 16 + 1024;
+    static_assert(kSmem <= 227 * 1024, "shared memory of the prompt attention kernel");
 };
 
 // QT: query tiles per CTA.  Two when that still gives every SM a CTA, one otherwise.
-template <int D, int QT>
+// DK, DV: elements of a key and of a value (DENSE: rounded up; the query's columns beyond its own are zeros, the output's
+// are not stored).  tm_cache is the cache, or the keys' rows when DENSE; tm_v and tm_r are read by the dense form only.
+template <int DK, int DV, int QT, bool DENSE>
 __global__ void __launch_bounds__(QT == 2 ? 352 : 192, 1)
-attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_cache, const PrefillParams p) {
-    constexpr int HF = D / 64;                                   // 64-column halves of a head
-    constexpr int CH = D / 8;                                    // 16-byte chunks per row
-    constexpr int KV_BYTES = BLOCK_N * D * 2;                    // K (or V) of one stage: [half][64 keys][128 B]
-    constexpr int STAGE_BYTES = 2 * KV_BYTES;
+attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_cache, const __grid_constant__ CUtensorMap tm_v,
+                       const __grid_constant__ CUtensorMap tm_r, const PrefillParams p) {
+    using Cfg = PrefillCfg<DK, DV, QT>;
+    static_assert(DENSE || DK == DV, "a slot of the cache holds a key or a value");
+    constexpr int NSTAGES = Cfg::kStages;
+    constexpr int KH = DK / 64, VH = DV / 64;                    // 64-column halves of a key and of a value
+    constexpr int CH = DV / 8;                                   // 16-byte chunks of a value row
+    constexpr int K_BYTES = BLOCK_N * DK * 2;                    // K of one stage: [half][64 keys][128 B]
+    constexpr int STAGE_BYTES = Cfg::kStageBytes;
     constexpr int P_BYTES = BLOCK_M * BLOCK_N * 2;               // one tile's probabilities: [128 rows][128 B]
+    constexpr int QT_COLS = DK < 128 ? DK : 128;                 // query elements a row that lie in tensor memory
     constexpr int TMEM_COLS = 512;
-    constexpr int NBARS = 2 * NSTAGES + BARS_PER_TILE * QT + 8;
+    constexpr int NBARS = Cfg::kBars;
     extern __shared__ uint8_t smem_raw[];
     const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
     uint8_t* gbase = smem_raw + (base - smem_u32(smem_raw));
     const uint32_t sP = base + NSTAGES * STAGE_BYTES;            // two buffers per tile: [tile][block % 2]
-    const uint32_t bars = sP + QT * 2 * P_BYTES;
+    const uint32_t sQ = sP + QT * 2 * P_BYTES;                   // the tiles' query columns beyond QT_COLS: [half][128 rows][128 B]
+    const uint32_t bars = sQ + QT * Cfg::kQExtra;
     uint8_t* gP = gbase + NSTAGES * STAGE_BYTES;
+    uint8_t* gQ = gP + QT * 2 * P_BYTES;
     // barriers: kv_full[NS], kv_empty[NS]; per tile x: s_full, s_free, p_full[0], pv_done[2], q_ready, p_full[1]
     auto kv_full = [&](int s) { return bars + 8u * s; };
     auto kv_empty = [&](int s) { return bars + 8u * (NSTAGES + s); };
@@ -204,7 +232,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_cache, const Prefi
     // whose turn it is at the special-function unit: the warps of the two tiles that share a scheduler (the same
     // lane quarter) take their exponential passes in turn
     auto turn = [&](int x, int q) { return bars + 8u * (2 * NSTAGES + BARS_PER_TILE * QT + 4 * x + q); };
-    volatile uint32_t* tmem_slot = (volatile uint32_t*)(gP + QT * 2 * P_BYTES + 8 * NBARS);
+    volatile uint32_t* tmem_slot = (volatile uint32_t*)(gQ + QT * Cfg::kQExtra + 8 * NBARS);
     volatile int* abort_flag = (volatile int*)(tmem_slot + 1);
 
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -213,7 +241,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_cache, const Prefi
     const int kvh = blockIdx.x;
     const int pair = (int)gridDim.y - 1 - (int)blockIdx.y;
     const int G = p.nq / p.nkv;
-    const int ps = 1 << p.page_shift;
+    const int ps = DENSE ? 0 : 1 << p.page_shift;
 
     if (tid == 0) {
         for (int s = 0; s < NSTAGES; ++s) mbar_init(kv_full(s), 1);
@@ -225,6 +253,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_cache, const Prefi
         *abort_flag = 0;
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
         asm volatile("prefetch.tensormap [%0];" ::"l"(&tm_cache) : "memory");
+        if (DENSE) asm volatile("prefetch.tensormap [%0];" ::"l"(&tm_v) : "memory");
     }
     if (warp == 1) tmem_alloc(smem_u32((const void*)tmem_slot), TMEM_COLS);
     tc_fence_before();
@@ -249,7 +278,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_cache, const Prefi
     const int lo_cta = p.window > 0 ? max(0, pos0 + first_tok - p.window + 1) : 0;   // first key any row sees
     const int kb_lo = lo_cta / BLOCK_N, kb_hi = hi / BLOCK_N;
     const int nb = active ? kb_hi - kb_lo + 1 : 0;
-    const int* table = p.block_table + (size_t)b * p.table_width;
+    const int* table = DENSE ? nullptr : p.block_table + (size_t)b * p.table_width;
     // a stage is free again when the PV products of every tile that has rows have read it
     if (tid == 0) {
         for (int s = 0; s < NSTAGES; ++s) mbar_init(kv_empty(s), (uint32_t)(n_act > 0 ? n_act : 1));
@@ -260,10 +289,10 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_cache, const Prefi
 
     if (warp == 0) {
         // ------------------------------------------------------------ TMA producer
-        const int ppb = BLOCK_N >> p.page_shift;
-        const int nloads = ppb * HF * 2;                          // boxes per stage (<= 32)
-        const int j = lane / (HF * 2), rem = lane % (HF * 2);
-        const int kv = rem / HF, hf = rem % HF;
+        const int ppb = DENSE ? 0 : BLOCK_N >> p.page_shift;
+        const int nloads = ppb * KH * 2;                          // boxes per stage (<= 32)
+        const int j = lane / (KH * 2), rem = lane % (KH * 2);
+        const int kv = rem / KH, hf = rem % KH;
         for (int i = 0; i < nb; ++i) {
             const int s = i % NSTAGES;
             const uint32_t round = i / NSTAGES;
@@ -273,6 +302,21 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_cache, const Prefi
                 ok = __shfl_sync(0xffffffffu, ok, 0);
             }
             if (!ok) break;
+            if constexpr (DENSE) {
+                // key n of the request is row q0 + n; rows beyond the request's are another's or zeros, and masked
+                if (lane == 0) mbar_expect_tx(kv_full(s), (uint32_t)STAGE_BYTES);
+                __syncwarp();
+                const int row = q0 + (kb_lo + i) * BLOCK_N;
+                if (lane < KH) {
+                    const uint32_t dst = base + s * STAGE_BYTES + lane * (BLOCK_N * 128);
+                    if (lane < p.k_halves) tma_load_2d(dst, &tm_cache, kv_full(s), kvh * p.k_head + lane * 64, row);
+                    else tma_load_2d(dst, &tm_r, kv_full(s), p.r_col + (lane - p.k_halves) * 64, row);
+                } else if (lane < KH + VH) {
+                    tma_load_2d(base + s * STAGE_BYTES + K_BYTES + (lane - KH) * (BLOCK_N * 128), &tm_v, kv_full(s),
+                                kvh * p.dv + (lane - KH) * 64, row);
+                }
+                continue;
+            }
             const int n0 = (kb_lo + i) * BLOCK_N + (j << p.page_shift);
             int page = -1;
             if (lane < nloads && n0 <= hi) page = table[n0 >> p.page_shift];
@@ -283,7 +327,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_cache, const Prefi
             if (valid) {
                 const long long row = ((((long long)page * p.cache_layers + p.layer) * 2 + kv) * p.nkv + kvh) << p.page_shift;
                 // stage layout: K then V, each [half][64 keys][128 B]
-                const uint32_t dst = base + s * STAGE_BYTES + kv * KV_BYTES + hf * (BLOCK_N * 128) +
+                const uint32_t dst = base + s * STAGE_BYTES + kv * K_BYTES + hf * (BLOCK_N * 128) +
                                      (uint32_t)((j << p.page_shift) * 128);
                 tma_load_2d(dst, &tm_cache, kv_full(s), hf * 64, (int)row);
             }
@@ -293,20 +337,24 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_cache, const Prefi
         const int x = warp == 1 ? 0 : 1;
         if (lane == 0 && x < n_act && nb > 0) {
             constexpr uint32_t idesc_s = make_idesc(BLOCK_M, BLOCK_N, 0);
-            constexpr uint32_t idesc_pv = make_idesc(BLOCK_M, D, 1);
+            constexpr uint32_t idesc_pv = make_idesc(BLOCK_M, DV, 1);
             const uint32_t t_o = tmem_base + x * 128, t_s = tmem_base + 256 + x * 64, t_q = tmem_base + 384 + x * 64;
             // descriptors are built once; a product costs one 64-bit add on each (the low bits of a
             // descriptor are the shared-memory address in units of 16 bytes)
             const uint64_t kdesc = make_smem_desc(base, 16);                       // + stage * STAGE_BYTES
-            const uint64_t vdesc = make_smem_desc(base + KV_BYTES, BLOCK_N * 128); // + stage * STAGE_BYTES
+            const uint64_t vdesc = make_smem_desc(base + K_BYTES, BLOCK_N * 128);  // + stage * STAGE_BYTES
             const uint64_t pdesc = make_smem_desc(sP + x * 2 * P_BYTES, 16);      // + (block % 2) * P_BYTES
             auto issue_s = [&](int jj) {                           // S(jj); K(jj) has landed, the S buffer is free
                 const uint64_t kd = kdesc + (uint64_t)((jj % NSTAGES) * (STAGE_BYTES >> 4));
 #pragma unroll
-                for (int kk = 0; kk < D / 16; ++kk) {
+                for (int kk = 0; kk < DK / 16; ++kk) {
                     // Q: 16 elements of a row = 8 columns of tensor memory; K: [half][64 keys][128 B], 32 bytes along a row
                     const uint32_t koff = ((kk / 4) * (BLOCK_N * 128) + (kk % 4) * 32) >> 4;
-                    umma_bf16_a_tmem(t_s, t_q + kk * 8, kd + koff, idesc_s, kk > 0 ? 1u : 0u);
+                    if (kk < QT_COLS / 16)
+                        umma_bf16_a_tmem(t_s, t_q + kk * 8, kd + koff, idesc_s, kk > 0 ? 1u : 0u);
+                    else
+                        umma_bf16(t_s, make_smem_desc(sQ + x * Cfg::kQExtra + ((kk * 16 - QT_COLS) / 64) * (BLOCK_M * 128), 16) +
+                                           (uint64_t)((kk % 4) * 2), kd + koff, idesc_s, 1u);
                 }
                 umma_commit(s_full(x));
             };
@@ -369,17 +417,26 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_cache, const Prefi
         const uint32_t t_q = t_row + 384 + x * 64;
         // the query tile: this thread's row, two elements a column, into tensor memory
         if (tile_active) {
-            const bf16* src = p.q + (size_t)(q0 + R / G) * p.q_row_stride + (size_t)(kvh * G + R % G) * D;
+            const bf16* src = p.q + (size_t)(q0 + R / G) * p.q_row_stride + (size_t)(kvh * G + R % G) * (DENSE ? p.d : DK);
 #pragma unroll
-            for (int c16 = 0; c16 < D / 32; ++c16) {
+            for (int c16 = 0; c16 < QT_COLS / 32; ++c16) {
                 uint32_t v[16];
 #pragma unroll
                 for (int c = 0; c < 4; ++c) {
                     uint4 u = make_uint4(0u, 0u, 0u, 0u);
-                    if (rv) u = *reinterpret_cast<const uint4*>(src + c16 * 32 + c * 8);
+                    if (rv && (!DENSE || c16 * 32 + c * 8 < p.d)) u = *reinterpret_cast<const uint4*>(src + c16 * 32 + c * 8);
                     v[4 * c] = u.x; v[4 * c + 1] = u.y; v[4 * c + 2] = u.z; v[4 * c + 3] = u.w;
                 }
                 tmem_st16(t_q + c16 * 16, v);
+            }
+            if constexpr (DK > QT_COLS) {                          // the columns beyond: K-major rows, swizzled as P is
+#pragma unroll
+                for (int c = 0; c < (DK - QT_COLS) / 8; ++c) {
+                    uint4 u = make_uint4(0u, 0u, 0u, 0u);
+                    if (rv && QT_COLS + c * 8 < p.d) u = *reinterpret_cast<const uint4*>(src + QT_COLS + c * 8);
+                    *reinterpret_cast<uint4*>(gQ + x * Cfg::kQExtra + (c >> 3) * (BLOCK_M * 128) + r * 128 + (((c & 7) ^ (r & 7)) << 4)) = u;
+                }
+                fence_async_smem();
             }
             tmem_st_wait();
             tc_fence_before();
@@ -404,7 +461,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_cache, const Prefi
                 // do it (the same zeros), so that each tile's products wait for its own warps only.
                 ok = mbar_wait_warp(kv_full(st), (j / NSTAGES) & 1, abort_flag);
                 if (!ok) break;
-                uint8_t* gV = gbase + st * STAGE_BYTES + KV_BYTES;
+                uint8_t* gV = gbase + st * STAGE_BYTES + K_BYTES;
                 for (int idx = tt; idx < BLOCK_N * CH; idx += 128) {
                     const int kr = idx / CH, c = idx % CH;
                     const int n = blk * BLOCK_N + kr;
@@ -471,7 +528,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_cache, const Prefi
                     if (!ok) break;
                     tc_fence_after();
 #pragma unroll 1
-                    for (int c0 = 0; c0 < D; c0 += 16) {
+                    for (int c0 = 0; c0 < DV; c0 += 16) {
                         uint32_t v[16];
                         tmem_ld16(t_o + c0, v);
                         tmem_ld_wait();
@@ -546,9 +603,10 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_cache, const Prefi
             if (p.sink && l > 0.f) l += exp2f(attn_sink_log2(p.sink_val, kvh * G + R % G) - m_used);   // the sink: a key without a value
             float inv = l > 0.f ? 1.f / l : 0.f;
             if (p.gate && rv) inv *= p.gate[(size_t)(q0 + R / G) * p.nq + (kvh * G + R % G)];
-            bf16* orow = p.out + ((size_t)(q0 + R / G) * p.nq + (kvh * G + R % G)) * D;
+            const int dv = DENSE ? p.dv : DV;
+            bf16* orow = p.out + ((size_t)(q0 + R / G) * p.nq + (kvh * G + R % G)) * dv;
 #pragma unroll 1
-            for (int c0 = 0; c0 < D; c0 += 16) {
+            for (int c0 = 0; c0 < DV; c0 += 16) {
                 uint32_t v[16];
                 tmem_ld16(t_o + c0, v);
                 tmem_ld_wait();
@@ -559,8 +617,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_cache, const Prefi
                         __nv_bfloat162 b2 = __floats2bfloat162_rn(__uint_as_float(v[2 * i]) * inv, __uint_as_float(v[2 * i + 1]) * inv);
                         w[i] = *reinterpret_cast<uint32_t*>(&b2);
                     }
-                    *reinterpret_cast<uint4*>(orow + c0) = make_uint4(w[0], w[1], w[2], w[3]);
-                    *reinterpret_cast<uint4*>(orow + c0 + 8) = make_uint4(w[4], w[5], w[6], w[7]);
+                    if (!DENSE || c0 < dv) *reinterpret_cast<uint4*>(orow + c0) = make_uint4(w[0], w[1], w[2], w[3]);
+                    if (!DENSE || c0 + 8 < dv) *reinterpret_cast<uint4*>(orow + c0 + 8) = make_uint4(w[4], w[5], w[6], w[7]);
                 }
             }
         }
@@ -580,20 +638,34 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_cache, const Prefi
     }
 }
 
-template <int D, int QT>
-int launch_prefill(const CUtensorMap& tm, const PrefillParams& p, int q_tiles, int B, cudaStream_t stream) {
+template <int DK, int DV, int QT, bool DENSE>
+int launch_prefill(const CUtensorMap& tm, const CUtensorMap& tv, const CUtensorMap& tr, const PrefillParams& p, int q_tiles,
+                   int B, cudaStream_t stream) {
     constexpr int NTHREADS = QT == 2 ? 352 : 192;
-    constexpr int smem = NSTAGES * 2 * BLOCK_N * D * 2 + QT * 2 * BLOCK_M * BLOCK_N * 2 +
-                         8 * (2 * NSTAGES + BARS_PER_TILE * QT + 8) + 16 + 1024;
-    static_assert(smem <= 227 * 1024, "shared memory of the prompt attention kernel");
-    auto kern = attn_prefill_tc_kernel<D, QT>;
+    constexpr int smem = PrefillCfg<DK, DV, QT>::kSmem;
+    auto kern = attn_prefill_tc_kernel<DK, DV, QT, DENSE>;
     static bool configured = false;
     if (!configured) {
         if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess)
             return TFF_ERR_LAUNCH;
         configured = true;
     }
-    return tff_launch_pdl(kern, dim3(p.nkv, q_tiles, B), dim3(NTHREADS), (size_t)smem, stream, tm, p);
+    return tff_launch_pdl(kern, dim3(p.nkv, q_tiles, B), dim3(NTHREADS), (size_t)smem, stream, tm, tv, tr, p);
+}
+
+// Two query tiles a CTA share one walk over the keys and take turns at the exponentials: a pair of tiles costs
+// 1.08 times what a single tile costs (512 new tokens behind 3,584 cached ones, 32/8 heads: 92 us as 128 CTAs
+// of one tile, 100 us as 64 CTAs of two).  So single tiles only while they all run at once, one an SM; as soon
+// as they would not, pairs (1,536 tokens from scratch: 61 us against 74 as single tiles; 2,816 tokens: 114
+// against 149; 1,536 behind 2,048 cached ones: 123 against 160).
+template <int DK, int DV, bool DENSE>
+int launch_prefill_tiles(const CUtensorMap& tm, const CUtensorMap& tv, const CUtensorMap& tr, const PrefillParams& p,
+                         int max_q_len, int B, cudaStream_t stream) {
+    const int tiles = (max_q_len * (p.nq / p.nkv) + BLOCK_M - 1) / BLOCK_M;
+    const long long sms = tff_num_sms() > 0 ? tff_num_sms() : 1;
+    if ((long long)tiles * p.nkv * B > sms)
+        return launch_prefill<DK, DV, 2, DENSE>(tm, tv, tr, p, (tiles + 1) / 2, B, stream);
+    return launch_prefill<DK, DV, 1, DENSE>(tm, tv, tr, p, tiles, B, stream);
 }
 
 }  // namespace
@@ -632,18 +704,50 @@ int tff_attention_prefill_launch(
     p.sink = extra.sink; p.gate = extra.gate; p.sink_val = extra.sink_val;
     p.error_flag = tff_device_error_flag();
     if (p.error_flag == nullptr) return TFF_ERR_LAUNCH;
-    const int G = nq / nkv;
-    const int tiles = (max_q_len * G + BLOCK_M - 1) / BLOCK_M;
-    const int pairs = (tiles + 1) / 2;
-    // Two query tiles a CTA share one walk over the keys and take turns at the exponentials: a pair of tiles costs
-    // 1.08 times what a single tile costs (512 new tokens behind 3,584 cached ones, 32/8 heads: 92 us as 128 CTAs
-    // of one tile, 100 us as 64 CTAs of two).  So single tiles only while they all run at once, one an SM; as soon
-    // as they would not, pairs (1,536 tokens from scratch: 61 us against 74 as single tiles; 2,816 tokens: 114
-    // against 149; 1,536 behind 2,048 cached ones: 123 against 160).
-    const long long sms = tff_num_sms() > 0 ? tff_num_sms() : 1;
-    if ((long long)tiles * nkv * num_requests > sms)
-        return d == 128 ? launch_prefill<128, 2>(tm, p, pairs, num_requests, stream)
-                        : launch_prefill<64, 2>(tm, p, pairs, num_requests, stream);
-    return d == 128 ? launch_prefill<128, 1>(tm, p, tiles, num_requests, stream)
-                    : launch_prefill<64, 1>(tm, p, tiles, num_requests, stream);
+    p.d = p.dv = d; p.k_halves = p.k_head = p.r_col = 0;
+    return d == 128 ? launch_prefill_tiles<128, 128, false>(tm, tm, tm, p, max_q_len, num_requests, stream)
+                    : launch_prefill_tiles<64, 64, false>(tm, tm, tm, p, max_q_len, num_requests, stream);
+}
+
+// The dense form: every request of the step starts at position 0, and the keys and values of its tokens are the rows
+// q_start .. of k [tokens, k_ld] (head h at columns h * k_head ..) and v [tokens, nkv * dv].  d elements of a query row
+// [nq * d]: with ``shared`` (bfloat16 [tokens, shared_ld], columns r_col .. of it) a key's last d - k_head elements are the
+// same for all heads and lie there, and k_head is a multiple of 64; without it k_head = d.  out [tokens, nq * dv].
+// TFF_ERR_UNSUPPORTED for sizes it does not take (d <= 192, dv <= 128, all multiples of 8).
+TFF_API int tff_attention_dense(const void* q, const int* q_start, const int* pos_start, const void* k, int k_ld, int k_head,
+                                const void* shared, int shared_ld, int r_col, const void* v, void* out, int num_tokens,
+                                int num_requests, int max_q_len, int nq, int nkv, int d, int dv, float scale, int window,
+                                float softcap, const float* sink, cudaStream_t stream) {
+    if (num_requests <= 0 || max_q_len <= 0 || num_tokens <= 0) return TFF_OK;
+    if (!q || !k || !v || !out || nq <= 0 || nkv <= 0 || nq % nkv || d <= 0 || dv <= 0 || window < 0 || k_head <= 0 || k_head > d)
+        return TFF_ERR_BAD_ARGUMENT;
+    const int rest = d - k_head;
+    if ((rest > 0) != (shared != nullptr) || k_ld < nkv * k_head || (shared && (r_col < 0 || r_col + rest > shared_ld)))
+        return TFF_ERR_BAD_ARGUMENT;
+    if (d > 192 || dv > 128 || (d & 7) || (dv & 7) || (k_ld & 7) || (k_head & 7) || !(scale > 0.f) || num_requests > 65535)
+        return TFF_ERR_UNSUPPORTED;
+    if (shared && (k_head % 64 || rest > 64 || (shared_ld & 7) || (r_col & 7))) return TFF_ERR_UNSUPPORTED;
+    if (((uintptr_t)q & 15) || ((uintptr_t)k & 15) || ((uintptr_t)v & 15) || ((uintptr_t)out & 15) || ((uintptr_t)shared & 15))
+        return TFF_ERR_UNSUPPORTED;
+    if ((long long)max_q_len * (nq / nkv) > 65535ll * 256) return TFF_ERR_UNSUPPORTED;
+    CUtensorMap tk, tv, tr;
+    if (!tff_tensor_map_2d(k, num_tokens, k_ld, BLOCK_N, 64, 2, &tk)) return TFF_ERR_DRIVER;
+    if (!tff_tensor_map_2d(v, num_tokens, (long long)nkv * dv, BLOCK_N, 64, 2, &tv)) return TFF_ERR_DRIVER;
+    tr = tk;
+    if (shared && !tff_tensor_map_2d(shared, num_tokens, shared_ld, BLOCK_N, 64, 2, &tr)) return TFF_ERR_DRIVER;
+    PrefillParams p = {};
+    p.q = (const bf16*)q; p.q_row_stride = nq * d; p.q_start = q_start; p.pos_start = pos_start;
+    p.out = (bf16*)out; p.nq = nq; p.nkv = nkv; p.scale_log2 = scale * 1.4426950408889634f; p.window = window;
+    p.scale_over_cap = softcap > 0.f ? scale / softcap : 0.f;
+    p.cap_log2 = softcap > 0.f ? softcap * 1.4426950408889634f : 0.f;
+    p.sink = sink ? 1 : 0; p.sink_val = sink;
+    p.d = d; p.dv = dv; p.k_head = k_head; p.r_col = r_col;
+    p.error_flag = tff_device_error_flag();
+    if (p.error_flag == nullptr) return TFF_ERR_LAUNCH;
+    if (d > 128) {
+        p.k_halves = shared ? k_head / 64 : 3;
+        return launch_prefill_tiles<192, 128, true>(tk, tv, tr, p, max_q_len, num_requests, stream);
+    }
+    p.k_halves = shared ? k_head / 64 : 2;
+    return launch_prefill_tiles<128, 128, true>(tk, tv, tr, p, max_q_len, num_requests, stream);
 }

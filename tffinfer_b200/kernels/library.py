@@ -804,6 +804,25 @@ class CudaKernels:
             _c_int(vd.shape[1] if vd is not None else 0), _c_float(softcap), _ptr(sink), self._stream()), "attention_tile")
         self.launches += 2 if splits > 1 else 1
 
+    def attention_dense(self, q, batch, keys, k_head: int, shared, r_col: int, values, out, nq, nkv, d, dv, scale,
+                        window: int = 0, softcap: float = 0.0, sink=None) -> None:
+        """Attention of whole prompts (every request of the step starts at position 0, bfloat16) over keys and values of
+        the step's own tokens in plain rows, on the tcgen05 kernel of csrc/attention_prefill.cu: q [T, nq*d], keys
+        [T, nkv*k_head], values [T, nkv*dv] -> out [T, nq*dv].  A key's last d - k_head elements lie in columns r_col .. of
+        ``shared`` [T, ...], the same for all heads (None: k_head = d).  d <= 192, dv <= 128, multiples of 8."""
+        self._need_cuda(q, keys, shared, values, out, sink)
+        T = q.shape[0]
+        for t in (q, keys, shared, values, out):
+            assert t is None or (t.dtype == torch.bfloat16 and t.shape[0] == T)
+        assert q.shape[1] == nq * d and keys.shape[1] == nkv * k_head and values.shape[1] == nkv * dv and out.shape[1] == nq * dv
+        assert sink is None or (sink.dtype == torch.float32 and sink.numel() == nq)
+        self._check(self.lib.tff_attention_dense(
+            _ptr(q), _ptr(batch.q_start), _ptr(batch.pos_start), _ptr(keys), _c_int(keys.shape[1]), _c_int(k_head), _ptr(shared),
+            _c_int(shared.shape[1] if shared is not None else 0), _c_int(r_col), _ptr(values), _ptr(out), _c_int(T),
+            _c_int(batch.num_requests), _c_int(batch.max_q_len), _c_int(nq), _c_int(nkv), _c_int(d), _c_int(dv),
+            _c_float(scale), _c_int(window), _c_float(softcap), _ptr(sink), self._stream()), "attention_dense")
+        self.launches += 1
+
     def tile_splits(self, batch, nq: int, nkv: int, window: int = 0, chunk: int = 0) -> int:
         """In how many shares attention_tile cuts every tile's key range: a power of two such that a step of few rows
         behind long contexts (decoded tokens above all) still gives every SM a CTA, with at least eight key blocks
@@ -1429,18 +1448,27 @@ class CudaKernels:
         if per_head:
             if q_rank:
                 self.latent_q_rot(q, q, f, batch, heads, dim, rot_dim, turn, dim)          # in place: the head's own row
-            keys = torch.empty((T, heads * (dim + rot_dim)), dtype=dt, device=dev)
+            # on the tcgen05 kernel a key's rotated part may stay where it is, in the latent rows, one for all heads
+            dense_tc = dim + rot_dim <= 192 and vdim <= 128 and scale > 0
+            apart = dense_tc and dim % 64 == 0 and 0 < rot_dim <= 64
+            k_head = dim if apart else dim + rot_dim
+            keys = torch.empty((T, heads * k_head), dtype=dt, device=dev)
             self.gemm_grouped(rows, w_uk, keys, heads, T, dim, kv_rank, slot, 0, kv_rank, dim * kv_rank,
-                              heads * (dim + rot_dim), dim + rot_dim)
-            self._check(self.lib.tff_latent_spread(_ptr(rows), _c_int(kv_rank), _c_int(rot_dim), _ptr(keys), _c_int(dim),
-                                                   _c_int(heads), _c_int(_dt(keys)), _c_int(T), self._stream()),
-                        "latent_spread")
-            self.launches += 1
+                              heads * k_head, k_head)
+            if not apart:
+                self._check(self.lib.tff_latent_spread(_ptr(rows), _c_int(kv_rank), _c_int(rot_dim), _ptr(keys), _c_int(dim),
+                                                       _c_int(heads), _c_int(_dt(keys)), _c_int(T), self._stream()),
+                            "latent_spread")
+                self.launches += 1
             values = torch.empty((T, heads * vdim), dtype=dt, device=dev)
             self.gemm_grouped(rows, w_uv, values, heads, T, vdim, kv_rank, slot, 0, kv_rank, vdim * kv_rank,
                               heads * vdim, vdim)
-            self.attention_tile(q, batch, block_table, kv_cache, kv_layer, page_size, out, heads, heads, dim + rot_dim,
-                                vdim, scale, window=window, sink=sink, dense=(keys, values))
+            if dense_tc:
+                self.attention_dense(q, batch, keys, k_head, rows if apart else None, kv_rank, values, out, heads, heads,
+                                     dim + rot_dim, vdim, scale, window=window, sink=sink)
+            else:
+                self.attention_tile(q, batch, block_table, kv_cache, kv_layer, page_size, out, heads, heads, dim + rot_dim,
+                                    vdim, scale, window=window, sink=sink, dense=(keys, values))
             return
         self.gemm_grouped(q, w_uk_t, q_lat, heads, T, kv_rank, dim, heads * q_ld, q_ld,
                           dim, kv_rank * dim, heads * slot, slot)

@@ -48,7 +48,7 @@ class LatentAttention(Mixer):
         self.sink_w = None
 
     def kernel_files(self):
-        return ("latent", "attention_tile", "gemm_grouped", "gemm_grouped_mma")
+        return ("latent", "attention_tile", "attention_prefill", "gemm_grouped", "gemm_grouped_mma")
 
     def cache_need(self):
         return KVNeed(1, self.kv_rank + self.rot_dim, self.window, planes=1)
