@@ -194,12 +194,14 @@ def ops():
 
 @pytest.mark.parametrize("H,D,V", [(2, 32, 16), (3, 12, 20), (1, 128, 128), (4, 7, 33), (2, 8, 130), (1, 200, 260), (1, 300, 40)])
 @pytest.mark.parametrize("silu", [True, False])
-def test_recurrence_steps_slots_and_a_far_key(ops, H, D, V, silu):
+@pytest.mark.parametrize("rounded", [False, True])
+def test_recurrence_steps_slots_and_a_far_key(ops, H, D, V, silu, rounded):
     """The recurrence through four steps (a long portion, short portions, one token each twice: the decode kernel), slots
     out of order, other slots poisoned and the requests' own slots full of NaN at the start (a request that brings
     position 0 starts from zeros), q, k and v column blocks of wider rows.  In the first request one key far back is
     planted under a decay near one, with a query aimed at it: its value must arrive at the last token.  The last sizes
-    do not fit the chunked form and run token by token."""
+    do not fit the chunked form and run token by token.  ``rounded`` is the chunk form on the tensor cores: behind the
+    rounding of q, k and v (inputs that bfloat16 holds exactly have none) it must be as close as the float32 form."""
     dev = "cuda"
     g = torch.Generator().manual_seed(H * D + V)
     cuts = [[150, 3, 1], [2, 70, 1], [1, 1, 1], [1, 1, 1]]
@@ -214,6 +216,7 @@ def test_recurrence_steps_slots_and_a_far_key(ops, H, D, V, silu):
     k0[4, 0] = 20.0
     q0[-1, :D] = 0.0
     q0[-1, 0] = 20.0
+    seqs = [[x.to(torch.bfloat16).float() for x in s] for s in seqs]
     f = P.silu if silu else (lambda x: x)
     want = []
     for q, k, v in seqs:
@@ -230,7 +233,7 @@ def test_recurrence_steps_slots_and_a_far_key(ops, H, D, V, silu):
         proj = torch.full((T, v_off + H * V + 5), float("nan"))
         proj[:, q_off:q_off + H * D], proj[:, k_off:k_off + H * D], proj[:, v_off:v_off + H * V] = part
         out = torch.full((T, H * V), float("nan"), device=dev)
-        ops.retention_raw(proj.to(dev), q_off, k_off, v_off, silu, state, b, decay.to(dev), out, H, D, V)
+        ops.retention_raw(proj.to(dev), q_off, k_off, v_off, silu, state, b, decay.to(dev), out, H, D, V, rounded=rounded)
         torch.cuda.synchronize()
         row = 0
         for i, n in enumerate(lens):
@@ -239,7 +242,7 @@ def test_recurrence_steps_slots_and_a_far_key(ops, H, D, V, silu):
         starts = [s + n for s, n in zip(starts, lens)]
     for i in range(3):
         err = float((torch.cat(got[i]) - want[i]).abs().max()) / float(want[i].abs().max())
-        assert err < 2e-5, f"request {i} off by {err:.3g}"
+        assert err < (1e-2 if rounded and silu else 2e-5), f"request {i} off by {err:.3g}"
     v4 = f(seqs[0][2][4, :V].double())                       # the far key's value is what the last output of head 0 holds
     last = torch.cat(got[0])[-1, :V]
     assert float(torch.dot(last, v4) / (last.norm() * v4.norm())) > 0.999

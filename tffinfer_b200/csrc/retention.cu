@@ -20,7 +20,11 @@
 //
 // The raw form (tff_retention_raw) is the recurrence alone: q, k and v are column blocks of float32 rows, optionally
 // with a silu applied where they are read, and the output is o itself in float32 (norms and gates are another kernel's
-// business).  Its decode kernel (steps of one token a request) streams the state through registers: a CTA per 32 value
+// business).  For engines that compute in bfloat16 its chunk form runs on the tensor cores (mma.sync): q, k and v, which
+// are projections behind an activation, are rounded to bfloat16; everything else stays 32-bit: the scores are float32
+// accumulators, and an operand that carries a decay or the state (the weighted scores, the values times decay^(n-1-j), the
+// chunk's start state) goes into its product as three bfloat16 terms whose sum is the float32 value to its last bits.
+// Its decode kernel (steps of one token a request) streams the state through registers: a CTA per 32 value
 // columns of a (head, request), four columns a thread, all rows of a thread asked for ahead of the arithmetic.
 #include "common.cuh"
 #include <type_traits>
@@ -509,6 +513,280 @@ retention_finish_kernel(RetParams p, int num_requests, const float* __restrict__
     }
 }
 
+// ------------------------------------------------------------------ chunk by chunk on the tensor cores (raw form)
+constexpr int MT = 256;                  // eight warps
+constexpr int SCOLS = 64, SST = SCOLS + 8;     // state columns a CTA of the finish kernel works on, and their row stride
+
+__host__ __device__ inline int pad16(int x) { return (x + 15) & ~15; }
+__device__ __forceinline__ uint32_t ret_smem(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
+__device__ __forceinline__ void ret_ldsm(uint32_t (&r)[4], const bf16* p) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(ret_smem(p)));
+}
+__device__ __forceinline__ void ret_ldsm_t(uint32_t (&r)[4], const bf16* p) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(ret_smem(p)));
+}
+__device__ __forceinline__ void ret_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ uint32_t pack_bf16(float a, float b) {
+    const __nv_bfloat162 v = __floats2bfloat162_rn(a, b);
+    return *reinterpret_cast<const uint32_t*>(&v);
+}
+// x and y as three bfloat16 terms each (a pair a register): 8 + 8 + 8 bits of significand
+__device__ __forceinline__ void split3(float x, float y, uint32_t& t1, uint32_t& t2, uint32_t& t3) {
+    const float x1 = __bfloat162float(__float2bfloat16_rn(x)), y1 = __bfloat162float(__float2bfloat16_rn(y));
+    const float xr = x - x1, yr = y - y1;
+    const float x2 = __bfloat162float(__float2bfloat16_rn(xr)), y2 = __bfloat162float(__float2bfloat16_rn(yr));
+    t1 = pack_bf16(x1, y1);
+    t2 = pack_bf16(x2, y2);
+    t3 = pack_bf16(xr - x2, yr - y2);
+}
+
+// C rows of ``width`` float32 columns (rows from n on and columns up to wP are zeros) -> bfloat16 rows of ``stride``
+__device__ __forceinline__ void load_rounded(bf16* dst, int stride, const float* __restrict__ src, int ld, int n, int width,
+                                             int wP, int silu) {
+    const int w4 = wP >> 2;
+    const bool vec = ((width | ld) & 3) == 0 && ((uintptr_t)src & 15) == 0;
+    for (int e = threadIdx.x; e < C * w4; e += MT) {
+        const int i = e / w4, c = (e % w4) << 2;
+        float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (i < n && c < width) {
+            const float* s = src + (size_t)i * ld + c;
+            if (vec) {
+                x = __ldcg(reinterpret_cast<const float4*>(s));
+            } else {
+                x.x = __ldcg(s);
+                if (c + 1 < width) x.y = __ldcg(s + 1);
+                if (c + 2 < width) x.z = __ldcg(s + 2);
+                if (c + 3 < width) x.w = __ldcg(s + 3);
+            }
+            x = ret_in4(x, silu);
+        }
+        uint2 v;
+        v.x = pack_bf16(x.x, x.y);
+        v.y = pack_bf16(x.z, x.w);
+        *reinterpret_cast<uint2*>(dst + i * stride + c) = v;
+    }
+}
+
+// local part of a chunk: acc (-> out [T, H*dv]) = mask(decay^(i-j) q_i . k_j) V and U = sum_j decay^(n-1-j) k_j v_j^T
+__global__ void __launch_bounds__(MT, 2)
+retention_local_mma_kernel(RetParams p, int num_requests, float* __restrict__ U) {
+    extern __shared__ __align__(16) unsigned char smraw[];
+    __shared__ float pw[C + 1];
+    pdl_launch_dependents();
+    const int h = blockIdx.y, d = p.d, dv = p.dv, dP = pad16(d), vP = pad16(dv), ks = dP + 8, vs = vP + 8;
+    bf16* Qs = (bf16*)smraw;             // [C][ks]
+    bf16* Ks = Qs + C * ks;              // [C][ks]
+    bf16* Vs = Ks + C * ks;              // [C][vs]
+    bf16* Ws = Vs + C * vs;              // [3][C][vs]: the values times decay^(n-1-j) in three terms
+    ChunkRef c;
+    const bool have = find_chunk(p, num_requests, blockIdx.x, c);
+    fill_powers(pw, p.decay[h]);
+    pdl_wait();
+    if (!have) return;
+    const int n = c.n, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    load_rounded(Qs, ks, p.q + (size_t)c.t * p.q_ld + (size_t)h * d, p.q_ld, n, d, dP, p.silu);
+    load_rounded(Ks, ks, p.k + (size_t)c.t * p.k_ld + (size_t)h * d, p.k_ld, n, d, dP, p.silu);
+    load_rounded(Vs, vs, p.vg + (size_t)c.t * p.ld + p.v_off + (size_t)h * dv, p.ld, n, dv, vP, p.silu);
+    __syncthreads();
+    for (int e = threadIdx.x; e < C * (vP >> 1); e += MT) {
+        const int j = e / (vP >> 1), cc = (e % (vP >> 1)) << 1;
+        const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(Vs + j * vs + cc));
+        const float w = j < n ? pw[n - 1 - j] : 0.f;
+        uint32_t t[3];
+        split3(v.x * w, v.y * w, t[0], t[1], t[2]);
+#pragma unroll
+        for (int s = 0; s < 3; ++s) *reinterpret_cast<uint32_t*>(Ws + ((size_t)s * C + j) * vs + cc) = t[s];
+    }
+    __syncthreads();
+    {   // a warp: 16 rows of the chunk (all their scores) and half of the value columns
+        const int rg = warp & 3, cg = warp >> 2;
+        float s[8][4];
+#pragma unroll
+        for (int t = 0; t < 8; ++t)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) s[t][e] = 0.f;
+        for (int kk = 0; kk < dP; kk += 16) {
+            uint32_t a[4], b[4];
+            ret_ldsm(a, Qs + (rg * 16 + (lane & 15)) * ks + kk + (lane >> 4) * 8);
+#pragma unroll
+            for (int t = 0; t < 4; ++t) {
+                if (t > rg) continue;                    // keys behind every row of the warp
+                ret_ldsm(b, Ks + (t * 16 + (lane & 7) + (lane >> 4) * 8) * ks + kk + ((lane >> 3) & 1) * 8);
+                ret_mma(s[2 * t], a, b[0], b[1]);
+                ret_mma(s[2 * t + 1], a, b[2], b[3]);
+            }
+        }
+        const int i0 = rg * 16 + (lane >> 2), i1 = i0 + 8;
+        uint32_t a3[4][3][4];                            // the weighted scores as A operands: [16 keys][term][register]
+#pragma unroll
+        for (int t = 0; t < 8; ++t) {
+            const int j = t * 8 + 2 * (lane & 3);
+            auto weigh = [&](float x, int i, int jj) { return jj <= i ? x * pw[i - jj] : 0.f; };
+            uint32_t (&r)[3][4] = a3[t >> 1];
+            const int hi = (t & 1) * 2;
+            split3(weigh(s[t][0], i0, j), weigh(s[t][1], i0, j + 1), r[0][hi], r[1][hi], r[2][hi]);
+            split3(weigh(s[t][2], i1, j), weigh(s[t][3], i1, j + 1), r[0][hi + 1], r[1][hi + 1], r[2][hi + 1]);
+        }
+        const int blocks = vP >> 4, half = (blocks + 1) >> 1;
+        const int b_lo = cg ? half : 0, b_hi = cg ? blocks : half;
+        float* orow = (float*)p.out + (size_t)c.t * p.H * dv + (size_t)h * dv;
+        for (int b0 = b_lo; b0 < b_hi; b0 += 4) {
+            float o[8][4];
+#pragma unroll
+            for (int t = 0; t < 8; ++t)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) o[t][e] = 0.f;
+#pragma unroll
+            for (int k2 = 0; k2 < 4; ++k2) {
+                if (k2 > rg) continue;
+#pragma unroll
+                for (int bb = 0; bb < 4; ++bb) {
+                    if (b0 + bb >= b_hi) continue;
+                    uint32_t b[4];
+                    ret_ldsm_t(b, Vs + (k2 * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * vs + (b0 + bb) * 16 + (lane >> 4) * 8);
+#pragma unroll
+                    for (int s3 = 2; s3 >= 0; --s3) {    // the small terms first
+                        ret_mma(o[2 * bb], a3[k2][s3], b[0], b[1]);
+                        ret_mma(o[2 * bb + 1], a3[k2][s3], b[2], b[3]);
+                    }
+                }
+            }
+#pragma unroll
+            for (int t = 0; t < 8; ++t) {
+                const int col = b0 * 16 + t * 8 + 2 * (lane & 3);
+                if (b0 + (t >> 1) >= b_hi) continue;
+#pragma unroll
+                for (int e = 0; e < 2; ++e)
+                    if (col + e < dv) {
+                        if (i0 < n) orow[(size_t)i0 * p.H * dv + col + e] = o[t][e];
+                        if (i1 < n) orow[(size_t)i1 * p.H * dv + col + e] = o[t][2 + e];
+                    }
+            }
+        }
+    }
+    // U: a warp takes 16 rows of the state at a time
+    float* Uc = U + ((size_t)blockIdx.x * p.H + h) * d * dv;
+    for (int m0 = warp * 16; m0 < dP; m0 += 128) {
+        for (int n0 = 0; n0 < vP; n0 += 128) {
+            float u[16][4];
+#pragma unroll
+            for (int t = 0; t < 16; ++t)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) u[t][e] = 0.f;
+            for (int k0 = 0; k0 < C && k0 < n; k0 += 16) {
+                uint32_t a[4];
+                ret_ldsm_t(a, Ks + (k0 + (lane & 7) + (lane >> 4) * 8) * ks + m0 + ((lane >> 3) & 1) * 8);
+#pragma unroll
+                for (int t = 0; t < 8; ++t) {
+                    if (n0 + t * 16 >= vP) continue;
+#pragma unroll
+                    for (int s3 = 2; s3 >= 0; --s3) {
+                        uint32_t b[4];
+                        ret_ldsm_t(b, Ws + ((size_t)s3 * C + k0 + (lane & 7) + ((lane >> 3) & 1) * 8) * vs + n0 + t * 16 + (lane >> 4) * 8);
+                        ret_mma(u[2 * t], a, b[0], b[1]);
+                        ret_mma(u[2 * t + 1], a, b[2], b[3]);
+                    }
+                }
+            }
+            const int r0 = m0 + (lane >> 2), r1 = r0 + 8;
+            const bool pairs = (dv & 1) == 0;
+#pragma unroll
+            for (int t = 0; t < 16; ++t) {
+                const int col = n0 + t * 8 + 2 * (lane & 3);
+                if (col >= dv) continue;
+                if (pairs) {
+                    if (r0 < d) *reinterpret_cast<float2*>(Uc + (size_t)r0 * dv + col) = make_float2(u[t][0], u[t][1]);
+                    if (r1 < d) *reinterpret_cast<float2*>(Uc + (size_t)r1 * dv + col) = make_float2(u[t][2], u[t][3]);
+                } else {
+#pragma unroll
+                    for (int e = 0; e < 2; ++e)
+                        if (col + e < dv) {
+                            if (r0 < d) Uc[(size_t)r0 * dv + col + e] = u[t][e];
+                            if (r1 < d) Uc[(size_t)r1 * dv + col + e] = u[t][2 + e];
+                        }
+                }
+            }
+        }
+    }
+}
+
+// out_i += decay^(i+1) S^T q_i for SCOLS value columns of a chunk, S the state it starts from (left in U by the scan)
+__global__ void __launch_bounds__(MT)
+retention_finish_mma_kernel(RetParams p, int num_requests, const float* __restrict__ U) {
+    extern __shared__ __align__(16) unsigned char smraw[];
+    __shared__ float pw[C + 1];
+    pdl_launch_dependents();
+    const int h = blockIdx.y, d = p.d, dv = p.dv, dP = pad16(d), ks = dP + 8, n0 = blockIdx.z * SCOLS;
+    bf16* Qs = (bf16*)smraw;             // [C][ks]
+    bf16* Ss = Qs + C * ks;              // [3][dP][SST]
+    ChunkRef c;
+    const bool have = find_chunk(p, num_requests, blockIdx.x, c);
+    fill_powers(pw, p.decay[h]);
+    pdl_wait();
+    if (!have || c.pos == 0) return;     // a sequence's first chunk starts from zeros: its local part is all of it
+    const int n = c.n, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    load_rounded(Qs, ks, p.q + (size_t)c.t * p.q_ld + (size_t)h * d, p.q_ld, n, d, dP, p.silu);
+    const float* Sc = U + ((size_t)blockIdx.x * p.H + h) * d * dv;
+    const bool vec = (dv & 3) == 0 && ((uintptr_t)U & 15) == 0;
+    for (int e = threadIdx.x; e < dP * (SCOLS / 4); e += MT) {
+        const int r = e / (SCOLS / 4), cc = (e % (SCOLS / 4)) << 2, col = n0 + cc;
+        float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (r < d && col < dv) {
+            const float* s = Sc + (size_t)r * dv + col;
+            if (vec) {
+                x = __ldcg(reinterpret_cast<const float4*>(s));
+            } else {
+                x.x = __ldcg(s);
+                if (col + 1 < dv) x.y = __ldcg(s + 1);
+                if (col + 2 < dv) x.z = __ldcg(s + 2);
+                if (col + 3 < dv) x.w = __ldcg(s + 3);
+            }
+        }
+        uint32_t t[3], v[3];
+        split3(x.x, x.y, t[0], t[1], t[2]);
+        split3(x.z, x.w, v[0], v[1], v[2]);
+#pragma unroll
+        for (int s3 = 0; s3 < 3; ++s3) *reinterpret_cast<uint2*>(Ss + ((size_t)s3 * dP + r) * SST + cc) = make_uint2(t[s3], v[s3]);
+    }
+    __syncthreads();
+    const int rg = warp & 3, cg = warp >> 2;             // 16 rows x 32 columns a warp
+    float o[4][4];
+#pragma unroll
+    for (int t = 0; t < 4; ++t)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) o[t][e] = 0.f;
+    for (int kk = 0; kk < dP; kk += 16) {
+        uint32_t a[4];
+        ret_ldsm(a, Qs + (rg * 16 + (lane & 15)) * ks + kk + (lane >> 4) * 8);
+#pragma unroll
+        for (int bb = 0; bb < 2; ++bb)
+#pragma unroll
+            for (int s3 = 2; s3 >= 0; --s3) {
+                uint32_t b[4];
+                ret_ldsm_t(b, Ss + ((size_t)s3 * dP + kk + (lane & 7) + ((lane >> 3) & 1) * 8) * SST + cg * 32 + bb * 16 + (lane >> 4) * 8);
+                ret_mma(o[2 * bb], a, b[0], b[1]);
+                ret_mma(o[2 * bb + 1], a, b[2], b[3]);
+            }
+    }
+    const int i0 = rg * 16 + (lane >> 2), i1 = i0 + 8;
+    float* orow = (float*)p.out + (size_t)c.t * p.H * dv + (size_t)h * dv;
+#pragma unroll
+    for (int t = 0; t < 4; ++t)
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+            const int col = n0 + cg * 32 + t * 8 + 2 * (lane & 3) + e;
+            if (col >= dv) continue;
+            if (i0 < n) { float* q = orow + (size_t)i0 * p.H * dv + col; *q = fmaf(pw[i0 + 1], o[t][e], __ldcg(q)); }
+            if (i1 < n) { float* q = orow + (size_t)i1 * p.H * dv + col; *q = fmaf(pw[i1 + 1], o[t][2 + e], __ldcg(q)); }
+        }
+}
+
 }  // namespace
 
 // Floats of workspace the chunked form needs for a step of ``num_tokens`` tokens in ``num_requests`` requests.
@@ -520,6 +798,15 @@ TFF_API long long tff_retention_workspace(int num_tokens, int num_requests, int 
 namespace {
 
 constexpr size_t MOST = 224 * 1024;        // dynamic shared memory a CTA may ask for here (the kernels have a little static on top)
+
+int launch_scan(const RetParams& p, int num_requests, float* U, cudaStream_t stream) {
+    const int d = p.d, dv = p.dv;
+    if ((d * dv) % 4 == 0 && ((uintptr_t)p.state & 15) == 0 && ((uintptr_t)U & 15) == 0)
+        return tff_launch_pdl(retention_scan_kernel<4>, dim3((d * dv / 4 + NT - 1) / NT, p.H, num_requests), dim3(NT), (size_t)0,
+                              stream, p, num_requests, U);
+    return tff_launch_pdl(retention_scan_kernel<1>, dim3((d * dv + NT - 1) / NT, p.H, num_requests), dim3(NT), (size_t)0,
+                          stream, p, num_requests, U);
+}
 
 // The three kernels of the chunked form; FIN the finish kernel of the form asked for.
 template <typename Fin>
@@ -537,14 +824,32 @@ int launch_chunked(const RetParams& p, int num_requests, float* workspace, int n
         return TFF_ERR_LAUNCH;
     int st = tff_launch_pdl(retention_local_kernel, dim3(chunks, H), dim3(NT), smem1, stream, p, num_requests, acc, U);
     if (st != TFF_OK) return st;
-    if ((d * dv) % 4 == 0 && ((uintptr_t)p.state & 15) == 0 && ((uintptr_t)U & 15) == 0)
-        st = tff_launch_pdl(retention_scan_kernel<4>, dim3((d * dv / 4 + NT - 1) / NT, H, num_requests), dim3(NT), (size_t)0,
-                            stream, p, num_requests, U);
-    else
-        st = tff_launch_pdl(retention_scan_kernel<1>, dim3((d * dv + NT - 1) / NT, H, num_requests), dim3(NT), (size_t)0,
-                            stream, p, num_requests, U);
+    st = launch_scan(p, num_requests, U, stream);
     if (st != TFF_OK) return st;
     return tff_launch_pdl(finish, dim3(chunks, H), dim3(NT), smem3, stream, p, num_requests, (const float*)acc, (const float*)U);
+}
+
+// The raw form on the tensor cores.
+int launch_chunked_mma(const RetParams& p, int num_requests, float* workspace, int num_tokens, cudaStream_t stream) {
+    if (!workspace || num_tokens <= 0) return TFF_ERR_BAD_ARGUMENT;
+    const int dP = pad16(p.d), vP = pad16(p.dv);
+    const size_t smem1 = sizeof(bf16) * ((size_t)2 * C * (dP + 8) + (size_t)4 * C * (vP + 8));
+    const size_t smem3 = sizeof(bf16) * ((size_t)C * (dP + 8) + (size_t)3 * dP * SST);
+    if (smem1 > MOST || smem3 > MOST) return TFF_ERR_UNSUPPORTED;
+    const int chunks = num_tokens / C + 2 * num_requests;
+    static bool configured = false;
+    if (!configured) {
+        if (cudaFuncSetAttribute(retention_local_mma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)MOST) != cudaSuccess ||
+            cudaFuncSetAttribute(retention_finish_mma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)MOST) != cudaSuccess)
+            return TFF_ERR_LAUNCH;
+        configured = true;
+    }
+    int st = tff_launch_pdl(retention_local_mma_kernel, dim3(chunks, p.H), dim3(MT), smem1, stream, p, num_requests, workspace);
+    if (st != TFF_OK) return st;
+    st = launch_scan(p, num_requests, workspace, stream);
+    if (st != TFF_OK) return st;
+    return tff_launch_pdl(retention_finish_mma_kernel, dim3(chunks, p.H, (p.dv + SCOLS - 1) / SCOLS), dim3(MT), smem3, stream, p,
+                          num_requests, (const float*)workspace);
 }
 
 }  // namespace
@@ -595,7 +900,8 @@ TFF_API int tff_retention(
 
 // The recurrence alone: q, k, v are column blocks of the float32 rows ``proj`` (leading dimension ld, first columns q_off,
 // k_off, v_off), passed through a silu when ``silu`` is set; out float32 [T, H*dv].  A request that brings position 0
-// starts from a zero state whatever its slot holds.  chunked as above.
+// starts from a zero state whatever its slot holds.  chunked as above; 2: chunk by chunk on the tensor cores, q, k and v
+// rounded to bfloat16 (the workspace is the same size).
 TFF_API int tff_retention_raw(
     const float* proj, int ld, int q_off, int k_off, int v_off, int silu, float* state, int num_slots, const int* q_start,
     const int* pos_start, const int* slots, const float* decay, float* out, int num_requests, int H, int d, int dv,
@@ -610,6 +916,7 @@ TFF_API int tff_retention_raw(
     p.v_off = v_off; p.g_off = 0; p.silu = silu;
     p.state = state; p.num_slots = num_slots; p.q_start = q_start; p.pos_start = pos_start; p.slots = slots;
     p.decay = decay; p.out = out; p.H = H; p.d = d; p.dv = dv; p.eps = 0.f;
+    if (chunked == 2) return launch_chunked_mma(p, num_requests, workspace, num_tokens, stream);
     if (chunked) return launch_chunked(p, num_requests, workspace, num_tokens, retention_finish_kernel<float, true>, stream);
     const bool vec = dv % 4 == 0 && ((uintptr_t)state & 15) == 0;
     const size_t smem = sizeof(float) * ((size_t)2 * d + 32 * 33);

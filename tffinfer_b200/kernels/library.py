@@ -714,15 +714,19 @@ class CudaKernels:
         proj = self.projection_buffer(T, w_in.shape[0], h.device, h.dtype)
         self.gemm(h, w_in, proj)
         o = torch.empty((T, H * dv), dtype=torch.float32, device=h.device)
-        self.retention_raw(proj, 0, H * d, 2 * H * d, True, state, batch, decay, o, H, d, dv)
+        self.retention_raw(proj, 0, H * d, 2 * H * d, True, state, batch, decay, o, H, d, dv,
+                           rounded=h.dtype == torch.bfloat16)
         self.gated_norm(o, H * dv, proj, 2 * H * d + H * dv, norm_w, eps, False, out, clear_cols=(0, proj.shape[1]),
                         last_reader=True, gate_act="sigmoid")
 
+    RETENTION_MMA = os.environ.get("TFFINFER_RETENTION_MMA", "1") != "0"   # 0: the chunk form as float32 FMAs
+
     def retention_raw(self, proj, q_off: int, k_off: int, v_off: int, silu: bool, state, batch, decay, out, H, d, dv,
-                      chunked: Optional[bool] = None) -> None:
+                      chunked: Optional[bool] = None, rounded: bool = False) -> None:
         """The recurrence S <- decay S + k v^T, o = S^T q per head over ``state`` [slots, H, d, dv] (float32) -> out
         float32 [T, H*dv]; q, k and v are columns q_off.., k_off.., v_off.. of the float32 rows ``proj``, passed through a
-        silu when ``silu``.  ``chunked`` as for ``retention``.  ``proj`` is left as it is."""
+        silu when ``silu``.  ``chunked`` as for ``retention``.  ``rounded``: q, k and v may be rounded to bfloat16, and the
+        chunk form runs on the tensor cores.  ``proj`` is left as it is."""
         self._need_cuda(proj, state, decay, out)
         T, ld = proj.shape
         assert proj.dtype == state.dtype == decay.dtype == out.dtype == torch.float32 and tuple(out.shape) == (T, H * dv)
@@ -730,7 +734,7 @@ class CudaKernels:
         if chunked is None:
             chunked = batch.max_q_len > 1
 
-        def run(ch: bool):
+        def run(ch: int):
             ws = None
             if ch:
                 self.lib.tff_retention_workspace.restype = ctypes.c_longlong
@@ -739,12 +743,14 @@ class CudaKernels:
             return self.lib.tff_retention_raw(
                 _ptr(proj), _c_int(ld), _c_int(q_off), _c_int(k_off), _c_int(v_off), _c_int(1 if silu else 0), _ptr(state),
                 _c_int(state.shape[0]), _ptr(batch.q_start), _ptr(batch.pos_start), _ptr(batch.slots), _ptr(decay), _ptr(out),
-                _c_int(batch.num_requests), _c_int(H), _c_int(d), _c_int(dv), _c_int(1 if ch else 0), _ptr(ws), _c_int(T),
+                _c_int(batch.num_requests), _c_int(H), _c_int(d), _c_int(dv), _c_int(ch), _ptr(ws), _c_int(T),
                 self._stream())
-        status = run(chunked)
-        if status == -2 and chunked:
-            chunked = False
-            status = run(False)                            # a head too large for the chunked form's shared memory
+        forms = ([2] if rounded and self.RETENTION_MMA else []) + [1, 0] if chunked else [0]
+        for form in forms:                                 # a head may be too large for a form's shared memory
+            status = run(form)
+            if status != -2:
+                break
+        chunked = form > 0
         self._check(status, "retention_raw")
         self.launches += 3 if chunked else 1
 
