@@ -88,7 +88,7 @@ def test_description_names_needs_and_schedule():
         assert names[n].shape == s, n
     assert not any(n in names for n in ("head", "l0.norm2", "l0.mix.dq", "l1.mlp.router", "l1.mlp.e5.up", "l2.mlp.up"))
     needs = model.cache_needs()
-    st = StateNeed((2, 10, 14), "float32")
+    st = StateNeed((2, 10, 14), "float32", self_starting=True)
     assert needs == [KVNeed(1, 24, 11, 1), st, KVNeed(1, 24, 1, 1), st, KVNeed(1, 24, 1, 1), st]   # every pass its own
     assert [(e.layer, e.add_embedding) for e in desc.schedule] == KadodraConfig.from_json_dict(sample_json()).runs()
     assert desc.logit_scale == 0.75 and desc.lm_head_name is None

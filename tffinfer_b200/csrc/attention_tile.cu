@@ -224,30 +224,43 @@ attention_tile_kernel(const TQ* __restrict__ q, const TC* __restrict__ cache, TQ
     }
 }
 
-// out[t, h] = out_scale * sum_s w_s o_s / sum_s w_s l_s with w_s = exp(m_s - max m): one warp per (token, head)
+// out[t, h] = out_scale * sum_s w_s o_s / sum_s w_s l_s with w_s = exp(m_s - max m): a block per (token, head), the
+// weights once by its first warp, then a thread a column with the shares' values asked for together
+constexpr int MERGE_THREADS = 128, MOST_SPLITS = 32;
+
 template <typename TQ>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(MERGE_THREADS)
 attention_tile_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, TQ* __restrict__ out,
-                            int out_ld, int out_off, long long rows, int nq, int dv, int splits, float out_scale) {
+                            int out_ld, int out_off, int nq, int dv, int splits, float out_scale) {
+    __shared__ float w_s[MOST_SPLITS];
     pdl_launch_dependents();
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const long long row = (long long)blockIdx.x * 4 + warp;
-    if (row >= rows) return;
+    const int lane = threadIdx.x & 31;
+    const long long row = blockIdx.x;
     pdl_wait();
-    const float* ml = part_ml + (size_t)row * splits * 2;
-    float M = -INFINITY;
-    for (int s = 0; s < splits; ++s) M = fmaxf(M, ml[2 * s]);
-    float L = 0.f;
-    for (int s = 0; s < splits; ++s) L += (ml[2 * s] == -INFINITY ? 0.f : expf(ml[2 * s] - M)) * ml[2 * s + 1];
-    const float inv = out_scale / L;
+    if (threadIdx.x < 32) {
+        const float* ml = part_ml + (size_t)row * splits * 2;
+        float m = -INFINITY, l = 0.f;
+        if (lane < splits) { m = __ldcg(ml + 2 * lane); l = __ldcg(ml + 2 * lane + 1); }
+        const float M = warp_max(m);
+        const float w = m == -INFINITY ? 0.f : expf(m - M);
+        const float L = warp_sum(w * l);
+        w_s[lane] = w * (out_scale / L);
+    }
+    __syncthreads();
     TQ* orow = out + (size_t)(row / nq) * out_ld + out_off + (size_t)(row % nq) * dv;
-    for (int c = lane; c < dv; c += 32) {
+    const float* po = part_o + (size_t)row * splits * dv;
+    for (int c = threadIdx.x; c < dv; c += MERGE_THREADS) {
         float acc = 0.f;
-        for (int s = 0; s < splits; ++s) {
-            const float w = ml[2 * s] == -INFINITY ? 0.f : expf(ml[2 * s] - M);
-            if (w != 0.f) acc = fmaf(w, part_o[((size_t)row * splits + s) * dv + c], acc);
+        for (int s0 = 0; s0 < splits; s0 += 8) {
+            float x[8];
+#pragma unroll
+            for (int u = 0; u < 8; ++u)              // a share whose weight is zero counts for nothing
+                x[u] = (s0 + u < splits && w_s[s0 + u] != 0.f) ? __ldcg(po + (size_t)(s0 + u) * dv + c) : 0.f;
+#pragma unroll
+            for (int u = 0; u < 8; ++u)
+                if (s0 + u < splits) acc = fmaf(w_s[s0 + u], x[u], acc);
         }
-        orow[c] = from_f32<TQ>(acc * inv);
+        orow[c] = from_f32<TQ>(acc);
     }
 }
 
@@ -270,8 +283,8 @@ int launch_tile(const void* q, const void* cache, void* out, const TileArgs& a, 
                                       (const TC*)cache, (TQ*)out, a);                                                \
         if (st != TFF_OK || a.splits == 1) return st;                                                                \
         const long long rows = (long long)num_tokens * a.nq;                                                         \
-        return tff_launch_pdl(attention_tile_merge_kernel<TQ>, dim3((unsigned)((rows + 3) / 4)), dim3(128), 0, stream, \
-                              (const float*)a.part_o, (const float*)a.part_ml, (TQ*)out, a.out_ld, a.out_off, rows,  \
+        return tff_launch_pdl(attention_tile_merge_kernel<TQ>, dim3((unsigned)rows), dim3(MERGE_THREADS), 0, stream, \
+                              (const float*)a.part_o, (const float*)a.part_ml, (TQ*)out, a.out_ld, a.out_off,  \
                               a.nq, a.dv, a.splits, a.out_scale);                                                    \
     } while (0)
     if (a.dv <= 64) TFF_TILE(4);
@@ -579,8 +592,8 @@ int launch_tile_mma(const void* q, const void* cache, void* out, const TileArgs&
                                       (const bf16*)cache, (bf16*)out, a, gm);                                        \
         if (st != TFF_OK || a.splits == 1) return st;                                                                \
         const long long rows = (long long)num_tokens * a.nq;                                                         \
-        return tff_launch_pdl(attention_tile_merge_kernel<bf16>, dim3((unsigned)((rows + 3) / 4)), dim3(128), 0, stream, \
-                              (const float*)a.part_o, (const float*)a.part_ml, (bf16*)out, a.out_ld, a.out_off, rows, \
+        return tff_launch_pdl(attention_tile_merge_kernel<bf16>, dim3((unsigned)rows), dim3(MERGE_THREADS), 0, stream, \
+                              (const float*)a.part_o, (const float*)a.part_ml, (bf16*)out, a.out_ld, a.out_off, \
                               a.nq, a.dv, a.splits, a.out_scale);                                                    \
     } while (0)
     if (nt == 2) TFF_TMMA(2);
@@ -622,7 +635,7 @@ TFF_API int tff_attention_tile(
     a.sink = sink;
     a.window = window; a.chunk = chunk; a.temp = temp; a.r1 = r1; a.r2 = r2; a.out_scale = out_scale;
     a.q_ld = q_ld; a.out_ld = out_ld; a.out_off = out_off;
-    if (splits < 1 || (splits > 1 && (!part_o || !part_ml))) return TFF_ERR_BAD_ARGUMENT;
+    if (splits < 1 || splits > MOST_SPLITS || (splits > 1 && (!part_o || !part_ml))) return TFF_ERR_BAD_ARGUMENT;
     a.splits = splits; a.part_o = part_o; a.part_ml = part_ml;
     a.k_dense = k_dense; a.v_dense = v_dense; a.k_ld = k_ld; a.v_ld = v_ld;
     if (k_dense) {                                   // the tensor-core form or nothing

@@ -19,6 +19,8 @@ __device__ __forceinline__ float norm_gate(float z, int act) {
     return (act == 0 ? z : 1.f) / (1.f + expf(-z));
 }
 
+constexpr int KEEP = 16;        // elements a thread keeps in registers
+
 template <typename TO, bool WIDE>
 __global__ void __launch_bounds__(256)
 gated_norm_kernel(const float* __restrict__ o, int width, int gs, float* __restrict__ gate, int g_ld, int g_off,
@@ -38,6 +40,33 @@ gated_norm_kernel(const float* __restrict__ o, int width, int gs, float* __restr
     if (!WIDE && g >= width / gs) return;
     const int c0 = g * gs;
     float ss = 0.f;
+    if (gs <= step * KEEP) {                     // the group's values and gates stay in registers, all loads in flight together
+        float u[KEEP], z[KEEP];
+#pragma unroll
+        for (int k = 0; k < KEEP; ++k) {
+            const int i = first + k * step;
+            u[k] = i < gs ? __ldcg(orow + c0 + i) : 0.f;
+            z[k] = i < gs ? __ldcg(grow + c0 + i) : 0.f;
+        }
+#pragma unroll
+        for (int k = 0; k < KEEP; ++k) {
+            if (first + k * step >= gs) continue;
+            z[k] = norm_gate(z[k], gate_act);
+            if (gate_first) u[k] *= z[k];
+            ss = fmaf(u[k], u[k], ss);
+        }
+        ss = WIDE ? block_sum<256>(ss, red) : warp_sum(ss);
+        const float inv = rsqrtf(ss / (float)gs + eps);
+#pragma unroll
+        for (int k = 0; k < KEEP; ++k) {
+            const int i = first + k * step, c = c0 + i;
+            if (i >= gs) continue;
+            if (g_off + c >= clear_lo && g_off + c < clear_hi) grow[c] = 0.f;
+            const float y = (u[k] * inv) * w[c % wlen];
+            dst[c] = from_f32<TO>((gate_first ? y : y * z[k]) * out_scale);
+        }
+        return;
+    }
     for (int c = c0 + first; c < c0 + gs; c += step) {
         float u = __ldcg(orow + c);
         if (gate_first) u *= norm_gate(__ldcg(grow + c), gate_act);

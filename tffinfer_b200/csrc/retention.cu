@@ -546,30 +546,41 @@ __device__ __forceinline__ void split3(float x, float y, uint32_t& t1, uint32_t&
     t3 = pack_bf16(xr - x2, yr - y2);
 }
 
+constexpr int LOADS = 8;
+
+// four neighbouring floats of which ``left`` (0 or less: none) are there, zeros for the rest
+__device__ __forceinline__ float4 load_four(const float* s, int left, bool vec) {
+    float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (left >= 4 && vec) return __ldcg(reinterpret_cast<const float4*>(s));
+    if (left > 0) x.x = __ldcg(s);
+    if (left > 1) x.y = __ldcg(s + 1);
+    if (left > 2) x.z = __ldcg(s + 2);
+    if (left > 3) x.w = __ldcg(s + 3);
+    return x;
+}
+
 // C rows of ``width`` float32 columns (rows from n on and columns up to wP are zeros) -> bfloat16 rows of ``stride``
 __device__ __forceinline__ void load_rounded(bf16* dst, int stride, const float* __restrict__ src, int ld, int n, int width,
                                              int wP, int silu) {
     const int w4 = wP >> 2;
     const bool vec = ((width | ld) & 3) == 0 && ((uintptr_t)src & 15) == 0;
-    for (int e = threadIdx.x; e < C * w4; e += MT) {
-        const int i = e / w4, c = (e % w4) << 2;
-        float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (i < n && c < width) {
-            const float* s = src + (size_t)i * ld + c;
-            if (vec) {
-                x = __ldcg(reinterpret_cast<const float4*>(s));
-            } else {
-                x.x = __ldcg(s);
-                if (c + 1 < width) x.y = __ldcg(s + 1);
-                if (c + 2 < width) x.z = __ldcg(s + 2);
-                if (c + 3 < width) x.w = __ldcg(s + 3);
-            }
-            x = ret_in4(x, silu);
+    for (int e0 = threadIdx.x; e0 < C * w4; e0 += MT * LOADS) {
+        float4 x[LOADS];                 // a thread's loads are in flight together
+#pragma unroll
+        for (int u = 0; u < LOADS; ++u) {
+            const int e = e0 + u * MT, i = e / w4, c = (e % w4) << 2;
+            x[u] = load_four(src + (size_t)i * ld + c, (i < n && c < width) ? width - c : 0, vec);
         }
-        uint2 v;
-        v.x = pack_bf16(x.x, x.y);
-        v.y = pack_bf16(x.z, x.w);
-        *reinterpret_cast<uint2*>(dst + i * stride + c) = v;
+#pragma unroll
+        for (int u = 0; u < LOADS; ++u) {
+            const int e = e0 + u * MT, i = e / w4, c = (e % w4) << 2;
+            if (e >= C * w4) continue;
+            x[u] = ret_in4(x[u], silu);  // (a silu of zero is zero)
+            uint2 v;
+            v.x = pack_bf16(x[u].x, x[u].y);
+            v.y = pack_bf16(x[u].z, x[u].w);
+            *reinterpret_cast<uint2*>(dst + i * stride + c) = v;
+        }
     }
 }
 
@@ -717,7 +728,7 @@ retention_local_mma_kernel(RetParams p, int num_requests, float* __restrict__ U)
 }
 
 // out_i += decay^(i+1) S^T q_i for SCOLS value columns of a chunk, S the state it starts from (left in U by the scan)
-__global__ void __launch_bounds__(MT)
+__global__ void __launch_bounds__(MT, 3)
 retention_finish_mma_kernel(RetParams p, int num_requests, const float* __restrict__ U) {
     extern __shared__ __align__(16) unsigned char smraw[];
     __shared__ float pw[C + 1];
@@ -734,33 +745,37 @@ retention_finish_mma_kernel(RetParams p, int num_requests, const float* __restri
     load_rounded(Qs, ks, p.q + (size_t)c.t * p.q_ld + (size_t)h * d, p.q_ld, n, d, dP, p.silu);
     const float* Sc = U + ((size_t)blockIdx.x * p.H + h) * d * dv;
     const bool vec = (dv & 3) == 0 && ((uintptr_t)U & 15) == 0;
-    for (int e = threadIdx.x; e < dP * (SCOLS / 4); e += MT) {
-        const int r = e / (SCOLS / 4), cc = (e % (SCOLS / 4)) << 2, col = n0 + cc;
-        float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (r < d && col < dv) {
-            const float* s = Sc + (size_t)r * dv + col;
-            if (vec) {
-                x = __ldcg(reinterpret_cast<const float4*>(s));
-            } else {
-                x.x = __ldcg(s);
-                if (col + 1 < dv) x.y = __ldcg(s + 1);
-                if (col + 2 < dv) x.z = __ldcg(s + 2);
-                if (col + 3 < dv) x.w = __ldcg(s + 3);
-            }
-        }
-        uint32_t t[3], v[3];
-        split3(x.x, x.y, t[0], t[1], t[2]);
-        split3(x.z, x.w, v[0], v[1], v[2]);
+    for (int e0 = threadIdx.x; e0 < dP * (SCOLS / 4); e0 += MT * LOADS) {
+        float4 x[LOADS];
 #pragma unroll
-        for (int s3 = 0; s3 < 3; ++s3) *reinterpret_cast<uint2*>(Ss + ((size_t)s3 * dP + r) * SST + cc) = make_uint2(t[s3], v[s3]);
+        for (int u = 0; u < LOADS; ++u) {
+            const int e = e0 + u * MT, r = e / (SCOLS / 4), col = n0 + ((e % (SCOLS / 4)) << 2);
+            x[u] = load_four(Sc + (size_t)r * dv + col, (r < d && col < dv) ? dv - col : 0, vec);
+        }
+#pragma unroll
+        for (int u = 0; u < LOADS; ++u) {
+            const int e = e0 + u * MT, r = e / (SCOLS / 4), cc = (e % (SCOLS / 4)) << 2;
+            if (r >= dP) continue;
+            uint32_t t[3], v[3];
+            split3(x[u].x, x[u].y, t[0], t[1], t[2]);
+            split3(x[u].z, x[u].w, v[0], v[1], v[2]);
+#pragma unroll
+            for (int s3 = 0; s3 < 3; ++s3) *reinterpret_cast<uint2*>(Ss + ((size_t)s3 * dP + r) * SST + cc) = make_uint2(t[s3], v[s3]);
+        }
     }
     __syncthreads();
     const int rg = warp & 3, cg = warp >> 2;             // 16 rows x 32 columns a warp
-    float o[4][4];
+    const int i0 = rg * 16 + (lane >> 2), i1 = i0 + 8;
+    float* orow = (float*)p.out + (size_t)c.t * p.H * dv + (size_t)h * dv;
+    float o[4][4], local[4][4];                          // (the local part is asked for ahead of the products)
 #pragma unroll
     for (int t = 0; t < 4; ++t)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) o[t][e] = 0.f;
+        for (int e = 0; e < 4; ++e) {
+            const int i = e < 2 ? i0 : i1, col = n0 + cg * 32 + t * 8 + 2 * (lane & 3) + (e & 1);
+            o[t][e] = 0.f;
+            local[t][e] = (i < n && col < dv) ? __ldcg(orow + (size_t)i * p.H * dv + col) : 0.f;
+        }
     for (int kk = 0; kk < dP; kk += 16) {
         uint32_t a[4];
         ret_ldsm(a, Qs + (rg * 16 + (lane & 15)) * ks + kk + (lane >> 4) * 8);
@@ -774,16 +789,12 @@ retention_finish_mma_kernel(RetParams p, int num_requests, const float* __restri
                 ret_mma(o[2 * bb + 1], a, b[2], b[3]);
             }
     }
-    const int i0 = rg * 16 + (lane >> 2), i1 = i0 + 8;
-    float* orow = (float*)p.out + (size_t)c.t * p.H * dv + (size_t)h * dv;
 #pragma unroll
     for (int t = 0; t < 4; ++t)
 #pragma unroll
-        for (int e = 0; e < 2; ++e) {
-            const int col = n0 + cg * 32 + t * 8 + 2 * (lane & 3) + e;
-            if (col >= dv) continue;
-            if (i0 < n) { float* q = orow + (size_t)i0 * p.H * dv + col; *q = fmaf(pw[i0 + 1], o[t][e], __ldcg(q)); }
-            if (i1 < n) { float* q = orow + (size_t)i1 * p.H * dv + col; *q = fmaf(pw[i1 + 1], o[t][2 + e], __ldcg(q)); }
+        for (int e = 0; e < 4; ++e) {
+            const int i = e < 2 ? i0 : i1, col = n0 + cg * 32 + t * 8 + 2 * (lane & 3) + (e & 1);
+            if (i < n && col < dv) orow[(size_t)i * p.H * dv + col] = fmaf(pw[i + 1], o[t][e], local[t][e]);
         }
 }
 

@@ -148,6 +148,7 @@ class ModelRunner:
         self.dummy_slot = self.ecfg.max_live_requests
         self.states = [torch.zeros((self.ecfg.max_live_requests + 1,) + tuple(s.shape),
                                    dtype=_STATE_DTYPES[s.dtype], device=self.device) for s in state_specs]
+        self._states_to_clear = [t for t, s in zip(self.states, state_specs) if not s.self_starting]
         self._graphs = {}
         self.last_h2d_bytes = 0
         self._graph_pool = None
@@ -308,7 +309,7 @@ class ModelRunner:
 
     def _forward(self, batch: StepBatch) -> torch.Tensor:
         try:
-            for state in self.states:       # requests that start (again) at position 0 start from zero state
+            for state in self._states_to_clear:       # requests that start (again) at position 0 start from zero state
                 self.ops.reset_state_slots(state, batch.slots, batch.pos_start)
             return self.model.forward(batch, self.ops, self.act_dtype, self.bindings, self.kv_caches,
                                       batch.block_tables, self.ecfg.page_size, self.states)

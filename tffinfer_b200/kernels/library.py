@@ -867,11 +867,14 @@ class CudaKernels:
         act = _c_int(code)
         clip = (_c_float(limit), _c_float(self.CLIPPED_SLOPE))
         ll = ctypes.c_longlong
-        if self.grouped_on_tensor_cores(a, b, K, lda, a_gs, ldb, b_gs, gated, N) and tile_rows in (0, self.grouped_tile_rows(True)):
+        if self.grouped_on_tensor_cores(a, b, K, lda, a_gs, ldb, b_gs, gated, N) and tile_rows in (
+                0, self.grouped_tile_rows(True), self.grouped_tile_rows(True, True)):
+            if not tile_rows:
+                tile_rows = self.grouped_tile_rows(True, M <= self.GROUPED_FEW_ROWS)
             status = self.lib.tff_gemm_grouped_mma(
                 _ptr(a), ll(lda), ll(a_gs), _ptr(b), ll(ldb), ll(b_gs), _ptr(c), _c_int(_dt(c)), ll(ldc), ll(c_gs),
                 _ptr(tg), _ptr(tr0), _ptr(tre), _ptr(nt), _c_int(max_tiles), _ptr(row_map), _ptr(a_rows), _c_int(groups), _c_int(M),
-                _c_int(2 * N if gated else N), _c_int(K), _c_int(1 if gated else 0), act, *clip, self._stream())
+                _c_int(2 * N if gated else N), _c_int(K), _c_int(1 if gated else 0), act, *clip, _c_int(tile_rows), self._stream())
             self._check(status, "gemm_grouped_mma")
             self.launches += 1
             return
@@ -894,8 +897,14 @@ class CudaKernels:
                 and all(v % 8 == 0 for v in (K, lda, a_gs, ldb, b_gs)) and a.data_ptr() % 16 == 0 and b.data_ptr() % 16 == 0
                 and (not gated or (gated == "interleaved" and N % self.GATE_UP_BLOCK == 0)))
 
-    def grouped_tile_rows(self, tensor_cores: bool) -> int:
-        return int(self.lib.tff_gemm_grouped_mma_tile_rows() if tensor_cores else self.lib.tff_gemm_grouped_tile_rows())
+    GROUPED_FEW_ROWS = 32    # up to this many rows a group the tensor-core kernel takes tiles of few rows
+
+    def grouped_tile_rows(self, tensor_cores: bool, few: bool = False) -> int:
+        """Rows of a tile of the grouped products: of the FMA kernel, or of the tensor-core kernel, which has tiles for
+        prompt-sized groups and for groups of ``few`` rows."""
+        if not tensor_cores:
+            return int(self.lib.tff_gemm_grouped_tile_rows())
+        return int(self.lib.tff_gemm_grouped_mma_tile_rows(_c_int(1 if few else 0)))
 
     GATE_UP_BLOCK = 64       # rows of a block of the "interleaved" gate/up layout (gate_up_block above: the same)
 
@@ -1113,12 +1122,13 @@ class CudaKernels:
                              identity=(pe[0], pair_weight, h) if pe else None)
             return
         a_rows = None
+        tile_rows = self.grouped_tile_rows(tc, P <= 12 * E)      # few pairs an expert on average: tiles of few rows
         if by_table:             # the product reads the tokens' rows where they are
-            pair_weight, row_map, tiles, a_rows = self.moe_table(router, T, top, E, self.grouped_tile_rows(tc))
+            pair_weight, row_map, tiles, a_rows = self.moe_table(router, T, top, E, tile_rows)
             x, pe = h, []
         else:
             pair_weight, row_map, tiles, x, *pe = self.moe_dispatch(h, w_router, top, renormalize, weight_on == "input",
-                                                                    self.grouped_tile_rows(tc), router=router)
+                                                                    tile_rows, router=router)
         act = torch.empty((P, ff), dtype=h.dtype, device=h.device)
         self.gemm_grouped(x, w_gate_up, act, E, 0, ff, W, W, 0, W, up_rows * W, ff, 0, gated="" if plain else layout,
                           activation=activation, tiles=tiles, a_rows=a_rows, limit=limit)

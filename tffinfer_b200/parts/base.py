@@ -46,6 +46,8 @@ class StateNeed:
     """A per-request state of fixed size (``shape`` elements of ``dtype`` per request)."""
     shape: Tuple[int, ...]
     dtype: str = "float32"
+    self_starting: bool = False      # the mixer's kernels start a request that brings position 0 from zeros whatever its
+                                     # slot holds: the runner need not clear it
 
 
 # --- run-time contexts ---------------------------------------------------------

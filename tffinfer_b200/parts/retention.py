@@ -112,7 +112,7 @@ class LightningAttention(Mixer):
         return ("retention", "gated_norm")
 
     def cache_need(self):
-        return StateNeed((self.num_heads, self.head_dim, self.v_head_dim), "float32")
+        return StateNeed((self.num_heads, self.head_dim, self.v_head_dim), "float32", self_starting=True)
 
     def weight_specs(self) -> Dict[str, WeightSpec]:
         n = self.names
