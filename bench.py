@@ -170,10 +170,12 @@ def decode_run(engine, batch: int, steps: int, warmup: int, seed: int, sampler=N
     launches = ops.launches - launches0
     ops.check_errors()
     h2d = engine.runner.last_h2d_bytes
+    # (the newest tokens have not been read back yet)
+    last_tokens = [engine.requests[i].generated[-min(4, len(engine.requests[i].generated))] for i in ids]
     for i in ids:                                   # stop the requests and give their pages back
         engine.abort(i)
     return {"tok_s": batch * steps / (dev_ms / 1e3), "ms_per_step": dev_ms / steps,
-            "e2e_tok_s": batch * steps / wall, "launches": launches, "mean_context": (ctx0 + ctx1) / 2,
+            "e2e_tok_s": batch * steps / wall, "launches": launches, "last_tokens": last_tokens, "mean_context": (ctx0 + ctx1) / 2,
             "h2d_bytes": h2d, "d2h_bytes": 4 * batch + 4,      # drawn tokens and the kernels' error word
             "p50_ms": per_step[len(per_step) // 2], "p99_ms": per_step[min(len(per_step) - 1, int(0.99 * len(per_step)))],
             "max_ms": per_step[-1]}
@@ -487,7 +489,7 @@ def traced_kinds(engine, prompt_len: int, batch: int):
     runner.step([StepEntry(rid, [1], [0]) for rid in ids])                   # and every decode-sized one
     torch.cuda.synchronize()
     with KernelTrace(runner.ops) as tr:
-        runner.step([StepEntry(rid, [2], [0]) for rid in ids])
+        runner.step([StepEntry(rid, [(7919 * i + 2) % vocab], [0]) for i, rid in enumerate(ids)])
     out["decode"] = {k: (c, round(ms, 4)) for k, c, ms in tr.summary()}
     for rid in ids:
         runner.finish_request(rid)
@@ -893,6 +895,15 @@ def kadodra_engine(size: str, max_live: int, cache_tokens: int, graphs: bool, st
     return tff.Engine(runner=runner), cfg
 
 
+def experts_of(engine, tokens):
+    """{"experts_touched": how many experts of a layer a step of these tokens reads, on average over the layers} where a
+    table of token ids chooses the experts; {} for other models."""
+    tables = [b.feed_forward.table for b in engine.runner.model.blocks if getattr(b.feed_forward, "table", None) is not None]
+    if not tables:
+        return {}
+    return {"experts_touched": round(sum(len(set(t[list(tokens)].flatten().tolist())) for t in tables) / len(tables), 1)}
+
+
 def run_kadodra(steps: int, warmup: int, sizes=None) -> int:
     """Prefill and decode throughput of the Kadodra design beside Nugosun at the same layer sizes, one JSON line a point,
     and for each model the device time of a step by kind of kernel call; for Kadodra also what its own kernels reach: the
@@ -918,8 +929,8 @@ def run_kadodra(steps: int, warmup: int, sizes=None) -> int:
                 run = decode_run(engine, b, steps, warmup, seed=b, prompt_len=P)
                 print(json.dumps({"point": "decode", "model": model, "size": size, "layers": TIPEZEN_LAYERS, "batch": b,
                                   "context": round(run["mean_context"]), "tok_s": round(run["tok_s"], 1),
-                                  "ms_per_step": round(run["ms_per_step"], 4), "launches_per_step": run["launches"] // steps}),
-                      flush=True)
+                                  "ms_per_step": round(run["ms_per_step"], 4), "launches_per_step": run["launches"] // steps,
+                                  **experts_of(engine, run["last_tokens"])}), flush=True)
             del engine
             torch.cuda.empty_cache()
             engine, cfg = make(size, 8, 8 * (P + 64), False, P)
@@ -962,9 +973,9 @@ def run_kadodra(steps: int, warmup: int, sizes=None) -> int:
                 if "attention_tile" in kd:
                     fr["decode_attention_tile_hbm_frac"] = round(nl * 8 * min(WIN, P) * (KR + R) * 2 / (kd["attention_tile"][1] / 1e3) / 1e9 / peaks["hbm_gbs"], 4)
                 if "gemm_grouped" in kd:          # the experts that 8 tokens of random ids touch, and the heads' projections
-                    touched = E * (1.0 - (1.0 - TOP / float(E)) ** 8)
+                    touched = experts_of(engine, [(7919 * i + 2) % TIPEZEN_VOCAB for i in range(8)])["experts_touched"]
                     w_b = nl * (touched * 3 * W * F * 2 + H * KR * (D + VD) * 2)
-                    fr["decode_experts_touched"] = round(touched, 1)
+                    fr["decode_experts_touched"] = touched
                     fr["decode_gemm_grouped_hbm_frac"] = round(w_b / (kd["gemm_grouped"][1] / 1e3) / 1e9 / peaks["hbm_gbs"], 4)
                 line["fractions"] = fr
             print(json.dumps(line), flush=True)
