@@ -955,10 +955,10 @@ def run_kadodra(steps: int, warmup: int, sizes=None) -> int:
                 if "retention_raw" in k:          # chunks of 64 tokens: A = Q K^T and A V, U = K^T V and Q S
                     flops = nl * LH * (P / 64.0) * 2.0 * 64 * (64 * LD + 64 * LV + 2 * LD * LV)
                     fr["prefill_retention_raw_fp32_tflops"] = round(flops / (k["retention_raw"][1] / 1e3) / 1e12, 2)
-                if "attention_tile" in k:
+                if "attention_dense" in k:
                     span = min(WIN, P)
                     pairs = span * (span + 1) / 2.0 + (P - span) * span
-                    fr["prefill_attention_tile_tflops"] = round(nl * H * pairs * 2.0 * (D + R + VD) / (k["attention_tile"][1] / 1e3) / 1e12, 2)
+                    fr["prefill_attention_dense_tflops"] = round(nl * H * pairs * 2.0 * (D + R + VD) / (k["attention_dense"][1] / 1e3) / 1e12, 2)
                 if "gemm_tc_grouped" in k:
                     fr["prefill_experts_tcgen05_tflops"] = round(nl * P * TOP * 3 * 2.0 * W * F / (k["gemm_tc_grouped"][1] / 1e3) / 1e12, 2)
                     fr["prefill_experts_tcgen05_frac"] = round(fr["prefill_experts_tcgen05_tflops"] / peaks["bf16_tflops"], 4)
