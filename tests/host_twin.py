@@ -198,10 +198,11 @@ class TwinCacheManager:
         for g in range(len(self.groups)):
             first = self._first_needed_block(g, rc.num_tokens)
             t = rc.tables[g]
-            gone = [t[b] for b in range(min(first, len(t))) if t[b] != NO_PAGE]
+            kept = -(-self.groups[g].keep_first // self.page_size)      # blocks that hold kept first tokens
+            gone = [t[b] for b in range(kept, min(first, len(t))) if t[b] != NO_PAGE]
             if gone:
                 self.pools[g].free(gone, req)
-                for b in range(min(first, len(t))):
+                for b in range(kept, min(first, len(t))):
                     t[b] = NO_PAGE
 
     def commit_step(self, reqs: Sequence[Hashable], counts: Sequence[int]) -> None:
@@ -257,7 +258,8 @@ class TwinCacheManager:
         for spec, pool in zip(self.groups, self.pools):
             most = length
             if spec.window > 0:
-                most = min(most, spec.window + budget_tokens + 2 * self.page_size)
+                kept = -(-spec.keep_first // self.page_size)
+                most = min(most, spec.window + budget_tokens + (kept + 2) * self.page_size)
             if most > pool.num_pages * self.page_size:
                 return False
         return True

@@ -30,7 +30,7 @@ def host_library():
     if _lib is None:
         lib = ctypes.CDLL(_build.host_library_path(build=True))
         lib.tffh_cache_create.restype = ctypes.c_void_p
-        lib.tffh_cache_create.argtypes = [ctypes.c_int, _i32p, ctypes.c_int, _i32p, ctypes.c_int]
+        lib.tffh_cache_create.argtypes = [ctypes.c_int, _i32p, _i32p, ctypes.c_int, _i32p, ctypes.c_int]
         lib.tffh_cache_destroy.argtypes = [ctypes.c_void_p]
         lib.tffh_cache_destroy.restype = None
         lib.tffh_last_error.argtypes = [ctypes.c_void_p]
@@ -115,8 +115,9 @@ class NativeCacheManager:
         self.groups = list(groups)
         self.page_size = int(page_size)
         windows = np.asarray([g.window for g in groups], dtype=np.int32)
+        keeps = np.asarray([g.keep_first for g in groups], dtype=np.int32)
         pages = np.asarray(list(pages_per_group), dtype=np.int32)
-        self._h = self.lib.tffh_cache_create(len(groups), _p32(windows), self.page_size, _p32(pages),
+        self._h = self.lib.tffh_cache_create(len(groups), _p32(windows), _p32(keeps), self.page_size, _p32(pages),
                                              int(max_live_requests))
         if not self._h:
             raise ValueError("the host runtime refused these cache sizes")

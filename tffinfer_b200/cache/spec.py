@@ -23,12 +23,14 @@ NO_PAGE = -1          # entry of a block table whose page was given back (a wind
 
 @dataclass(frozen=True)
 class GroupSpec:
-    """A group of schedule entries with one need.  ``window`` 0 = all keys are kept."""
+    """A group of schedule entries with one need.  ``window`` 0 = all keys are kept; beside a window, the pages of the
+    first ``keep_first`` tokens are kept too."""
     num_layers: int
     num_kv_heads: int
     head_dim: int
     window: int = 0
     planes: int = 2      # planes of a page: keys and values, or 1 for a cache of one vector per token
+    keep_first: int = 0
 
 
 class CacheAccountingError(RuntimeError):

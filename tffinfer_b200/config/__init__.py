@@ -5,4 +5,5 @@ from .dominex_config import DominexConfig, DominexLayer, DominexExperts
 from .sadupel_config import SadupelConfig, SadupelLayer, SadupelExperts
 from .nugosun_config import NugosunConfig, NugosunLayer, NugosunMlp
 from .kadodra_config import KadodraConfig, KadodraLayer, KadodraMlp
+from .gumodra_config import GumodraConfig, GumodraLayer, GumodraMlp
 from .engine_config import EngineConfig

@@ -66,6 +66,7 @@ struct AttnParams {
     bf16* out; float* part_o; float* part_ml; int num_splits;
     int nq, nkv; float scale_log2; int window;
     float scale_over_cap, cap_log2; int sink; const float* gate; const float* sink_val;   // AttnExtra, ready for the kernel
+    int keep;
 };
 
 template <int D, bool KEYS_MODE>
@@ -96,11 +97,10 @@ attn_fwd_kernel(const AttnParams p) {
     const int last_tok = min(q_len - 1, (tile * BLOCK_M + BLOCK_M - 1) / G);
     const int hi = pos0 + last_tok;
     const int lo_tile = p.window > 0 ? max(0, pos0 + first_tok - p.window + 1) : 0;
-    const int kb_lo = lo_tile / BLOCK_N, kb_hi = hi / BLOCK_N;
-    const int nblk = kb_hi - kb_lo + 1;
-    const int per = (nblk + p.num_splits - 1) / p.num_splits;
-    const int kb_begin = kb_lo + split * per;
-    const int kb_end = min(kb_hi + 1, kb_begin + per);           // may be <= kb_begin: an empty split
+    const KeyWalk walk(p.keep, BLOCK_N, lo_tile / BLOCK_N, hi / BLOCK_N);
+    const int per = (walk.count + p.num_splits - 1) / p.num_splits;
+    const int w_begin = split * per;                             // this split's share of the walk
+    const int w_end = min(walk.count, w_begin + per);            // may be <= w_begin: an empty split
     const int* table = p.block_table + (size_t)b * p.table_width;
     const bf16* cache_k = p.cache + (size_t)p.layer * p.L.layer_stride + (size_t)kvh * p.L.head_stride;
 
@@ -139,7 +139,7 @@ attn_fwd_kernel(const AttnParams p) {
         }
         cp_async16(smem_u32(sQ + swz<D>(row, chunk)), src, bytes);
     }
-    if (kb_begin < kb_end) load_kv(kb_begin, 0);
+    if (w_begin < w_end) load_kv(walk.block(w_begin), 0);
     cp_async_commit();
 
     // ------------------------------------------------------- per-thread rows
@@ -158,13 +158,13 @@ attn_fwd_kernel(const AttnParams p) {
     float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
     uint32_t qf[D / 16][4];
 
-    for (int blk = kb_begin; blk < kb_end; ++blk) {
-        const int stage = (blk - kb_begin) & 1;
-        if (blk + 1 < kb_end) load_kv(blk + 1, stage ^ 1);
+    for (int w = w_begin; w < w_end; ++w) {
+        const int blk = walk.block(w), stage = (w - w_begin) & 1;
+        if (w + 1 < w_end) load_kv(walk.block(w + 1), stage ^ 1);
         cp_async_commit();
         cp_async_wait<1>();
         __syncthreads();
-        if (blk == kb_begin) {
+        if (w == w_begin) {
             // query fragments once: matrices (rows 0-7 | 8-15) x (k 0-7 | 8-15)
 #pragma unroll
             for (int kk = 0; kk < D / 16; ++kk) {
@@ -201,7 +201,7 @@ attn_fwd_kernel(const AttnParams p) {
             for (int e = 0; e < 4; ++e) {
                 const int n = nbase + nt * 8 + (e & 1);
                 const bool up = e < 2;
-                const bool ok = up ? (v0 && n <= pr0 && n >= lo0) : (v1 && n <= pr1 && n >= lo1);
+                const bool ok = up ? (v0 && n <= pr0 && (n >= lo0 || n < p.keep)) : (v1 && n <= pr1 && (n >= lo1 || n < p.keep));
                 const float x = ok ? attn_score_log2(s[nt][e], p.scale_log2, p.scale_over_cap, p.cap_log2) : -INFINITY;
                 s[nt][e] = x;
                 if (up) bm0 = fmaxf(bm0, x); else bm1 = fmaxf(bm1, x);
@@ -429,7 +429,7 @@ static int attention_bf16_impl(
     void* out, void* workspace, int num_tokens, int num_requests, int max_q_len, int num_splits,
     int nq, int nkv, int d, float scale, int window, AttnExtra extra, cudaStream_t stream) {
     if (num_tokens <= 0 || num_requests <= 0) return TFF_OK;
-    if (extra.softcap < 0.f) return TFF_ERR_BAD_ARGUMENT;
+    if (extra.softcap < 0.f || extra.keep < 0) return TFF_ERR_BAD_ARGUMENT;
     if (nq <= 0 || nkv <= 0 || nq % nkv != 0 || page_size <= 0 || max_q_len <= 0 || num_splits < 1)
         return TFF_ERR_BAD_ARGUMENT;
     if (d != 64 && d != 128) return TFF_ERR_UNSUPPORTED;
@@ -452,6 +452,7 @@ static int attention_bf16_impl(
     p.scale_over_cap = extra.softcap > 0.f ? scale / extra.softcap : 0.f;
     p.cap_log2 = extra.softcap > 0.f ? extra.softcap * 1.4426950408889634f : 0.f;
     p.sink = extra.sink; p.gate = extra.gate; p.sink_val = extra.sink_val;
+    p.keep = window > 0 ? extra.keep : 0;
     const bool keys_mode = (long long)max_q_len * G <= 16;
     const int block_m = keys_mode ? 16 : 64;
     const int q_tiles = (max_q_len * G + block_m - 1) / block_m;
@@ -490,7 +491,7 @@ TFF_API int tff_attention_bf16(
     int nq, int nkv, int d, float scale, int window, cudaStream_t stream) {
     return attention_bf16_impl(q, q_start, pos_start, nullptr, block_table, table_width, cache, 0, cache_layers, layer,
                                page_size, out, workspace, num_tokens, num_requests, max_q_len, num_splits, nq, nkv, d,
-                               scale, window, AttnExtra{0.f, 0, nullptr, nullptr}, stream);
+                               scale, window, AttnExtra{0.f, 0, nullptr, nullptr, 0}, stream);
 }
 
 // The same with the number of pages of the cache tensor given, which lets decode-sized calls
@@ -504,18 +505,20 @@ TFF_API int tff_attention_bf16_paged(
     int nq, int nkv, int d, float scale, int window, cudaStream_t stream) {
     return attention_bf16_impl(q, q_start, pos_start, req_ids, block_table, table_width, cache, cache_pages, cache_layers,
                                layer, page_size, out, workspace, num_tokens, num_requests, max_q_len, num_splits, nq,
-                               nkv, d, scale, window, AttnExtra{0.f, 0, nullptr, nullptr}, stream);
+                               nkv, d, scale, window, AttnExtra{0.f, 0, nullptr, nullptr, 0}, stream);
 }
 
-// The same with a cap on the scores, a sink in the softmax and a multiplier per (token, head) (attention_common.h).
+// The same with a cap on the scores, a sink in the softmax, a multiplier per (token, head) and kept first positions beside
+// the window (attention_common.h).
 TFF_API int tff_attention_bf16_paged_ext(
     const void* q, const int* q_start, const int* pos_start, const int* req_ids, const int* block_table, int table_width,
     const void* cache, long long cache_pages, int cache_layers, int layer, int page_size,
     void* out, void* workspace, int num_tokens, int num_requests, int max_q_len, int num_splits,
-    int nq, int nkv, int d, float scale, int window, float softcap, int sink, const float* sink_val, const float* gate, cudaStream_t stream) {
+    int nq, int nkv, int d, float scale, int window, float softcap, int sink, const float* sink_val, const float* gate, int keep,
+    cudaStream_t stream) {
     return attention_bf16_impl(q, q_start, pos_start, req_ids, block_table, table_width, cache, cache_pages, cache_layers,
                                layer, page_size, out, workspace, num_tokens, num_requests, max_q_len, num_splits, nq,
-                               nkv, d, scale, window, AttnExtra{softcap, sink, gate, sink_val}, stream);
+                               nkv, d, scale, window, AttnExtra{softcap, sink, gate, sink_val, keep}, stream);
 }
 
 // ------------------------------------------------------- allocation-free variant

@@ -6,15 +6,31 @@
 //   softcap  > 0: a score s (after the scale) becomes softcap * tanh(s / softcap)
 //   sink     != 0: the softmax's denominator has one more term, a key that has no value; its score (not scaled, not
 //                 capped) is sink_val[head] (float32 [nq]) or, with sink_val null, 0
+//   keep     > 0, with a window: the first ``keep`` positions of the sequence stay visible however far the window has
+//                 moved on (a query at position p sees key n <= p if n > p - window or n < keep)
 //   gate     float32 [tokens, nq]: the output of head h of token t is multiplied by gate[t, h] (null: by 1)
 struct AttnExtra {
     float softcap;
     int sink;
     const float* gate;
     const float* sink_val;
+    int keep;
 };
 
 #ifdef __CUDACC__
+// The key blocks that a tile walks, in order: first the ``kept`` blocks from position 0 that hold kept positions and lie
+// ahead of the window's, then blocks lo, lo + 1, ... of the window.
+struct KeyWalk {
+    int kept, lo, count;
+    __device__ __forceinline__ KeyWalk(int keep, int block, int lo_block, int hi_block) {
+        kept = keep > 0 ? min((keep + block - 1) / block, lo_block) : 0;
+        lo = lo_block;
+        count = kept + hi_block - lo_block + 1;
+    }
+    __device__ __forceinline__ int block(int i) const { return i < kept ? i : lo + i - kept; }
+    // whether some key of the block (its last ones, or those ahead of the window) may be one that no row sees
+    __device__ __forceinline__ bool ragged(int i) const { return i == count - 1 || i == kept || i == kept - 1; }
+};
 // tanh from one exponential and one division: 1 - 2 / (1 + 2^(2 x log2 e)); absolute error near 1e-7, so that a
 // capped score keeps the accuracy of an uncapped one (tanh.approx is good to 5e-4 only, times the cap).
 __device__ __forceinline__ float attn_tanh(float x) {

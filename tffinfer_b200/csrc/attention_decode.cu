@@ -69,6 +69,7 @@ struct DecodeParams {
     bf16* out; float* part_o; float* part_ml; int num_splits;
     int nq, nkv; float scale_log2; int window;
     float scale_over_cap, cap_log2; int sink; const float* gate; const float* sink_val;   // AttnExtra, ready for the kernel
+    int keep;
     int* error_flag;
 };
 
@@ -129,11 +130,10 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tm_cache, const DecodePar
     const int pos0 = p.pos_start[b];
     const int hi = pos0 + q_len - 1;
     const int lo_tile = p.window > 0 ? max(0, pos0 - p.window + 1) : 0;
-    const int kb_lo = lo_tile / BLOCK_N, kb_hi = hi / BLOCK_N;
-    const int nblk = kb_hi - kb_lo + 1;
-    const int per = (nblk + p.num_splits - 1) / p.num_splits;
-    const int kb_begin = kb_lo + split * per;
-    const int kb_end = min(kb_hi + 1, kb_begin + per);             // may be <= kb_begin: an empty split
+    const KeyWalk walk(p.keep, BLOCK_N, lo_tile / BLOCK_N, hi / BLOCK_N);
+    const int per = (walk.count + p.num_splits - 1) / p.num_splits;
+    const int w_begin = split * per;                               // this split's share of the walk
+    const int w_end = min(walk.count, w_begin + per);              // may be <= w_begin: an empty split
     const int* table = p.block_table + (size_t)b * p.table_width;
 
     if (warp == 4) {
@@ -143,8 +143,8 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tm_cache, const DecodePar
         const uint32_t box_bytes = (uint32_t)(2 * D * 2) << p.page_shift;      // K and V of one page
         const int first_new_blk = pos0 / BLOCK_N;                  // key blocks from here on hold slots written just now
         bool waited = false;
-        for (int blk = kb_begin; blk < kb_end; ++blk) {
-            const int i = blk - kb_begin, s = i % NSTAGES;
+        for (int w = w_begin; w < w_end; ++w) {
+            const int blk = walk.block(w), i = w - w_begin, s = i % NSTAGES;
             const uint32_t round = i / NSTAGES;
             bool ok = true;
             if (!waited && (blk >= first_new_blk || round > 0)) { pdl_wait(); waited = true; }
@@ -201,21 +201,21 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tm_cache, const DecodePar
     for (int i = 0; i < D / 8; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
     float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
 
-    for (int blk = kb_begin; blk < kb_end; ++blk) {
-        const int i = blk - kb_begin, s = i % NSTAGES;
+    for (int w = w_begin; w < w_end; ++w) {
+        const int blk = walk.block(w), i = w - w_begin, s = i % NSTAGES;
         const uint32_t round = i / NSTAGES;
         if (!mbar_wait(full_bar(s), round & 1, abort_flag)) break;
         const uint32_t tS = base + s * STAGE_BYTES;
-        if (blk == kb_hi || blk == kb_lo) {
-            // This warp's value rows that no query row may see -- beyond the last key, or before
-            // the window -- are cleared: their page slots may hold anything, and pages that were
+        if (walk.ragged(w)) {
+            // This warp's value rows that no query row may see -- beyond the last key, or between the kept
+            // ones and the window -- are cleared: their page slots may hold anything, and pages that were
             // not fetched leave whatever shared memory held.  (Such key rows only produce scores
             // that the mask discards.)
             uint8_t* gS = gbase + s * STAGE_BYTES;
             for (int idx = lane; idx < 16 * CH; idx += 32) {
                 const int kr = key_off + idx / CH, c = idx % CH;
                 const int n = blk * BLOCK_N + kr;
-                if (n > hi || n < lo_tile)
+                if (n > hi || (n < lo_tile && n >= p.keep))
                     *reinterpret_cast<uint4*>(gS + kv_off<D>(kr, c, 1, p.page_shift)) = make_uint4(0u, 0u, 0u, 0u);
             }
             __syncwarp();
@@ -242,7 +242,7 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tm_cache, const DecodePar
             for (int e = 0; e < 4; ++e) {
                 const int n = nbase + nt * 8 + (e & 1);
                 const bool up = e < 2;
-                const bool ok = up ? (v0 && n <= pr0 && n >= lo0) : (v1 && n <= pr1 && n >= lo1);
+                const bool ok = up ? (v0 && n <= pr0 && (n >= lo0 || n < p.keep)) : (v1 && n <= pr1 && (n >= lo1 || n < p.keep));
                 const float x = ok ? attn_score_log2(sc[nt][e], p.scale_log2, p.scale_over_cap, p.cap_log2) : -INFINITY;
                 sc[nt][e] = x;
                 if (up) bm0 = fmaxf(bm0, x); else bm1 = fmaxf(bm1, x);
@@ -378,6 +378,7 @@ int tff_attention_decode_launch(
     p.scale_over_cap = extra.softcap > 0.f ? scale / extra.softcap : 0.f;
     p.cap_log2 = extra.softcap > 0.f ? extra.softcap * 1.4426950408889634f : 0.f;
     p.sink = extra.sink; p.gate = extra.gate; p.sink_val = extra.sink_val;
+    p.keep = window > 0 ? extra.keep : 0;
     p.error_flag = tff_device_error_flag();
     if (p.error_flag == nullptr) return TFF_ERR_LAUNCH;
     return d == 128 ? launch_decode<128>(tm, p, num_requests, stream) : launch_decode<64>(tm, p, num_requests, stream);

@@ -5,7 +5,7 @@
 //
 // For the token at position p of request b and query head h (kv head h / (nq/nkv),
 // src/kernel/cuda/paged_flash_attention.cu:891-892):
-//   s[n] = (q . k[n]) * scale for lo <= n <= p, lo = window ? max(0, p-window+1) : 0
+//   s[n] = (q . k[n]) * scale for lo <= n <= p, lo = window ? max(0, p-window+1) : 0; with ``keep`` > 0 also for n < keep
 //   s[n] = softcap * tanh(s[n] / softcap)                      when softcap > 0
 //   out  = sum_n softmax(s)[n] * v[n]
 // with the running-maximum ("online") softmax of the reference
@@ -16,6 +16,7 @@
 // scaled nor capped) is sink_val[h], or 0 when sink_val is null: weights exp(s[n]) / (exp(sink) + sum exp(s)).  With ``gate`` (float32 [tokens, nq]) the head's output is multiplied by
 // gate[t, h].  Keys have d elements and values dv; both lie in cache slots of dc >= max(d, dv) elements.
 #include "common.cuh"
+#include "attention_common.h"
 
 namespace {
 
@@ -29,7 +30,7 @@ attention_generic_kernel(const T* __restrict__ q_in, int row_stride,
                          const T* __restrict__ cache, KvLayout L, int layer,
                          T* __restrict__ out, int num_tokens, int nq, int nkv, int d, int dv,
                          float scale, int window, float softcap, int sink, const float* __restrict__ sink_val,
-                         const float* __restrict__ gate) {
+                         const float* __restrict__ gate, int keep) {
     extern __shared__ float smem[];            // WARPS * d floats: the warp's query row
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const long long item = (long long)blockIdx.x * WARPS + warp;
@@ -54,9 +55,10 @@ attention_generic_kernel(const T* __restrict__ q_in, int row_stride,
     float m = sink ? (sink_val ? sink_val[h] : 0.f) : -INFINITY, l = sink ? 1.f : 0.f;
     const float inv_cap = softcap > 0.f ? 1.f / softcap : 0.f;
 
-    for (int k0 = (lo / 32) * 32; k0 <= p; k0 += 32) {
-        const int n = k0 + lane;
-        const bool valid = n >= lo && n <= p;
+    const KeyWalk walk(keep, 32, lo / 32, p / 32);
+    for (int w = 0; w < walk.count; ++w) {
+        const int n = walk.block(w) * 32 + lane;
+        const bool valid = n <= p && (n >= lo || n < keep);
         float s = -INFINITY;
         const T* vbase = nullptr;
         if (valid) {
@@ -110,11 +112,12 @@ TFF_API int tff_attention_generic_ext(
     const int* positions, const int* tok_req, const int* block_table, int table_width,
     const void* cache, int cache_layers, int layer, int page_size,
     void* out, int num_tokens, int nq, int nkv, int d, int dv, int dc, float scale, int window,
-    float softcap, int sink, const float* sink_val, const float* gate, cudaStream_t stream) {
+    float softcap, int sink, const float* sink_val, const float* gate, int keep, cudaStream_t stream) {
     if (num_tokens <= 0) return TFF_OK;
-    if (nq <= 0 || nkv <= 0 || nq % nkv != 0 || d <= 0 || dv <= 0 || dc < d || dc < dv || page_size <= 0 || softcap < 0.f)
+    if (nq <= 0 || nkv <= 0 || nq % nkv != 0 || d <= 0 || dv <= 0 || dc < d || dc < dv || page_size <= 0 || softcap < 0.f || keep < 0)
         return TFF_ERR_BAD_ARGUMENT;
     if (d > 512 || dv > 512) return TFF_ERR_UNSUPPORTED;
+    if (window <= 0) keep = 0;
     const KvLayout L = make_kv_layout(cache_layers, nkv, page_size, dc);
     const long long items = (long long)num_tokens * nq;
     const unsigned blocks = (unsigned)((items + WARPS - 1) / WARPS);
@@ -122,11 +125,11 @@ TFF_API int tff_attention_generic_ext(
     if (is_bf16)
         attention_generic_kernel<bf16><<<blocks, WARPS * 32, smem, stream>>>(
             (const bf16*)qkv, row_stride, positions, tok_req, block_table, table_width,
-            (const bf16*)cache, L, layer, (bf16*)out, num_tokens, nq, nkv, d, dv, scale, window, softcap, sink, sink_val, gate);
+            (const bf16*)cache, L, layer, (bf16*)out, num_tokens, nq, nkv, d, dv, scale, window, softcap, sink, sink_val, gate, keep);
     else
         attention_generic_kernel<float><<<blocks, WARPS * 32, smem, stream>>>(
             (const float*)qkv, row_stride, positions, tok_req, block_table, table_width,
-            (const float*)cache, L, layer, (float*)out, num_tokens, nq, nkv, d, dv, scale, window, softcap, sink, sink_val, gate);
+            (const float*)cache, L, layer, (float*)out, num_tokens, nq, nkv, d, dv, scale, window, softcap, sink, sink_val, gate, keep);
     return tff_launch_status();
 }
 
@@ -137,5 +140,5 @@ TFF_API int tff_attention_generic(
     void* out, int num_tokens, int nq, int nkv, int d, float scale, int window, cudaStream_t stream) {
     return tff_attention_generic_ext(qkv, is_bf16, row_stride, positions, tok_req, block_table, table_width, cache,
                                      cache_layers, layer, page_size, out, num_tokens, nq, nkv, d, d, d, scale, window,
-                                     0.f, 0, nullptr, nullptr, stream);
+                                     0.f, 0, nullptr, nullptr, 0, stream);
 }

@@ -173,6 +173,7 @@ struct PrefillParams {
     bf16* out;
     int nq, nkv; float scale_log2; int window;
     float scale_over_cap, cap_log2; int sink; const float* gate; const float* sink_val;   // AttnExtra, ready for the kernel
+    int keep;
     int* error_flag;
     int d, dv;                           // elements of a query row and of an output row (DENSE; at most DK and DV)
     int k_halves, k_head;                // DENSE: 64-column halves of a key that come from tm_k, columns between its heads
@@ -276,8 +277,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_cache, const __gri
     const int last_tok = min(q_len - 1, (row0 + QT * BLOCK_M - 1) / G);
     const int hi = pos0 + last_tok;                               // last key any row of the CTA sees
     const int lo_cta = p.window > 0 ? max(0, pos0 + first_tok - p.window + 1) : 0;   // first key any row sees
-    const int kb_lo = lo_cta / BLOCK_N, kb_hi = hi / BLOCK_N;
-    const int nb = active ? kb_hi - kb_lo + 1 : 0;
+    const KeyWalk walk(p.keep, BLOCK_N, lo_cta / BLOCK_N, hi / BLOCK_N);
+    const int nb = active ? walk.count : 0;
     const int* table = DENSE ? nullptr : p.block_table + (size_t)b * p.table_width;
     // a stage is free again when the PV products of every tile that has rows have read it
     if (tid == 0) {
@@ -306,7 +307,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_cache, const __gri
                 // key n of the request is row q0 + n; rows beyond the request's are another's or zeros, and masked
                 if (lane == 0) mbar_expect_tx(kv_full(s), (uint32_t)STAGE_BYTES);
                 __syncwarp();
-                const int row = q0 + (kb_lo + i) * BLOCK_N;
+                const int row = q0 + walk.block(i) * BLOCK_N;
                 if (lane < KH) {
                     const uint32_t dst = base + s * STAGE_BYTES + lane * (BLOCK_N * 128);
                     if (lane < p.k_halves) tma_load_2d(dst, &tm_cache, kv_full(s), kvh * p.k_head + lane * 64, row);
@@ -317,7 +318,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_cache, const __gri
                 }
                 continue;
             }
-            const int n0 = (kb_lo + i) * BLOCK_N + (j << p.page_shift);
+            const int n0 = walk.block(i) * BLOCK_N + (j << p.page_shift);
             int page = -1;
             if (lane < nloads && n0 <= hi) page = table[n0 >> p.page_shift];
             const bool valid = page >= 0;
@@ -454,10 +455,10 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_cache, const __gri
 #endif
         for (int j = 0; j < nb_x && ok; ++j) {
             const int st = j % NSTAGES;
-            const int blk = kb_lo + j;
-            if (blk == kb_hi || blk == kb_lo) {
-                // value rows no query row of the CTA may see (beyond the last key, before the first window) are
-                // cleared, since page slots and unfetched shared memory may hold anything; the warps of both tiles
+            const int blk = walk.block(j);
+            if (walk.ragged(j)) {
+                // value rows no query row of the CTA may see (beyond the last key, between the kept ones and the first
+                // window) are cleared, since page slots and unfetched shared memory may hold anything; the warps of both tiles
                 // do it (the same zeros), so that each tile's products wait for its own warps only.
                 ok = mbar_wait_warp(kv_full(st), (j / NSTAGES) & 1, abort_flag);
                 if (!ok) break;
@@ -465,7 +466,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_cache, const __gri
                 for (int idx = tt; idx < BLOCK_N * CH; idx += 128) {
                     const int kr = idx / CH, c = idx % CH;
                     const int n = blk * BLOCK_N + kr;
-                    if (n > hi || n < lo_cta)
+                    if (n > hi || (n < lo_cta && n >= p.keep))
                         *reinterpret_cast<uint4*>(gV + (c >> 3) * (BLOCK_N * 128) + kr * 128 + (((c & 7) ^ (kr & 7)) << 4)) =
                             make_uint4(0u, 0u, 0u, 0u);
                 }
@@ -494,14 +495,14 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_cache, const __gri
             // (four running maxima and, below, four partial sums: chains of 16 dependent operations, not 64)
             float m4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
             const int n_first = blk * BLOCK_N;
-            if (__all_sync(0xffffffffu, rv && n_first + BLOCK_N - 1 <= pr && n_first >= lo_r)) {
+            if (__all_sync(0xffffffffu, rv && n_first + BLOCK_N - 1 <= pr && (n_first >= lo_r || n_first + BLOCK_N <= p.keep))) {
 #pragma unroll
                 for (int i = 0; i < BLOCK_N; i += 2) m4[(i >> 1) & 3] = fmax3(m4[(i >> 1) & 3], s[i], s[i + 1]);
             } else {
 #pragma unroll
                 for (int i = 0; i < BLOCK_N; ++i) {
                     const int n = n_first + i;
-                    const bool vis = rv && n <= pr && n >= lo_r;
+                    const bool vis = rv && n <= pr && (n >= lo_r || n < p.keep);
                     s[i] = vis ? s[i] : -INFINITY;
                     m4[i & 3] = fmaxf(m4[i & 3], s[i]);
                 }
@@ -702,6 +703,7 @@ int tff_attention_prefill_launch(
     p.scale_over_cap = extra.softcap > 0.f ? scale / extra.softcap : 0.f;
     p.cap_log2 = extra.softcap > 0.f ? extra.softcap * 1.4426950408889634f : 0.f;
     p.sink = extra.sink; p.gate = extra.gate; p.sink_val = extra.sink_val;
+    p.keep = window > 0 ? extra.keep : 0;
     p.error_flag = tff_device_error_flag();
     if (p.error_flag == nullptr) return TFF_ERR_LAUNCH;
     p.d = p.dv = d; p.k_halves = p.k_head = p.r_col = 0;

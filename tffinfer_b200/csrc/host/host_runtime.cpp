@@ -74,6 +74,7 @@ struct RequestCache {
 struct Cache {
     int page_size = 0;
     std::vector<int> windows;                // per group; 0 = all keys are kept
+    std::vector<int> keeps;                  // per group: so many first tokens stay behind whatever the window
     std::vector<Pool> pools;
     Pool slots;
     std::unordered_map<int64_t, RequestCache> requests;
@@ -90,6 +91,7 @@ struct Cache {
         if (w <= 0) return 0;
         return std::max(0, num_tokens - w + 1) / page_size;      // a query at p sees keys p-w+1 .. p
     }
+    int kept_blocks(int g) const { return (keeps[g] + page_size - 1) / page_size; }
     void pages_needed(const RequestCache& rc, int n_new, int* per_group) const {
         const int blocks = (rc.num_tokens + n_new + page_size - 1) / page_size;
         for (size_t g = 0; g < pools.size(); ++g)
@@ -101,14 +103,15 @@ Cache* as_cache(void* p) { return static_cast<Cache*>(p); }
 
 }  // namespace
 
-TFFH_API void* tffh_cache_create(int num_groups, const int* windows, int page_size, const int* pages_per_group,
-                                 int max_live_requests) {
+TFFH_API void* tffh_cache_create(int num_groups, const int* windows, const int* keeps, int page_size,
+                                 const int* pages_per_group, int max_live_requests) {
     if (num_groups < 0 || page_size <= 0 || max_live_requests <= 0) return nullptr;
     for (int g = 0; g < num_groups; ++g)
-        if (pages_per_group[g] <= 0) return nullptr;
+        if (pages_per_group[g] <= 0 || windows[g] < 0 || keeps[g] < 0) return nullptr;
     Cache* c = new Cache();
     c->page_size = page_size;
     c->windows.assign(windows, windows + num_groups);
+    c->keeps.assign(keeps, keeps + num_groups);
     c->pools.resize(num_groups);
     for (int g = 0; g < num_groups; ++g) c->pools[g].init(pages_per_group[g]);
     c->slots.init(max_live_requests);
@@ -185,11 +188,11 @@ TFFH_API int tffh_commit(void* cache, int64_t req, int n_new) {
                                                 " tokens committed beyond the " + std::to_string(rc->reserved_tokens) +
                                                 " reserved");
     rc->num_tokens += n_new;
-    // pages that the window of every later query has passed go back to their pool
+    // pages that the window of every later query has passed, and that hold none of the kept first tokens, go back
     for (size_t g = 0; g < c->pools.size(); ++g) {
         std::vector<int>& t = rc->tables[g];
         const int first = std::min(c->first_needed_block((int)g, rc->num_tokens), (int)t.size());
-        for (int b = 0; b < first; ++b) {
+        for (int b = c->kept_blocks((int)g); b < first; ++b) {
             if (t[b] == NO_PAGE) continue;
             if (!c->pools[g].give_back(t[b], req, c->error)) return TFFH_ERR_ACCOUNTING;
             t[b] = NO_PAGE;
@@ -408,13 +411,13 @@ TFFH_API int tffh_plan_step(void* cache, int budget_tokens, int max_model_len,
     };
     const char* too_many = "more events than the buffer given holds";
     // Whether a request of ``len`` tokens can ever run, alone: in a group that keeps all keys it holds pages for
-    // all of them; in a group that keeps a window, for the window and one step's tokens (whose pages are taken
-    // before those behind the window go back), with a page of slack at either ragged end.
+    // all of them; in a group that keeps a window, for the window, the kept first tokens and one step's tokens (whose
+    // pages are taken before those behind the window go back), with a page of slack at every ragged end.
     auto fits_alone = [&](int len) -> bool {
         for (int g = 0; g < G; ++g) {
             const int w = c->windows[g];
             int64_t most = len;
-            if (w > 0) most = std::min<int64_t>(most, (int64_t)w + budget_tokens + 2 * (int64_t)c->page_size);
+            if (w > 0) most = std::min<int64_t>(most, (int64_t)w + budget_tokens + ((int64_t)c->kept_blocks(g) + 2) * c->page_size);
             if (most > (int64_t)c->pools[g].total * c->page_size) return false;
         }
         return true;

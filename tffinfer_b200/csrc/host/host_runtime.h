@@ -30,8 +30,10 @@ enum {
 };
 
 // ---- cache manager
-TFFH_API void* tffh_cache_create(int num_groups, const int* windows, int page_size, const int* pages_per_group,
-                                 int max_live_requests);
+// windows[g]: tokens a query of the group's layers sees (0: all); keeps[g]: the first tokens of a sequence that stay
+// visible, and whose pages stay, beside a window
+TFFH_API void* tffh_cache_create(int num_groups, const int* windows, const int* keeps, int page_size,
+                                 const int* pages_per_group, int max_live_requests);
 TFFH_API void tffh_cache_destroy(void* cache);
 TFFH_API const char* tffh_last_error(void* cache);
 

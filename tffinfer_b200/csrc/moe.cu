@@ -29,7 +29,8 @@ template <typename TH, typename TW>
 __global__ void __launch_bounds__(ROUTE_THREADS)
 moe_route_kernel(const TH* __restrict__ h, const TW* __restrict__ w_router, const float* __restrict__ bias, int T, int W, int E,
                  int top, int renormalize, int softmax_scores, const float* __restrict__ correction, int groups, int keep, int num_real,
-                 int* __restrict__ pair_expert, float* __restrict__ pair_weight, int* __restrict__ counts) {
+                 int* __restrict__ pair_expert, float* __restrict__ pair_weight, int* __restrict__ counts,
+                 const TW* __restrict__ row_w, float* __restrict__ row_out) {
     // A block takes ROUTE_TOK tokens: the router's rows are read once for all of them (2,048 tokens re-read a 64 KB router
     // 2,048 times otherwise), every token keeps sums of its own, and behind the products warp i does token i's choice.
     extern __shared__ float sm[];              // per token W floats (its row) and 3 E: the scores, the choice scores, groups
@@ -65,9 +66,10 @@ moe_route_kernel(const TH* __restrict__ h, const TW* __restrict__ w_router, cons
     __syncthreads();
     // A warp an output; a lane takes eight neighbouring elements a load where the rows allow it (16-byte loads, several in
     // flight), else one.  Either way the order of a dot product's additions is fixed by W alone.
-    const bool wide = (W & 7) == 0 && ((size_t)w_router & 15) == 0;
-    for (int e = warp; e < E; e += ROUTE_THREADS / 32) {
-        const TW* wr = w_router + (size_t)e * W;
+    // (Index E is the row beside the router's, when there is one.)
+    const bool wide = (W & 7) == 0 && (((size_t)w_router | (size_t)row_w) & 15) == 0;
+    for (int e = warp; e < E + (row_w ? 1 : 0); e += ROUTE_THREADS / 32) {
+        const TW* wr = e < E ? w_router + (size_t)e * W : row_w;
         float acc[ROUTE_TOK];
 #pragma unroll
         for (int k = 0; k < ROUTE_TOK; ++k) acc[k] = 0.f;
@@ -103,6 +105,11 @@ moe_route_kernel(const TH* __restrict__ h, const TW* __restrict__ w_router, cons
         }
 #pragma unroll
         for (int k = 0; k < ROUTE_TOK; ++k) {
+            if (e == E) {
+                const float z = warp_sum(acc[k]);
+                if (lane == 0 && k < nt) row_out[t0 + k] = 1.0f / (1.0f + expf(-z));
+                continue;
+            }
             const float z = warp_sum(acc[k]) + (bias ? bias[e] : 0.f);
             if (lane == 0) scores[(size_t)k * 3 * E + e] = softmax_scores ? z : 1.0f / (1.0f + expf(-z));
         }
@@ -190,7 +197,7 @@ moe_route_kernel(const TH* __restrict__ h, const TW* __restrict__ w_router, cons
         return;
     }
     if (renormalize && lane == 0)
-        for (int k = 0; k < top; ++k) pair_weight[(size_t)t * top + k] /= total;
+        for (int k = 0; k < top; ++k) pair_weight[(size_t)t * top + k] /= total + 1e-20f;   // (all chosen scores may be zero)
 }
 
 // pad_rows > 0: every expert's rows start at a multiple of pad_rows (= tile_rows): the sorted order then consists of
@@ -337,7 +344,8 @@ template <typename TH>
 __global__ void __launch_bounds__(256)
 moe_combine_kernel(const float* __restrict__ y, int W, int top, const float* __restrict__ pair_weight,
                    int weight_on_output, const int* __restrict__ place_of_pair, float* __restrict__ residual,
-                   float* __restrict__ out, const int* __restrict__ pair_expert, const TH* __restrict__ h) {
+                   float* __restrict__ out, const int* __restrict__ pair_expert, const TH* __restrict__ h,
+                   float* __restrict__ shared, const float* __restrict__ shared_w, int clear_shared) {
     pdl_launch_dependents();
     pdl_wait();
     const int t = blockIdx.x;
@@ -354,6 +362,10 @@ moe_combine_kernel(const float* __restrict__ y, int W, int top, const float* __r
         acc = fmaf(w, __ldcg(y + (place_of_pair ? (size_t)__ldcg(place_of_pair + pair) : pair) * W + i), acc);
     }
     const size_t at = (size_t)t * W + i;
+    if (shared) {                                             // an expert that every token uses, times the token's weight
+        acc = fmaf(__ldcg(shared_w + t), __ldcg(shared + at), acc);
+        if (clear_shared) shared[at] = 0.f;
+    }
     out[at] = residual ? residual[at] + acc : acc;
 }
 
@@ -362,13 +374,14 @@ moe_combine_kernel(const float* __restrict__ y, int W, int top, const float* __r
 // E router outputs, of which the last E - num_real are identity experts (pair_expert -1).  softmax_scores: the scores are
 // softmax(z) over all E outputs instead of sigmoid(z); 2: the scores are the logits z, and the weights of the chosen are the
 // softmax over the chosen logits alone.  bias [E] float32 or null: added to the router's product.  correction [E] float32 or null: added to the scores for the
-// choice only.  groups > 1 with keep < groups: E / groups neighbours form a group, and only the ``keep`` groups whose best
+// choice only.  row_w [W] (the router's type) or null: one more row, row_out[t] = sigmoid(row_w . h[t]).  groups > 1 with keep < groups: E / groups neighbours form a group, and only the ``keep`` groups whose best
 // choice score is largest can be chosen from.
 TFF_API int tff_moe_route(const void* h, int h_dt, const void* w_router, int w_dt, const float* bias, int T, int W, int E, int top,
                           int renormalize, int softmax_scores, const float* correction, int groups, int keep,
-                          int num_real, int* pair_expert, float* pair_weight, int* counts, cudaStream_t stream) {
+                          int num_real, int* pair_expert, float* pair_weight, int* counts, const void* row_w, float* row_out,
+                          cudaStream_t stream) {
     if (T <= 0) return TFF_OK;
-    if (W <= 0 || E <= 0 || top <= 0 || top > E || !h || !w_router || num_real < 0 || num_real > E)
+    if (W <= 0 || E <= 0 || top <= 0 || top > E || !h || !w_router || num_real < 0 || num_real > E || (row_w && !row_out))
         return TFF_ERR_BAD_ARGUMENT;
     if (groups > 1 && (E % groups != 0 || keep <= 0 || keep > groups || top > keep * (E / groups))) return TFF_ERR_BAD_ARGUMENT;
     const size_t smem = (size_t)ROUTE_TOK * (W + 3 * E) * sizeof(float);
@@ -379,7 +392,7 @@ TFF_API int tff_moe_route(const void* h, int h_dt, const void* w_router, int w_d
             cudaFuncSetAttribute(moe_route_kernel<TH, TW>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);   \
         return tff_launch_pdl(moe_route_kernel<TH, TW>, dim3((T + ROUTE_TOK - 1) / ROUTE_TOK), dim3(ROUTE_THREADS), smem, stream, (const TH*)h, \
                               (const TW*)w_router, bias, T, W, E, top, renormalize, softmax_scores, correction, groups, keep, \
-                              num_real, pair_expert, pair_weight, counts);         \
+                              num_real, pair_expert, pair_weight, counts, (const TW*)row_w, row_out);         \
     } while (0)
     if (h_dt == 0 && w_dt == 0) TFF_ROUTE(float, float);
     if (h_dt == 0 && w_dt == 1) TFF_ROUTE(float, bf16);
@@ -437,16 +450,19 @@ TFF_API int tff_moe_gather(const void* h, int h_dt, int pairs, int W, int top, c
 }
 
 // pair_expert (null: every pair has a row in y) and h [T, W] (h_dt 0 float32, 1 bfloat16): pairs whose expert is -1 are
-// identity experts and add pair_weight * h[t]; pair_weight must then be given.
+// identity experts and add pair_weight * h[t]; pair_weight must then be given.  shared [T, W] and shared_w [T] (or null): the
+// rows of an expert that every token uses and their weights; clear_shared: the rows are set to zero behind the read.
 TFF_API int tff_moe_combine(const float* y, int T, int W, int top, const float* pair_weight, int weight_on_output,
                             const int* place_of_pair, float* residual, float* out, const int* pair_expert,
-                            const void* h, int h_dt, cudaStream_t stream) {
+                            const void* h, int h_dt, float* shared, const float* shared_w, int clear_shared,
+                            cudaStream_t stream) {
     if (T <= 0) return TFF_OK;
+    if (shared && !shared_w) return TFF_ERR_BAD_ARGUMENT;
     if (pair_expert && (!h || !pair_weight)) return TFF_ERR_BAD_ARGUMENT;
     dim3 grid(T, (W + 255) / 256);
     if (h_dt == 1)
         return tff_launch_pdl(moe_combine_kernel<bf16>, grid, dim3(256), 0, stream, y, W, top, pair_weight, weight_on_output,
-                              place_of_pair, residual, out, pair_expert, (const bf16*)h);
+                              place_of_pair, residual, out, pair_expert, (const bf16*)h, shared, shared_w, clear_shared);
     return tff_launch_pdl(moe_combine_kernel<float>, grid, dim3(256), 0, stream, y, W, top, pair_weight, weight_on_output,
-                          place_of_pair, residual, out, pair_expert, (const float*)h);
+                          place_of_pair, residual, out, pair_expert, (const float*)h, shared, shared_w, clear_shared);
 }

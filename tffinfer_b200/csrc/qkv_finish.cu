@@ -125,7 +125,123 @@ qkv_finish_kernel(TIN* __restrict__ proj, int clear_input, int ld, TQ* __restric
     }
 }
 
+// The form for attentions that norm their heads: row = [q (nq*d) | k (nkv*d) | v (nkv*dv)] of float32 accumulators, a warp per
+// (token, head), the head in registers, so that the row is read once and everything asked for together:
+//   u = row + bias;   q and k: u / rms(u) * norm weight (rms over the head's d elements with ``eps``, weights [d] shared by
+//   heads; null: no norm), then turned as above;   v: u of the value columns or, with ``v_is_k`` (no such columns), the key's u
+// Cosines and sines of the token are made once a block, ahead of the wait for the kernel before.
+constexpr int QF_WARPS = 8, QF_MOST_D = 512;
+
+template <typename TQ, int RJ>        // RJ: registers an element array takes, d <= 32 * RJ
+__global__ void __launch_bounds__(QF_WARPS * 32)
+qk_finish_kernel(float* __restrict__ proj, int clear_input, int ld, TQ* __restrict__ q_out, const float* __restrict__ qw,
+                 const float* __restrict__ kw, float eps, const float* __restrict__ bias, int v_is_k,
+                 const float* __restrict__ freq, int rot_dims, float magnitude, int interleaved,
+                 const int* __restrict__ positions, const int* __restrict__ tok_req, const int* __restrict__ block_table,
+                 int table_width, TQ* __restrict__ cache, KvLayout L, int layer, int dc, int nq, int nkv, int d, int dv) {
+    __shared__ float cs[QF_MOST_D / 2], sn[QF_MOST_D / 2];
+    constexpr int PJ = (RJ + 1) / 2;
+    pdl_launch_dependents();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int t = blockIdx.y, head = blockIdx.x * QF_WARPS + warp;
+    const int half = rot_dims >> 1, pos = positions[t];
+    for (int i = threadIdx.x; i < half; i += QF_WARPS * 32) {
+        float s, c;
+        sincosf((float)pos * freq[i], &s, &c);
+        sn[i] = s * magnitude; cs[i] = c * magnitude;
+    }
+    __syncthreads();
+    const bool is_q = head < nq, is_k = !is_q && head < nq + nkv;
+    TQ* slot = nullptr;                                           // the head's key slot (a value lies kv_stride further)
+    if (!is_q && head < nq + (v_is_k ? nkv : 2 * nkv)) {
+        const int page = block_table[(size_t)tok_req[t] * table_width + pos / L.page_size];
+        if (page >= 0)                                            // no page: the host never schedules this
+            slot = cache + (size_t)page * L.page_stride + (size_t)layer * L.layer_stride +
+                   (size_t)(is_k ? head - nq : head - nq - nkv) * L.head_stride + (size_t)(pos % L.page_size) * dc;
+    }
+    pdl_wait();
+    if (!is_q && !slot) return;
+    float* row = proj + (size_t)t * ld;
+    if (!is_q && !is_k) {                                         // a value head
+        const int col = (nq + nkv) * d + (head - nq - nkv) * dv;
+        for (int i = lane; i < dv; i += 32) {
+            const float v = __ldcg(row + col + i) + (bias ? bias[col + i] : 0.f);
+            if (clear_input) row[col + i] = 0.f;
+            slot[L.kv_stride + i] = from_f32<TQ>(v);
+        }
+        return;
+    }
+    float* src = row + (size_t)head * d;
+    const float* hb = bias ? bias + (size_t)head * d : nullptr;
+    const float* hw = is_q ? qw : kw;
+    float a[PJ], b[PJ], c[RJ];                                    // the turned pairs and the elements that pass
+    float ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < PJ; ++j) {
+        const int i = lane + 32 * j, ia = interleaved ? 2 * i : i, ib = interleaved ? 2 * i + 1 : i + half;
+        a[j] = i < half ? __ldcg(src + ia) + (hb ? hb[ia] : 0.f) : 0.f;
+        b[j] = i < half ? __ldcg(src + ib) + (hb ? hb[ib] : 0.f) : 0.f;
+    }
+#pragma unroll
+    for (int j = 0; j < RJ; ++j) {
+        const int i = 2 * half + lane + 32 * j;
+        c[j] = i < d ? __ldcg(src + i) + (hb ? hb[i] : 0.f) : 0.f;
+    }
+#pragma unroll
+    for (int j = 0; j < PJ; ++j) { ss = fmaf(a[j], a[j], ss); ss = fmaf(b[j], b[j], ss); }
+#pragma unroll
+    for (int j = 0; j < RJ; ++j) ss = fmaf(c[j], c[j], ss);
+    float rs = 1.f;
+    if (hw) rs = rsqrtf(warp_sum(ss) / (float)d + eps);
+    TQ* dst = is_q ? q_out + (size_t)t * nq * d + (size_t)head * d : slot;
+    TQ* val = !is_q && v_is_k ? slot + L.kv_stride : nullptr;
+#pragma unroll
+    for (int j = 0; j < PJ; ++j) {
+        const int i = lane + 32 * j, ia = interleaved ? 2 * i : i, ib = interleaved ? 2 * i + 1 : i + half;
+        if (i >= half) continue;
+        if (clear_input) { src[ia] = 0.f; src[ib] = 0.f; }
+        if (val) { val[ia] = from_f32<TQ>(a[j]); val[ib] = from_f32<TQ>(b[j]); }
+        const float u = hw ? a[j] * rs * hw[ia] : a[j], v = hw ? b[j] * rs * hw[ib] : b[j];
+        dst[ia] = from_f32<TQ>(u * cs[i] - v * sn[i]);
+        dst[ib] = from_f32<TQ>(v * cs[i] + u * sn[i]);
+    }
+#pragma unroll
+    for (int j = 0; j < RJ; ++j) {
+        const int i = 2 * half + lane + 32 * j;
+        if (i >= d) continue;
+        if (clear_input) src[i] = 0.f;
+        if (val) val[i] = from_f32<TQ>(c[j]);
+        dst[i] = from_f32<TQ>(hw ? c[j] * rs * hw[i] : c[j]);
+    }
+}
+
 }  // namespace
+
+// proj float32 [num_tokens, ld]; q_out and the cache have q_dt (0 float32, 1 bfloat16); qw, kw float32 [d] or both null;
+// bias float32 over the row's columns or null; v_is_k: the row has no value columns, dv = d.
+TFF_API int tff_qk_finish(
+    float* proj, int clear_input, int ld, void* q_out, int q_dt, const float* qw, const float* kw, float eps, const float* bias,
+    int v_is_k, const float* freq, int rot_dims, float magnitude, int interleaved, const int* positions, const int* tok_req,
+    const int* block_table, int table_width, void* cache, int cache_layers, int layer, int page_size, int dc,
+    int num_tokens, int nq, int nkv, int d, int dv, cudaStream_t stream) {
+    if (num_tokens <= 0) return TFF_OK;
+    if (!proj || !q_out || !cache || !block_table || !positions || !tok_req || nq <= 0 || nkv <= 0 || d <= 0 || dv <= 0 ||
+        rot_dims < 0 || rot_dims > d || (rot_dims & 1) || (rot_dims > 0 && !freq) || page_size <= 0 || dc < d || dc < dv ||
+        (v_is_k && dv != d) || (qw != nullptr) != (kw != nullptr) || (qw && !(eps > 0.f)))
+        return TFF_ERR_BAD_ARGUMENT;
+    if (d > QF_MOST_D || num_tokens > 65535) return TFF_ERR_UNSUPPORTED;
+    const KvLayout L = make_kv_layout(cache_layers, nkv, page_size, dc);
+    const int heads = nq + (v_is_k ? nkv : 2 * nkv);
+    const dim3 grid((heads + QF_WARPS - 1) / QF_WARPS, num_tokens);
+#define TFF_QF(TQ, RJ)                                                                                                \
+    return tff_launch_pdl(qk_finish_kernel<TQ, RJ>, grid, dim3(QF_WARPS * 32), 0, stream, proj, clear_input, ld, (TQ*)q_out, \
+                          qw, kw, eps, bias, v_is_k, freq, rot_dims, magnitude, interleaved, positions, tok_req,      \
+                          block_table, table_width, (TQ*)cache, L, layer, dc, nq, nkv, d, dv)
+    if (q_dt == 1) { if (d <= 128) TFF_QF(bf16, 4); TFF_QF(bf16, 16); }
+    if (d <= 128) TFF_QF(float, 4);
+    TFF_QF(float, 16);
+#undef TFF_QF
+}
 
 // in_dt, q_dt, cache_dt: 0 = float32, 1 = bfloat16.  bias: float32 [nq*d + nkv*d + nkv*dv] or null; unit_eps: 0 = no norm.  q_out has q_dt; the cache cache_dt; k_out and v_share are float32.
 TFF_API int tff_qkv_finish(

@@ -26,7 +26,7 @@
 // chunk's start state) goes into its product as three bfloat16 terms whose sum is the float32 value to its last bits.
 // Its decode kernel (steps of one token a request) streams the state through registers: a CTA per 32 value
 // columns of a (head, request), four columns a thread, all rows of a thread asked for ahead of the arithmetic.
-#include "common.cuh"
+#include "chunk_recurrence.cuh"
 #include <type_traits>
 
 namespace {
@@ -55,11 +55,6 @@ struct RetParams {
     const float* decay;                // [H] on the device
     void* out; int H, d, dv; float eps;
 };
-
-__device__ __forceinline__ float ret_in(float x, int silu) { return silu ? x / (1.0f + expf(-x)) : x; }
-__device__ __forceinline__ float4 ret_in4(float4 x, int silu) {
-    return make_float4(ret_in(x.x, silu), ret_in(x.y, silu), ret_in(x.z, silu), ret_in(x.w, silu));
-}
 
 // ------------------------------------------------------------------ token by token
 // IN_SMEM: the head's state fits shared memory beside the rest (else it is worked on where it lies)
@@ -217,28 +212,6 @@ retention_decode_kernel(RetParams p) {
 //   3. finish: o_i = acc_i + decay^(i+1) S^T q_i (S in blocks of 64 value columns), then the head's RMS norm and
 //              the gate -> out
 // The products are float32 FMAs on 4 x 4 register tiles out of shared memory (operands zero-padded to multiples of 4).
-constexpr int C = 64;
-
-__host__ __device__ inline int pad4(int x) { return (x + 3) & ~3; }
-
-// Which chunk is CTA ``index``: request b, first row t, tokens n, position of the first token; false beyond the last.
-struct ChunkRef { int b, t, n, pos; };
-__device__ inline bool find_chunk(const RetParams& p, int num_requests, int index, ChunkRef& c) {
-    for (int b = 0; b < num_requests; ++b) {
-        const int t0 = p.q_start[b], len = p.q_start[b + 1] - t0;
-        if (len <= 0) continue;
-        const int pos0 = p.pos_start[b];
-        const int first = pos0 / C, count = (pos0 + len - 1) / C - first + 1;
-        if (index < count) {
-            const int lo = max(pos0, (first + index) * C), hi = min(pos0 + len, (first + index + 1) * C);
-            c.b = b; c.pos = lo; c.t = t0 + (lo - pos0); c.n = hi - lo;
-            return true;
-        }
-        index -= count;
-    }
-    return false;
-}
-
 // out(m, n) = sum_k A[m][k] B[k][n] for m < M, n < N; K a multiple of 4; rows of A up to pad4(M) and columns of B up
 // to pad4(N) are readable.  Consecutive threads take consecutive column tiles.
 // ``lower``: 0 = nothing known; 1 = only outputs with n <= m are wanted (tiles above the diagonal are left out);
@@ -297,7 +270,7 @@ retention_local_kernel(RetParams p, int num_requests, float* __restrict__ acc, f
     float* sv = skT + dP * C;            // [C][vP]
     float* sA = sv + C * vP;             // [C][C]
     ChunkRef c;
-    const bool have = find_chunk(p, num_requests, blockIdx.x, c);
+    const bool have = find_chunk(p.q_start, p.pos_start, num_requests, blockIdx.x, c);
     fill_powers(pw, p.decay[h]);
     pdl_wait();
     if (!have) return;
@@ -399,7 +372,7 @@ retention_finish_kernel(RetParams p, int num_requests, const float* __restrict__
     float* sS = sq + C * dP;             // [dP][NB]
     float* so = sS + dP * NB;            // [C][vP]
     ChunkRef c;
-    const bool have = find_chunk(p, num_requests, blockIdx.x, c);
+    const bool have = find_chunk(p.q_start, p.pos_start, num_requests, blockIdx.x, c);
     fill_powers(pw, p.decay[h]);
     pdl_wait();
     if (!have) return;
@@ -514,75 +487,16 @@ retention_finish_kernel(RetParams p, int num_requests, const float* __restrict__
 }
 
 // ------------------------------------------------------------------ chunk by chunk on the tensor cores (raw form)
-constexpr int MT = 256;                  // eight warps
-constexpr int SCOLS = 64, SST = SCOLS + 8;     // state columns a CTA of the finish kernel works on, and their row stride
-
-__host__ __device__ inline int pad16(int x) { return (x + 15) & ~15; }
-__device__ __forceinline__ uint32_t ret_smem(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
-__device__ __forceinline__ void ret_ldsm(uint32_t (&r)[4], const bf16* p) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
-                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(ret_smem(p)));
-}
-__device__ __forceinline__ void ret_ldsm_t(uint32_t (&r)[4], const bf16* p) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
-                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(ret_smem(p)));
-}
-__device__ __forceinline__ void ret_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ uint32_t pack_bf16(float a, float b) {
-    const __nv_bfloat162 v = __floats2bfloat162_rn(a, b);
-    return *reinterpret_cast<const uint32_t*>(&v);
-}
-// x and y as three bfloat16 terms each (a pair a register): 8 + 8 + 8 bits of significand
-__device__ __forceinline__ void split3(float x, float y, uint32_t& t1, uint32_t& t2, uint32_t& t3) {
-    const float x1 = __bfloat162float(__float2bfloat16_rn(x)), y1 = __bfloat162float(__float2bfloat16_rn(y));
-    const float xr = x - x1, yr = y - y1;
-    const float x2 = __bfloat162float(__float2bfloat16_rn(xr)), y2 = __bfloat162float(__float2bfloat16_rn(yr));
-    t1 = pack_bf16(x1, y1);
-    t2 = pack_bf16(x2, y2);
-    t3 = pack_bf16(xr - x2, yr - y2);
-}
-
-constexpr int LOADS = 8;
-
-// four neighbouring floats of which ``left`` (0 or less: none) are there, zeros for the rest
-__device__ __forceinline__ float4 load_four(const float* s, int left, bool vec) {
-    float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (left >= 4 && vec) return __ldcg(reinterpret_cast<const float4*>(s));
-    if (left > 0) x.x = __ldcg(s);
-    if (left > 1) x.y = __ldcg(s + 1);
-    if (left > 2) x.z = __ldcg(s + 2);
-    if (left > 3) x.w = __ldcg(s + 3);
-    return x;
-}
-
-// C rows of ``width`` float32 columns (rows from n on and columns up to wP are zeros) -> bfloat16 rows of ``stride``
-__device__ __forceinline__ void load_rounded(bf16* dst, int stride, const float* __restrict__ src, int ld, int n, int width,
-                                             int wP, int silu) {
-    const int w4 = wP >> 2;
-    const bool vec = ((width | ld) & 3) == 0 && ((uintptr_t)src & 15) == 0;
-    for (int e0 = threadIdx.x; e0 < C * w4; e0 += MT * LOADS) {
-        float4 x[LOADS];                 // a thread's loads are in flight together
-#pragma unroll
-        for (int u = 0; u < LOADS; ++u) {
-            const int e = e0 + u * MT, i = e / w4, c = (e % w4) << 2;
-            x[u] = load_four(src + (size_t)i * ld + c, (i < n && c < width) ? width - c : 0, vec);
-        }
-#pragma unroll
-        for (int u = 0; u < LOADS; ++u) {
-            const int e = e0 + u * MT, i = e / w4, c = (e % w4) << 2;
-            if (e >= C * w4) continue;
-            x[u] = ret_in4(x[u], silu);  // (a silu of zero is zero)
-            uint2 v;
-            v.x = pack_bf16(x[u].x, x[u].y);
-            v.y = pack_bf16(x[u].z, x[u].w);
-            *reinterpret_cast<uint2*>(dst + i * stride + c) = v;
-        }
-    }
-}
+// q, k and v with a fixed decay per head: pair (i, j) weighs decay^(i-j), the end state decay^(n-1-j), the start state decay^(i+1).
+struct FixedDecay {
+    static constexpr bool SUMS = false;
+    const float* pw;                     // powers of the decay
+    int n;
+    __device__ __forceinline__ float pair(int i, int j) const { return pw[i - j]; }
+    __device__ __forceinline__ float tail(int j) const { return pw[n - 1 - j]; }
+    __device__ __forceinline__ void row_sum(int, float) const {}
+    __device__ __forceinline__ float join(int i, float dot, float local) const { return fmaf(pw[i + 1], dot, local); }
+};
 
 // local part of a chunk: acc (-> out [T, H*dv]) = mask(decay^(i-j) q_i . k_j) V and U = sum_j decay^(n-1-j) k_j v_j^T
 __global__ void __launch_bounds__(MT, 2)
@@ -590,141 +504,16 @@ retention_local_mma_kernel(RetParams p, int num_requests, float* __restrict__ U)
     extern __shared__ __align__(16) unsigned char smraw[];
     __shared__ float pw[C + 1];
     pdl_launch_dependents();
-    const int h = blockIdx.y, d = p.d, dv = p.dv, dP = pad16(d), vP = pad16(dv), ks = dP + 8, vs = vP + 8;
-    bf16* Qs = (bf16*)smraw;             // [C][ks]
-    bf16* Ks = Qs + C * ks;              // [C][ks]
-    bf16* Vs = Ks + C * ks;              // [C][vs]
-    bf16* Ws = Vs + C * vs;              // [3][C][vs]: the values times decay^(n-1-j) in three terms
+    const int h = blockIdx.y, d = p.d, dv = p.dv;
     ChunkRef c;
-    const bool have = find_chunk(p, num_requests, blockIdx.x, c);
+    const bool have = find_chunk(p.q_start, p.pos_start, num_requests, blockIdx.x, c);
     fill_powers(pw, p.decay[h]);
     pdl_wait();
     if (!have) return;
-    const int n = c.n, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    load_rounded(Qs, ks, p.q + (size_t)c.t * p.q_ld + (size_t)h * d, p.q_ld, n, d, dP, p.silu);
-    load_rounded(Ks, ks, p.k + (size_t)c.t * p.k_ld + (size_t)h * d, p.k_ld, n, d, dP, p.silu);
-    load_rounded(Vs, vs, p.vg + (size_t)c.t * p.ld + p.v_off + (size_t)h * dv, p.ld, n, dv, vP, p.silu);
-    __syncthreads();
-    for (int e = threadIdx.x; e < C * (vP >> 1); e += MT) {
-        const int j = e / (vP >> 1), cc = (e % (vP >> 1)) << 1;
-        const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(Vs + j * vs + cc));
-        const float w = j < n ? pw[n - 1 - j] : 0.f;
-        uint32_t t[3];
-        split3(v.x * w, v.y * w, t[0], t[1], t[2]);
-#pragma unroll
-        for (int s = 0; s < 3; ++s) *reinterpret_cast<uint32_t*>(Ws + ((size_t)s * C + j) * vs + cc) = t[s];
-    }
-    __syncthreads();
-    {   // a warp: 16 rows of the chunk (all their scores) and half of the value columns
-        const int rg = warp & 3, cg = warp >> 2;
-        float s[8][4];
-#pragma unroll
-        for (int t = 0; t < 8; ++t)
-#pragma unroll
-            for (int e = 0; e < 4; ++e) s[t][e] = 0.f;
-        for (int kk = 0; kk < dP; kk += 16) {
-            uint32_t a[4], b[4];
-            ret_ldsm(a, Qs + (rg * 16 + (lane & 15)) * ks + kk + (lane >> 4) * 8);
-#pragma unroll
-            for (int t = 0; t < 4; ++t) {
-                if (t > rg) continue;                    // keys behind every row of the warp
-                ret_ldsm(b, Ks + (t * 16 + (lane & 7) + (lane >> 4) * 8) * ks + kk + ((lane >> 3) & 1) * 8);
-                ret_mma(s[2 * t], a, b[0], b[1]);
-                ret_mma(s[2 * t + 1], a, b[2], b[3]);
-            }
-        }
-        const int i0 = rg * 16 + (lane >> 2), i1 = i0 + 8;
-        uint32_t a3[4][3][4];                            // the weighted scores as A operands: [16 keys][term][register]
-#pragma unroll
-        for (int t = 0; t < 8; ++t) {
-            const int j = t * 8 + 2 * (lane & 3);
-            auto weigh = [&](float x, int i, int jj) { return jj <= i ? x * pw[i - jj] : 0.f; };
-            uint32_t (&r)[3][4] = a3[t >> 1];
-            const int hi = (t & 1) * 2;
-            split3(weigh(s[t][0], i0, j), weigh(s[t][1], i0, j + 1), r[0][hi], r[1][hi], r[2][hi]);
-            split3(weigh(s[t][2], i1, j), weigh(s[t][3], i1, j + 1), r[0][hi + 1], r[1][hi + 1], r[2][hi + 1]);
-        }
-        const int blocks = vP >> 4, half = (blocks + 1) >> 1;
-        const int b_lo = cg ? half : 0, b_hi = cg ? blocks : half;
-        float* orow = (float*)p.out + (size_t)c.t * p.H * dv + (size_t)h * dv;
-        for (int b0 = b_lo; b0 < b_hi; b0 += 4) {
-            float o[8][4];
-#pragma unroll
-            for (int t = 0; t < 8; ++t)
-#pragma unroll
-                for (int e = 0; e < 4; ++e) o[t][e] = 0.f;
-#pragma unroll
-            for (int k2 = 0; k2 < 4; ++k2) {
-                if (k2 > rg) continue;
-#pragma unroll
-                for (int bb = 0; bb < 4; ++bb) {
-                    if (b0 + bb >= b_hi) continue;
-                    uint32_t b[4];
-                    ret_ldsm_t(b, Vs + (k2 * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * vs + (b0 + bb) * 16 + (lane >> 4) * 8);
-#pragma unroll
-                    for (int s3 = 2; s3 >= 0; --s3) {    // the small terms first
-                        ret_mma(o[2 * bb], a3[k2][s3], b[0], b[1]);
-                        ret_mma(o[2 * bb + 1], a3[k2][s3], b[2], b[3]);
-                    }
-                }
-            }
-#pragma unroll
-            for (int t = 0; t < 8; ++t) {
-                const int col = b0 * 16 + t * 8 + 2 * (lane & 3);
-                if (b0 + (t >> 1) >= b_hi) continue;
-#pragma unroll
-                for (int e = 0; e < 2; ++e)
-                    if (col + e < dv) {
-                        if (i0 < n) orow[(size_t)i0 * p.H * dv + col + e] = o[t][e];
-                        if (i1 < n) orow[(size_t)i1 * p.H * dv + col + e] = o[t][2 + e];
-                    }
-            }
-        }
-    }
-    // U: a warp takes 16 rows of the state at a time
-    float* Uc = U + ((size_t)blockIdx.x * p.H + h) * d * dv;
-    for (int m0 = warp * 16; m0 < dP; m0 += 128) {
-        for (int n0 = 0; n0 < vP; n0 += 128) {
-            float u[16][4];
-#pragma unroll
-            for (int t = 0; t < 16; ++t)
-#pragma unroll
-                for (int e = 0; e < 4; ++e) u[t][e] = 0.f;
-            for (int k0 = 0; k0 < C && k0 < n; k0 += 16) {
-                uint32_t a[4];
-                ret_ldsm_t(a, Ks + (k0 + (lane & 7) + (lane >> 4) * 8) * ks + m0 + ((lane >> 3) & 1) * 8);
-#pragma unroll
-                for (int t = 0; t < 8; ++t) {
-                    if (n0 + t * 16 >= vP) continue;
-#pragma unroll
-                    for (int s3 = 2; s3 >= 0; --s3) {
-                        uint32_t b[4];
-                        ret_ldsm_t(b, Ws + ((size_t)s3 * C + k0 + (lane & 7) + ((lane >> 3) & 1) * 8) * vs + n0 + t * 16 + (lane >> 4) * 8);
-                        ret_mma(u[2 * t], a, b[0], b[1]);
-                        ret_mma(u[2 * t + 1], a, b[2], b[3]);
-                    }
-                }
-            }
-            const int r0 = m0 + (lane >> 2), r1 = r0 + 8;
-            const bool pairs = (dv & 1) == 0;
-#pragma unroll
-            for (int t = 0; t < 16; ++t) {
-                const int col = n0 + t * 8 + 2 * (lane & 3);
-                if (col >= dv) continue;
-                if (pairs) {
-                    if (r0 < d) *reinterpret_cast<float2*>(Uc + (size_t)r0 * dv + col) = make_float2(u[t][0], u[t][1]);
-                    if (r1 < d) *reinterpret_cast<float2*>(Uc + (size_t)r1 * dv + col) = make_float2(u[t][2], u[t][3]);
-                } else {
-#pragma unroll
-                    for (int e = 0; e < 2; ++e)
-                        if (col + e < dv) {
-                            if (r0 < d) Uc[(size_t)r0 * dv + col + e] = u[t][e];
-                            if (r1 < d) Uc[(size_t)r1 * dv + col + e] = u[t][2 + e];
-                        }
-                }
-            }
-        }
-    }
+    chunk_local_mma(smraw, p.q + (size_t)c.t * p.q_ld + (size_t)h * d, p.q_ld, p.k + (size_t)c.t * p.k_ld + (size_t)h * d, p.k_ld,
+                    p.vg + (size_t)c.t * p.ld + p.v_off + (size_t)h * dv, p.ld, p.silu, c.n, d, dv, FixedDecay{pw, c.n},
+                    (float*)p.out + (size_t)c.t * p.H * dv + (size_t)h * dv, p.H * dv,
+                    U + ((size_t)blockIdx.x * p.H + h) * d * dv);
 }
 
 // out_i += decay^(i+1) S^T q_i for SCOLS value columns of a chunk, S the state it starts from (left in U by the scan)
@@ -733,69 +522,15 @@ retention_finish_mma_kernel(RetParams p, int num_requests, const float* __restri
     extern __shared__ __align__(16) unsigned char smraw[];
     __shared__ float pw[C + 1];
     pdl_launch_dependents();
-    const int h = blockIdx.y, d = p.d, dv = p.dv, dP = pad16(d), ks = dP + 8, n0 = blockIdx.z * SCOLS;
-    bf16* Qs = (bf16*)smraw;             // [C][ks]
-    bf16* Ss = Qs + C * ks;              // [3][dP][SST]
+    const int h = blockIdx.y, d = p.d, dv = p.dv, n0 = blockIdx.z * SCOLS;
     ChunkRef c;
-    const bool have = find_chunk(p, num_requests, blockIdx.x, c);
+    const bool have = find_chunk(p.q_start, p.pos_start, num_requests, blockIdx.x, c);
     fill_powers(pw, p.decay[h]);
     pdl_wait();
     if (!have || c.pos == 0) return;     // a sequence's first chunk starts from zeros: its local part is all of it
-    const int n = c.n, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    load_rounded(Qs, ks, p.q + (size_t)c.t * p.q_ld + (size_t)h * d, p.q_ld, n, d, dP, p.silu);
-    const float* Sc = U + ((size_t)blockIdx.x * p.H + h) * d * dv;
-    const bool vec = (dv & 3) == 0 && ((uintptr_t)U & 15) == 0;
-    for (int e0 = threadIdx.x; e0 < dP * (SCOLS / 4); e0 += MT * LOADS) {
-        float4 x[LOADS];
-#pragma unroll
-        for (int u = 0; u < LOADS; ++u) {
-            const int e = e0 + u * MT, r = e / (SCOLS / 4), col = n0 + ((e % (SCOLS / 4)) << 2);
-            x[u] = load_four(Sc + (size_t)r * dv + col, (r < d && col < dv) ? dv - col : 0, vec);
-        }
-#pragma unroll
-        for (int u = 0; u < LOADS; ++u) {
-            const int e = e0 + u * MT, r = e / (SCOLS / 4), cc = (e % (SCOLS / 4)) << 2;
-            if (r >= dP) continue;
-            uint32_t t[3], v[3];
-            split3(x[u].x, x[u].y, t[0], t[1], t[2]);
-            split3(x[u].z, x[u].w, v[0], v[1], v[2]);
-#pragma unroll
-            for (int s3 = 0; s3 < 3; ++s3) *reinterpret_cast<uint2*>(Ss + ((size_t)s3 * dP + r) * SST + cc) = make_uint2(t[s3], v[s3]);
-        }
-    }
-    __syncthreads();
-    const int rg = warp & 3, cg = warp >> 2;             // 16 rows x 32 columns a warp
-    const int i0 = rg * 16 + (lane >> 2), i1 = i0 + 8;
-    float* orow = (float*)p.out + (size_t)c.t * p.H * dv + (size_t)h * dv;
-    float o[4][4], local[4][4];                          // (the local part is asked for ahead of the products)
-#pragma unroll
-    for (int t = 0; t < 4; ++t)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-            const int i = e < 2 ? i0 : i1, col = n0 + cg * 32 + t * 8 + 2 * (lane & 3) + (e & 1);
-            o[t][e] = 0.f;
-            local[t][e] = (i < n && col < dv) ? __ldcg(orow + (size_t)i * p.H * dv + col) : 0.f;
-        }
-    for (int kk = 0; kk < dP; kk += 16) {
-        uint32_t a[4];
-        ret_ldsm(a, Qs + (rg * 16 + (lane & 15)) * ks + kk + (lane >> 4) * 8);
-#pragma unroll
-        for (int bb = 0; bb < 2; ++bb)
-#pragma unroll
-            for (int s3 = 2; s3 >= 0; --s3) {
-                uint32_t b[4];
-                ret_ldsm_t(b, Ss + ((size_t)s3 * dP + kk + (lane & 7) + ((lane >> 3) & 1) * 8) * SST + cg * 32 + bb * 16 + (lane >> 4) * 8);
-                ret_mma(o[2 * bb], a, b[0], b[1]);
-                ret_mma(o[2 * bb + 1], a, b[2], b[3]);
-            }
-    }
-#pragma unroll
-    for (int t = 0; t < 4; ++t)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-            const int i = e < 2 ? i0 : i1, col = n0 + cg * 32 + t * 8 + 2 * (lane & 3) + (e & 1);
-            if (i < n && col < dv) orow[(size_t)i * p.H * dv + col] = fmaf(pw[i + 1], o[t][e], local[t][e]);
-        }
+    chunk_finish_load(smraw, p.q + (size_t)c.t * p.q_ld + (size_t)h * d, p.q_ld, p.silu, c.n, d, dv, n0,
+                      U + ((size_t)blockIdx.x * p.H + h) * d * dv);
+    chunk_finish_mma(smraw, c.n, d, dv, n0, FixedDecay{pw, c.n}, (float*)p.out + (size_t)c.t * p.H * dv + (size_t)h * dv, p.H * dv);
 }
 
 }  // namespace
@@ -843,9 +578,7 @@ int launch_chunked(const RetParams& p, int num_requests, float* workspace, int n
 // The raw form on the tensor cores.
 int launch_chunked_mma(const RetParams& p, int num_requests, float* workspace, int num_tokens, cudaStream_t stream) {
     if (!workspace || num_tokens <= 0) return TFF_ERR_BAD_ARGUMENT;
-    const int dP = pad16(p.d), vP = pad16(p.dv);
-    const size_t smem1 = sizeof(bf16) * ((size_t)2 * C * (dP + 8) + (size_t)4 * C * (vP + 8));
-    const size_t smem3 = sizeof(bf16) * ((size_t)C * (dP + 8) + (size_t)3 * dP * SST);
+    const size_t smem1 = local_mma_smem(p.d, p.dv), smem3 = finish_mma_smem(p.d);
     if (smem1 > MOST || smem3 > MOST) return TFF_ERR_UNSUPPORTED;
     const int chunks = num_tokens / C + 2 * num_requests;
     static bool configured = false;

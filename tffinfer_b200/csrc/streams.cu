@@ -178,6 +178,98 @@ stream_step_kernel(float* __restrict__ x, int S, int W,
     }
 }
 
+// The join of a gated residual: what the sublayers of a layer gave, each times its gate, onto the residual, and the next
+// reader's norm.
+//   x[r] += (y1[r] + c1) * s(z[r, :W] + b[:W]) + y2[r] * s(z[r, W:] + b[W:]),   s the sigmoid (y2 null: no second term)
+//   h[r] = x[r] * rsqrt(mean(x[r]^2) + eps) * w                                 (h null: not wanted)
+// Everything in float32.  y1, y2 and z may be accumulator buffers, which are set to zero behind the read (bits 1, 2 and 4 of
+// ``clear``).  With row_index, CTA r works on row row_index[r], h is written to row r and x is left as it was.
+__device__ __forceinline__ float gate_of(float z) { return 1.0f / (1.0f + expf(-z)); }
+template <typename TZ> __device__ __forceinline__ float4 load_z4(const TZ* p);
+template <> __device__ __forceinline__ float4 load_z4<float>(const float* p) { return __ldcg(reinterpret_cast<const float4*>(p)); }
+template <> __device__ __forceinline__ float4 load_z4<bf16>(const bf16* p) {
+    const uint2 raw = __ldcg(reinterpret_cast<const uint2*>(p));
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+    return make_float4(a.x, a.y, b.x, b.y);
+}
+
+template <typename TO, typename TZ, int NT>
+__global__ void __launch_bounds__(NT)
+gated_join_kernel(float* __restrict__ x, int W, TZ* __restrict__ z, const float* __restrict__ b, float* __restrict__ y1,
+                  const float* __restrict__ c1, float* __restrict__ y2, int clear, const float* __restrict__ w, float eps,
+                  const int* __restrict__ row_index, TO* __restrict__ h) {
+    extern __shared__ __align__(16) float u_row[];   // W floats: the new row, kept between the two passes
+    __shared__ float red[32];
+    pdl_launch_dependents();
+    const int r = blockIdx.x, row = row_index ? row_index[r] : r;
+    const int zw = y2 ? 2 * W : W;
+    float* xr = x + (size_t)row * W;
+    float* y1r = y1 + (size_t)row * W;
+    float* y2r = y2 ? y2 + (size_t)row * W : nullptr;
+    TZ* zr = z + (size_t)row * zw;
+    const bool store_x = row_index == nullptr;
+    pdl_wait();
+    float ss = 0.f;
+    const bool vec = (W & 3) == 0 && (((uintptr_t)x | (uintptr_t)y1 | (uintptr_t)y2 | (uintptr_t)b | (uintptr_t)c1 | (uintptr_t)w) & 15) == 0 &&
+                     ((uintptr_t)z & (4 * sizeof(TZ) - 1)) == 0 && ((uintptr_t)h & (4 * sizeof(TO) - 1)) == 0;
+    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (vec) {
+        const int W4 = W >> 2;
+#pragma unroll 2
+        for (int i = threadIdx.x; i < W4; i += NT) {
+            float4 v = __ldcg(reinterpret_cast<const float4*>(xr) + i);
+            const float4 a = __ldcg(reinterpret_cast<const float4*>(y1r) + i);
+            const float4 za = load_z4<TZ>(zr + 4 * i);
+            const float4 ba = reinterpret_cast<const float4*>(b)[i];
+            const float4 ca = c1 ? reinterpret_cast<const float4*>(c1)[i] : zero;
+            if (y2r) {
+                const float4 f = __ldcg(reinterpret_cast<const float4*>(y2r) + i);
+                const float4 zf = load_z4<TZ>(zr + W + 4 * i);
+                const float4 bf = reinterpret_cast<const float4*>(b + W)[i];
+                v.x = fmaf(f.x, gate_of(zf.x + bf.x), v.x); v.y = fmaf(f.y, gate_of(zf.y + bf.y), v.y);
+                v.z = fmaf(f.z, gate_of(zf.z + bf.z), v.z); v.w = fmaf(f.w, gate_of(zf.w + bf.w), v.w);
+            }
+            v.x = fmaf(a.x + ca.x, gate_of(za.x + ba.x), v.x); v.y = fmaf(a.y + ca.y, gate_of(za.y + ba.y), v.y);
+            v.z = fmaf(a.z + ca.z, gate_of(za.z + ba.z), v.z); v.w = fmaf(a.w + ca.w, gate_of(za.w + ba.w), v.w);
+            if (store_x) reinterpret_cast<float4*>(xr)[i] = v;
+            if (clear & 1) reinterpret_cast<float4*>(y1r)[i] = zero;
+            if (clear & 2) reinterpret_cast<float4*>(y2r)[i] = zero;
+            if constexpr (sizeof(TZ) == 4)
+                if (clear & 4) {
+                    reinterpret_cast<float4*>(zr)[i] = zero;
+                    if (y2r) reinterpret_cast<float4*>(zr + W)[i] = zero;
+                }
+            reinterpret_cast<float4*>(u_row)[i] = v;
+            ss = fmaf(v.x, v.x, ss); ss = fmaf(v.y, v.y, ss); ss = fmaf(v.z, v.z, ss); ss = fmaf(v.w, v.w, ss);
+        }
+        if (!h) return;
+        ss = block_sum<NT>(ss, red);
+        const float rs = rsqrtf(ss / (float)W + eps);
+        for (int i = threadIdx.x; i < W4; i += NT) {  // a thread reads back what it wrote itself
+            const float4 u = reinterpret_cast<const float4*>(u_row)[i];
+            const float4 g = reinterpret_cast<const float4*>(w)[i];
+            store4<TO>(h + (size_t)r * W + 4 * i, (u.x * rs) * g.x, (u.y * rs) * g.y, (u.z * rs) * g.z, (u.w * rs) * g.w);
+        }
+        return;
+    }
+    for (int i = threadIdx.x; i < W; i += NT) {
+        float v = __ldcg(xr + i);
+        if (y2r) v = fmaf(__ldcg(y2r + i), gate_of(to_f32<TZ>(zr[W + i]) + b[W + i]), v);
+        v = fmaf(__ldcg(y1r + i) + (c1 ? c1[i] : 0.f), gate_of(to_f32<TZ>(zr[i]) + b[i]), v);
+        if (store_x) xr[i] = v;
+        if (clear & 1) y1r[i] = 0.f;
+        if (clear & 2) y2r[i] = 0.f;
+        if (clear & 4) { zr[i] = from_f32<TZ>(0.f); if (y2r) zr[W + i] = from_f32<TZ>(0.f); }
+        u_row[i] = v;
+        ss = fmaf(v, v, ss);
+    }
+    if (!h) return;
+    ss = block_sum<NT>(ss, red);
+    const float rs = rsqrtf(ss / (float)W + eps);
+    for (int i = threadIdx.x; i < W; i += NT) h[(size_t)r * W + i] = from_f32<TO>((u_row[i] * rs) * w[i]);
+}
+
 // out[t, c, :] = E[token[t], :] * scale for c < copies: the embedding output as the start of every stream.
 template <typename TW>
 __global__ void embed_streams_kernel(const int* __restrict__ tokens, const TW* __restrict__ table,
@@ -237,6 +329,34 @@ TFF_API int tff_stream_step(float* x, int S, int W, float* y, int clear_y, const
     TFF_STREAM_LAUNCH(float, 64);
 #undef TFF_STREAM_LAUNCH
 #undef TFF_STREAM_LAUNCH_S
+}
+
+// x [rows_total, W] float32, updated in place; z [rows_total, 2 W] (W without y2), z_is_bf16; b float32 of z's width; y1, y2
+// [rows_total, W] float32 (y2 may be null); c1 [W] or null; h [rows, W] or null, then w [W] may be null too.
+TFF_API int tff_gated_join(float* x, int W, void* z, int z_is_bf16, const float* b, float* y1, const float* c1, float* y2,
+                           int clear, const float* w, float eps, const int* row_index, void* h, int h_is_bf16, int rows,
+                           cudaStream_t stream) {
+    if (rows <= 0) return TFF_OK;
+    if (!x || !z || !b || !y1 || W <= 0 || (h && !w) || (row_index && clear) || ((clear & 4) && z_is_bf16) ||
+        ((clear & 2) && !y2))
+        return TFF_ERR_BAD_ARGUMENT;
+    const size_t smem = (size_t)W * sizeof(float);
+    if (smem > 96 * 1024) return TFF_ERR_UNSUPPORTED;
+#define TFF_JOIN(TO, TZ, NT)                                                                                        \
+    do {                                                                                                            \
+        auto kern = gated_join_kernel<TO, TZ, NT>;                                                                  \
+        if (smem > 48 * 1024 && cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 96 * 1024) != cudaSuccess) \
+            return TFF_ERR_LAUNCH;                                                                                  \
+        return tff_launch_pdl(kern, dim3(rows), dim3(NT), smem, stream, x, W, (TZ*)z, b, y1, c1, y2, clear, w, eps,  \
+                              row_index, (TO*)h);                                                                   \
+    } while (0)
+#define TFF_JOIN_N(TO, TZ)                                                                                          \
+    do { if (W >= 2048) TFF_JOIN(TO, TZ, 512); if (W >= 512) TFF_JOIN(TO, TZ, 128); TFF_JOIN(TO, TZ, 64); } while (0)
+    if (h_is_bf16) { if (z_is_bf16) TFF_JOIN_N(bf16, bf16); TFF_JOIN_N(bf16, float); }
+    if (z_is_bf16) TFF_JOIN_N(float, bf16);
+    TFF_JOIN_N(float, float);
+#undef TFF_JOIN_N
+#undef TFF_JOIN
 }
 
 TFF_API int tff_embed_streams(const int* tokens, const void* table, int table_is_bf16, float* out, int num_tokens,

@@ -10,6 +10,7 @@ sequence at a time and return logits of every row to the host.
 """
 from __future__ import annotations
 
+from dataclasses import replace
 from typing import Dict, Hashable, List, Optional, Sequence
 
 import torch
@@ -95,12 +96,12 @@ class ModelRunner:
             # a mixer may keep pages, a state, or both (a tuple): the binding carries a group and a state index
             for one in (need if isinstance(need, (tuple, list)) else (need,)):
                 if isinstance(one, KVNeed):
-                    key = (one.num_kv_heads, one.head_dim, one.window, one.planes)
+                    key = (one.num_kv_heads, one.head_dim, one.window, one.planes, one.keep_first)
                     for g, spec in enumerate(groups):
-                        if (spec.num_kv_heads, spec.head_dim, spec.window, spec.planes) == key:
+                        if (spec.num_kv_heads, spec.head_dim, spec.window, spec.planes, spec.keep_first) == key:
                             break
                     else:
-                        groups.append(GroupSpec(0, one.num_kv_heads, one.head_dim, one.window, one.planes))
+                        groups.append(GroupSpec(0, *key))
                         members.append([])
                         g = len(groups) - 1
                     self.bindings[e].group, self.bindings[e].layer_in_group, self.bindings[e].write = g, len(members[g]), True
@@ -117,7 +118,7 @@ class ModelRunner:
                 src = self.bindings[entry.cache_of]
                 self.bindings[e] = CacheBinding(group=src.group, layer_in_group=src.layer_in_group,
                                                 write=False, state_index=src.state_index)
-        groups = [GroupSpec(len(m), s.num_kv_heads, s.head_dim, s.window, s.planes) for s, m in zip(groups, members)]
+        groups = [replace(s, num_layers=len(m)) for s, m in zip(groups, members)]
         ps = self.ecfg.page_size
         elt = torch.empty((), dtype=self.act_dtype).element_size()
         page_bytes = [g.num_layers * g.planes * g.num_kv_heads * ps * g.head_dim * elt for g in groups]
@@ -164,7 +165,7 @@ class ModelRunner:
             # the reference logs the size of its cache the same way (src/core/runtime/InferRuntime.cu:109-140)
             log.info("cache group %d: %d layers, %d kv heads of %d, %s: %d pages of %d tokens (%.1f MiB), %s",
                      g, spec.num_layers, spec.num_kv_heads, spec.head_dim,
-                     f"window {spec.window}" if spec.window else "all keys", n, ps, n * pb / 2 ** 20, self.ecfg.dtype)
+                     f"window {spec.window}" + (f" and the first {spec.keep_first}" if spec.keep_first else "") if spec.window else "all keys", n, ps, n * pb / 2 ** 20, self.ecfg.dtype)
         if self.states:
             log.info("%d state tensors of %d slots", len(self.states), self.ecfg.max_live_requests)
 

@@ -61,6 +61,12 @@ def effective_requests(kv_lens) -> float:
     return float(kv.sum() / kv.max())
 
 
+def mlstm_state_size(H: int, K: int, V: int) -> int:
+    """float32 elements a request's mLSTM state takes in its slot: the heads' S [H, K, V], their n [H, K], their m [H],
+    rounded up to whole groups of four (csrc/mlstm.cu)."""
+    return -(-(H * K * V + H * K + H) // 4) * 4
+
+
 def nearest_power_of_two(x: float) -> int:
     b = 1
     while b * 1.4142 < x:
@@ -400,11 +406,46 @@ class CudaKernels:
             self._acc_zero[buf.data_ptr()] = True
         return buf
 
-    def sublayer_output(self, rows: int, width: int, device, act_dtype) -> torch.Tensor:
+    def sublayer_output(self, rows: int, width: int, device, act_dtype, use: str = "") -> torch.Tensor:
         """A float32 [rows, width] buffer for a sublayer's output that a connector consumes (``stream_step`` clears it
         behind the read): for decode-sized bfloat16 steps one of the accumulator buffers, so that the split product
-        that writes it needs no clearing kernel; else plain scratch."""
-        return self.projection_buffer(rows, width, device, act_dtype)
+        that writes it needs no clearing kernel; else plain scratch.  Outputs that wait side by side have a ``use`` each."""
+        return self.projection_buffer(rows, width, device, act_dtype, use)
+
+    def gate_rows(self, rows: int, width: int, device, act_dtype) -> torch.Tensor:
+        """A [rows, width] buffer for the gates of a gated residual, which ``gated_join`` reads (and clears): float32
+        accumulators in decode-sized steps, the activation type above."""
+        if act_dtype == torch.bfloat16 and rows > self.SWAP_MAX_M:
+            return torch.empty((rows, width), dtype=act_dtype, device=device)
+        return self.projection_buffer(rows, width, device, act_dtype, use="residual gates")
+
+    def gated_join(self, x, gates, gate_bias, y1, y1_bias=None, y2=None, norm_weight=None, eps: float = 0.0, h=None,
+                   row_index=None) -> None:
+        """x float32 [T, W] += (y1 + y1_bias) * sigmoid(gates[:, :W] + b) + y2 * sigmoid(gates[:, W:] + b') in place, and,
+        with ``h`` ([rows, W], activation type), h = rmsnorm(x) with ``norm_weight`` and ``eps``.  ``gates`` [T, W or 2W]
+        float32 or bfloat16, ``gate_bias`` float32 of its width; y1, y2 float32 [T, W].  ``row_index`` (int32 [rows]): only
+        those rows feed h, and x stays as it was.  Accumulator buffers that are kept at zero are cleared behind the read."""
+        self._need_cuda(x, gates, gate_bias, y1, y1_bias, y2, norm_weight, h, row_index)
+        T, W = x.shape
+        width = 2 * W if y2 is not None else W
+        assert x.dtype == y1.dtype == gate_bias.dtype == torch.float32 and tuple(y1.shape) == (T, W)
+        assert y2 is None or (y2.dtype == torch.float32 and tuple(y2.shape) == (T, W))
+        assert tuple(gates.shape) == (T, width) and gate_bias.numel() == width
+        assert y1_bias is None or (y1_bias.dtype == torch.float32 and y1_bias.numel() == W)
+        rows = T if row_index is None else row_index.numel()
+        assert row_index is None or row_index.dtype == torch.int32
+        assert h is None or (tuple(h.shape) == (rows, W) and norm_weight.dtype == torch.float32 and norm_weight.numel() == W)
+        clear = 0
+        for bit, t in ((1, y1), (2, y2), (4, gates)):
+            if t is not None and t.data_ptr() in self._acc_zero:
+                if row_index is None:
+                    clear |= bit
+                self._acc_zero[t.data_ptr()] = row_index is None
+        self._check(self.lib.tff_gated_join(
+            _ptr(x), _c_int(W), _ptr(gates), _c_int(_dt(gates)), _ptr(gate_bias), _ptr(y1), _ptr(y1_bias), _ptr(y2),
+            _c_int(clear), _ptr(norm_weight), _c_float(eps), _ptr(row_index), _ptr(h),
+            _c_int(_dt(h)) if h is not None else _c_int(0), _c_int(rows), self._stream()), "gated_join")
+        self.launches += 1
 
     def reset_accumulators(self) -> None:
         """After a step that was cut short: every accumulator buffer back to zero."""
@@ -573,14 +614,46 @@ class CudaKernels:
             self._acc_zero[proj.data_ptr()] = True
         self.launches += 1
 
+    def qk_finish(self, proj, q_out, norm, eps: float, bias, values_are_keys: bool, freq, batch, block_table, kv_cache,
+                  kv_layer, page_size, nq, nkv, d, dv) -> None:
+        """proj float32 [T, ld] = [q (nq*d) | k (nkv*d) | v (nkv*dv), unless ``values_are_keys``] -> the queries, each head
+        normed (``norm`` = (q, k weights float32 [d]) or None) and turned, in ``q_out`` [T, nq*d]; keys the same way and
+        values into the tokens' cache slots, the values of ``values_are_keys`` being the keys as projected.  ``bias`` float32
+        over the columns, added first; ``freq`` = (frequencies, rot_dim, magnitude, interleaved) or None.  An accumulator
+        buffer that is kept at zero is cleared."""
+        qw, kw = norm if norm is not None else (None, None)
+        self._need_cuda(proj, q_out, qw, kw, bias, block_table)
+        T, ld = proj.shape
+        used = (nq + nkv) * d + (0 if values_are_keys else nkv * dv)
+        assert proj.dtype == torch.float32 and ld >= used and tuple(q_out.shape) == (T, nq * d)
+        assert bias is None or (bias.dtype == torch.float32 and bias.numel() == used)
+        for w in (qw, kw):
+            assert w is None or (w.dtype == torch.float32 and w.numel() == d)
+        assert tuple(kv_cache.shape[2:5]) == (2, nkv, page_size) and kv_cache.dtype == q_out.dtype
+        f, rot, mag, inter = freq if freq is not None else (None, 0, 1.0, False)
+        c_ptr, _, c_layers, c_layer = self._cache_args(kv_cache, kv_layer)
+        clear = 1 if proj.data_ptr() in self._acc_zero else 0
+        self._check(self.lib.tff_qk_finish(
+            _ptr(proj), _c_int(clear), _c_int(ld), _ptr(q_out), _c_int(_dt(q_out)), _ptr(qw), _ptr(kw), _c_float(eps),
+            _ptr(bias), _c_int(1 if values_are_keys else 0), _ptr(f), _c_int(rot), _c_float(mag), _c_int(1 if inter else 0),
+            _ptr(batch.positions), _ptr(batch.tok_req), _ptr(block_table), _c_int(block_table.shape[1]), c_ptr,
+            _c_int(c_layers), _c_int(c_layer), _c_int(page_size), _c_int(kv_cache.shape[-1]), _c_int(T), _c_int(nq),
+            _c_int(nkv), _c_int(d), _c_int(dv), self._stream()), "qk_finish")
+        if clear:
+            self._acc_zero[proj.data_ptr()] = True
+        self.launches += 1
+
     def attend_gated(self, h, w_in, freq, batch, block_table, kv_cache, kv_layer, page_size, out, nq, nkv, d, dv,
-                     scale, window, softcap, sink, v_mode, v_share, lam, gate_off, write_cache, pre=None) -> None:
+                     scale, window, softcap, sink, v_mode, v_share, lam, gate_off, write_cache, pre=None, heads=None,
+                     keep: int = 0) -> None:
         """The whole of a gated, capped, sink attention between its input rows and its output projection: one product
         for q, k, v and the head gates (``w_in`` rows [q | k | v | gates | padding]); rotation, value mixing, cache
         write and sigmoid of the gates; attention over the paged cache with the cap, the window, the sink and the
         gates -> out [T, nq*dv].  ``pre`` = dict(taps, conv=(q, k, v weights [channels, taps] or None), norm=(q, k weights
         over the whole projection or None), eps, state): a short causal convolution over time on the projected q, k, v
-        and an RMS norm of all of q and of all of k, between the product and the rotation (short_conv_norm)."""
+        and an RMS norm of all of q and of all of k, between the product and the rotation (short_conv_norm).  ``heads`` =
+        dict(bias, norm=(q, k weights [d] or None), eps, values_are_keys): biases, per-head norms and values that are the
+        keys as projected (qk_finish).  ``keep``: the first so many positions stay visible beside the window."""
         if not write_cache:
             raise KernelError("attend_gated writes the keys and values it attends to; a borrowed cache is not supported")
         T = h.shape[0]
@@ -590,6 +663,13 @@ class CudaKernels:
         self.gemm(h, w_in, proj)
         q = torch.empty((T, nq * d), dtype=out.dtype, device=out.device)
         gates = torch.empty((T, nq), dtype=torch.float32, device=out.device) if gate_off >= 0 else None
+        if heads is not None:
+            self.qk_finish(proj, q, heads.get("norm"), float(heads.get("eps", 0.0)), heads.get("bias"),
+                           bool(heads.get("values_are_keys")), freq, batch, block_table, kv_cache, kv_layer, page_size, nq,
+                           nkv, d, dv)
+            self.attention_ext(q, batch, block_table, kv_cache, kv_layer, page_size, out, nq, nkv, d, dv, scale, window,
+                               softcap, sink, gates, keep)
+            return
         if pre is not None:
             taps = int(pre.get("taps") or 1)
             conv = pre.get("conv") or (None, None, None)
@@ -625,10 +705,10 @@ class CudaKernels:
         return bool(sink), None
 
     def attention_ext(self, q, batch, block_table, kv_cache, kv_layer, page_size, out, nq, nkv, d, dv, scale, window,
-                      softcap: float = 0.0, sink=False, gates=None) -> None:
+                      softcap: float = 0.0, sink=False, gates=None, keep: int = 0) -> None:
         """q [T, nq*d] against the paged cache (slots of kv_cache.shape[-1] >= max(d, dv) elements) -> out [T, nq*dv],
         with a cap on the scores, a sink in the softmax (True: of score 0; a float32 tensor [nq]: of that score per head)
-        and a multiplier per (token, head)."""
+        and a multiplier per (token, head).  ``keep``: beside a window, the first so many positions stay visible."""
         self._need_cuda(q, block_table, out, gates)
         T = q.shape[0]
         dc = kv_cache.shape[-1]
@@ -639,7 +719,7 @@ class CudaKernels:
         if q.dtype == torch.bfloat16 and d == dv == dc and d in (64, 128) and hasattr(batch, "h_sorted_q_lens"):
             # the kernels of plain attention take the cap, the sink and the gates as well
             self.attention_bf16(q, batch, block_table, kv_cache, kv_layer, page_size, out, nq, nkv, d, scale, window,
-                                extra=(float(softcap), sink, gates))
+                                extra=(float(softcap), sink, gates, int(keep)))
             return
         c_ptr, _, c_layers, c_layer = self._cache_args(kv_cache, kv_layer)
         sink_on, sink_val = self._sink_args(sink, nq)
@@ -648,7 +728,7 @@ class CudaKernels:
             _ptr(batch.positions), _ptr(batch.tok_req), _ptr(block_table), _c_int(block_table.shape[1]),
             c_ptr, _c_int(c_layers), _c_int(c_layer), _c_int(page_size),
             _ptr(out), _c_int(T), _c_int(nq), _c_int(nkv), _c_int(d), _c_int(dv), _c_int(dc), _c_float(scale),
-            _c_int(window), _c_float(softcap), _c_int(1 if sink_on else 0), _ptr(sink_val), _ptr(gates), self._stream()),
+            _c_int(window), _c_float(softcap), _c_int(1 if sink_on else 0), _ptr(sink_val), _ptr(gates), _c_int(keep), self._stream()),
             "attention_generic_ext")
         self.launches += 1
 
@@ -752,6 +832,56 @@ class CudaKernels:
                 break
         chunked = form > 0
         self._check(status, "retention_raw")
+        self.launches += 3 if chunked else 1
+
+    MLSTM_MMA = os.environ.get("TFFINFER_MLSTM_MMA", "1") != "0"   # 0: prompts token by token, as float32 FMAs
+
+    def mlstm(self, h, w_in, batch, state, gate_bias, cap: float, norm_w, eps: float, out, H, K, V) -> None:
+        """The whole of an mLSTM mixer between its input rows and its output projection -> out [T, H*V]: one product
+        (``w_in`` rows [q | k | v | gate | input gates | forget gates | padding]) into float32; the recurrence over ``state``
+        (mlstm_recurrence); per-head RMS norm, weight and sigmoid gate."""
+        T = h.shape[0]
+        if isinstance(h, DeferredNorm):
+            h = h.materialize()
+        proj = self.projection_buffer(T, w_in.shape[0], h.device, h.dtype)
+        self.gemm(h, w_in, proj)
+        o = torch.empty((T, H * V), dtype=torch.float32, device=h.device)
+        self.mlstm_recurrence(proj, state, batch, gate_bias, cap, o, H, K, V, rounded=h.dtype == torch.bfloat16)
+        self.gated_norm(o, V, proj, 2 * H * K + H * V, norm_w, eps, False, out, clear_cols=(0, proj.shape[1]),
+                        last_reader=True, gate_act="sigmoid")
+
+    def mlstm_recurrence(self, proj, state, batch, gate_bias, cap: float, out, H, K, V, rounded: bool = False,
+                         chunked: Optional[bool] = None) -> None:
+        """proj float32 [T, ld] = [q H*K | k H*K | v H*V | H*V others | input gates H | forget gates H | ...] -> o float32
+        [T, H*V] of the recurrence that parts/mlstm.py states, q scaled by K^-1/2; ``gate_bias`` float32 [2H], ``state``
+        float32 [slots, mlstm_state_size(H, K, V)].  ``rounded``: q, k and v may be rounded to bfloat16, and portions of
+        prompts run chunk by chunk on the tensor cores (``chunked`` None: when some request brings more than one token);
+        everything else runs token by token in float32.  ``proj`` is left as it is."""
+        self._need_cuda(proj, state, gate_bias, out)
+        T, ld = proj.shape
+        assert proj.dtype == state.dtype == gate_bias.dtype == out.dtype == torch.float32 and tuple(out.shape) == (T, H * V)
+        assert state.dim() == 2 and state.shape[1] == mlstm_state_size(H, K, V) and gate_bias.numel() == 2 * H
+        gates = 2 * H * K + 2 * H * V
+        assert ld >= gates + 2 * H
+        if chunked is None:
+            chunked = rounded and self.MLSTM_MMA and batch.max_q_len > 1
+
+        def run(ch: int):
+            ws = None
+            if ch:
+                self.lib.tff_mlstm_workspace.restype = ctypes.c_longlong
+                need = int(self.lib.tff_mlstm_workspace(_c_int(T), _c_int(batch.num_requests), _c_int(H), _c_int(K), _c_int(V)))
+                ws = torch.empty(need, dtype=torch.float32, device=proj.device)
+            return self.lib.tff_mlstm(
+                _ptr(proj), _c_int(ld), _c_int(0), _c_int(H * K), _c_int(2 * H * K), _c_int(gates), _c_int(gates + H),
+                _ptr(gate_bias), _c_float(cap), _c_float(float(K) ** -0.5), _ptr(state), _c_int(state.shape[0]),
+                _c_int(state.shape[1]), _ptr(batch.q_start), _ptr(batch.pos_start), _ptr(batch.slots), _ptr(out),
+                _c_int(batch.num_requests), _c_int(H), _c_int(K), _c_int(V), _c_int(ch), _ptr(ws), _c_int(T), self._stream())
+        status = run(1) if chunked else -2
+        if status == -2:                     # a head may be too large for the chunk form's shared memory
+            chunked = False
+            status = run(0)
+        self._check(status, "mlstm")
         self.launches += 3 if chunked else 1
 
     # ------------------------------------------------------- attention in float32 tiles (any sizes, latent caches, biases)
@@ -1063,7 +1193,8 @@ class CudaKernels:
 
     # ------------------------------------------------------- routed feed-forward (mixture of experts)
     def routed_mlp(self, h, w_router, w_gate_up, layout: str, w_down, residual, top: int, renormalize: bool = False,
-                   weight_on: str = "output", activation: str = "silu", out=None, router=None, limit: float = 0.0) -> None:
+                   weight_on: str = "output", activation: str = "silu", out=None, router=None, limit: float = 0.0,
+                   shared=None) -> None:
         """residual += sum over a token's ``top`` experts of down_e(act(gate_e(x)) * up_e(x)), the experts chosen by
         the largest sigmoid(W_r h) (computed in float32), weights the scores themselves or renormalised to sum 1;
         ``weight_on`` "input": x = w h and the outputs are summed as they are; "output": x = h and the outputs are
@@ -1072,7 +1203,9 @@ class CudaKernels:
         ``activation`` a function of one product ("relu2").  ``router`` (see moe_dispatch): softmax scores, a correction of
         the choice, groups of experts, identity experts (router outputs beyond the E experts: weight times the input);
         with score "table" there is no router (``w_router`` None): an integer table gives every token id its experts, each
-        with weight 1/top (moe_table).  ``limit``: the clipping of the activation "clipped_swish".
+        with weight 1/top (moe_table).  ``limit``: the clipping of the activation "clipped_swish".  ``shared`` = (y float32
+        [T, W], w [1, W]): the rows of an expert that every token uses, which join the sum times sigmoid(w h) (computed in
+        float32 by the router's kernel).
         With ``residual`` None the sum goes to ``out``.  Six launches, no host synchronisation: route, plan, gather, two
         grouped products over the tokens sorted by expert, combine (a token's experts are added in the order of their
         rank)."""
@@ -1098,6 +1231,10 @@ class CudaKernels:
         target = residual if residual is not None else out
         assert target.dtype == torch.float32 and tuple(target.shape) == (T, W)
         P = T * top
+        if shared is not None:
+            assert not by_table and shared[0].dtype == torch.float32 and tuple(shared[0].shape) == (T, W)
+            router = dict(router or {}, row=shared[1], row_out=torch.empty(T, dtype=torch.float32, device=h.device))
+            shared = (shared[0], router["row_out"])
         # both products run on the same kernel (one tile table): the tensor-core one if both can
         tc = (self.grouped_on_tensor_cores(h, w_gate_up, W, W, 0, W, up_rows * W, "" if plain else layout, ff)
               and self.grouped_on_tensor_cores(h, w_down, ff, ff, 0, ff, W * ff, "", W))
@@ -1119,7 +1256,7 @@ class CudaKernels:
             y = torch.empty((rows, W), dtype=torch.float32, device=h.device)
             self.gemm_tc_grouped(act, w_down, y, E, W, ff, lane_group)
             self.moe_combine(y, pair_weight if weight_on == "output" else None, top, residual, target, place,
-                             identity=(pe[0], pair_weight, h) if pe else None)
+                             identity=(pe[0], pair_weight, h) if pe else None, shared=shared)
             return
         a_rows = None
         tile_rows = self.grouped_tile_rows(tc, P <= 12 * E)      # few pairs an expert on average: tiles of few rows
@@ -1135,7 +1272,7 @@ class CudaKernels:
         y = torch.empty((P, W), dtype=torch.float32, device=h.device)
         self.gemm_grouped(act, w_down, y, E, 0, W, ff, ff, 0, ff, W * ff, W, 0, tiles=tiles, row_map=row_map)
         self.moe_combine(y, pair_weight if weight_on == "output" else None, top, residual, target,
-                         identity=(pe[0], pair_weight, h) if pe else None)
+                         identity=(pe[0], pair_weight, h) if pe else None, shared=shared)
 
     GROUPED_TCGEN05 = os.environ.get("TFFINFER_GROUPED_TCGEN05", "1") != "0"
     GROUPED_TCGEN05_FROM = 1024      # (token, expert) pairs of a step from which the experts run on the tcgen05 product
@@ -1170,7 +1307,8 @@ class CudaKernels:
         every tile of x, -1 for tiles nobody uses) and place_of_pair (int32 [T*top]).  ``router`` = dict(score="sigmoid" |
         "softmax" | "softmax_chosen" (the logits choose, the chosen are weighted by a softmax among themselves),
         bias=float32 [outputs] or None (added to the logits), correction=float32 [outputs] or None, groups=(count, keep), identity=n): the router's last n outputs are
-        identity experts, whose pairs get no row (pair_expert -1; returned as a last, further value when n > 0)."""
+        identity experts, whose pairs get no row (pair_expert -1; returned as a last, further value when n > 0).  ``row``
+        [1, W] and ``row_out`` float32 [T]: one more row beside the router's, row_out[t] = sigmoid(row . h[t])."""
         T, W = h.shape
         r = router or {}
         identity = int(r.get("identity", 0))
@@ -1199,11 +1337,14 @@ class CudaKernels:
         bias = r.get("bias")
         self._need_cuda(bias)
         assert bias is None or (bias.dtype == torch.float32 and bias.numel() == E + identity)
+        row, row_out = r.get("row"), r.get("row_out")
+        self._need_cuda(row, row_out)
+        assert row is None or (row.dtype == w_router.dtype and row.numel() == W and row_out.numel() == T)
         self._check(self.lib.tff_moe_route(_ptr(h), _c_int(_dt(h)), _ptr(w_router), _c_int(_dt(w_router)), _ptr(bias), _c_int(T), _c_int(W),
                                            _c_int(E + identity), _c_int(top), _c_int(1 if renormalize else 0),
                                            _c_int({"sigmoid": 0, "softmax": 1, "softmax_chosen": 2}[r.get("score", "sigmoid")]), _ptr(correction),
                                            _c_int(int(groups)), _c_int(int(keep)), _c_int(E), _ptr(pair_expert),
-                                           _ptr(pair_weight), _ptr(counts), self._stream()), "moe_route")
+                                           _ptr(pair_weight), _ptr(counts), _ptr(row), _ptr(row_out), self._stream()), "moe_route")
         self._check(self.lib.tff_moe_plan(_ptr(counts), _c_int(E), _c_int(bm), _ptr(cursor), _ptr(tile_group), _ptr(tile_row0),
                                           _ptr(tile_row_end), _ptr(num_tiles), _c_int(bm if padded_rows else 0),
                                           _ptr(lane_group), _c_int(lane_tiles), self._stream()), "moe_plan")
@@ -1251,11 +1392,16 @@ class CudaKernels:
                                             _c_int(top), _ptr(place_of_pair), _ptr(x), self._stream()), "moe_spread")
         self.launches += 1
 
-    def moe_combine(self, y, pair_weight, top: int, residual, out, place_of_pair=None, identity=None) -> None:
+    def moe_combine(self, y, pair_weight, top: int, residual, out, place_of_pair=None, identity=None, shared=None) -> None:
         """out[t] = residual[t] + sum_k w[t, k] * y[t*top + k] in the order of k (pair_weight None: plain sum); with
         ``place_of_pair`` the row of pair t*top + k is y[place_of_pair[t*top + k]] (y in the sorted order).  ``identity`` =
-        (pair_expert, pair_weight, h): pairs whose expert is -1 add their weight times the token's row of ``h`` instead."""
+        (pair_expert, pair_weight, h): pairs whose expert is -1 add their weight times the token's row of ``h`` instead.
+        ``shared`` = (rows float32 [T, W], weights float32 [T]): the token's row times its weight joins the sum; an
+        accumulator buffer that is kept at zero is cleared."""
         T, W = out.shape
+        ys, ws = shared if shared is not None else (None, None)
+        self._need_cuda(ys, ws)
+        clear = 1 if ys is not None and ys.data_ptr() in self._acc_zero else 0
         pe, iw, h = identity if identity is not None else (None, None, None)
         if identity is not None and pair_weight is None:
             weights, on_output = iw, 0            # the weights are read for the identity pairs only
@@ -1264,7 +1410,10 @@ class CudaKernels:
         self._check(self.lib.tff_moe_combine(_ptr(y), _c_int(T), _c_int(W), _c_int(top), _ptr(weights),
                                              _c_int(on_output), _ptr(place_of_pair),
                                              _ptr(residual), _ptr(out), _ptr(pe), _ptr(h),
-                                             _c_int(_dt(h)) if h is not None else _c_int(0), self._stream()), "moe_combine")
+                                             _c_int(_dt(h)) if h is not None else _c_int(0), _ptr(ys), _ptr(ws),
+                                             _c_int(clear), self._stream()), "moe_combine")
+        if clear:
+            self._acc_zero[ys.data_ptr()] = True
         self.launches += 1
 
     # ------------------------------------------------------- gated recurrence over a state of one vector
@@ -1718,11 +1867,12 @@ class CudaKernels:
         return self.attention_splits(eff, max_q_len, nq, nkv)
 
     def attention_bf16(self, q, batch, block_table, kv_cache, kv_layer, page_size, out,
-                       nq, nkv, d, scale, window, num_splits=None, extra=(0.0, False, None)) -> None:
+                       nq, nkv, d, scale, window, num_splits=None, extra=(0.0, False, None, 0)) -> None:
         """Flash attention over the paged cache (head sizes 64 and 128).  Requests that bring so few
         tokens that they fit a 16-row tile (decoded tokens) and requests that bring long portions are
         launched apart when a step holds both, each with the kernel made for it.  ``extra`` = (softcap, sink,
-        gates): a cap on the scores, a sink in the softmax, a float32 [T, nq] multiplier of the heads' outputs."""
+        gates, keep): a cap on the scores, a sink in the softmax, a float32 [T, nq] multiplier of the heads' outputs, and how
+        many first positions stay visible beside the window."""
         G = nq // nkv
         sq = batch.h_sorted_q_lens
         B = batch.num_requests
@@ -1770,7 +1920,7 @@ class CudaKernels:
                                         window, num_splits, order, B, batch.max_q_len, extra)
 
     def _attention_bf16_launch(self, q, batch, block_table, kv_cache, kv_layer, page_size, out, nq, nkv, d, scale,
-                               window, num_splits, req_ids, num_requests, max_q_len, extra=(0.0, False, None)) -> None:
+                               window, num_splits, req_ids, num_requests, max_q_len, extra=(0.0, False, None, 0)) -> None:
         T = q.shape[0]
         splits = num_splits
         c_ptr, c_pages, c_layers, c_layer = self._cache_args(kv_cache, kv_layer)
@@ -1786,7 +1936,7 @@ class CudaKernels:
                     self._portion_ws = ws
             else:
                 ws = torch.empty(need, dtype=torch.float32, device=q.device)
-        softcap, sink, gates = extra
+        softcap, sink, gates, keep = extra
         sink_on, sink_val = self._sink_args(sink, nq)
         self._check(self.lib.tff_attention_bf16_paged_ext(
             _ptr(q), _ptr(batch.q_start), _ptr(batch.pos_start), _ptr(req_ids), _ptr(block_table),
@@ -1795,7 +1945,7 @@ class CudaKernels:
             _c_int(page_size),
             _ptr(out), _ptr(ws), _c_int(T), _c_int(num_requests), _c_int(max_q_len), _c_int(splits),
             _c_int(nq), _c_int(nkv), _c_int(d), _c_float(scale), _c_int(window), _c_float(softcap),
-            _c_int(1 if sink_on else 0), _ptr(sink_val), _ptr(gates), self._stream()), "attention_bf16")
+            _c_int(1 if sink_on else 0), _ptr(sink_val), _ptr(gates), _c_int(keep), self._stream()), "attention_bf16")
         self.launches += 2 if splits > 1 else 1
 
     def attention_generic(self, q, batch, block_table, kv_cache, kv_layer, page_size, out,

@@ -5,3 +5,4 @@ from . import dominex  # noqa: F401  (registration)
 from . import sadupel  # noqa: F401  (registration)
 from . import nugosun  # noqa: F401  (registration)
 from . import kadodra  # noqa: F401  (registration)
+from . import gumodra  # noqa: F401  (registration)

@@ -105,6 +105,13 @@ class GatedSinkAttention(Mixer):
     * ``value_mix``: "source" leaves this layer's values of the step's tokens in ``ctx.shared[value_key]``;
       "mix" replaces its own by ``(1 - lambda) v + lambda v_source`` with a learned scalar lambda before they are
       cached; "none" does neither;
+    * ``qk_norm`` "head": an RMS norm over every head's q and over every head's k with plain weights "q_norm" and "k_norm"
+      [head_dim] that all heads share and ``qk_norm_eps``, ahead of the rotation;
+    * ``projection_bias``: biases of the q, k (and v) projections and of the output projection (tensors "q_bias", "k_bias",
+      "v_bias", "o_bias"), added in the projection;
+    * ``values_are_keys``: there is no value projection; a token's values are its keys as projected, ahead of norm and
+      rotation;
+    * ``keep_first``: beside a window, the first so many tokens of the sequence stay visible (and their pages stay);
     * ``head_gate``: every head's output is multiplied by ``sigmoid(W_g h)`` of that head, W_g [heads, hidden], read
       from the mixer's input like the projections.
 
@@ -115,6 +122,7 @@ class GatedSinkAttention(Mixer):
                  softmax_scale: Optional[float] = None, softcap: float = 0.0, window: int = 0, sink: bool = False,
                  value_mix: str = "none", value_key: str = "values", head_gate: bool = False,
                  lambda_tensor: bool = False, conv_taps: int = 0, qk_norm: str = "none", qk_norm_eps: float = 0.0,
+                 projection_bias: bool = False, values_are_keys: bool = False, keep_first: int = 0,
                  names: Optional[Dict[str, str]] = None, prefix: str = ""):
         super().__init__(prefix)
         self.hidden_size, self.num_heads, self.num_kv_heads = int(hidden_size), int(num_heads), int(num_kv_heads)
@@ -122,15 +130,26 @@ class GatedSinkAttention(Mixer):
         self.v_head_dim = int(v_head_dim) if v_head_dim else int(head_dim)
         self.scale = float(softmax_scale) if softmax_scale is not None else 1.0 / math.sqrt(self.head_dim)
         self.softcap, self.window = float(softcap), int(window)
+        self.keep_first = int(keep_first) if self.window > 0 else 0
+        self.projection_bias, self.values_are_keys = bool(projection_bias), bool(values_are_keys)
+        if self.keep_first < 0:
+            raise ValueError("keep_first must not be negative")
+        if self.values_are_keys and self.v_head_dim != self.head_dim:
+            raise ValueError("values that are the keys have the keys' size")
+        # what runs in the kernel that norms heads (qk_finish): it has no value mixing, no convolution and no head gates
+        self.head_finish = qk_norm == "head" or self.projection_bias or self.values_are_keys
+        if self.head_finish and (conv_taps or value_mix != "none" or head_gate or qk_norm == "whole"):
+            raise ValueError("norms of heads, biases and values that are the keys are not built together with a convolution, "
+                             "value mixing, head gates or a norm of the whole projection")
         if sink not in (False, True, "learned"):
             raise ValueError(f"sink must be False, True or 'learned', got {sink!r}")
         self.sink = sink
         self.conv_taps = int(conv_taps)
         if self.conv_taps < 0 or self.conv_taps > 8:
             raise ValueError(f"conv_taps must lie in 0 .. 8, got {self.conv_taps}")
-        if qk_norm not in ("none", "whole"):
-            raise ValueError(f"qk_norm must be 'none' or 'whole', got '{qk_norm}'")
-        if qk_norm == "whole" and not qk_norm_eps > 0:
+        if qk_norm not in ("none", "whole", "head"):
+            raise ValueError(f"qk_norm must be 'none', 'whole' or 'head', got '{qk_norm}'")
+        if qk_norm != "none" and not qk_norm_eps > 0:
             raise ValueError("qk_norm needs qk_norm_eps > 0")
         self.qk_norm, self.qk_norm_eps = qk_norm, float(qk_norm_eps)
         if value_mix not in ("none", "source", "mix"):
@@ -141,21 +160,22 @@ class GatedSinkAttention(Mixer):
             raise ValueError("num_heads must be a multiple of num_kv_heads")
         self.names = {"q": "q_proj.weight", "k": "k_proj.weight", "v": "v_proj.weight", "o": "o_proj.weight",
                       "gate": "gate_proj.weight", "lambda": "value_lambda", "sink": "sink", "q_conv": "q_conv",
-                      "k_conv": "k_conv", "v_conv": "v_conv", "q_norm": "q_norm", "k_norm": "k_norm"}
+                      "k_conv": "k_conv", "v_conv": "v_conv", "q_norm": "q_norm", "k_norm": "k_norm",
+                      "q_bias": "q_bias", "k_bias": "k_bias", "v_bias": "v_bias", "o_bias": "o_bias"}
         self.names.update(names or {})
         self.q_width = self.num_heads * self.head_dim
         self.k_width = self.num_kv_heads * self.head_dim
         self.v_width = self.num_kv_heads * self.v_head_dim
         self.cache_dim = max(self.head_dim, self.v_head_dim)     # a cache slot holds a key or a value
         self.w_in = self.w_o = self.lam = self.sink_w = None
-        self.conv_w = self.conv_wt = self.norm_w = None
+        self.conv_w = self.conv_wt = self.norm_w = self.bias = None
 
     def kernel_files(self):
         return ("attention_bf16", "attention_decode", "attention_prefill", "attention_generic",
-                "qkv_finish", "short_conv")
+                "qkv_finish", "short_conv", "streams")
 
     def cache_need(self):
-        kv = KVNeed(self.num_kv_heads, self.cache_dim, self.window)
+        kv = KVNeed(self.num_kv_heads, self.cache_dim, self.window, keep_first=self.keep_first)
         if self.conv_taps > 1:        # the projected rows the convolution still needs when the next step comes
             return kv, StateNeed((self.conv_taps - 1, self.q_width + self.k_width + self.v_width), "float32")
         return kv
@@ -164,12 +184,18 @@ class GatedSinkAttention(Mixer):
         n = self.names
         s = {n["q"]: WeightSpec((self.q_width, self.hidden_size), MATRIX),
              n["k"]: WeightSpec((self.k_width, self.hidden_size), MATRIX),
-             n["v"]: WeightSpec((self.v_width, self.hidden_size), MATRIX),
              n["o"]: WeightSpec((self.hidden_size, self.num_heads * self.v_head_dim), MATRIX)}
+        if not self.values_are_keys:
+            s[n["v"]] = WeightSpec((self.v_width, self.hidden_size), MATRIX)
+        if self.projection_bias:
+            widths = [("q_bias", self.q_width), ("k_bias", self.k_width), ("o_bias", self.hidden_size)]
+            for which, width in widths + ([] if self.values_are_keys else [("v_bias", self.v_width)]):
+                s[n[which]] = WeightSpec((width,), VECTOR, init="normal", init_scale=0.3)
         if self.head_gate:
             s[n["gate"]] = WeightSpec((self.num_heads, self.hidden_size), MATRIX)
         # a layer that mixes nothing may still carry the scalar in a file: it is accepted and not used
-        s[n["lambda"]] = WeightSpec((), VECTOR, init="normal", init_scale=0.3, optional=not self.lambda_tensor)
+        if not self.head_finish:
+            s[n["lambda"]] = WeightSpec((), VECTOR, init="normal", init_scale=0.3, optional=not self.lambda_tensor)
         if self.sink == "learned":
             s[n["sink"]] = WeightSpec((self.num_heads,), VECTOR, init="normal", init_scale=1.0)
         if self.conv_taps > 0:
@@ -178,11 +204,16 @@ class GatedSinkAttention(Mixer):
         if self.qk_norm == "whole":
             s[n["q_norm"]] = WeightSpec((self.q_width,), VECTOR, init="one_plus_normal")
             s[n["k_norm"]] = WeightSpec((self.k_width,), VECTOR, init="one_plus_normal")
+        elif self.qk_norm == "head":
+            s[n["q_norm"]] = WeightSpec((self.head_dim,), VECTOR, init="one_plus_normal")
+            s[n["k_norm"]] = WeightSpec((self.head_dim,), VECTOR, init="one_plus_normal")
         return s
 
     def load(self, tensors, ops, act_dtype) -> None:
         n = self.names
-        rows = [tensors[n["q"]], tensors[n["k"]], tensors[n["v"]]]
+        rows = [tensors[n["q"]], tensors[n["k"]]]
+        if not self.values_are_keys:
+            rows.append(tensors[n["v"]])
         if self.head_gate:
             rows.append(tensors[n["gate"]])
         dt = rows[0].dtype if all(r.dtype == rows[0].dtype for r in rows) else torch.float32
@@ -200,7 +231,11 @@ class GatedSinkAttention(Mixer):
         if self.conv_taps > 0:
             self.conv_w = tuple(tensors[n[w]].to(torch.float32).contiguous() for w in ("q_conv", "k_conv", "v_conv"))
             self.conv_wt = tuple(w.t().contiguous() for w in self.conv_w)     # [taps, channels]: the fused kernel's layout
-        if self.qk_norm == "whole":
+        if self.projection_bias:                     # one vector laid out like the product's q | k | v columns
+            which = ("q_bias", "k_bias") + (() if self.values_are_keys else ("v_bias",))
+            self.bias = torch.cat([tensors[n[w]].to(torch.float32) for w in which]).contiguous()
+            self.output_bias = tensors[n["o_bias"]].to(torch.float32).contiguous()
+        if self.qk_norm != "none":
             self.norm_w = (tensors[n["q_norm"]].to(torch.float32).contiguous(), tensors[n["k_norm"]].to(torch.float32).contiguous())
 
     def forward(self, h, ctx: LayerContext, residual):
@@ -217,7 +252,9 @@ class GatedSinkAttention(Mixer):
                 raise ValueError(f"value_mix='mix' needs the values of an earlier layer of this step under "
                                  f"'{self.value_key}' with {self.v_width} elements a token")
         attn = torch.empty((T, self.num_heads * self.v_head_dim), dtype=h.dtype, device=h.device)
-        pre = None
+        pre = heads = None
+        if self.head_finish:
+            heads = dict(bias=self.bias, norm=self.norm_w, eps=self.qk_norm_eps, values_are_keys=self.values_are_keys)
         if self.conv_taps > 0 or self.qk_norm == "whole":
             pre = dict(taps=max(self.conv_taps, 1), conv=self.conv_w, conv_t=self.conv_wt, norm=self.norm_w, eps=self.qk_norm_eps,
                        state=ctx.state if self.conv_taps > 1 else None)
@@ -226,12 +263,14 @@ class GatedSinkAttention(Mixer):
                          self.softcap, self.sink_w if self.sink == "learned" else self.sink,
                          {"none": 0, "source": 1, "mix": 2}[self.value_mix], share,
                          self.lam if self.value_mix == "mix" else None,
-                         self.gate_off if self.head_gate else -1, ctx.write_cache, pre=pre)
+                         self.gate_off if self.head_gate else -1, ctx.write_cache, pre=pre, heads=heads, keep=self.keep_first)
         if residual is None:
-            out = ops.sublayer_output(T, self.hidden_size, h.device, h.dtype)
+            out = ops.sublayer_output(T, self.hidden_size, h.device, h.dtype, self.output_use)
             ops.gemm(attn, self.w_o, out)
             return out
         ops.gemm(attn, self.w_o, residual, residual=residual)
+        if self.output_bias is not None:
+            ops.stream_step(residual.view(T, 1, self.hidden_size), bias=self.output_bias)
         return residual
 
 

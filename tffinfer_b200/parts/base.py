@@ -34,11 +34,13 @@ class WeightSpec:
 class KVNeed:
     """Keys and values of every token (window == 0) or of the last ``window`` tokens.  ``planes`` 2: a page holds a
     plane of keys and a plane of values, slots of ``head_dim`` elements each; 1: one plane, a token's slot is one
-    vector of ``head_dim`` elements from which the mixer makes both (a latent cache)."""
+    vector of ``head_dim`` elements from which the mixer makes both (a latent cache).  ``keep_first``: the first so many
+    tokens of the sequence are kept beside a window."""
     num_kv_heads: int
     head_dim: int
     window: int = 0
     planes: int = 2
+    keep_first: int = 0
 
 
 @dataclass(frozen=True)
@@ -140,6 +142,11 @@ class Mixer(Part):
     forward(h, ctx, residual) -> float32 [T, hidden]: residual + mixer(h); with ``residual`` None, mixer(h)
     alone in a tensor of its own (arrangements that do something else with it than add it to one stream).
     """
+    output_use = ""       # with ``residual`` None: the use the output's accumulator buffer is kept for (an arrangement whose
+                          # sublayers' outputs wait side by side names one each)
+    output_bias = None    # float32 [hidden] of the output projection, or None.  With ``residual`` None the output comes
+                          # WITHOUT it: the arrangement adds it where it joins the output to the residual
+
     def cache_need(self):
         return None
 
@@ -192,7 +199,7 @@ class SplitMixer(Mixer):
         mixed = torch.empty((T, self.mixed_width()), dtype=h.dtype, device=h.device)
         self.mix(proj, 0, ctx, mixed, 0, 1.0, True)
         if residual is None:
-            out = ops.sublayer_output(T, self.output_cols().shape[0], h.device, h.dtype)
+            out = ops.sublayer_output(T, self.output_cols().shape[0], h.device, h.dtype, self.output_use)
             ops.gemm(mixed, self.output_cols(), out)
             return out
         ops.gemm(mixed, self.output_cols(), residual, residual=residual)
@@ -201,6 +208,8 @@ class SplitMixer(Mixer):
 
 class FeedForward(Part):
     """forward(h, ctx, residual) -> float32 [T, hidden]: residual + f(h); with ``residual`` None, f(h) alone."""
+    output_use = ""       # as a mixer's
+
     def forward(self, h: torch.Tensor, ctx: LayerContext, residual: torch.Tensor) -> torch.Tensor:
         raise NotImplementedError
 

@@ -106,7 +106,7 @@ class LatentAttention(Mixer):
                           self.scale, ctx.write_cache, w_uk=self.w_uk, shared=ctx.shared,
                           window=self.window, sink=self.sink_w)
         if residual is None:
-            out = ops.sublayer_output(T, self.hidden_size, h.device, h.dtype)
+            out = ops.sublayer_output(T, self.hidden_size, h.device, h.dtype, self.output_use)
             ops.gemm(mixed, self.w_o, out)
             return out
         ops.gemm(mixed, self.w_o, residual, residual=residual)

@@ -104,7 +104,7 @@ class GatedLinearAttention(Mixer):
         ops.gated_norm(o, V, proj, self.gate_off, self.norm_w, self.eps, False, mixed, clear_cols=(0, proj.shape[1]),
                        last_reader=True)
         if residual is None:
-            out = ops.sublayer_output(T, self.hidden_size, h.device, h.dtype)
+            out = ops.sublayer_output(T, self.hidden_size, h.device, h.dtype, self.output_use)
             ops.gemm(mixed, self.w_o, out)
             return out
         ops.gemm(mixed, self.w_o, residual, residual=residual)

@@ -53,7 +53,7 @@ class SwiGLU(FeedForward):
 
     def forward(self, h, ctx, residual):
         if residual is None:              # f(h) alone, for arrangements that do more with it than add it
-            out = ctx.ops.sublayer_output(h.shape[0], self.hidden_size, h.device, h.dtype)
+            out = ctx.ops.sublayer_output(h.shape[0], self.hidden_size, h.device, h.dtype, self.output_use)
             ctx.ops.gated_mlp(h, self.w_gate_up, self.w_down, None, self.intermediate_size,
                               activation=self.activation, out=out)
             return out
@@ -91,6 +91,6 @@ class PlainMLP(FeedForward):
     def forward(self, h, ctx, residual):
         out = None
         if residual is None:
-            out = ctx.ops.sublayer_output(h.shape[0], self.hidden_size, h.device, h.dtype)
+            out = ctx.ops.sublayer_output(h.shape[0], self.hidden_size, h.device, h.dtype, self.output_use)
         ctx.ops.plain_mlp(h, self.w_up, self.w_down, residual, self.activation, out=out)
         return residual if residual is not None else out

@@ -18,7 +18,9 @@ token uses ``top``.
     f_e(x) = down_e( act(up_e(x)) )                      not gated (activation "relu2", the square of relu)
 
 The last ``identity_experts`` router outputs have no tensors: f_e(x) = x.  ``shared_intermediate`` > 0 adds one more
-expert of the same form that every token uses with weight 1 (tensors under ``names["shared"]``).
+expert of the same form that every token uses with weight 1 (tensors under ``names["shared"]``) or, with ``shared_gate``, with
+weight sigmoid(w_sg h), one number per token from a row of its own (tensor ``<shared>.sg`` [1, hidden], computed in float32
+beside the router).
 
 The experts' tensors are ``<prefix>.e<i>.{gate,up,down}`` and the router ``<prefix>.router`` unless ``names`` says
 otherwise; they are stacked into [E, 2 ff, hidden] (gate and up; [E, ff, hidden] when not gated) and [E, hidden, ff]
@@ -42,7 +44,8 @@ class RoutedExperts(FeedForward):
     def __init__(self, hidden_size: int, intermediate_size: int, num_experts: int, top: int, activation: str = "silu",
                  renormalize: bool = False, weight_on: str = "output", gated: bool = True, router_score: str = "sigmoid",
                  correction: bool = False, groups=None, identity_experts: int = 0, shared_intermediate: int = 0,
-                 router_bias: bool = False, activation_limit: float = 0.0, table_rows: int = 0, names=None, prefix: str = ""):
+                 router_bias: bool = False, activation_limit: float = 0.0, table_rows: int = 0, shared_gate: bool = False,
+                 names=None, prefix: str = ""):
         super().__init__(prefix)
         self.hidden_size, self.intermediate_size = int(hidden_size), int(intermediate_size)
         self.num_experts, self.top = int(num_experts), int(top)
@@ -77,11 +80,14 @@ class RoutedExperts(FeedForward):
                              f"leave at least top ({self.top}) of them")
         self.groups = (count, keep)
         self.shared_intermediate = int(shared_intermediate)
-        self.names = {"router": "router", "router_bias": "router.b", "expert": "e{}", "gate": "gate", "up": "up", "down": "down",
+        self.shared_gate = bool(shared_gate)
+        if self.shared_gate and (self.shared_intermediate <= 0 or not self.gated or router_score == "table"):
+            raise ValueError("a gate of the shared expert needs a gated shared expert and a router")
+        self.names = {"shared_gate": "sg", "router": "router", "router_bias": "router.b", "expert": "e{}", "gate": "gate", "up": "up", "down": "down",
                       "correction": "correction", "shared": "shared", "table": "table"}
         self.names.update(names or {})
         self.w_router = self.w_gate_up = self.w_down = self.correction_w = self.router_bias_w = None
-        self.shared_up = self.shared_down = self.table = None
+        self.shared_up = self.shared_down = self.table = self.shared_gate_w = None
         self.gate_up_layout = "blocked"
 
     def _expert(self, e: int, which: str) -> str:
@@ -113,6 +119,8 @@ class RoutedExperts(FeedForward):
                 s[self._shared("gate")] = WeightSpec((self.shared_intermediate, self.hidden_size), MATRIX)
             s[self._shared("up")] = WeightSpec((self.shared_intermediate, self.hidden_size), MATRIX)
             s[self._shared("down")] = WeightSpec((self.hidden_size, self.shared_intermediate), MATRIX)
+            if self.shared_gate:
+                s[self._shared("shared_gate")] = WeightSpec((1, self.hidden_size), MATRIX)
         return s
 
     def load(self, tensors, ops, act_dtype) -> None:
@@ -145,6 +153,10 @@ class RoutedExperts(FeedForward):
             else:
                 self.shared_up = tensors[self._shared("up")]
             self.shared_down = tensors[self._shared("down")]
+            if self.shared_gate:                      # a row beside the router's, in the router's type
+                self.shared_gate_w = tensors[self._shared("shared_gate")]
+                if self.shared_gate_w.dtype != self.w_router.dtype:
+                    self.shared_gate_w, self.w_router = self.shared_gate_w.to(torch.float32), self.w_router.to(torch.float32)
 
     def _router(self, ctx):
         if self.router_score == "table":
@@ -160,6 +172,14 @@ class RoutedExperts(FeedForward):
         target = residual
         if target is None:
             target = torch.empty((h.shape[0], self.hidden_size), dtype=torch.float32, device=h.device)
+        if self.shared_gate:          # the shared expert first: its rows join the sum, times their gate, in the sum's kernel
+            shared = ops.sublayer_output(h.shape[0], self.hidden_size, h.device, h.dtype, "shared expert")
+            ops.gated_mlp(h, self.shared_up, self.shared_down, None, self.shared_intermediate, activation=self.activation,
+                          out=shared)
+            ops.routed_mlp(h, self.w_router, self.w_gate_up, self.gate_up_layout, self.w_down, residual, self.top,
+                           self.renormalize, self.weight_on, self.activation, out=None if residual is not None else target,
+                           router=self._router(ctx), limit=self.activation_limit, shared=(shared, self.shared_gate_w))
+            return target
         ops.routed_mlp(h, self.w_router, self.w_gate_up, self.gate_up_layout, self.w_down, residual, self.top,
                        self.renormalize, self.weight_on, self.activation, out=None if residual is not None else target,
                        router=self._router(ctx), limit=self.activation_limit)

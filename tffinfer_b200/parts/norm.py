@@ -14,7 +14,8 @@ from .base import Norm, WeightSpec, VECTOR
 
 @register_part("norm", "rms_norm")
 class RMSNorm(Norm):
-    def __init__(self, dim: int, eps: float, name: str = "weight", weight_offset: float = 0.0, prefix: str = ""):
+    def __init__(self, dim: int, eps: float, name: str = "weight", weight_offset: float = 0.0, one_number: bool = False,
+                 prefix: str = ""):
         super().__init__(prefix)
         self.dim = int(dim)
         self.eps = float(eps)
@@ -22,17 +23,21 @@ class RMSNorm(Norm):
         # a weight stored around zero: the multiplier is weight_offset + w (1 + w in the designs that do this); the sum
         # is taken once, in float32, when the tensor is loaded
         self.weight_offset = float(weight_offset)
+        self.one_number = bool(one_number)        # the weight is a single number (a tensor of no dimensions) for all columns
         self.weight: Optional[torch.Tensor] = None
 
     def weight_specs(self) -> Dict[str, WeightSpec]:
+        shape = () if self.one_number else (self.dim,)
         if self.weight_offset != 0.0:
-            return {self.name: WeightSpec((self.dim,), VECTOR, init="normal", init_scale=0.1)}
-        return {self.name: WeightSpec((self.dim,), VECTOR, init="one_plus_normal")}
+            return {self.name: WeightSpec(shape, VECTOR, init="normal", init_scale=0.1)}
+        return {self.name: WeightSpec(shape, VECTOR, init="one_plus_normal")}
 
     def load(self, tensors, ops, act_dtype) -> None:
         self.weight = tensors[self.name]
         if self.weight_offset != 0.0:
             self.weight = (self.weight.to(torch.float32) + self.weight_offset).contiguous()
+        if self.one_number:
+            self.weight = self.weight.reshape(1).expand(self.dim).contiguous()
 
     def deferred(self, x, ops, out_dtype):
         """The norm of ``x`` as an object that the kernel library's products can fold in, or None when the

@@ -83,7 +83,7 @@ class ParallelMixers(Mixer):
         for i, m in enumerate(self.branches):
             m.mix(proj, self.in_cols[i], ctx, mixed, self.mixed_cols[i], self.scales[i], i == last)
         if residual is None:
-            out = ops.sublayer_output(T, self.hidden_size, h.device, h.dtype)
+            out = ops.sublayer_output(T, self.hidden_size, h.device, h.dtype, self.output_use)
             ops.gemm(mixed, self.w_out, out)
             return out
         ops.gemm(mixed, self.w_out, residual, residual=residual)

@@ -74,7 +74,7 @@ class Retention(Mixer):
         ops.retain(h, self.w_in, freq, ctx.batch, ctx.state, self.decay_dev, mixed, self.num_heads, self.head_dim,
                    self.v_head_dim, float(self.head_dim) ** -0.5, self.eps)
         if residual is None:
-            out = ops.sublayer_output(T, self.hidden_size, h.device, h.dtype)
+            out = ops.sublayer_output(T, self.hidden_size, h.device, h.dtype, self.output_use)
             ops.gemm(mixed, self.w_o, out)
             return out
         ops.gemm(mixed, self.w_o, residual, residual=residual)
@@ -141,7 +141,7 @@ class LightningAttention(Mixer):
         ops.lightning(h, self.w_in, ctx.batch, ctx.state, self.decay_dev, self.norm_w, self.eps, mixed, self.num_heads,
                       self.head_dim, self.v_head_dim)
         if residual is None:
-            out = ops.sublayer_output(T, self.hidden_size, h.device, h.dtype)
+            out = ops.sublayer_output(T, self.hidden_size, h.device, h.dtype, self.output_use)
             ops.gemm(mixed, self.w_o, out)
             return out
         ops.gemm(mixed, self.w_o, residual, residual=residual)

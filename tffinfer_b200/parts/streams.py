@@ -34,6 +34,7 @@ class ResidualStreams:
         self.streams = x.shape[1]
         self.pending = None            # (y, scale, mix, out) of the write that is still to come
         self.pending_bias = None       # a vector [hidden] that is still to be added to every stream, behind that write
+        self.pending_gated = None      # the gated outputs of a layer's sublayers, still to be added (one stream only)
 
     @classmethod
     def from_embedding(cls, token_ids, table, scale: float, streams: int, ops) -> "ResidualStreams":
@@ -55,7 +56,21 @@ class ResidualStreams:
             self.flush()
         self.pending_bias = vec
 
+    def write_gated(self, gates, gate_bias, y_mixer, mixer_bias, y_ff) -> None:
+        """x <- x + (y_mixer + mixer_bias) * sigmoid(gates[:, :W] + b) + y_ff * sigmoid(gates[:, W:] + b'), for a residual of
+        one stream; like a write, it runs with the next read (ops.gated_join)."""
+        if self.x.shape[1] != 1:
+            raise ValueError("gated writes are built for one stream")
+        self.flush()
+        self.pending_gated = dict(gates=gates, gate_bias=gate_bias, y1=y_mixer, y1_bias=mixer_bias, y2=y_ff)
+
+    def _rows(self) -> torch.Tensor:
+        return self.x.view(self.x.shape[0], self.x.shape[2])
+
     def flush(self) -> None:
+        if self.pending_gated is not None:
+            join, self.pending_gated = self.pending_gated, None
+            self.ops.gated_join(self._rows(), **join)
         if self.pending is not None or self.pending_bias is not None:
             y, scale, mix, out = self.pending if self.pending is not None else (None, None, None, None)
             bias, self.pending, self.pending_bias = self.pending_bias, None, None
@@ -67,6 +82,12 @@ class ResidualStreams:
         streams are not updated: that is the model's last read, nothing looks at them afterwards."""
         rows = self.x.shape[0] if row_index is None else row_index.shape[0]
         h = torch.empty((rows, self.x.shape[2]), dtype=out_dtype, device=self.x.device)
+        if self.pending_gated is not None and self.pending is None and self.pending_bias is None and read_w is None:
+            join, self.pending_gated = self.pending_gated, None
+            ops.gated_join(self._rows(), **join, norm_weight=norm.weight, eps=norm.eps, h=h, row_index=row_index)
+            return h
+        if self.pending_gated is not None:
+            self.flush()
         y, scale, mix, out = self.pending if self.pending is not None else (None, None, None, None)
         bias, self.pending, self.pending_bias = self.pending_bias, None, None
         ops.stream_step(self.x, y=y, scale=scale, mix=mix, out=out, read=read_w, norm_weight=norm.weight,
