@@ -986,19 +986,122 @@ def run_kadodra(steps: int, warmup: int, sizes=None) -> int:
     return 0
 
 
+# The Gumodra design beside Kadodra (the closest of the other models: one norm for two sublayers side by side, a windowed
+# attention with a learned sink and linear attention over matrix states in turn, dense and routed feed-forwards) at the same
+# width: (width, attention heads, kv heads, dim, window, kept first tokens, mlstm heads, key size, value size, experts, chosen,
+# groups, kept groups, expert ff, shared ff, dense ff).  Eight layers, mlstm with a dense feed-forward and attention with experts
+# in turn; the dense feed-forward is gated, so its ff is two thirds of the twin's for the same arithmetic.  What the twin has no
+# like of: the gates of the residual (two width x width products a layer) and the shared expert.
+GUMODRA_SIZES = {"2k": (2048, 16, 4, 128, 1024, 64, 16, 128, 128, 16, 2, 4, 2, 3072, 3072, 6144),
+                 "4k": (4096, 32, 8, 128, 1024, 64, 32, 128, 128, 16, 2, 4, 2, 6144, 6144, 12288)}
+
+
+def gumodra_engine(size: str, max_live: int, cache_tokens: int, graphs: bool, step_tokens: int):
+    import torch
+    import tffinfer_b200 as tff
+    from tffinfer_b200.config.gumodra_config import GumodraConfig, GumodraLayer, GumodraMlp, GumodraAttention, GumodraMlstm
+    from tffinfer_b200.config.tipezen_config import RotaryConfig
+    from tffinfer_b200.weights import random_tensors_on_device
+    W, H, G, D, WIN, KEEP, MH, MD, MV, E, TOP, NG, KG, F, SF, DF = GUMODRA_SIZES[size]
+    memory = GumodraLayer("mlstm", mlp=GumodraMlp("dense", DF), mlstm=GumodraMlstm(MH, MD, MV, 15.0))
+    attention = GumodraLayer("attention", mlp=GumodraMlp("moe", F, E, TOP, (NG, KG), SF), attention=GumodraAttention(
+        H, G, D, D ** -0.5, RotaryConfig(5e5, D // 2), WIN, KEEP))
+    cfg = GumodraConfig("Gumodra", vocab_size=TIPEZEN_VOCAB, hidden_size=W, norm_eps=1e-6, embed_scale=W ** 0.5,
+                        layers=(memory, attention) * (TIPEZEN_LAYERS // 2))
+    tensors = random_tensors_on_device(cfg, 0, "cuda", "bfloat16")
+    ecfg = tff.EngineConfig(dtype="bfloat16", page_size=PAGE_SIZE, max_cache_tokens=cache_tokens, max_live_requests=max_live,
+                            max_tokens_per_step=step_tokens, max_model_len=8192, use_cuda_graphs=graphs)
+    runner = tff.ModelRunner(config=cfg, tensors=tensors, engine_config=ecfg)
+    del tensors
+    torch.cuda.empty_cache()
+    return tff.Engine(runner=runner), cfg
+
+
+def run_gumodra(steps: int, warmup: int, sizes=None) -> int:
+    """Prefill and decode throughput of the Gumodra design beside Kadodra at the same layer sizes, one JSON line a point, and
+    for each model the device time of a step by kind of kernel call; for Gumodra also what its own kernels reach: the mLSTM
+    recurrence in TFLOP/s of its chunk form (prompt step) and as a fraction of the measured copy rate for the states it reads
+    and writes (decode step), the windowed attention, the kernels of the residual's gates, of the heads, of the norm behind the
+    recurrence and of the experts' sum as fractions of the copy rate, the products of the measured bfloat16 rate."""
+    import torch
+    peaks = load_peaks()
+    steps = min(steps, 32)
+    P = PROMPT_LEN
+    clocks = ClockSampler()
+    clocks.start()
+    for size in (sizes or GUMODRA_SIZES):
+        W, H, G, D, WIN, KEEP, MH, MD, MV, E, TOP, NG, KG, F, SF, DF = GUMODRA_SIZES[size]
+        for model, make in (("gumodra", gumodra_engine), ("kadodra", kadodra_engine)):
+            need = 64 * (P + warmup + steps + 64 + 72)
+            engine, cfg = make(size, 64, need, True, P)
+            pms = prefill_run(engine, iters=3, warmup=2, seed=1, prompt_len=P)
+            print(json.dumps({"point": "prefill", "model": model, "size": size, "layers": TIPEZEN_LAYERS, "tokens": P,
+                              "ms": round(pms, 3), "tok_s": round(P / (pms / 1e3), 1)}), flush=True)
+            for b in (8, 64):
+                run = decode_run(engine, b, steps, warmup, seed=b, prompt_len=P)
+                print(json.dumps({"point": "decode", "model": model, "size": size, "layers": TIPEZEN_LAYERS, "batch": b,
+                                  "context": round(run["mean_context"]), "tok_s": round(run["tok_s"], 1),
+                                  "ms_per_step": round(run["ms_per_step"], 4), "launches_per_step": run["launches"] // steps,
+                                  **experts_of(engine, run["last_tokens"])}), flush=True)
+            del engine
+            torch.cuda.empty_cache()
+            engine, cfg = make(size, 8, 8 * (P + 64), False, P)
+            kinds = traced_kinds(engine, P, 8)
+            line = {"point": "kernels", "model": model, "size": size, "prefill_tokens": P, "decode_batch": 8,
+                    "prefill_ms_by_kind": kinds.get("prefill"), "decode_ms_by_kind": kinds.get("decode"), "peaks": peaks["source"]}
+            if model == "gumodra":
+                nl = TIPEZEN_LAYERS // 2                        # layers of either kind
+                fr = {}
+                for step, T in (("prefill", P), ("decode", 8)):
+                    k = kinds.get(step) or {}
+                    z = 2 if T == P else 4                      # bytes of a gate: bfloat16 in prompts, accumulators in decode steps
+                    for kind, nbytes in (("gated_join", (2 * nl - 1) * T * W * (4 + 4 + 4 + 4 + 2 * z + 2)),
+                                         ("gated_norm", nl * T * MH * MV * (4 + 4 + 2)),
+                                         ("qk_finish", nl * T * D * ((H + G) * 4 + (H + 2 * G) * 2)),
+                                         ("moe_combine", nl * T * W * (TOP * 4 + 4 + 4))):
+                        if kind in k:
+                            fr[f"{step}_{kind}_hbm_frac"] = round(nbytes / (k[kind][1] / 1e3) / 1e9 / peaks["hbm_gbs"], 4)
+                k, kd = kinds.get("prefill") or {}, kinds.get("decode") or {}
+                if "mlstm_recurrence" in k:       # chunks of 64 tokens: A = Q K^T and A V, U = K^T V and Q S
+                    flops = nl * MH * (P / 64.0) * 2.0 * 64 * (64 * MD + 64 * MV + 2 * MD * MV)
+                    fr["prefill_mlstm_recurrence_tflops"] = round(flops / (k["mlstm_recurrence"][1] / 1e3) / 1e12, 2)
+                if "attention_bf16" in k:
+                    span = min(WIN, P)
+                    pairs = span * (span + 1) / 2.0 + (P - span) * (span + KEEP)
+                    fr["prefill_attention_bf16_tflops"] = round(nl * H * pairs * 4.0 * D / (k["attention_bf16"][1] / 1e3) / 1e12, 2)
+                if "gemm_tc_grouped" in k:
+                    fr["prefill_experts_tcgen05_frac"] = round(nl * P * TOP * 6.0 * W * F / (k["gemm_tc_grouped"][1] / 1e3) / 1e12 / peaks["bf16_tflops"], 4)
+                if "gemm_tc" in k:                # mlstm in and out, attention in and out, gates, both down products
+                    flops = P * 2.0 * W * (nl * (2 * MH * MD + 3 * MH * MV + 2 * MH + (2 * H + G) * D + SF + DF) + 2 * nl * 2 * W)
+                    fr["prefill_dense_products_frac"] = round(flops / (k["gemm_tc"][1] / 1e3) / 1e12 / peaks["bf16_tflops"], 4)
+                if "gemm_gated_act" in k:
+                    fr["prefill_gemm_gated_act_frac"] = round(nl * P * 4.0 * W * (DF + SF) / (k["gemm_gated_act"][1] / 1e3) / 1e12 / peaks["bf16_tflops"], 4)
+                if "mlstm_recurrence" in kd:
+                    fr["decode_mlstm_recurrence_hbm_frac"] = round(nl * 8 * MH * MD * (MV + 1) * 4 * 2 / (kd["mlstm_recurrence"][1] / 1e3) / 1e9 / peaks["hbm_gbs"], 4)
+                if "attention_bf16" in kd:
+                    fr["decode_attention_bf16_hbm_frac"] = round(nl * 8 * min(WIN + KEEP, P) * 2 * G * D * 2 / (kd["attention_bf16"][1] / 1e3) / 1e9 / peaks["hbm_gbs"], 4)
+                line["fractions"] = fr
+            print(json.dumps(line), flush=True)
+            del engine
+            torch.cuda.empty_cache()
+    clocks.stop()
+    print(json.dumps({"point": "clocks", "clocks": clocks.summary()}), flush=True)
+    return 0
+
+
 def main() -> int:
     ap = argparse.ArgumentParser()
-    ap.add_argument("--workload", default="headline", choices=["headline", "sweep", "attn_decode", "shapes", "tipezen", "dominex", "sadupel", "nugosun", "kadodra"] + sorted(WORKLOADS),
+    ap.add_argument("--workload", default="headline", choices=["headline", "sweep", "attn_decode", "shapes", "tipezen", "dominex", "sadupel", "nugosun", "kadodra", "gumodra"] + sorted(WORKLOADS),
                     help="headline: the decode/prefill benchmark; sweep: the same shape at further batch sizes and "
                          "context lengths; attn_decode: the decode attention alone; shapes: the layer sizes of the other "
-                         "models of the family; tipezen: the Tipezen design beside Qwen3 at equal layer sizes; dominex: the Dominex design beside Tipezen at equal layer sizes; sadupel: the Sadupel design beside Dominex at equal layer sizes; nugosun: the Nugosun design beside Dominex at equal layer sizes; kadodra: the Kadodra design beside Nugosun at equal layer sizes; else a whole workload through "
+                         "models of the family; tipezen: the Tipezen design beside Qwen3 at equal layer sizes; dominex: the Dominex design beside Tipezen at equal layer sizes; sadupel: the Sadupel design beside Dominex at equal layer sizes; nugosun: the Nugosun design beside Dominex at equal layer sizes; kadodra: the Kadodra design beside Nugosun at equal layer sizes; gumodra: the Gumodra design beside Kadodra at equal layer sizes; else a whole workload through "
                          "the scheduler")
     ap.add_argument("--gpus", type=int, default=1)
     ap.add_argument("--steps", type=int, default=64)
     ap.add_argument("--warmup", type=int, default=4)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--batch", type=int, default=8)
-    ap.add_argument("--size", default="", help="with --workload dominex, sadupel, nugosun or kadodra: one of its layer sizes (2k, 4k) instead of all")
+    ap.add_argument("--size", default="", help="with --workload dominex, sadupel, nugosun, kadodra or gumodra: one of its layer sizes (2k, 4k) instead of all")
     ap.add_argument("--layers", type=int, default=SHAPE["num_layers"],
                     help="fewer layers than the shape has (both numbers are reported)")
     ap.add_argument("--skip-points", action="store_true", help="only the headline batch (no batch 1 / 64, no prefill)")
@@ -1031,6 +1134,8 @@ def main() -> int:
         return run_nugosun(args.steps, warmup, [args.size] if args.size else None)
     if args.workload == "kadodra":
         return run_kadodra(args.steps, warmup, [args.size] if args.size else None)
+    if args.workload == "gumodra":
+        return run_gumodra(args.steps, warmup, [args.size] if args.size else None)
     if args.workload != "headline":
         return run_workload(args.workload, 0 if args.layers == SHAPE["num_layers"] else args.layers)
 
