@@ -68,7 +68,7 @@ def sink_softmax(scores, seen, sink):
 
 def attention_mixer(h, positions, w, p: str, m: dict, eps: float):
     T, H, G, D = h.shape[0], int(m["heads"]), int(m["kv_heads"]), int(m["dim"])
-    rot = m["rot"]
+    rot = m.get("rot") or {"dims": 0, "base": 1.0}
     q = lin(h, w[p + ".q"], w[p + ".q.b"]).reshape(T, H, D)
     u = lin(h, w[p + ".k"], w[p + ".k.b"]).reshape(T, G, D)
     q = turn_halves(q / rms(q, eps) * w[p + ".q.norm"], positions, int(rot["dims"]), float(rot["base"]))

@@ -96,6 +96,25 @@ def test_window_gives_pages_back_when_passed(Manager):
     m.check()
 
 
+def test_kept_first_tokens_keep_their_pages_behind_a_window(Manager):
+    """Pages that hold one of the first ``keep_first`` tokens stay while the window moves on; everything goes back at the end."""
+    for keep, kept in ((0, 0), (1, 1), (4, 1), (5, 2), (12, 3), (100, 25)):
+        m = Manager([GroupSpec(1, 1, 16, 6, keep_first=keep)], 4, [40], 2)
+        m.admit("a")
+        n = 0
+        for part in (3, 20, 1, 1, 30, 1, 20):
+            assert m.reserve("a", part)
+            m.commit("a", part)
+            n += part
+            first = max(0, n - 6 + 1) // 4
+            table = m.block_table("a", 0)
+            assert [p != NO_PAGE for p in table] == [b < kept or b >= first for b in range(len(table))], (keep, n)
+            m.check()
+        m.release("a")
+        m.check()
+        assert m.pools[0].num_free == 40
+
+
 def test_random_orders_never_lose_or_double_book_a_page(Manager):
     rng = random.Random(11)
     m = Manager([GroupSpec(3, 2, 16, 0), GroupSpec(2, 2, 16, 10)], 4, [24, 12], 5)

@@ -14,7 +14,7 @@ from tffinfer_b200.engine.batch import StepEntry
 @pytest.mark.parametrize("seed", [0, 1, 2])
 def test_native_manager_and_packer_equal_the_python_twins(seed):
     rng = random.Random(seed)
-    groups = [GroupSpec(2, 2, 16, 0), GroupSpec(1, 2, 16, rng.choice([5, 9, 30]))]
+    groups = [GroupSpec(2, 2, 16, 0), GroupSpec(1, 2, 16, rng.choice([5, 9, 30]), keep_first=(0, 3, 17)[seed])]
     page = rng.choice([2, 4, 16])
     sizes = [rng.randint(20, 60), rng.randint(8, 20)]
     a = CacheManager(groups, page, sizes, 5)
@@ -112,7 +112,7 @@ def test_native_planning_equals_the_python_scheduler_in_lockstep(seed):
     live = rng.randint(1, 4)
     budget = rng.choice([3, 8, 20])
     max_len = rng.choice([40, 200])
-    groups = [GroupSpec(2, 2, 16, 0)] + ([GroupSpec(1, 2, 16, 7)] if seed % 2 else [])
+    groups = [GroupSpec(2, 2, 16, 0)] + ([GroupSpec(1, 2, 16, 7, keep_first=seed % 3 * 5)] if seed % 2 else [])
     sizes = [pages] + ([max(3, pages // 2)] if seed % 2 else [])
     sa = Scheduler(CacheManager(groups, page, sizes, live), budget, max_len)
     sb = Scheduler(NativeCacheManager(groups, page, sizes, live), budget, max_len)
