@@ -83,6 +83,64 @@ gated_norm_kernel(const float* __restrict__ o, int width, int gs, float* __restr
     }
 }
 
+// Narrow groups in whole fours: a lane holds G4 times four neighbouring elements (16-byte accesses), a warp a group.
+template <typename TO, int G4>
+__global__ void __launch_bounds__(256)
+gated_norm4_kernel(const float* __restrict__ o, int width, int gs, float* __restrict__ gate, int g_ld, int g_off,
+                   const float* __restrict__ w, int wlen, float eps, int gate_first, int gate_act, int clear_lo, int clear_hi,
+                   TO* __restrict__ out, int out_ld, int out_off, float out_scale) {
+    pdl_launch_dependents();
+    const int t = blockIdx.x, lane = threadIdx.x & 31, g = blockIdx.y * 8 + (threadIdx.x >> 5), n4 = gs >> 2;
+    float* grow = gate + (size_t)t * g_ld;
+    pdl_wait();
+    for (int c = clear_lo + blockIdx.y * 256 + threadIdx.x; c < clear_hi; c += gridDim.y * 256)
+        if (c < g_off || c >= g_off + width) grow[c] = 0.f;
+    if (g >= width / gs) return;
+    const float4* o4 = reinterpret_cast<const float4*>(o + (size_t)t * width + g * gs);
+    float4* z4 = reinterpret_cast<float4*>(grow + g_off + g * gs);
+    float u[G4][4], z[G4][4];
+#pragma unroll
+    for (int k = 0; k < G4; ++k) {
+        const int i = lane + 32 * k;
+        const float4 a = i < n4 ? __ldcg(o4 + i) : make_float4(0.f, 0.f, 0.f, 0.f), b = i < n4 ? __ldcg(z4 + i) : a;
+        u[k][0] = a.x; u[k][1] = a.y; u[k][2] = a.z; u[k][3] = a.w;
+        z[k][0] = b.x; z[k][1] = b.y; z[k][2] = b.z; z[k][3] = b.w;
+    }
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < G4; ++k)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            z[k][e] = norm_gate(z[k][e], gate_act);
+            if (gate_first) u[k][e] *= z[k][e];
+            ss = fmaf(u[k][e], u[k][e], ss);             // (elements beyond the group are zeros)
+        }
+    const float inv = rsqrtf(warp_sum(ss) / (float)gs + eps);
+#pragma unroll
+    for (int k = 0; k < G4; ++k) {
+        const int i = lane + 32 * k, c = g * gs + 4 * i;
+        if (i >= n4) continue;
+        if (g_off + c >= clear_lo && g_off + c < clear_hi) z4[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+        const float4 ww = *reinterpret_cast<const float4*>(w + c % wlen);
+        const float wv[4] = {ww.x, ww.y, ww.z, ww.w};
+        float r[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const float y = (u[k][e] * inv) * wv[e];
+            r[e] = (gate_first ? y : y * z[k][e]) * out_scale;
+        }
+        TO* dst = out + (size_t)t * out_ld + out_off + c;
+        if constexpr (sizeof(TO) == 2) {
+            __nv_bfloat162 lo = __floats2bfloat162_rn(r[0], r[1]), hi = __floats2bfloat162_rn(r[2], r[3]);
+            uint2 v;
+            v.x = *reinterpret_cast<uint32_t*>(&lo); v.y = *reinterpret_cast<uint32_t*>(&hi);
+            *reinterpret_cast<uint2*>(dst) = v;
+        } else {
+            *reinterpret_cast<float4*>(dst) = make_float4(r[0], r[1], r[2], r[3]);
+        }
+    }
+}
+
 }  // namespace
 
 // out_dt: 0 = float32, 1 = bfloat16.
@@ -98,6 +156,18 @@ TFF_API int tff_gated_norm(const float* o, int width, int gs, float* gate, int g
     const dim3 grid(num_tokens, wide ? width / gs : (width / gs + 7) / 8);
     int st;
     if (!clear) clear_lo = clear_hi = 0;
+    const int elt = out_dt == 1 ? 2 : 4;
+    if (!wide && gs % 4 == 0 && wlen % 4 == 0 && g_ld % 4 == 0 && g_off % 4 == 0 && out_ld % 4 == 0 && out_off % 4 == 0 &&
+        clear_lo % 4 == 0 && clear_hi % 4 == 0 && (((uintptr_t)o | (uintptr_t)gate | (uintptr_t)w) & 15) == 0 &&
+        ((uintptr_t)out & (4 * elt - 1)) == 0) {
+#define TFF_GN4(TO, G4)                                                                                               \
+        return tff_launch_pdl(gated_norm4_kernel<TO, G4>, grid, dim3(256), 0, stream, o, width, gs, gate, g_ld, g_off, w, wlen, \
+                              eps, gate_first, gate_act, clear_lo, clear_hi, (TO*)out, out_ld, out_off, out_scale)
+        if (out_dt == 1) { if (gs <= 128) TFF_GN4(bf16, 1); TFF_GN4(bf16, 4); }
+        if (gs <= 128) TFF_GN4(float, 1);
+        TFF_GN4(float, 4);
+#undef TFF_GN4
+    }
 #define TFF_GN(TO, WIDE)                                                                                              \
     st = tff_launch_pdl(gated_norm_kernel<TO, WIDE>, grid, dim3(256), 0, stream, o, width, gs, gate, g_ld,            \
                         g_off, w, wlen, eps, gate_first, gate_act, clear_lo, clear_hi, (TO*)out, out_ld, out_off, out_scale)

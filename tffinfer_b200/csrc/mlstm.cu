@@ -32,6 +32,9 @@ struct MlstmParams {
     float* state; int num_slots, slot_len;
     const int* q_start; const int* pos_start; const int* slots;
     float* out; int H, d, dv;
+    // The step kernel may go on to the mixer's output: mixed[t, h*dv + j] = o_j / rms(o) * norm_w[h*dv + j] * sigmoid(g), g the
+    // row's columns g_off .. (norm_w null: o itself to ``out``); with ``clear`` it sets what it has read of the row to zero.
+    float* rows; int g_off; const float* norm_w; float eps; void* mixed; int mixed_is_bf16, clear;
 };
 
 __device__ __forceinline__ float in_gate(float z, float cap) { return cap * tanhf(z / cap); }
@@ -56,7 +59,8 @@ mlstm_step_kernel(MlstmParams p) {
     float* sq = sm;                     // [d]
     float* sk = sq + d;                 // [d]
     float* sn = sk + d;                 // [d]
-    float* part = sn + d;               // [NY][groups * VEC]
+    float* so = sn + d;                 // [dv]
+    float* part = so + dv;              // [NY][groups * VEC]
     const int groups = (dv + VEC - 1) / VEC, LX = min(groups, ST), NY = ST / LX;
     const int lx = tid % LX, ty = tid / LX;
     const int t0 = p.q_start[b], t1 = p.q_start[b + 1];
@@ -129,12 +133,32 @@ mlstm_step_kernel(MlstmParams p) {
             for (int c = 0; c < VEC; ++c) part[(size_t)ty * groups * VEC + g * VEC + c] = acc[c];
         }
         nq = block_sum<ST>(nq, red);                     // (a barrier behind the partial sums too)
+        float ss = 0.f;
         for (int j = tid; j < dv; j += ST) {
             float o = 0.f;
             for (int y = 0; y < NY; ++y) o += part[(size_t)y * groups * VEC + j];
-            p.out[(size_t)t * p.H * dv + (size_t)h * dv + j] = divide(o, nq, m);
+            o = divide(o, nq, m);
+            if (!p.norm_w) { p.out[(size_t)t * p.H * dv + (size_t)h * dv + j] = o; continue; }
+            so[j] = o;                                   // (this thread alone reads it back)
+            ss = fmaf(o, o, ss);
         }
         fresh = false;
+        if (!p.norm_w) continue;
+        const float inv = rsqrtf(block_sum<ST>(ss, red) / (float)dv + p.eps);
+        float* wrow = p.rows + (size_t)t * p.ld;
+        for (int j = tid; j < dv; j += ST) {
+            const int c = h * dv + j;
+            const float g = __ldcg(row + p.g_off + c);
+            const float y = (so[j] * inv) * p.norm_w[c] / (1.0f + expf(-g));
+            const size_t at = (size_t)t * p.H * dv + c;
+            if (p.mixed_is_bf16) ((bf16*)p.mixed)[at] = __float2bfloat16_rn(y);
+            else ((float*)p.mixed)[at] = y;
+            if (p.clear) { wrow[p.g_off + c] = 0.f; wrow[p.v_off + c] = 0.f; }
+        }
+        if (p.clear) {                                   // (everything of the row that this head reads has been read)
+            for (int i = tid; i < d; i += ST) { wrow[p.q_off + h * d + i] = 0.f; wrow[p.k_off + h * d + i] = 0.f; }
+            if (tid == 0) { wrow[p.i_off + h] = 0.f; wrow[p.f_off + h] = 0.f; }
+        }
     }
     if (KEEP && ty < NY && lx < groups)
 #pragma unroll
@@ -379,25 +403,28 @@ TFF_API long long tff_mlstm_workspace(int num_tokens, int num_requests, int H, i
 }
 
 // chunked != 0: chunk by chunk on the tensor cores, q, k and v rounded to bfloat16 (``workspace`` of tff_mlstm_workspace
-// floats); else token by token in float32.  TFF_ERR_UNSUPPORTED when a head does not fit the form's shared memory.
+// floats); else token by token in float32, and with norm_w (float32 [H*dv]) on to the mixer's output ``mixed`` [T, H*dv], where
+// ``rows`` is proj again and ``clear`` sets the columns that were read to zero.  TFF_ERR_UNSUPPORTED when a head does not fit the form's shared memory.
 TFF_API int tff_mlstm(const float* proj, int ld, int q_off, int k_off, int v_off, int i_off, int f_off, const float* gate_bias,
                       float cap, float q_scale, float* state, int num_slots, int slot_len, const int* q_start,
                       const int* pos_start, const int* slots, float* out, int num_requests, int H, int d, int dv, int chunked,
-                      float* workspace, int num_tokens, cudaStream_t stream) {
+                      float* workspace, int num_tokens, float* rows, int g_off, const float* norm_w, float eps, void* mixed,
+                      int mixed_is_bf16, int clear, cudaStream_t stream) {
     if (num_requests <= 0) return TFF_OK;
-    if (!proj || !gate_bias || !state || !q_start || !pos_start || !slots || !out || H <= 0 || d <= 0 || dv <= 0 || !(cap > 0.f) ||
+    if (norm_w && (chunked || !mixed || g_off < 0 || g_off + H * dv > ld || !(eps > 0.f) || (clear && !rows))) return TFF_ERR_BAD_ARGUMENT;
+    if (!proj || !gate_bias || !state || !q_start || !pos_start || !slots || (!out && !norm_w) || H <= 0 || d <= 0 || dv <= 0 || !(cap > 0.f) ||
         q_off < 0 || k_off < 0 || v_off < 0 || i_off < 0 || f_off < 0 || q_off + H * d > ld || k_off + H * d > ld ||
         v_off + H * dv > ld || i_off + H > ld || f_off + H > ld || (slot_len & 3) ||
         (long long)slot_len < (long long)H * d * dv + (long long)H * d + H)
         return TFF_ERR_BAD_ARGUMENT;
     if (num_requests > 65535 || H > 65535) return TFF_ERR_UNSUPPORTED;
     const MlstmParams p{proj, ld, q_off, k_off, v_off, i_off, f_off, gate_bias, cap, q_scale, state, num_slots, slot_len,
-                        q_start, pos_start, slots, out, H, d, dv};
+                        q_start, pos_start, slots, out, H, d, dv, rows, g_off, norm_w, eps, mixed, mixed_is_bf16, clear};
     if (chunked) return launch_chunked(p, num_requests, workspace, num_tokens, stream);
     const bool vec = dv % 4 == 0 && ((uintptr_t)state & 15) == 0 && (H * d * dv) % 4 == 0;
     const int width = vec ? 4 : 1, groups = dv / width, lx = groups < ST ? groups : ST, ny = ST / lx;
     const bool keep = groups <= ST && ny * ROWS >= d;
-    const size_t smem = sizeof(float) * ((size_t)3 * d + (size_t)ny * groups * width);
+    const size_t smem = sizeof(float) * ((size_t)3 * d + dv + (size_t)ny * groups * width);
     if (smem > 48 * 1024) return TFF_ERR_UNSUPPORTED;
     const dim3 grid(H, num_requests);
     if (vec && keep) return tff_launch_pdl(mlstm_step_kernel<4, true>, grid, dim3(ST), smem, stream, p);

@@ -12,7 +12,9 @@
 //            ``tile_rows`` rows that never span two experts), and the counters back to zero for the next call
 //   table    instead of route and plan where a table gives every token id its experts (no router): one block counts the
 //            experts' pairs in shared memory, lays out their rows and tiles as plan does, and gives every pair its place
-//            (an atomic cursor in shared memory, as gather's), its weight 1/top, and every place its token row
+//            (an atomic cursor in shared memory, as gather's), its weight 1/top, and every place its token row.  Behind
+//            the router's kernel (no table) it stands for plan and gather in steps of few pairs, whose products read
+//            the tokens' rows where they are
 //   gather   per pair: its place among its expert's rows (an atomic cursor: the order within an expert is not fixed,
 //            but a row's result does not depend on its place), row_map[place] = pair, and the expert's input row
 //            x[place] = w * h[token] (weight on the input) or h[token]
@@ -22,10 +24,11 @@
 
 namespace {
 
-constexpr int ROUTE_TOK = 4;                   // tokens a block of moe_route_kernel, one warp each for the choice
-constexpr int ROUTE_THREADS = 256;
+// Tokens a block of moe_route_kernel takes (one warp each for the choice) and its threads: steps of many tokens share the
+// reading of the router's rows, steps of few give every output a warp of its own.
+constexpr int ROUTE_MANY_TOK = 4, ROUTE_MANY_THREADS = 256, ROUTE_FEW_TOK = 1, ROUTE_FEW_THREADS = 512, ROUTE_FEW = 256;
 
-template <typename TH, typename TW>
+template <typename TH, typename TW, int ROUTE_TOK, int ROUTE_THREADS>
 __global__ void __launch_bounds__(ROUTE_THREADS)
 moe_route_kernel(const TH* __restrict__ h, const TW* __restrict__ w_router, const float* __restrict__ bias, int T, int W, int E,
                  int top, int renormalize, int softmax_scores, const float* __restrict__ correction, int groups, int keep, int num_real,
@@ -64,54 +67,75 @@ moe_route_kernel(const TH* __restrict__ h, const TW* __restrict__ w_router, cons
     for (int k = nt; k < ROUTE_TOK; ++k)
         for (int i = threadIdx.x; i < W; i += ROUTE_THREADS) rows[(size_t)k * W + i] = 0.f;
     __syncthreads();
-    // A warp an output; a lane takes eight neighbouring elements a load where the rows allow it (16-byte loads, several in
-    // flight), else one.  Either way the order of a dot product's additions is fixed by W alone.
-    // (Index E is the row beside the router's, when there is one.)
+    // A warp takes up to RE outputs side by side (a row's elements are read once for them), a lane eight neighbouring
+    // elements a load where the rows allow it (16-byte loads, several in flight), else one.  Either way the order of a dot
+    // product's additions is fixed by W alone.  (Index E is the row beside the router's, when there is one.)
+    constexpr int RE = ROUTE_TOK > 1 ? 3 : 1, RW = ROUTE_THREADS / 32;
     const bool wide = (W & 7) == 0 && (((size_t)w_router | (size_t)row_w) & 15) == 0;
-    for (int e = warp; e < E + (row_w ? 1 : 0); e += ROUTE_THREADS / 32) {
-        const TW* wr = e < E ? w_router + (size_t)e * W : row_w;
-        float acc[ROUTE_TOK];
+    const int outputs = E + (row_w ? 1 : 0);
+    for (int e0 = warp; e0 < outputs; e0 += RW * RE) {
+        const TW* wr[RE];
+        float acc[RE][ROUTE_TOK];
 #pragma unroll
-        for (int k = 0; k < ROUTE_TOK; ++k) acc[k] = 0.f;
+        for (int x = 0; x < RE; ++x) {
+            const int e = min(e0 + x * RW, outputs - 1);
+            wr[x] = e < E ? w_router + (size_t)e * W : row_w;
+#pragma unroll
+            for (int k = 0; k < ROUTE_TOK; ++k) acc[x][k] = 0.f;
+        }
         if (wide) {
-#pragma unroll 4
+#pragma unroll 2
             for (int i = lane * 8; i < W; i += 256) {
-                float w8[8];
-                if constexpr (sizeof(TW) == 2) {
-                    const uint4 raw = *reinterpret_cast<const uint4*>(wr + i);
-                    const __nv_bfloat162* p2 = reinterpret_cast<const __nv_bfloat162*>(&raw);
+                float w8[RE][8];
 #pragma unroll
-                    for (int k = 0; k < 4; ++k) { const float2 f = __bfloat1622float2(p2[k]); w8[2 * k] = f.x; w8[2 * k + 1] = f.y; }
-                } else {
-                    const float4 a = *reinterpret_cast<const float4*>(wr + i), b = *reinterpret_cast<const float4*>(wr + i + 4);
-                    w8[0] = a.x; w8[1] = a.y; w8[2] = a.z; w8[3] = a.w; w8[4] = b.x; w8[5] = b.y; w8[6] = b.z; w8[7] = b.w;
+                for (int x = 0; x < RE; ++x) {
+                    if constexpr (sizeof(TW) == 2) {
+                        const uint4 raw = *reinterpret_cast<const uint4*>(wr[x] + i);
+                        const __nv_bfloat162* p2 = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+                        for (int k = 0; k < 4; ++k) { const float2 f = __bfloat1622float2(p2[k]); w8[x][2 * k] = f.x; w8[x][2 * k + 1] = f.y; }
+                    } else {
+                        const float4 a = *reinterpret_cast<const float4*>(wr[x] + i), b = *reinterpret_cast<const float4*>(wr[x] + i + 4);
+                        w8[x][0] = a.x; w8[x][1] = a.y; w8[x][2] = a.z; w8[x][3] = a.w; w8[x][4] = b.x; w8[x][5] = b.y; w8[x][6] = b.z; w8[x][7] = b.w;
+                    }
                 }
 #pragma unroll
                 for (int k = 0; k < ROUTE_TOK; ++k) {
                     const float* row = rows + (size_t)k * W + i;
                     const float4 r0 = *reinterpret_cast<const float4*>(row), r1 = *reinterpret_cast<const float4*>(row + 4);
-                    float a = acc[k];
-                    a = fmaf(r0.x, w8[0], a); a = fmaf(r0.y, w8[1], a); a = fmaf(r0.z, w8[2], a); a = fmaf(r0.w, w8[3], a);
-                    a = fmaf(r1.x, w8[4], a); a = fmaf(r1.y, w8[5], a); a = fmaf(r1.z, w8[6], a); a = fmaf(r1.w, w8[7], a);
-                    acc[k] = a;
+#pragma unroll
+                    for (int x = 0; x < RE; ++x) {
+                        float a = acc[x][k];
+                        a = fmaf(r0.x, w8[x][0], a); a = fmaf(r0.y, w8[x][1], a); a = fmaf(r0.z, w8[x][2], a); a = fmaf(r0.w, w8[x][3], a);
+                        a = fmaf(r1.x, w8[x][4], a); a = fmaf(r1.y, w8[x][5], a); a = fmaf(r1.z, w8[x][6], a); a = fmaf(r1.w, w8[x][7], a);
+                        acc[x][k] = a;
+                    }
                 }
             }
         } else {
             for (int i = lane; i < W; i += 32) {
-                const float wv = to_f32<TW>(wr[i]);
 #pragma unroll
-                for (int k = 0; k < ROUTE_TOK; ++k) acc[k] = fmaf(rows[(size_t)k * W + i], wv, acc[k]);
+                for (int x = 0; x < RE; ++x) {
+                    const float wv = to_f32<TW>(wr[x][i]);
+#pragma unroll
+                    for (int k = 0; k < ROUTE_TOK; ++k) acc[x][k] = fmaf(rows[(size_t)k * W + i], wv, acc[x][k]);
+                }
             }
         }
 #pragma unroll
-        for (int k = 0; k < ROUTE_TOK; ++k) {
-            if (e == E) {
-                const float z = warp_sum(acc[k]);
-                if (lane == 0 && k < nt) row_out[t0 + k] = 1.0f / (1.0f + expf(-z));
-                continue;
+        for (int x = 0; x < RE; ++x) {
+            const int e = e0 + x * RW;
+            if (e >= outputs) continue;
+#pragma unroll
+            for (int k = 0; k < ROUTE_TOK; ++k) {
+                if (e == E) {
+                    const float z = warp_sum(acc[x][k]);
+                    if (lane == 0 && k < nt) row_out[t0 + k] = 1.0f / (1.0f + expf(-z));
+                    continue;
+                }
+                const float z = warp_sum(acc[x][k]) + (bias ? bias[e] : 0.f);
+                if (lane == 0) scores[(size_t)k * 3 * E + e] = softmax_scores ? z : 1.0f / (1.0f + expf(-z));
             }
-            const float z = warp_sum(acc[k]) + (bias ? bias[e] : 0.f);
-            if (lane == 0) scores[(size_t)k * 3 * E + e] = softmax_scores ? z : 1.0f / (1.0f + expf(-z));
         }
     }
     __syncthreads();
@@ -203,28 +227,53 @@ moe_route_kernel(const TH* __restrict__ h, const TW* __restrict__ w_router, cons
 // pad_rows > 0: every expert's rows start at a multiple of pad_rows (= tile_rows): the sorted order then consists of
 // whole tiles of one expert each, and lane_group[row / pad_rows] names it (-1: a tile nobody uses), which is what the
 // grouped tcgen05 product reads.
-__global__ void moe_plan_kernel(int* __restrict__ counts, int E, int tile_rows, int* __restrict__ cursor,
-                                int* __restrict__ tile_group, int* __restrict__ tile_row0, int* __restrict__ tile_row_end,
-                                int* __restrict__ num_tiles, int pad_rows, int* __restrict__ lane_group, int lane_tiles) {
+// The first row and the first tile of every expert from the experts' counts, by one warp, 32 experts at a time.
+__device__ __forceinline__ void layout_experts(const int* count, int E, int tile_rows, int pad_rows, int* first, int* tile0,
+                                               int* num_tiles) {
+    const int lane = threadIdx.x & 31;
+    int rows = 0, tiles = 0;
+    for (int e0 = 0; e0 < E; e0 += 32) {
+        const int e = e0 + lane;
+        const int c = e < E ? count[e] : 0;
+        int r = pad_rows > 0 ? (c + pad_rows - 1) / pad_rows * pad_rows : c, n = (c + tile_rows - 1) / tile_rows;
+        const int own_r = r, own_n = n;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const int a = __shfl_up_sync(0xffffffffu, r, o), b = __shfl_up_sync(0xffffffffu, n, o);
+            if (lane >= o) { r += a; n += b; }
+        }
+        if (e < E) { first[e] = rows + r - own_r; tile0[e] = tiles + n - own_n; }
+        rows += __shfl_sync(0xffffffffu, r, 31);
+        tiles += __shfl_sync(0xffffffffu, n, 31);
+    }
+    if (lane == 0) *num_tiles = tiles;
+}
+
+__global__ void __launch_bounds__(256)
+moe_plan_kernel(int* __restrict__ counts, int E, int tile_rows, int* __restrict__ cursor,
+                int* __restrict__ tile_group, int* __restrict__ tile_row0, int* __restrict__ tile_row_end,
+                int* __restrict__ num_tiles, int pad_rows, int* __restrict__ lane_group, int lane_tiles) {
+    extern __shared__ int smi[];
+    int* count = smi;                          // [E]
+    int* first = smi + E;                      // [E]
+    int* tile0 = first + E;                    // [E]
     pdl_launch_dependents();
     pdl_wait();
+    for (int e = threadIdx.x; e < E; e += 256) { count[e] = __ldcg(counts + e); counts[e] = 0; }
     if (lane_group)
-        for (int i = threadIdx.x; i < lane_tiles; i += blockDim.x) lane_group[i] = -1;
+        for (int i = threadIdx.x; i < lane_tiles; i += 256) lane_group[i] = -1;
     __syncthreads();
-    if (threadIdx.x != 0) return;
-    int off = 0, n = 0;
-    for (int e = 0; e < E; ++e) {
-        const int c = counts[e];
-        counts[e] = 0;
-        if (pad_rows > 0) off = (off + pad_rows - 1) / pad_rows * pad_rows;
+    if (threadIdx.x < 32) layout_experts(count, E, tile_rows, pad_rows, first, tile0, num_tiles);
+    __syncthreads();
+    for (int e = threadIdx.x; e < E; e += 256) {
+        const int c = count[e], off = first[e];
+        int n = tile0[e];
         cursor[e] = off;
-        for (int r = off; r < off + c; r += tile_rows) {
-            tile_group[n] = e; tile_row0[n] = r; tile_row_end[n] = off + c; ++n;
+        for (int r = off; r < off + c; r += tile_rows, ++n) {
+            tile_group[n] = e; tile_row0[n] = r; tile_row_end[n] = off + c;
             if (lane_group) lane_group[r / pad_rows] = e;
         }
-        off += c;
     }
-    *num_tiles = n;
 }
 
 constexpr int TABLE_THREADS = 1024;
@@ -234,7 +283,7 @@ moe_table_kernel(const int* __restrict__ tokens, const int* __restrict__ table, 
                  int tile_rows, int pad_rows, int* __restrict__ pair_expert, float* __restrict__ pair_weight,
                  int* __restrict__ row_map, int* __restrict__ token_of_row, int* __restrict__ place_of_pair,
                  int* __restrict__ tile_group, int* __restrict__ tile_row0, int* __restrict__ tile_row_end,
-                 int* __restrict__ num_tiles, int* __restrict__ lane_group, int lane_tiles) {
+                 int* __restrict__ num_tiles, int* __restrict__ lane_group, int lane_tiles, int* __restrict__ counts) {
     extern __shared__ int smi[];
     int* count = smi;                          // [E] pairs of the expert, later its cursor
     int* first = smi + E;                      // [E] its first row
@@ -246,8 +295,15 @@ moe_table_kernel(const int* __restrict__ tokens, const int* __restrict__ table, 
     pdl_wait();
     if (lane_group)
         for (int i = tid; i < lane_tiles; i += TABLE_THREADS) lane_group[i] = -1;
+    if (!table) {                              // the router's choice: count it; its counters go back to zero
+        for (int e = tid; e < E; e += TABLE_THREADS) counts[e] = 0;
+        for (int i = tid; i < P; i += TABLE_THREADS) {
+            const int e = __ldcg(pair_expert + i);
+            if (e >= 0) atomicAdd(&count[e], 1);
+        }
+    }
     const float w = 1.0f / (float)top;
-    for (int i = tid; i < P; i += TABLE_THREADS) {
+    for (int i = tid; table && i < P; i += TABLE_THREADS) {
         const int tok = tokens[i / top];
         int e = (tok >= 0 && tok < table_rows) ? table[(size_t)tok * top + i % top] : -1;
         if (e < 0 || e >= E) e = -1;           // the host refuses such ids and tables; never a wrong row
@@ -256,24 +312,7 @@ moe_table_kernel(const int* __restrict__ tokens, const int* __restrict__ table, 
         if (e >= 0) atomicAdd(&count[e], 1);
     }
     __syncthreads();
-    if (tid < 32) {                            // rows and tiles of the experts ahead, 32 experts at a time
-        int rows = 0, tiles = 0;
-        for (int e0 = 0; e0 < E; e0 += 32) {
-            const int e = e0 + tid;
-            const int c = e < E ? count[e] : 0;
-            int r = pad_rows > 0 ? (c + pad_rows - 1) / pad_rows * pad_rows : c, n = (c + tile_rows - 1) / tile_rows;
-            const int own_r = r, own_n = n;
-#pragma unroll
-            for (int o = 1; o < 32; o <<= 1) {
-                const int a = __shfl_up_sync(0xffffffffu, r, o), b = __shfl_up_sync(0xffffffffu, n, o);
-                if (tid >= o) { r += a; n += b; }
-            }
-            if (e < E) { first[e] = rows + r - own_r; tile0[e] = tiles + n - own_n; }
-            rows += __shfl_sync(0xffffffffu, r, 31);
-            tiles += __shfl_sync(0xffffffffu, n, 31);
-        }
-        if (tid == 0) *num_tiles = tiles;
-    }
+    if (tid < 32) layout_experts(count, E, tile_rows, pad_rows, first, tile0, num_tiles);
     __syncthreads();
     for (int e = tid; e < E; e += TABLE_THREADS) {
         const int c = count[e], r0 = first[e];
@@ -286,7 +325,7 @@ moe_table_kernel(const int* __restrict__ tokens, const int* __restrict__ table, 
     }
     __syncthreads();
     for (int i = tid; i < P; i += TABLE_THREADS) {
-        const int e = pair_expert[i];          // this thread wrote it
+        const int e = table ? pair_expert[i] : __ldcg(pair_expert + i);        // (this thread wrote it, or the router's kernel)
         const int place = e >= 0 ? atomicAdd(&count[e], 1) : -1;
         if (place >= 0) { row_map[place] = i; token_of_row[place] = i / top; }
         if (place_of_pair) place_of_pair[i] = place;
@@ -340,7 +379,17 @@ moe_gather_kernel(const TH* __restrict__ h, int W, int top, const int* __restric
     for (int i = threadIdx.x; i < W; i += 128) dst[i] = from_f32<TH>(w * to_f32<TH>(src[i]));
 }
 
-template <typename TH>
+// four neighbouring elements as float32
+__device__ __forceinline__ float4 load_row4(const float* p) { return __ldcg(reinterpret_cast<const float4*>(p)); }
+__device__ __forceinline__ float4 load_row4(const bf16* p) {
+    const uint2 raw = __ldcg(reinterpret_cast<const uint2*>(p));
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+    return make_float4(a.x, a.y, b.x, b.y);
+}
+
+// VEC columns a thread (4: 16-byte accesses); pairs are asked for eight at a time
+template <typename TH, int VEC>
 __global__ void __launch_bounds__(256)
 moe_combine_kernel(const float* __restrict__ y, int W, int top, const float* __restrict__ pair_weight,
                    int weight_on_output, const int* __restrict__ place_of_pair, float* __restrict__ residual,
@@ -349,24 +398,54 @@ moe_combine_kernel(const float* __restrict__ y, int W, int top, const float* __r
     pdl_launch_dependents();
     pdl_wait();
     const int t = blockIdx.x;
-    const int i = blockIdx.y * 256 + threadIdx.x;
+    const int i = (blockIdx.y * 256 + threadIdx.x) * VEC;
     if (i >= W) return;
-    float acc = 0.f;
-    for (int k = 0; k < top; ++k) {
-        const size_t pair = (size_t)t * top + k;              // y in (token, rank) order, or in the sorted order
-        if (pair_expert && __ldcg(pair_expert + pair) < 0) {           // an identity expert: the weight times the input itself
-            acc = fmaf(pair_weight[pair], to_f32<TH>(h[(size_t)t * W + i]), acc);
-            continue;
-        }
-        const float w = weight_on_output ? __ldcg(pair_weight + pair) : 1.f;
-        acc = fmaf(w, __ldcg(y + (place_of_pair ? (size_t)__ldcg(place_of_pair + pair) : pair) * W + i), acc);
-    }
+    auto load = [&](const auto* p, float (&v)[VEC]) {
+        if constexpr (VEC == 4) { const float4 x = load_row4(p); v[0] = x.x; v[1] = x.y; v[2] = x.z; v[3] = x.w; }
+        else v[0] = to_f32(*p);
+    };
+    float acc[VEC];
+#pragma unroll
+    for (int c = 0; c < VEC; ++c) acc[c] = 0.f;
     const size_t at = (size_t)t * W + i;
-    if (shared) {                                             // an expert that every token uses, times the token's weight
-        acc = fmaf(__ldcg(shared_w + t), __ldcg(shared + at), acc);
-        if (clear_shared) shared[at] = 0.f;
+    for (int k0 = 0; k0 < top; k0 += 4) {
+        float v[4][VEC], w[4];
+#pragma unroll
+        for (int u = 0; u < 4; ++u) {
+            if (k0 + u >= top) continue;
+            const size_t pair = (size_t)t * top + k0 + u;     // y in (token, rank) order, or in the sorted order
+            if (pair_expert && __ldcg(pair_expert + pair) < 0) {       // an identity expert: the weight times the input itself
+                w[u] = __ldcg(pair_weight + pair);
+                load(h + at, v[u]);
+                continue;
+            }
+            w[u] = weight_on_output ? __ldcg(pair_weight + pair) : 1.f;
+            load(y + (place_of_pair ? (size_t)__ldcg(place_of_pair + pair) : pair) * W + i, v[u]);
+        }
+#pragma unroll
+        for (int u = 0; u < 4; ++u)
+            if (k0 + u < top)
+#pragma unroll
+                for (int c = 0; c < VEC; ++c) acc[c] = fmaf(w[u], v[u][c], acc[c]);
     }
-    out[at] = residual ? residual[at] + acc : acc;
+    if (shared) {                                             // an expert that every token uses, times the token's weight
+        float v[VEC];
+        load(shared + at, v);
+        const float w = __ldcg(shared_w + t);
+#pragma unroll
+        for (int c = 0; c < VEC; ++c) acc[c] = fmaf(w, v[c], acc[c]);
+        if (clear_shared)
+#pragma unroll
+            for (int c = 0; c < VEC; ++c) shared[at + c] = 0.f;
+    }
+    if (residual) {
+        float v[VEC];
+        load(residual + at, v);
+#pragma unroll
+        for (int c = 0; c < VEC; ++c) acc[c] += v[c];
+    }
+    if constexpr (VEC == 4) *reinterpret_cast<float4*>(out + at) = make_float4(acc[0], acc[1], acc[2], acc[3]);
+    else out[at] = acc[0];
 }
 
 }  // namespace
@@ -384,21 +463,29 @@ TFF_API int tff_moe_route(const void* h, int h_dt, const void* w_router, int w_d
     if (W <= 0 || E <= 0 || top <= 0 || top > E || !h || !w_router || num_real < 0 || num_real > E || (row_w && !row_out))
         return TFF_ERR_BAD_ARGUMENT;
     if (groups > 1 && (E % groups != 0 || keep <= 0 || keep > groups || top > keep * (E / groups))) return TFF_ERR_BAD_ARGUMENT;
-    const size_t smem = (size_t)ROUTE_TOK * (W + 3 * E) * sizeof(float);
+    const bool few = T <= ROUTE_FEW;
+    const int tok = few ? ROUTE_FEW_TOK : ROUTE_MANY_TOK;
+    const size_t smem = (size_t)tok * (W + 3 * E) * sizeof(float);
     if (smem > 200 * 1024) return TFF_ERR_UNSUPPORTED;
-#define TFF_ROUTE(TH, TW)                                                                                             \
+#define TFF_ROUTE_N(TH, TW, TOK, THREADS)                                                                             \
     do {                                                                                                              \
         if (smem > 48 * 1024)                                                                                         \
-            cudaFuncSetAttribute(moe_route_kernel<TH, TW>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);   \
-        return tff_launch_pdl(moe_route_kernel<TH, TW>, dim3((T + ROUTE_TOK - 1) / ROUTE_TOK), dim3(ROUTE_THREADS), smem, stream, (const TH*)h, \
+            cudaFuncSetAttribute(moe_route_kernel<TH, TW, TOK, THREADS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+        return tff_launch_pdl(moe_route_kernel<TH, TW, TOK, THREADS>, dim3((T + TOK - 1) / TOK), dim3(THREADS), smem, stream, (const TH*)h, \
                               (const TW*)w_router, bias, T, W, E, top, renormalize, softmax_scores, correction, groups, keep, \
                               num_real, pair_expert, pair_weight, counts, (const TW*)row_w, row_out);         \
+    } while (0)
+#define TFF_ROUTE(TH, TW)                                                                                             \
+    do {                                                                                                              \
+        if (few) TFF_ROUTE_N(TH, TW, ROUTE_FEW_TOK, ROUTE_FEW_THREADS);                                               \
+        TFF_ROUTE_N(TH, TW, ROUTE_MANY_TOK, ROUTE_MANY_THREADS);                                                      \
     } while (0)
     if (h_dt == 0 && w_dt == 0) TFF_ROUTE(float, float);
     if (h_dt == 0 && w_dt == 1) TFF_ROUTE(float, bf16);
     if (h_dt == 1 && w_dt == 1) TFF_ROUTE(bf16, bf16);
     if (h_dt == 1 && w_dt == 0) TFF_ROUTE(bf16, float);
 #undef TFF_ROUTE
+#undef TFF_ROUTE_N
     return TFF_ERR_BAD_ARGUMENT;
 }
 
@@ -407,18 +494,20 @@ TFF_API int tff_moe_plan(int* counts, int E, int tile_rows, int* cursor, int* ti
                          cudaStream_t stream) {
     if (E <= 0 || tile_rows <= 0 || pad_rows < 0 || (pad_rows > 0 && pad_rows != tile_rows) || (lane_group && pad_rows <= 0))
         return TFF_ERR_BAD_ARGUMENT;
-    return tff_launch_pdl(moe_plan_kernel, dim3(1), dim3(128), 0, stream, counts, E, tile_rows, cursor, tile_group,
+    if (E > 4096) return TFF_ERR_UNSUPPORTED;
+    return tff_launch_pdl(moe_plan_kernel, dim3(1), dim3(256), (size_t)3 * E * sizeof(int), stream, counts, E, tile_rows, cursor, tile_group,
                           tile_row0, tile_row_end, num_tiles, pad_rows, lane_group, lane_tiles);
 }
 
 // tokens [P / top] int32, table [table_rows, top] int32.  Outputs as tff_moe_route, tff_moe_plan and tff_moe_gather leave
-// them (place_of_pair and lane_group may be null), and token_of_row: sorted place -> row of the step's tokens.
+// them (place_of_pair and lane_group may be null), and token_of_row: sorted place -> row of the step's tokens.  With table null
+// pair_expert is the choice that tff_moe_route left, and its ``counts`` are set back to zero.
 TFF_API int tff_moe_table(const int* tokens, const int* table, int table_rows, int P, int top, int E, int tile_rows,
                           int pad_rows, int* pair_expert, float* pair_weight, int* row_map, int* token_of_row,
                           int* place_of_pair, int* tile_group, int* tile_row0, int* tile_row_end, int* num_tiles,
-                          int* lane_group, int lane_tiles, cudaStream_t stream) {
+                          int* lane_group, int lane_tiles, int* counts, cudaStream_t stream) {
     if (P <= 0) return TFF_OK;
-    if (!tokens || !table || table_rows <= 0 || top <= 0 || P % top || E <= 0 || tile_rows <= 0 || pad_rows < 0 ||
+    if ((table ? !tokens || table_rows <= 0 : !counts) || top <= 0 || P % top || E <= 0 || tile_rows <= 0 || pad_rows < 0 ||
         (pad_rows > 0 && pad_rows != tile_rows) || (lane_group && pad_rows <= 0) || !pair_expert || !pair_weight || !row_map ||
         !token_of_row || !tile_group || !tile_row0 || !tile_row_end || !num_tiles)
         return TFF_ERR_BAD_ARGUMENT;
@@ -426,7 +515,7 @@ TFF_API int tff_moe_table(const int* tokens, const int* table, int table_rows, i
     if (smem > 48 * 1024) return TFF_ERR_UNSUPPORTED;
     return tff_launch_pdl(moe_table_kernel, dim3(1), dim3(TABLE_THREADS), smem, stream, tokens, table, table_rows, P, top, E,
                           tile_rows, pad_rows, pair_expert, pair_weight, row_map, token_of_row, place_of_pair, tile_group,
-                          tile_row0, tile_row_end, num_tiles, lane_group, lane_tiles);
+                          tile_row0, tile_row_end, num_tiles, lane_group, lane_tiles, counts);
 }
 
 TFF_API int tff_moe_spread(const void* h, int h_dt, int pairs, int W, int top, const int* place_of_pair, void* x,
@@ -459,10 +548,14 @@ TFF_API int tff_moe_combine(const float* y, int T, int W, int top, const float* 
     if (T <= 0) return TFF_OK;
     if (shared && !shared_w) return TFF_ERR_BAD_ARGUMENT;
     if (pair_expert && (!h || !pair_weight)) return TFF_ERR_BAD_ARGUMENT;
-    dim3 grid(T, (W + 255) / 256);
-    if (h_dt == 1)
-        return tff_launch_pdl(moe_combine_kernel<bf16>, grid, dim3(256), 0, stream, y, W, top, pair_weight, weight_on_output,
-                              place_of_pair, residual, out, pair_expert, (const bf16*)h, shared, shared_w, clear_shared);
-    return tff_launch_pdl(moe_combine_kernel<float>, grid, dim3(256), 0, stream, y, W, top, pair_weight, weight_on_output,
-                          place_of_pair, residual, out, pair_expert, (const float*)h, shared, shared_w, clear_shared);
+    const bool vec = W % 4 == 0 && (((uintptr_t)y | (uintptr_t)residual | (uintptr_t)out | (uintptr_t)h | (uintptr_t)shared) & 15) == 0;
+    const int cols = vec ? W / 4 : W;
+    const dim3 grid(T, (cols + 255) / 256), block(cols < 256 ? (cols + 31) / 32 * 32 : 256);
+#define TFF_COMBINE(TH, VEC)                                                                                          \
+    return tff_launch_pdl(moe_combine_kernel<TH, VEC>, grid, block, 0, stream, y, W, top, pair_weight, weight_on_output, \
+                          place_of_pair, residual, out, pair_expert, (const TH*)h, shared, shared_w, clear_shared)
+    if (h_dt == 1) { if (vec) TFF_COMBINE(bf16, 4); TFF_COMBINE(bf16, 1); }
+    if (vec) TFF_COMBINE(float, 4);
+    TFF_COMBINE(float, 1);
+#undef TFF_COMBINE
 }

@@ -132,6 +132,101 @@ qkv_finish_kernel(TIN* __restrict__ proj, int clear_input, int ld, TQ* __restric
 // Cosines and sines of the token are made once a block, ahead of the wait for the kernel before.
 constexpr int QF_WARPS = 8, QF_MOST_D = 512;
 
+// Heads of at most 128 elements in groups of four: a lane holds four neighbouring elements (16-byte accesses), a pair's other
+// member comes from the lane half/4 away.  A block takes a token, its warps heads in turn.
+template <typename TQ>
+__global__ void __launch_bounds__(QF_WARPS * 32)
+qk_finish4_kernel(float* __restrict__ proj, int clear_input, int ld, TQ* __restrict__ q_out, const float* __restrict__ qw,
+                  const float* __restrict__ kw, float eps, const float* __restrict__ bias, int v_is_k,
+                  const float* __restrict__ freq, int rot_dims, float magnitude,
+                  const int* __restrict__ positions, const int* __restrict__ tok_req, const int* __restrict__ block_table,
+                  int table_width, TQ* __restrict__ cache, KvLayout L, int layer, int dc, int nq, int nkv, int d) {
+    __shared__ float4 cs[16], sn[16];
+    pdl_launch_dependents();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int t = blockIdx.y, half = rot_dims >> 1, h4 = half >> 2, pos = positions[t], d4 = d >> 2;
+    if (threadIdx.x < half) {
+        float s, c;
+        sincosf((float)pos * freq[threadIdx.x], &s, &c);
+        reinterpret_cast<float*>(sn)[threadIdx.x] = s * magnitude; reinterpret_cast<float*>(cs)[threadIdx.x] = c * magnitude;
+    }
+    const int page = block_table[(size_t)tok_req[t] * table_width + pos / L.page_size];
+    TQ* slots = cache + (size_t)page * L.page_stride + (size_t)layer * L.layer_stride + (size_t)(pos % L.page_size) * dc;
+    const bool on = lane < d4;
+    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f), one = make_float4(1.f, 1.f, 1.f, 1.f);
+    const float4 wq = on && qw ? reinterpret_cast<const float4*>(qw)[lane] : one;
+    const float4 wk = on && kw ? reinterpret_cast<const float4*>(kw)[lane] : one;
+    __syncthreads();
+    const bool turned = lane < 2 * h4, first = lane < h4;
+    const float4 c4 = turned ? cs[first ? lane : lane - h4] : one, s4 = turned ? sn[first ? lane : lane - h4] : zero;
+    const int partner = first ? lane + h4 : lane - h4;
+    const int heads = nq + nkv;
+    pdl_wait();
+    float4* row = reinterpret_cast<float4*>(proj + (size_t)t * ld);
+    auto store = [](TQ* p, float4 v) {
+        if constexpr (sizeof(TQ) == 2) {
+            __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+            uint2 u;
+            u.x = *reinterpret_cast<uint32_t*>(&lo); u.y = *reinterpret_cast<uint32_t*>(&hi);
+            *reinterpret_cast<uint2*>(p) = u;
+        } else {
+            *reinterpret_cast<float4*>(p) = v;
+        }
+    };
+    constexpr int N = 4;                                          // heads of a warp in flight
+    for (int h0 = blockIdx.x * QF_WARPS + warp; h0 < heads; h0 += N * gridDim.x * QF_WARPS) {
+        float4 u[N];
+#pragma unroll
+        for (int n = 0; n < N; ++n) {
+            const int head = h0 + n * gridDim.x * QF_WARPS;
+            u[n] = on && head < heads ? __ldcg(row + head * d4 + lane) : zero;
+        }
+#pragma unroll
+        for (int n = 0; n < N; ++n) {
+            const int head = h0 + n * gridDim.x * QF_WARPS;
+            if (head >= heads) continue;                          // (the same for the whole warp)
+            if (on && bias) {
+                const float4 b = reinterpret_cast<const float4*>(bias)[head * d4 + lane];
+                u[n].x += b.x; u[n].y += b.y; u[n].z += b.z; u[n].w += b.w;
+            }
+            if (on && clear_input) row[head * d4 + lane] = zero;
+            const bool is_q = head < nq;
+            float4 v = u[n];
+            if (qw) {
+                const float ss = warp_sum(v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w);
+                const float rs = rsqrtf(ss / (float)d + eps);
+                const float4 w = is_q ? wq : wk;
+                v = make_float4(v.x * rs * w.x, v.y * rs * w.y, v.z * rs * w.z, v.w * rs * w.w);
+            }
+            float4 o;                                             // (every lane takes part in the exchange)
+            o.x = __shfl_sync(0xffffffffu, v.x, partner & 31); o.y = __shfl_sync(0xffffffffu, v.y, partner & 31);
+            o.z = __shfl_sync(0xffffffffu, v.z, partner & 31); o.w = __shfl_sync(0xffffffffu, v.w, partner & 31);
+            if (turned) {
+                const float sg = first ? -1.f : 1.f;
+                v = make_float4(v.x * c4.x + sg * o.x * s4.x, v.y * c4.y + sg * o.y * s4.y, v.z * c4.z + sg * o.z * s4.z,
+                                v.w * c4.w + sg * o.w * s4.w);
+            }
+            if (!on) continue;
+            if (is_q) { store(q_out + ((size_t)t * nq + head) * d + 4 * lane, v); continue; }
+            if (page < 0) continue;                               // no page: the host never schedules this
+            TQ* slot = slots + (size_t)(head - nq) * L.head_stride;
+            store(slot + 4 * lane, v);
+            if (v_is_k) store(slot + L.kv_stride + 4 * lane, u[n]);
+        }
+    }
+    if (v_is_k || page < 0) return;
+    for (int g = blockIdx.x * QF_WARPS + warp; g < nkv; g += gridDim.x * QF_WARPS) {          // values of their own, of d elements
+        if (!on) continue;
+        float4 u = __ldcg(row + (heads + g) * d4 + lane);
+        if (bias) {
+            const float4 b = reinterpret_cast<const float4*>(bias)[(heads + g) * d4 + lane];
+            u.x += b.x; u.y += b.y; u.z += b.z; u.w += b.w;
+        }
+        if (clear_input) row[(heads + g) * d4 + lane] = zero;
+        store(slots + (size_t)g * L.head_stride + L.kv_stride + 4 * lane, u);
+    }
+}
+
 template <typename TQ, int RJ>        // RJ: registers an element array takes, d <= 32 * RJ
 __global__ void __launch_bounds__(QF_WARPS * 32)
 qk_finish_kernel(float* __restrict__ proj, int clear_input, int ld, TQ* __restrict__ q_out, const float* __restrict__ qw,
@@ -233,6 +328,19 @@ TFF_API int tff_qk_finish(
     const KvLayout L = make_kv_layout(cache_layers, nkv, page_size, dc);
     const int heads = nq + (v_is_k ? nkv : 2 * nkv);
     const dim3 grid((heads + QF_WARPS - 1) / QF_WARPS, num_tokens);
+    const int elt = q_dt == 1 ? 2 : 4;
+    if (d <= 128 && d % 4 == 0 && dv == d && rot_dims % 8 == 0 && !interleaved && ld % 4 == 0 && dc % 4 == 0 &&
+        (((uintptr_t)proj | (uintptr_t)bias | (uintptr_t)qw | (uintptr_t)kw) & 15) == 0 &&
+        (((uintptr_t)q_out | (uintptr_t)cache) & (4 * elt - 1)) == 0) {
+        const dim3 grid4(num_tokens > 256 ? 1 : (nq + nkv + QF_WARPS - 1) / QF_WARPS, num_tokens);
+#define TFF_QF4(TQ)                                                                                                   \
+        return tff_launch_pdl(qk_finish4_kernel<TQ>, grid4, dim3(QF_WARPS * 32), 0, stream, proj, clear_input, ld, (TQ*)q_out, \
+                              qw, kw, eps, bias, v_is_k, freq, rot_dims, magnitude, positions, tok_req, block_table,  \
+                              table_width, (TQ*)cache, L, layer, dc, nq, nkv, d)
+        if (q_dt == 1) TFF_QF4(bf16);
+        TFF_QF4(float);
+#undef TFF_QF4
+    }
 #define TFF_QF(TQ, RJ)                                                                                                \
     return tff_launch_pdl(qk_finish_kernel<TQ, RJ>, grid, dim3(QF_WARPS * 32), 0, stream, proj, clear_input, ld, (TQ*)q_out, \
                           qw, kw, eps, bias, v_is_k, freq, rot_dims, magnitude, interleaved, positions, tok_req,      \

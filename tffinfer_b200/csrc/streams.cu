@@ -196,23 +196,22 @@ template <> __device__ __forceinline__ float4 load_z4<bf16>(const bf16* p) {
 
 template <typename TO, typename TZ, int NT>
 __global__ void __launch_bounds__(NT)
-gated_join_kernel(float* __restrict__ x, int W, TZ* __restrict__ z, const float* __restrict__ b, float* __restrict__ y1,
+gated_join_kernel(float* __restrict__ x, int W, TZ* __restrict__ z, int zld, const float* __restrict__ b, float* __restrict__ y1,
                   const float* __restrict__ c1, float* __restrict__ y2, int clear, const float* __restrict__ w, float eps,
                   const int* __restrict__ row_index, TO* __restrict__ h) {
     extern __shared__ __align__(16) float u_row[];   // W floats: the new row, kept between the two passes
     __shared__ float red[32];
     pdl_launch_dependents();
     const int r = blockIdx.x, row = row_index ? row_index[r] : r;
-    const int zw = y2 ? 2 * W : W;
     float* xr = x + (size_t)row * W;
     float* y1r = y1 + (size_t)row * W;
     float* y2r = y2 ? y2 + (size_t)row * W : nullptr;
-    TZ* zr = z + (size_t)row * zw;
+    TZ* zr = z + (size_t)row * zld;
     const bool store_x = row_index == nullptr;
     pdl_wait();
     float ss = 0.f;
     const bool vec = (W & 3) == 0 && (((uintptr_t)x | (uintptr_t)y1 | (uintptr_t)y2 | (uintptr_t)b | (uintptr_t)c1 | (uintptr_t)w) & 15) == 0 &&
-                     ((uintptr_t)z & (4 * sizeof(TZ) - 1)) == 0 && ((uintptr_t)h & (4 * sizeof(TO) - 1)) == 0;
+                     ((uintptr_t)z & (4 * sizeof(TZ) - 1)) == 0 && (zld & 3) == 0 && ((uintptr_t)h & (4 * sizeof(TO) - 1)) == 0;
     const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
     if (vec) {
         const int W4 = W >> 2;
@@ -331,13 +330,13 @@ TFF_API int tff_stream_step(float* x, int S, int W, float* y, int clear_y, const
 #undef TFF_STREAM_LAUNCH_S
 }
 
-// x [rows_total, W] float32, updated in place; z [rows_total, 2 W] (W without y2), z_is_bf16; b float32 of z's width; y1, y2
+// x [rows_total, W] float32, updated in place; z [rows_total, 2 W] (W without y2), rows zld apart, z_is_bf16; b float32 of z's width; y1, y2
 // [rows_total, W] float32 (y2 may be null); c1 [W] or null; h [rows, W] or null, then w [W] may be null too.
-TFF_API int tff_gated_join(float* x, int W, void* z, int z_is_bf16, const float* b, float* y1, const float* c1, float* y2,
+TFF_API int tff_gated_join(float* x, int W, void* z, int zld, int z_is_bf16, const float* b, float* y1, const float* c1, float* y2,
                            int clear, const float* w, float eps, const int* row_index, void* h, int h_is_bf16, int rows,
                            cudaStream_t stream) {
     if (rows <= 0) return TFF_OK;
-    if (!x || !z || !b || !y1 || W <= 0 || (h && !w) || (row_index && clear) || ((clear & 4) && z_is_bf16) ||
+    if (!x || !z || !b || !y1 || W <= 0 || zld < (y2 ? 2 * W : W) || (h && !w) || (row_index && clear) || ((clear & 4) && z_is_bf16) ||
         ((clear & 2) && !y2))
         return TFF_ERR_BAD_ARGUMENT;
     const size_t smem = (size_t)W * sizeof(float);
@@ -347,7 +346,7 @@ TFF_API int tff_gated_join(float* x, int W, void* z, int z_is_bf16, const float*
         auto kern = gated_join_kernel<TO, TZ, NT>;                                                                  \
         if (smem > 48 * 1024 && cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 96 * 1024) != cudaSuccess) \
             return TFF_ERR_LAUNCH;                                                                                  \
-        return tff_launch_pdl(kern, dim3(rows), dim3(NT), smem, stream, x, W, (TZ*)z, b, y1, c1, y2, clear, w, eps,  \
+        return tff_launch_pdl(kern, dim3(rows), dim3(NT), smem, stream, x, W, (TZ*)z, zld, b, y1, c1, y2, clear, w, eps,  \
                               row_index, (TO*)h);                                                                   \
     } while (0)
 #define TFF_JOIN_N(TO, TZ)                                                                                          \

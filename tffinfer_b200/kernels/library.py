@@ -412,6 +412,11 @@ class CudaKernels:
         that writes it needs no clearing kernel; else plain scratch.  Outputs that wait side by side have a ``use`` each."""
         return self.projection_buffer(rows, width, device, act_dtype, use)
 
+    def joins_products(self, h) -> bool:
+        """Whether products of these rows with several matrices are better run as one: in decode-sized steps, which are
+        passes over the weights."""
+        return h.dtype == torch.bfloat16 and h.shape[0] <= self.SWAP_MAX_M
+
     def gate_rows(self, rows: int, width: int, device, act_dtype) -> torch.Tensor:
         """A [rows, width] buffer for the gates of a gated residual, which ``gated_join`` reads (and clears): float32
         accumulators in decode-sized steps, the activation type above."""
@@ -420,17 +425,17 @@ class CudaKernels:
         return self.projection_buffer(rows, width, device, act_dtype, use="residual gates")
 
     def gated_join(self, x, gates, gate_bias, y1, y1_bias=None, y2=None, norm_weight=None, eps: float = 0.0, h=None,
-                   row_index=None) -> None:
+                   row_index=None, gate_col: int = 0) -> None:
         """x float32 [T, W] += (y1 + y1_bias) * sigmoid(gates[:, :W] + b) + y2 * sigmoid(gates[:, W:] + b') in place, and,
-        with ``h`` ([rows, W], activation type), h = rmsnorm(x) with ``norm_weight`` and ``eps``.  ``gates`` [T, W or 2W]
-        float32 or bfloat16, ``gate_bias`` float32 of its width; y1, y2 float32 [T, W].  ``row_index`` (int32 [rows]): only
+        with ``h`` ([rows, W], activation type), h = rmsnorm(x) with ``norm_weight`` and ``eps``.  ``gates`` [T, >= W or 2W]
+        float32 or bfloat16 from column ``gate_col`` on (the last columns of its rows), ``gate_bias`` float32 of its width; y1, y2 float32 [T, W].  ``row_index`` (int32 [rows]): only
         those rows feed h, and x stays as it was.  Accumulator buffers that are kept at zero are cleared behind the read."""
         self._need_cuda(x, gates, gate_bias, y1, y1_bias, y2, norm_weight, h, row_index)
         T, W = x.shape
         width = 2 * W if y2 is not None else W
         assert x.dtype == y1.dtype == gate_bias.dtype == torch.float32 and tuple(y1.shape) == (T, W)
         assert y2 is None or (y2.dtype == torch.float32 and tuple(y2.shape) == (T, W))
-        assert tuple(gates.shape) == (T, width) and gate_bias.numel() == width
+        assert gates.shape[0] == T and gates.shape[1] == gate_col + width and gate_bias.numel() == width
         assert y1_bias is None or (y1_bias.dtype == torch.float32 and y1_bias.numel() == W)
         rows = T if row_index is None else row_index.numel()
         assert row_index is None or row_index.dtype == torch.int32
@@ -442,7 +447,8 @@ class CudaKernels:
                     clear |= bit
                 self._acc_zero[t.data_ptr()] = row_index is None
         self._check(self.lib.tff_gated_join(
-            _ptr(x), _c_int(W), _ptr(gates), _c_int(_dt(gates)), _ptr(gate_bias), _ptr(y1), _ptr(y1_bias), _ptr(y2),
+            _ptr(x), _c_int(W), _vp(gates.data_ptr() + gate_col * gates.element_size()), _c_int(gates.shape[1]),
+            _c_int(_dt(gates)), _ptr(gate_bias), _ptr(y1), _ptr(y1_bias), _ptr(y2),
             _c_int(clear), _ptr(norm_weight), _c_float(eps), _ptr(row_index), _ptr(h),
             _c_int(_dt(h)) if h is not None else _c_int(0), _c_int(rows), self._stream()), "gated_join")
         self.launches += 1
@@ -615,12 +621,12 @@ class CudaKernels:
         self.launches += 1
 
     def qk_finish(self, proj, q_out, norm, eps: float, bias, values_are_keys: bool, freq, batch, block_table, kv_cache,
-                  kv_layer, page_size, nq, nkv, d, dv) -> None:
+                  kv_layer, page_size, nq, nkv, d, dv, last_reader: bool = True) -> None:
         """proj float32 [T, ld] = [q (nq*d) | k (nkv*d) | v (nkv*dv), unless ``values_are_keys``] -> the queries, each head
         normed (``norm`` = (q, k weights float32 [d]) or None) and turned, in ``q_out`` [T, nq*d]; keys the same way and
         values into the tokens' cache slots, the values of ``values_are_keys`` being the keys as projected.  ``bias`` float32
         over the columns, added first; ``freq`` = (frequencies, rot_dim, magnitude, interleaved) or None.  An accumulator
-        buffer that is kept at zero is cleared."""
+        buffer that is kept at zero is cleared (``last_reader``: nobody reads columns behind these)."""
         qw, kw = norm if norm is not None else (None, None)
         self._need_cuda(proj, q_out, qw, kw, bias, block_table)
         T, ld = proj.shape
@@ -639,13 +645,13 @@ class CudaKernels:
             _ptr(batch.positions), _ptr(batch.tok_req), _ptr(block_table), _c_int(block_table.shape[1]), c_ptr,
             _c_int(c_layers), _c_int(c_layer), _c_int(page_size), _c_int(kv_cache.shape[-1]), _c_int(T), _c_int(nq),
             _c_int(nkv), _c_int(d), _c_int(dv), self._stream()), "qk_finish")
-        if clear:
+        if clear and last_reader:
             self._acc_zero[proj.data_ptr()] = True
         self.launches += 1
 
     def attend_gated(self, h, w_in, freq, batch, block_table, kv_cache, kv_layer, page_size, out, nq, nkv, d, dv,
                      scale, window, softcap, sink, v_mode, v_share, lam, gate_off, write_cache, pre=None, heads=None,
-                     keep: int = 0) -> None:
+                     keep: int = 0, proj=None) -> None:
         """The whole of a gated, capped, sink attention between its input rows and its output projection: one product
         for q, k, v and the head gates (``w_in`` rows [q | k | v | gates | padding]); rotation, value mixing, cache
         write and sigmoid of the gates; attention over the paged cache with the cap, the window, the sink and the
@@ -653,20 +659,23 @@ class CudaKernels:
         over the whole projection or None), eps, state): a short causal convolution over time on the projected q, k, v
         and an RMS norm of all of q and of all of k, between the product and the rotation (short_conv_norm).  ``heads`` =
         dict(bias, norm=(q, k weights [d] or None), eps, values_are_keys): biases, per-head norms and values that are the
-        keys as projected (qk_finish).  ``keep``: the first so many positions stay visible beside the window."""
+        keys as projected (qk_finish).  ``keep``: the first so many positions stay visible beside the window.  ``proj``
+        (with ``heads``): rows whose first columns hold the product already; somebody else reads the others behind this."""
         if not write_cache:
             raise KernelError("attend_gated writes the keys and values it attends to; a borrowed cache is not supported")
         T = h.shape[0]
         if isinstance(h, DeferredNorm):
             h = h.materialize()
-        proj = self.projection_buffer(T, w_in.shape[0], h.device, h.dtype)
-        self.gemm(h, w_in, proj)
+        last_reader = proj is None
+        if proj is None:
+            proj = self.projection_buffer(T, w_in.shape[0], h.device, h.dtype)
+            self.gemm(h, w_in, proj)
         q = torch.empty((T, nq * d), dtype=out.dtype, device=out.device)
         gates = torch.empty((T, nq), dtype=torch.float32, device=out.device) if gate_off >= 0 else None
         if heads is not None:
             self.qk_finish(proj, q, heads.get("norm"), float(heads.get("eps", 0.0)), heads.get("bias"),
                            bool(heads.get("values_are_keys")), freq, batch, block_table, kv_cache, kv_layer, page_size, nq,
-                           nkv, d, dv)
+                           nkv, d, dv, last_reader)
             self.attention_ext(q, batch, block_table, kv_cache, kv_layer, page_size, out, nq, nkv, d, dv, scale, window,
                                softcap, sink, gates, keep)
             return
@@ -836,30 +845,47 @@ class CudaKernels:
 
     MLSTM_MMA = os.environ.get("TFFINFER_MLSTM_MMA", "1") != "0"   # 0: prompts token by token, as float32 FMAs
 
-    def mlstm(self, h, w_in, batch, state, gate_bias, cap: float, norm_w, eps: float, out, H, K, V) -> None:
+    def mlstm(self, h, w_in, batch, state, gate_bias, cap: float, norm_w, eps: float, out, H, K, V, proj=None) -> None:
         """The whole of an mLSTM mixer between its input rows and its output projection -> out [T, H*V]: one product
         (``w_in`` rows [q | k | v | gate | input gates | forget gates | padding]) into float32; the recurrence over ``state``
-        (mlstm_recurrence); per-head RMS norm, weight and sigmoid gate."""
+        (mlstm_recurrence); per-head RMS norm, weight and sigmoid gate, in the recurrence's kernel where that runs token by
+        token.  ``proj``: rows whose first columns hold that product already; somebody else reads the others behind this."""
         T = h.shape[0]
         if isinstance(h, DeferredNorm):
             h = h.materialize()
-        proj = self.projection_buffer(T, w_in.shape[0], h.device, h.dtype)
-        self.gemm(h, w_in, proj)
+        last_reader = proj is None
+        if proj is None:
+            proj = self.projection_buffer(T, w_in.shape[0], h.device, h.dtype)
+            self.gemm(h, w_in, proj)
+        g_off = 2 * H * K + H * V
+        if not (h.dtype == torch.bfloat16 and self.MLSTM_MMA and batch.max_q_len > 1):
+            self.mlstm_recurrence(proj, state, batch, gate_bias, cap, None, H, K, V, finish=(g_off, norm_w, eps, out))
+            if last_reader and proj.data_ptr() in self._acc_zero:
+                self._acc_zero[proj.data_ptr()] = True
+            return
         o = torch.empty((T, H * V), dtype=torch.float32, device=h.device)
-        self.mlstm_recurrence(proj, state, batch, gate_bias, cap, o, H, K, V, rounded=h.dtype == torch.bfloat16)
-        self.gated_norm(o, V, proj, 2 * H * K + H * V, norm_w, eps, False, out, clear_cols=(0, proj.shape[1]),
-                        last_reader=True, gate_act="sigmoid")
+        self.mlstm_recurrence(proj, state, batch, gate_bias, cap, o, H, K, V, rounded=True)
+        self.gated_norm(o, V, proj, g_off, norm_w, eps, False, out, clear_cols=(0, w_in.shape[0]), last_reader=last_reader,
+                        gate_act="sigmoid")
 
     def mlstm_recurrence(self, proj, state, batch, gate_bias, cap: float, out, H, K, V, rounded: bool = False,
-                         chunked: Optional[bool] = None) -> None:
+                         chunked: Optional[bool] = None, finish=None) -> None:
         """proj float32 [T, ld] = [q H*K | k H*K | v H*V | H*V others | input gates H | forget gates H | ...] -> o float32
         [T, H*V] of the recurrence that parts/mlstm.py states, q scaled by K^-1/2; ``gate_bias`` float32 [2H], ``state``
         float32 [slots, mlstm_state_size(H, K, V)].  ``rounded``: q, k and v may be rounded to bfloat16, and portions of
         prompts run chunk by chunk on the tensor cores (``chunked`` None: when some request brings more than one token);
-        everything else runs token by token in float32.  ``proj`` is left as it is."""
-        self._need_cuda(proj, state, gate_bias, out)
+        everything else runs token by token in float32.  ``proj`` is left as it is.  ``finish`` = (first gate column, norm_w,
+        eps, mixed [T, H*V]): token by token only, on to the mixer's output (``out`` None), and an accumulator buffer that is
+        kept at zero is cleared where it was read."""
+        g_off, norm_w, eps, mixed = finish if finish is not None else (0, None, 0.0, None)
+        self._need_cuda(proj, state, gate_bias, out, norm_w, mixed)
         T, ld = proj.shape
-        assert proj.dtype == state.dtype == gate_bias.dtype == out.dtype == torch.float32 and tuple(out.shape) == (T, H * V)
+        assert proj.dtype == state.dtype == gate_bias.dtype == torch.float32
+        if finish is None:
+            assert out.dtype == torch.float32 and tuple(out.shape) == (T, H * V)
+        else:
+            assert not rounded and not chunked and tuple(mixed.shape) == (T, H * V) and norm_w.numel() == H * V
+        clear = 1 if finish is not None and proj.data_ptr() in self._acc_zero else 0
         assert state.dim() == 2 and state.shape[1] == mlstm_state_size(H, K, V) and gate_bias.numel() == 2 * H
         gates = 2 * H * K + 2 * H * V
         assert ld >= gates + 2 * H
@@ -876,7 +902,9 @@ class CudaKernels:
                 _ptr(proj), _c_int(ld), _c_int(0), _c_int(H * K), _c_int(2 * H * K), _c_int(gates), _c_int(gates + H),
                 _ptr(gate_bias), _c_float(cap), _c_float(float(K) ** -0.5), _ptr(state), _c_int(state.shape[0]),
                 _c_int(state.shape[1]), _ptr(batch.q_start), _ptr(batch.pos_start), _ptr(batch.slots), _ptr(out),
-                _c_int(batch.num_requests), _c_int(H), _c_int(K), _c_int(V), _c_int(ch), _ptr(ws), _c_int(T), self._stream())
+                _c_int(batch.num_requests), _c_int(H), _c_int(K), _c_int(V), _c_int(ch), _ptr(ws), _c_int(T), _ptr(proj),
+                _c_int(g_off), _ptr(norm_w), _c_float(eps), _ptr(mixed), _c_int(_dt(mixed) if mixed is not None else 0),
+                _c_int(clear), self._stream())
         status = run(1) if chunked else -2
         if status == -2:                     # a head may be too large for the chunk form's shared memory
             chunked = False
@@ -1263,6 +1291,9 @@ class CudaKernels:
         if by_table:             # the product reads the tokens' rows where they are
             pair_weight, row_map, tiles, a_rows = self.moe_table(router, T, top, E, tile_rows)
             x, pe = h, []
+        elif weight_on == "output" and not identity and P <= self.CHOOSE_MOST:
+            pair_weight, row_map, tiles, a_rows = self.moe_choose(h, w_router, top, renormalize, tile_rows, router)
+            x, pe = h, []
         else:
             pair_weight, row_map, tiles, x, *pe = self.moe_dispatch(h, w_router, top, renormalize, weight_on == "input",
                                                                     tile_rows, router=router)
@@ -1313,15 +1344,7 @@ class CudaKernels:
         r = router or {}
         identity = int(r.get("identity", 0))
         E = w_router.shape[0] - identity                          # experts that have rows
-        groups, keep = r.get("groups") or (1, 1)
-        correction = r.get("correction")
-        self._need_cuda(correction)
-        assert correction is None or (correction.dtype == torch.float32 and correction.numel() == E + identity)
         dev, P = h.device, T * top
-        counts = self._moe_counts.get((E, str(dev)))
-        if counts is None:
-            counts = torch.zeros(E, dtype=torch.int32, device=dev)       # set back to zero by the plan kernel
-            self._moe_counts[(E, str(dev))] = counts
         bm = tile_rows or self.grouped_tile_rows(False)      # rows of a tile of the grouped product that follows
         max_tiles = -(-P // bm) + E
         R = max(P, padded_rows)                              # rows of the sorted order
@@ -1333,18 +1356,7 @@ class CudaKernels:
         num_tiles = ints[o + 3 * max_tiles:o + 3 * max_tiles + 1]
         lane_group = ints[o + 3 * max_tiles + 1:o + 3 * max_tiles + 1 + lane_tiles] if padded_rows else None
         place = ints[o + 3 * max_tiles + 1 + lane_tiles:] if padded_rows else None
-        pair_weight = torch.empty(P, dtype=torch.float32, device=dev)
-        bias = r.get("bias")
-        self._need_cuda(bias)
-        assert bias is None or (bias.dtype == torch.float32 and bias.numel() == E + identity)
-        row, row_out = r.get("row"), r.get("row_out")
-        self._need_cuda(row, row_out)
-        assert row is None or (row.dtype == w_router.dtype and row.numel() == W and row_out.numel() == T)
-        self._check(self.lib.tff_moe_route(_ptr(h), _c_int(_dt(h)), _ptr(w_router), _c_int(_dt(w_router)), _ptr(bias), _c_int(T), _c_int(W),
-                                           _c_int(E + identity), _c_int(top), _c_int(1 if renormalize else 0),
-                                           _c_int({"sigmoid": 0, "softmax": 1, "softmax_chosen": 2}[r.get("score", "sigmoid")]), _ptr(correction),
-                                           _c_int(int(groups)), _c_int(int(keep)), _c_int(E), _ptr(pair_expert),
-                                           _ptr(pair_weight), _ptr(counts), _ptr(row), _ptr(row_out), self._stream()), "moe_route")
+        pair_weight, counts = self._moe_route(h, w_router, top, renormalize, r, pair_expert)
         self._check(self.lib.tff_moe_plan(_ptr(counts), _c_int(E), _c_int(bm), _ptr(cursor), _ptr(tile_group), _ptr(tile_row0),
                                           _ptr(tile_row_end), _ptr(num_tiles), _c_int(bm if padded_rows else 0),
                                           _ptr(lane_group), _c_int(lane_tiles), self._stream()), "moe_plan")
@@ -1352,12 +1364,55 @@ class CudaKernels:
         self._check(self.lib.tff_moe_gather(_ptr(h), _c_int(_dt(h)), _c_int(P), _c_int(W), _c_int(top), _ptr(pair_expert),
                                             _ptr(pair_weight), _c_int(1 if scale_rows else 0), _ptr(cursor),
                                             _ptr(row_map), _ptr(place), _ptr(x), self._stream()), "moe_gather")
-        self.launches += 3
+        self.launches += 2
         tiles = (tile_group, tile_row0, tile_row_end, num_tiles, max_tiles, bm)
         extra = (pair_expert,) if identity else ()
         if padded_rows:
             return (pair_weight, row_map, tiles, x, lane_group, place) + extra
         return (pair_weight, row_map, tiles, x) + extra
+
+    def _moe_route(self, h, w_router, top: int, renormalize: bool, r: dict, pair_expert):
+        """Scores and choice (csrc/moe.cu: route) into ``pair_expert`` int32 [T*top]: (pair_weight, the experts' counters)."""
+        T, W = h.shape
+        identity = int(r.get("identity", 0))
+        E = w_router.shape[0] - identity                          # experts that have rows
+        groups, keep = r.get("groups") or (1, 1)
+        correction, bias, row, row_out = r.get("correction"), r.get("bias"), r.get("row"), r.get("row_out")
+        self._need_cuda(correction, bias, row, row_out)
+        for v in (correction, bias):
+            assert v is None or (v.dtype == torch.float32 and v.numel() == E + identity)
+        assert row is None or (row.dtype == w_router.dtype and row.numel() == W and row_out.numel() == T)
+        counts = self._moe_counts.get((E, str(h.device)))
+        if counts is None:
+            counts = torch.zeros(E, dtype=torch.int32, device=h.device)  # set back to zero by the kernel behind the route
+            self._moe_counts[(E, str(h.device))] = counts
+        pair_weight = torch.empty(T * top, dtype=torch.float32, device=h.device)
+        self._check(self.lib.tff_moe_route(_ptr(h), _c_int(_dt(h)), _ptr(w_router), _c_int(_dt(w_router)), _ptr(bias), _c_int(T), _c_int(W),
+                                           _c_int(E + identity), _c_int(top), _c_int(1 if renormalize else 0),
+                                           _c_int({"sigmoid": 0, "softmax": 1, "softmax_chosen": 2}[r.get("score", "sigmoid")]), _ptr(correction),
+                                           _c_int(int(groups)), _c_int(int(keep)), _c_int(E), _ptr(pair_expert),
+                                           _ptr(pair_weight), _ptr(counts), _ptr(row), _ptr(row_out), self._stream()), "moe_route")
+        self.launches += 1
+        return pair_weight, counts
+
+    CHOOSE_MOST = 8192       # pairs that one block sorts by expert
+
+    def moe_choose(self, h, w_router, top: int, renormalize: bool, tile_rows: int, router=None):
+        """moe_dispatch for steps of few pairs whose products read the tokens' rows where they are: (pair_weight, row_map, the
+        tile table, a_rows int32: sorted place -> token row).  Two launches: route, and one block that sorts."""
+        r = router or {}
+        assert not r.get("identity")
+        T, P, E, dev = h.shape[0], h.shape[0] * top, w_router.shape[0], h.device
+        max_tiles = -(-P // tile_rows) + E
+        ints = torch.empty(3 * P + 3 * max_tiles + 1, dtype=torch.int32, device=dev)
+        pair_expert, row_map, a_rows, tg, tr0, tre, nt = ints.split([P, P, P, max_tiles, max_tiles, max_tiles, 1])
+        pair_weight, counts = self._moe_route(h, w_router, top, renormalize, r, pair_expert)
+        self._check(self.lib.tff_moe_table(
+            _vp(0), _vp(0), _c_int(0), _c_int(P), _c_int(top), _c_int(E), _c_int(tile_rows), _c_int(0), _ptr(pair_expert),
+            _ptr(pair_weight), _ptr(row_map), _ptr(a_rows), _vp(0), _ptr(tg), _ptr(tr0), _ptr(tre), _ptr(nt), _vp(0), _c_int(0),
+            _ptr(counts), self._stream()), "moe_table")
+        self.launches += 1
+        return pair_weight, row_map, (tg, tr0, tre, nt, max_tiles, tile_rows), a_rows
 
     def moe_table(self, router, T: int, top: int, E: int, tile_rows: int, padded_rows: int = 0):
         """The choice and sorting of a routed feed-forward whose experts a table gives: ``router`` = dict(table=int32
@@ -1379,7 +1434,7 @@ class CudaKernels:
         self._check(self.lib.tff_moe_table(
             _ptr(tokens), _ptr(table), _c_int(table.shape[0]), _c_int(P), _c_int(top), _c_int(E), _c_int(bm),
             _c_int(bm if padded_rows else 0), _ptr(pair_expert), _ptr(pair_weight), _ptr(row_map), _ptr(a_rows), _ptr(place),
-            _ptr(tg), _ptr(tr0), _ptr(tre), _ptr(nt), _ptr(lane_group), _c_int(lane_tiles), self._stream()), "moe_table")
+            _ptr(tg), _ptr(tr0), _ptr(tre), _ptr(nt), _ptr(lane_group), _c_int(lane_tiles), _vp(0), self._stream()), "moe_table")
         self.launches += 1
         tiles = (tg, tr0, tre, nt, max_tiles, bm)
         return (pair_weight, row_map, tiles, a_rows) + ((lane_group, place) if padded_rows else ())

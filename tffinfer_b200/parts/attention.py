@@ -238,7 +238,11 @@ class GatedSinkAttention(Mixer):
         if self.qk_norm != "none":
             self.norm_w = (tensors[n["q_norm"]].to(torch.float32).contiguous(), tensors[n["k_norm"]].to(torch.float32).contiguous())
 
-    def forward(self, h, ctx: LayerContext, residual):
+    @property
+    def takes_projection(self) -> bool:
+        return self.head_finish
+
+    def forward(self, h, ctx: LayerContext, residual, proj=None):
         ops, batch = ctx.ops, ctx.batch
         T = h.shape[0]
         freq = ctx.position.frequencies() if ctx.position is not None else None
@@ -263,7 +267,7 @@ class GatedSinkAttention(Mixer):
                          self.softcap, self.sink_w if self.sink == "learned" else self.sink,
                          {"none": 0, "source": 1, "mix": 2}[self.value_mix], share,
                          self.lam if self.value_mix == "mix" else None,
-                         self.gate_off if self.head_gate else -1, ctx.write_cache, pre=pre, heads=heads, keep=self.keep_first)
+                         self.gate_off if self.head_gate else -1, ctx.write_cache, pre=pre, heads=heads, keep=self.keep_first, proj=proj)
         if residual is None:
             out = ops.sublayer_output(T, self.hidden_size, h.device, h.dtype, self.output_use)
             ops.gemm(attn, self.w_o, out)

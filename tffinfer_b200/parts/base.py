@@ -147,6 +147,11 @@ class Mixer(Part):
     output_bias = None    # float32 [hidden] of the output projection, or None.  With ``residual`` None the output comes
                           # WITHOUT it: the arrangement adds it where it joins the output to the residual
 
+    w_in = None           # the rows of the mixer's input product, where it ...
+    takes_projection = False     # ... says that forward(h, ctx, None, proj=rows) takes that product from the first columns of
+                                 # ``rows`` (an arrangement that runs it together with products of its own; the other columns
+                                 # are read behind the mixer)
+
     def cache_need(self):
         return None
 
@@ -258,6 +263,9 @@ class Block:
         self.ffn_norm = ffn_norm
         self.extra_norms = dict(extra_norms or {})
         self.connectors = dict(connectors or {})  # by a name of the arrangement's choosing
+
+    def loaded(self) -> None:
+        """Called when every part has its tensors: an arrangement may put weights of several parts side by side."""
 
     def parts(self):
         named = [self.mixer_norm, self.mixer, self.ffn_norm, self.feed_forward] + list(self.extra_norms.values()) + \

@@ -65,14 +65,16 @@ class MLstm(Mixer):
         self.norm_w = tensors[n["norm"]].to(torch.float32).contiguous()
         self.gate_bias = torch.cat([tensors[n["in_bias"]].to(torch.float32), tensors[n["forget_bias"]].to(torch.float32)]).contiguous()
 
-    def forward(self, h, ctx: LayerContext, residual):
+    takes_projection = True
+
+    def forward(self, h, ctx: LayerContext, residual, proj=None):
         if ctx.state is None:
             raise ValueError("mlstm needs a state tensor (StateNeed)")
         ops = ctx.ops
         T = h.shape[0]
         mixed = torch.empty((T, self.v_width), dtype=h.dtype, device=h.device)
         ops.mlstm(h, self.w_in, ctx.batch, ctx.state, self.gate_bias, self.gate_cap, self.norm_w, self.eps, mixed,
-                  self.num_heads, self.head_dim, self.v_head_dim)
+                  self.num_heads, self.head_dim, self.v_head_dim, proj=proj)
         if residual is None:
             out = ops.sublayer_output(T, self.hidden_size, h.device, h.dtype, self.output_use)
             ops.gemm(mixed, self.w_o, out)

@@ -93,6 +93,8 @@ class Model:
         self.vector_tables = {name: tensors[name].to(torch.float32).contiguous() for name in d.vector_tables}
         for p in self.all_parts():
             p.load({rel: tensors[p.full_name(rel)] for rel in p.weight_specs() if p.full_name(rel) in tensors}, ops, act_dtype)
+        for b in self.blocks:
+            b.loaded()
         for pos in self.positions.values():
             pos.prepare(ops, device, d.max_position)
 
@@ -160,7 +162,10 @@ class Model:
         if R == 0:
             return torch.empty((0, d.vocab_size), dtype=torch.float32, device=self.embed.device)
         if d.streams > 0:
-            hn = x.read(None, self.final_norm, ops, act_dtype, row_index=batch.logit_rows)
+            # a decode step of fixed size asks for every row once, in order: the read may then go on to all rows (and clear
+            # what it reads)
+            rows = None if getattr(batch, "graph_bucket", None) is not None and R == T else batch.logit_rows
+            hn = x.read(None, self.final_norm, ops, act_dtype, row_index=rows)
         else:
             hn = self.final_norm.forward(x, ops, act_dtype, row_index=batch.logit_rows)
         logits = torch.empty((R, d.vocab_size), dtype=torch.float32, device=self.embed.device)

@@ -27,7 +27,7 @@ class ResidualGates(Connector):
         self.hidden_size, self.feed_forward = int(hidden_size), bool(feed_forward)
         self.names = {"mixer": "rg1", "mixer_bias": "rg1.b", "ffn": "rg2", "ffn_bias": "rg2.b"}
         self.names.update(names or {})
-        self.w = self.bias = None
+        self.w = self.bias = self.w_all = None
 
     def weight_specs(self) -> Dict[str, WeightSpec]:
         n, W = self.names, self.hidden_size
@@ -45,6 +45,15 @@ class ResidualGates(Connector):
         self.w = torch.cat([r.to(dt) for r in rows], dim=0).contiguous()
         self.bias = torch.cat([b.to(torch.float32) for b in bias]).contiguous()
 
+    def share_rows(self, mixer) -> None:
+        """Puts the rows of the mixer's input product and those of the gates side by side in one matrix, of which both keep
+        their part: where few tokens make every product a pass over its weights, the two run as one."""
+        if not getattr(mixer, "takes_projection", False) or mixer.w_in.dtype != self.w.dtype:
+            return
+        n = mixer.w_in.shape[0]
+        self.w_all = torch.cat([mixer.w_in, self.w], dim=0).contiguous()
+        mixer.w_in, self.w = self.w_all[:n], self.w_all[n:]
+
     def gates(self, h, ops) -> torch.Tensor:
         """The gates ahead of bias and sigmoid, [T, hidden] or [T, 2 * hidden]."""
         z = ops.gate_rows(h.shape[0], self.w.shape[0], h.device, h.dtype)
@@ -54,8 +63,8 @@ class ResidualGates(Connector):
     def read(self, x: ResidualStreams, norm, ops, out_dtype):
         return x.read(None, norm, ops, out_dtype)
 
-    def write(self, x: ResidualStreams, y, z=None, mixer_bias=None, y_ff=None) -> None:
-        x.write_gated(z, self.bias, y, mixer_bias, y_ff)
+    def write(self, x: ResidualStreams, y, z=None, mixer_bias=None, y_ff=None, gate_col: int = 0) -> None:
+        x.write_gated(z, self.bias, y, mixer_bias, y_ff, gate_col)
 
 
 @register_part("block", "gated_parallel")
@@ -71,11 +80,19 @@ class GatedParallelBlock(Block):
         if feed_forward is not None:
             feed_forward.output_use = "feed-forward behind a gate"
 
+    def loaded(self) -> None:
+        self.connectors["gates"].share_rows(self.mixer)
+
     def forward(self, x: ResidualStreams, ctx: LayerContext, act_dtype):
-        join = self.connectors["gates"]
-        h = join.read(x, self.mixer_norm, ctx.ops, act_dtype)
-        z = join.gates(h, ctx.ops)
-        y = self.mixer.forward(h, ctx, residual=None)
+        join, ops = self.connectors["gates"], ctx.ops
+        h = join.read(x, self.mixer_norm, ops, act_dtype)
+        if join.w_all is not None and ops.joins_products(h):        # one product for the mixer's input and the gates
+            z, col = ops.projection_buffer(h.shape[0], join.w_all.shape[0], h.device, h.dtype, "with gates"), self.mixer.w_in.shape[0]
+            ops.gemm(h, join.w_all, z)
+            y = self.mixer.forward(h, ctx, residual=None, proj=z)
+        else:
+            z, col = join.gates(h, ops), 0
+            y = self.mixer.forward(h, ctx, residual=None)
         f = self.feed_forward.forward(h, ctx, residual=None) if self.feed_forward is not None else None
-        join.write(x, y, z, self.mixer.output_bias, f)
+        join.write(x, y, z, self.mixer.output_bias, f, col)
         return x

@@ -56,13 +56,14 @@ class ResidualStreams:
             self.flush()
         self.pending_bias = vec
 
-    def write_gated(self, gates, gate_bias, y_mixer, mixer_bias, y_ff) -> None:
+    def write_gated(self, gates, gate_bias, y_mixer, mixer_bias, y_ff, gate_col: int = 0) -> None:
         """x <- x + (y_mixer + mixer_bias) * sigmoid(gates[:, :W] + b) + y_ff * sigmoid(gates[:, W:] + b'), for a residual of
-        one stream; like a write, it runs with the next read (ops.gated_join)."""
+        one stream; like a write, it runs with the next read (ops.gated_join).  The gates are the columns of ``gates`` from
+        ``gate_col`` on."""
         if self.x.shape[1] != 1:
             raise ValueError("gated writes are built for one stream")
         self.flush()
-        self.pending_gated = dict(gates=gates, gate_bias=gate_bias, y1=y_mixer, y1_bias=mixer_bias, y2=y_ff)
+        self.pending_gated = dict(gates=gates, gate_bias=gate_bias, y1=y_mixer, y1_bias=mixer_bias, y2=y_ff, gate_col=gate_col)
 
     def _rows(self) -> torch.Tensor:
         return self.x.view(self.x.shape[0], self.x.shape[2])
