@@ -40,7 +40,7 @@ __device__ inline bool find_chunk(const int* __restrict__ q_start, const int* __
 
 
 constexpr int MT = 256;                  // eight warps
-constexpr int SCOLS = 64, SST = SCOLS + 8;     // state columns a CTA of the finish kernel works on, and their row stride
+constexpr int SCOLS = 64;                // state columns a CTA of the finish kernel works on
 
 __host__ __device__ inline int pad16(int x) { return (x + 15) & ~15; }
 __device__ __forceinline__ uint32_t ret_smem(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
@@ -114,7 +114,7 @@ __device__ __forceinline__ void load_rounded(bf16* dst, int stride, const float*
 // and, for weights that ask for them (SUMS), weights.row_sum(i, sum_j weights.pair(i, j) (q_i . k_j)).  The rounded k rows
 // stay in shared memory at local_keys().  A chunk's weights are ready in shared memory when this is called.
 static inline size_t local_mma_smem(int d, int dv) {
-    return sizeof(bf16) * ((size_t)2 * C * (pad16(d) + 8) + (size_t)4 * C * (pad16(dv) + 8));
+    return sizeof(bf16) * ((size_t)2 * C * (pad16(d) + 8) + (size_t)C * (pad16(dv) + 8));
 }
 __device__ __forceinline__ bf16* local_keys(unsigned char* smraw, int d) { return (bf16*)smraw + C * (pad16(d) + 8); }
 
@@ -127,21 +127,10 @@ __device__ __forceinline__ void chunk_local_mma(unsigned char* smraw, const floa
     bf16* Qs = (bf16*)smraw;             // [C][ks]
     bf16* Ks = local_keys(smraw, d);     // [C][ks]
     bf16* Vs = Ks + C * ks;              // [C][vs]
-    bf16* Ws = Vs + C * vs;              // [3][C][vs]: the values times weights.tail(j) in three terms
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     load_rounded(Qs, ks, q, q_ld, n, d, dP, silu);
     load_rounded(Ks, ks, k, k_ld, n, d, dP, silu);
     load_rounded(Vs, vs, v, v_ld, n, dv, vP, silu);
-    __syncthreads();
-    for (int e = threadIdx.x; e < C * (vP >> 1); e += MT) {
-        const int j = e / (vP >> 1), cc = (e % (vP >> 1)) << 1;
-        const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(Vs + j * vs + cc));
-        const float w = j < n ? weights.tail(j) : 0.f;
-        uint32_t t[3];
-        split3(v.x * w, v.y * w, t[0], t[1], t[2]);
-#pragma unroll
-        for (int s = 0; s < 3; ++s) *reinterpret_cast<uint32_t*>(Ws + ((size_t)s * C + j) * vs + cc) = t[s];
-    }
     __syncthreads();
     {   // a warp: 16 rows of the chunk (all their scores) and half of the value columns
         const int rg = warp & 3, cg = warp >> 2;
@@ -166,6 +155,7 @@ __device__ __forceinline__ void chunk_local_mma(unsigned char* smraw, const floa
         uint32_t a3[4][3][4];                            // the weighted scores as A operands: [16 keys][term][register]
 #pragma unroll
         for (int t = 0; t < 8; ++t) {
+            if ((t >> 1) > rg) continue;                 // (their terms are not used either)
             const int j = t * 8 + 2 * (lane & 3);
             auto weigh = [&](float x, int i, int jj) { return (jj <= i && jj < n) ? x * weights.pair(i, jj) : 0.f; };
             uint32_t (&r)[3][4] = a3[t >> 1];
@@ -185,6 +175,7 @@ __device__ __forceinline__ void chunk_local_mma(unsigned char* smraw, const floa
             }
         }
         const int blocks = vP >> 4, half = (blocks + 1) >> 1;
+        const bool out2 = ((dv | o_ld) & 1) == 0 && ((uintptr_t)orow & 7) == 0;
         const int b_lo = cg ? half : 0, b_hi = cg ? blocks : half;
         for (int b0 = b_lo; b0 < b_hi; b0 += 4) {
             float o[8][4];
@@ -211,6 +202,11 @@ __device__ __forceinline__ void chunk_local_mma(unsigned char* smraw, const floa
             for (int t = 0; t < 8; ++t) {
                 const int col = b0 * 16 + t * 8 + 2 * (lane & 3);
                 if (b0 + (t >> 1) >= b_hi) continue;
+                if (out2 && col < dv) {
+                    if (i0 < n) *reinterpret_cast<float2*>(orow + (size_t)i0 * o_ld + col) = make_float2(o[t][0], o[t][1]);
+                    if (i1 < n) *reinterpret_cast<float2*>(orow + (size_t)i1 * o_ld + col) = make_float2(o[t][2], o[t][3]);
+                    continue;
+                }
 #pragma unroll
                 for (int e = 0; e < 2; ++e)
                     if (col + e < dv) {
@@ -231,15 +227,23 @@ __device__ __forceinline__ void chunk_local_mma(unsigned char* smraw, const floa
             for (int k0 = 0; k0 < C && k0 < n; k0 += 16) {
                 uint32_t a[4];
                 ret_ldsm_t(a, Ks + (k0 + (lane & 7) + (lane >> 4) * 8) * ks + m0 + ((lane >> 3) & 1) * 8);
+                uint32_t a3[3][4];                       // the keys times weights.tail(j) in three terms
+                const int j = k0 + 2 * (lane & 3);
+#pragma unroll
+                for (int r = 0; r < 4; ++r) {
+                    const int jj = j + (r >> 1) * 8;
+                    const float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&a[r]));
+                    split3(jj < n ? x.x * weights.tail(jj) : 0.f, jj + 1 < n ? x.y * weights.tail(jj + 1) : 0.f, a3[0][r], a3[1][r], a3[2][r]);
+                }
 #pragma unroll
                 for (int t = 0; t < 8; ++t) {
                     if (n0 + t * 16 >= vP) continue;
+                    uint32_t b[4];
+                    ret_ldsm_t(b, Vs + (k0 + (lane & 7) + ((lane >> 3) & 1) * 8) * vs + n0 + t * 16 + (lane >> 4) * 8);
 #pragma unroll
-                    for (int s3 = 2; s3 >= 0; --s3) {
-                        uint32_t b[4];
-                        ret_ldsm_t(b, Ws + ((size_t)s3 * C + k0 + (lane & 7) + ((lane >> 3) & 1) * 8) * vs + n0 + t * 16 + (lane >> 4) * 8);
-                        ret_mma(u[2 * t], a, b[0], b[1]);
-                        ret_mma(u[2 * t + 1], a, b[2], b[3]);
+                    for (int s3 = 2; s3 >= 0; --s3) {    // the small terms first
+                        ret_mma(u[2 * t], a3[s3], b[0], b[1]);
+                        ret_mma(u[2 * t + 1], a3[s3], b[2], b[3]);
                     }
                 }
             }
@@ -266,76 +270,88 @@ __device__ __forceinline__ void chunk_local_mma(unsigned char* smraw, const floa
 }
 
 
-// The start state's part, SCOLS value columns from n0 on: q_i and the state Sc [d, dv] into shared memory ...
-static inline size_t finish_mma_smem(int d) { return sizeof(bf16) * ((size_t)C * (pad16(d) + 8) + (size_t)3 * pad16(d) * SST); }
+// The start state's part, SCOLS value columns from n0 on: orow_i = weights.join(i, (Sc^T q_i), orow_i).  A warp takes eight
+// columns of the state Sc [d, dv] and all rows of the chunk: every element of the state is loaded once, straight into the
+// registers of the product's B operand (three bfloat16 terms), ahead of the queries where d reaches no further than
+// FINISH_ROWS.  Two steps, between which the includer may use the rounded queries in shared memory:
+constexpr int FINISH_ROWS = 64, FK = FINISH_ROWS / 16;
+static inline size_t finish_mma_smem(int d) { return sizeof(bf16) * (size_t)C * (pad16(d) + 8); }
 
-__device__ __forceinline__ void chunk_finish_load(unsigned char* smraw, const float* __restrict__ q, int q_ld, int silu, int n,
-                                                  int d, int dv, int n0, const float* __restrict__ Sc) {
-    const int dP = pad16(d), ks = dP + 8;
-    bf16* Qs = (bf16*)smraw;             // [C][ks]
-    bf16* Ss = Qs + C * ks;              // [3][dP][SST]
-    load_rounded(Qs, ks, q, q_ld, n, d, dP, silu);
-    const bool vec = (dv & 3) == 0 && ((uintptr_t)Sc & 15) == 0;
-    for (int e0 = threadIdx.x; e0 < dP * (SCOLS / 4); e0 += MT * LOADS) {
-        float4 x[LOADS];
+struct FinishRegs { float s[FK][4]; float local[4][4]; };
+
+__device__ __forceinline__ void finish_load_state(FinishRegs& f, const float* __restrict__ Sc, int d, int dv, int col, int r0) {
+    const int kb = 2 * (threadIdx.x & 3);
 #pragma unroll
-        for (int u = 0; u < LOADS; ++u) {
-            const int e = e0 + u * MT, r = e / (SCOLS / 4), col = n0 + ((e % (SCOLS / 4)) << 2);
-            x[u] = load_four(Sc + (size_t)r * dv + col, (r < d && col < dv) ? dv - col : 0, vec);
+    for (int kk = 0; kk < FK; ++kk)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const int r = r0 + kk * 16 + kb + (e & 1) + (e >> 1) * 8;
+            f.s[kk][e] = (r < d && col < dv) ? __ldcg(Sc + (size_t)r * dv + col) : 0.f;
         }
+}
+
+__device__ __forceinline__ void chunk_finish_load(FinishRegs& f, unsigned char* smraw, const float* __restrict__ q, int q_ld, int silu,
+                                                  int n, int d, int dv, int n0, const float* __restrict__ Sc,
+                                                  const float* __restrict__ orow, int o_ld) {
+    const int dP = pad16(d), warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    finish_load_state(f, Sc, d, dv, n0 + warp * 8 + (lane >> 2), 0);
+    const int col = n0 + warp * 8 + 2 * (lane & 3);
+    const bool two = ((dv | o_ld) & 1) == 0 && ((uintptr_t)orow & 7) == 0;
 #pragma unroll
-        for (int u = 0; u < LOADS; ++u) {
-            const int e = e0 + u * MT, r = e / (SCOLS / 4), cc = (e % (SCOLS / 4)) << 2;
-            if (r >= dP) continue;
-            uint32_t t[3], v[3];
-            split3(x[u].x, x[u].y, t[0], t[1], t[2]);
-            split3(x[u].z, x[u].w, v[0], v[1], v[2]);
+    for (int rg = 0; rg < 4; ++rg)
 #pragma unroll
-            for (int s3 = 0; s3 < 3; ++s3) *reinterpret_cast<uint2*>(Ss + ((size_t)s3 * dP + r) * SST + cc) = make_uint2(t[s3], v[s3]);
+        for (int hi = 0; hi < 2; ++hi) {                 // (the local part is asked for ahead of the products)
+            const int i = rg * 16 + (lane >> 2) + hi * 8;
+            const float* p = orow + (size_t)i * o_ld + col;
+            float2 x = make_float2(0.f, 0.f);
+            if (i < n && two && col < dv) x = __ldcg(reinterpret_cast<const float2*>(p));
+            else if (i < n) { if (col < dv) x.x = __ldcg(p); if (col + 1 < dv) x.y = __ldcg(p + 1); }
+            f.local[rg][2 * hi] = x.x; f.local[rg][2 * hi + 1] = x.y;
         }
-    }
+    load_rounded((bf16*)smraw, dP + 8, q, q_ld, n, d, dP, silu);
     __syncthreads();
 }
 
-// ... and orow_i = weights.join(i, (Sc^T q_i), orow_i).
 template <class W>
-__device__ __forceinline__ void chunk_finish_mma(const unsigned char* smraw, int n, int d, int dv, int n0, const W& weights,
-                                                 float* __restrict__ orow, int o_ld) {
+__device__ __forceinline__ void chunk_finish_mma(FinishRegs& f, const unsigned char* smraw, int n, int d, int dv, int n0,
+                                                 const float* __restrict__ Sc, const W& weights, float* __restrict__ orow, int o_ld) {
     const int dP = pad16(d), ks = dP + 8, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const bf16* Qs = (const bf16*)smraw;
-    const bf16* Ss = Qs + C * ks;
-    const int rg = warp & 3, cg = warp >> 2;             // 16 rows x 32 columns a warp
-    const int i0 = rg * 16 + (lane >> 2), i1 = i0 + 8;
-    float o[4][4], local[4][4];                          // (the local part is asked for ahead of the products)
+    float o[4][4];
 #pragma unroll
-    for (int t = 0; t < 4; ++t)
+    for (int rg = 0; rg < 4; ++rg)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-            const int i = e < 2 ? i0 : i1, col = n0 + cg * 32 + t * 8 + 2 * (lane & 3) + (e & 1);
-            o[t][e] = 0.f;
-            local[t][e] = (i < n && col < dv) ? __ldcg(orow + (size_t)i * o_ld + col) : 0.f;
-        }
-    for (int kk = 0; kk < dP; kk += 16) {
-        uint32_t a[4];
-        ret_ldsm(a, Qs + (rg * 16 + (lane & 15)) * ks + kk + (lane >> 4) * 8);
+        for (int e = 0; e < 4; ++e) o[rg][e] = 0.f;
+    for (int r0 = 0; r0 < dP; r0 += FINISH_ROWS) {
+        if (r0 > 0) finish_load_state(f, Sc, d, dv, n0 + warp * 8 + (lane >> 2), r0);
 #pragma unroll
-        for (int bb = 0; bb < 2; ++bb)
+        for (int kk = 0; kk < FK; ++kk) {
+            if (r0 + kk * 16 >= dP) continue;
+            uint32_t t0[3], t1[3];
+            split3(f.s[kk][0], f.s[kk][1], t0[0], t0[1], t0[2]);
+            split3(f.s[kk][2], f.s[kk][3], t1[0], t1[1], t1[2]);
 #pragma unroll
-            for (int s3 = 2; s3 >= 0; --s3) {
-                uint32_t b[4];
-                ret_ldsm_t(b, Ss + ((size_t)s3 * dP + kk + (lane & 7) + ((lane >> 3) & 1) * 8) * SST + cg * 32 + bb * 16 + (lane >> 4) * 8);
-                ret_mma(o[2 * bb], a, b[0], b[1]);
-                ret_mma(o[2 * bb + 1], a, b[2], b[3]);
+            for (int rg = 0; rg < 4; ++rg) {
+                uint32_t a[4];
+                ret_ldsm(a, Qs + (rg * 16 + (lane & 15)) * ks + r0 + kk * 16 + (lane >> 4) * 8);
+#pragma unroll
+                for (int s3 = 2; s3 >= 0; --s3) ret_mma(o[rg], a, t0[s3], t1[s3]);          // the small terms first
             }
+        }
     }
+    const int col = n0 + warp * 8 + 2 * (lane & 3);
+    const bool two = ((dv | o_ld) & 1) == 0 && ((uintptr_t)orow & 7) == 0;
 #pragma unroll
-    for (int t = 0; t < 4; ++t)
+    for (int rg = 0; rg < 4; ++rg)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-            const int i = e < 2 ? i0 : i1, col = n0 + cg * 32 + t * 8 + 2 * (lane & 3) + (e & 1);
-            if (i < n && col < dv) orow[(size_t)i * o_ld + col] = weights.join(i, o[t][e], local[t][e]);
+        for (int hi = 0; hi < 2; ++hi) {
+            const int i = rg * 16 + (lane >> 2) + hi * 8;
+            if (i >= n) continue;
+            float* p = orow + (size_t)i * o_ld + col;
+            const float x = weights.join(i, o[rg][2 * hi], f.local[rg][2 * hi]), y = weights.join(i, o[rg][2 * hi + 1], f.local[rg][2 * hi + 1]);
+            if (two && col < dv) *reinterpret_cast<float2*>(p) = make_float2(x, y);
+            else { if (col < dv) p[0] = x; if (col + 1 < dv) p[1] = y; }
         }
 }
-
 
 }  // namespace

@@ -184,11 +184,11 @@ __host__ __device__ inline Workspace workspace_of(float* ws, long long chunks, i
 
 struct LocalWeights {
     static constexpr bool SUMS = true;
-    const float* a; const float* M;
-    float scale, M_end;
+    const float* a; const float* M; const float* tails;
+    float scale;
     float* sums;
     __device__ __forceinline__ float pair(int i, int j) const { return scale * expf(a[j] - M[i]); }
-    __device__ __forceinline__ float tail(int j) const { return expf(a[j] - M_end); }
+    __device__ __forceinline__ float tail(int j) const { return tails[j]; }
     __device__ __forceinline__ void row_sum(int i, float x) const { sums[i] = x; }
 };
 
@@ -249,8 +249,8 @@ mlstm_local_kernel(MlstmParams p, int num_requests, Workspace w) {
     __syncthreads();
     const float* row = p.proj + (size_t)c.t * p.ld;
     float* Uc = w.U + at * chunk_floats(d, dv);
-    const LocalWeights weights{sa, sM, p.q_scale, sM[c.n - 1], nums + 2 * C};
-    if (threadIdx.x < C) tails[threadIdx.x] = threadIdx.x < c.n ? weights.tail(threadIdx.x) : 0.f;
+    const LocalWeights weights{sa, sM, tails, p.q_scale, nums + 2 * C};
+    if (threadIdx.x < C) tails[threadIdx.x] = threadIdx.x < c.n ? expf(sa[threadIdx.x] - sM[c.n - 1]) : 0.f;
     chunk_local_mma(smraw, row + p.q_off + (size_t)h * d, p.ld, row + p.k_off + (size_t)h * d, p.ld, row + p.v_off + (size_t)h * dv,
                     p.ld, 0, c.n, d, dv, weights, p.out + (size_t)c.t * p.H * dv + (size_t)h * dv, p.H * dv, Uc);
     const bf16* Ks = local_keys(smraw, d);
@@ -331,7 +331,7 @@ struct FinishWeights {
     }
 };
 
-__global__ void __launch_bounds__(MT, 3)
+__global__ void __launch_bounds__(MT, 2)
 mlstm_finish_kernel(MlstmParams p, int num_requests, Workspace w) {
     extern __shared__ __align__(16) unsigned char smraw[];
     __shared__ float wl[C], ws[C], inv[C];
@@ -344,7 +344,9 @@ mlstm_finish_kernel(MlstmParams p, int num_requests, Workspace w) {
     const size_t at = (size_t)blockIdx.x * p.H + h;
     const float* Sc = w.U + at * chunk_floats(d, dv);
     const float* Nc = Sc + round4(d * dv);
-    chunk_finish_load(smraw, p.proj + (size_t)c.t * p.ld + p.q_off + (size_t)h * d, p.ld, 0, c.n, d, dv, n0, Sc);
+    float* orow = p.out + (size_t)c.t * p.H * dv + (size_t)h * dv;
+    FinishRegs f;
+    chunk_finish_load(f, smraw, p.proj + (size_t)c.t * p.ld + p.q_off + (size_t)h * d, p.ld, 0, c.n, d, dv, n0, Sc, orow, p.H * dv);
     {   // the denominators: four threads a token
         const bf16* q = (const bf16*)smraw + (threadIdx.x >> 2) * (pad16(d) + 8);
         const int i = threadIdx.x >> 2;
@@ -362,7 +364,7 @@ mlstm_finish_kernel(MlstmParams p, int num_requests, Workspace w) {
         }
     }
     __syncthreads();
-    chunk_finish_mma(smraw, c.n, d, dv, n0, FinishWeights{wl, ws, inv}, p.out + (size_t)c.t * p.H * dv + (size_t)h * dv, p.H * dv);
+    chunk_finish_mma(f, smraw, c.n, d, dv, n0, Sc, FinishWeights{wl, ws, inv}, orow, p.H * dv);
 }
 
 constexpr size_t MOST = 224 * 1024;    // dynamic shared memory a CTA may ask for here (the kernels have a little static on top)

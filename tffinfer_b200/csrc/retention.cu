@@ -517,7 +517,7 @@ retention_local_mma_kernel(RetParams p, int num_requests, float* __restrict__ U)
 }
 
 // out_i += decay^(i+1) S^T q_i for SCOLS value columns of a chunk, S the state it starts from (left in U by the scan)
-__global__ void __launch_bounds__(MT, 3)
+__global__ void __launch_bounds__(MT, 2)
 retention_finish_mma_kernel(RetParams p, int num_requests, const float* __restrict__ U) {
     extern __shared__ __align__(16) unsigned char smraw[];
     __shared__ float pw[C + 1];
@@ -528,9 +528,11 @@ retention_finish_mma_kernel(RetParams p, int num_requests, const float* __restri
     fill_powers(pw, p.decay[h]);
     pdl_wait();
     if (!have || c.pos == 0) return;     // a sequence's first chunk starts from zeros: its local part is all of it
-    chunk_finish_load(smraw, p.q + (size_t)c.t * p.q_ld + (size_t)h * d, p.q_ld, p.silu, c.n, d, dv, n0,
-                      U + ((size_t)blockIdx.x * p.H + h) * d * dv);
-    chunk_finish_mma(smraw, c.n, d, dv, n0, FixedDecay{pw, c.n}, (float*)p.out + (size_t)c.t * p.H * dv + (size_t)h * dv, p.H * dv);
+    float* orow = (float*)p.out + (size_t)c.t * p.H * dv + (size_t)h * dv;
+    const float* Sc = U + ((size_t)blockIdx.x * p.H + h) * d * dv;
+    FinishRegs f;
+    chunk_finish_load(f, smraw, p.q + (size_t)c.t * p.q_ld + (size_t)h * d, p.q_ld, p.silu, c.n, d, dv, n0, Sc, orow, p.H * dv);
+    chunk_finish_mma(f, smraw, c.n, d, dv, n0, Sc, FixedDecay{pw, c.n}, orow, p.H * dv);
 }
 
 }  // namespace

@@ -184,7 +184,7 @@ stream_step_kernel(float* __restrict__ x, int S, int W,
 //   h[r] = x[r] * rsqrt(mean(x[r]^2) + eps) * w                                 (h null: not wanted)
 // Everything in float32.  y1, y2 and z may be accumulator buffers, which are set to zero behind the read (bits 1, 2 and 4 of
 // ``clear``).  With row_index, CTA r works on row row_index[r], h is written to row r and x is left as it was.
-__device__ __forceinline__ float gate_of(float z) { return 1.0f / (1.0f + expf(-z)); }
+__device__ __forceinline__ float gate_of(float z) { return __fdividef(1.0f, 1.0f + expf(-z)); }
 template <typename TZ> __device__ __forceinline__ float4 load_z4(const TZ* p);
 template <> __device__ __forceinline__ float4 load_z4<float>(const float* p) { return __ldcg(reinterpret_cast<const float4*>(p)); }
 template <> __device__ __forceinline__ float4 load_z4<bf16>(const bf16* p) {
@@ -215,32 +215,42 @@ gated_join_kernel(float* __restrict__ x, int W, TZ* __restrict__ z, int zld, con
     const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
     if (vec) {
         const int W4 = W >> 2;
-#pragma unroll 2
-        for (int i = threadIdx.x; i < W4; i += NT) {
-            float4 v = __ldcg(reinterpret_cast<const float4*>(xr) + i);
-            const float4 a = __ldcg(reinterpret_cast<const float4*>(y1r) + i);
-            const float4 za = load_z4<TZ>(zr + 4 * i);
-            const float4 ba = reinterpret_cast<const float4*>(b)[i];
-            const float4 ca = c1 ? reinterpret_cast<const float4*>(c1)[i] : zero;
-            if (y2r) {
-                const float4 f = __ldcg(reinterpret_cast<const float4*>(y2r) + i);
-                const float4 zf = load_z4<TZ>(zr + W + 4 * i);
-                const float4 bf = reinterpret_cast<const float4*>(b + W)[i];
-                v.x = fmaf(f.x, gate_of(zf.x + bf.x), v.x); v.y = fmaf(f.y, gate_of(zf.y + bf.y), v.y);
-                v.z = fmaf(f.z, gate_of(zf.z + bf.z), v.z); v.w = fmaf(f.w, gate_of(zf.w + bf.w), v.w);
+        for (int i0 = threadIdx.x; i0 < W4; i0 += 2 * NT) {
+            float4 v[2], a[2], za[2], f[2], zf[2];       // both columns' loads are in flight together
+#pragma unroll
+            for (int u = 0; u < 2; ++u) {
+                const int i = i0 + u * NT;
+                if (i >= W4) continue;
+                v[u] = __ldcg(reinterpret_cast<const float4*>(xr) + i);
+                a[u] = __ldcg(reinterpret_cast<const float4*>(y1r) + i);
+                za[u] = load_z4<TZ>(zr + 4 * i);
+                f[u] = y2r ? __ldcg(reinterpret_cast<const float4*>(y2r) + i) : zero;
+                zf[u] = y2r ? load_z4<TZ>(zr + W + 4 * i) : zero;
             }
-            v.x = fmaf(a.x + ca.x, gate_of(za.x + ba.x), v.x); v.y = fmaf(a.y + ca.y, gate_of(za.y + ba.y), v.y);
-            v.z = fmaf(a.z + ca.z, gate_of(za.z + ba.z), v.z); v.w = fmaf(a.w + ca.w, gate_of(za.w + ba.w), v.w);
-            if (store_x) reinterpret_cast<float4*>(xr)[i] = v;
-            if (clear & 1) reinterpret_cast<float4*>(y1r)[i] = zero;
-            if (clear & 2) reinterpret_cast<float4*>(y2r)[i] = zero;
-            if constexpr (sizeof(TZ) == 4)
-                if (clear & 4) {
-                    reinterpret_cast<float4*>(zr)[i] = zero;
-                    if (y2r) reinterpret_cast<float4*>(zr + W)[i] = zero;
+#pragma unroll
+            for (int u = 0; u < 2; ++u) {
+                const int i = i0 + u * NT;
+                if (i >= W4) continue;
+                if (y2r) {
+                    const float4 bf = reinterpret_cast<const float4*>(b + W)[i];
+                    v[u].x = fmaf(f[u].x, gate_of(zf[u].x + bf.x), v[u].x); v[u].y = fmaf(f[u].y, gate_of(zf[u].y + bf.y), v[u].y);
+                    v[u].z = fmaf(f[u].z, gate_of(zf[u].z + bf.z), v[u].z); v[u].w = fmaf(f[u].w, gate_of(zf[u].w + bf.w), v[u].w);
                 }
-            reinterpret_cast<float4*>(u_row)[i] = v;
-            ss = fmaf(v.x, v.x, ss); ss = fmaf(v.y, v.y, ss); ss = fmaf(v.z, v.z, ss); ss = fmaf(v.w, v.w, ss);
+                const float4 ba = reinterpret_cast<const float4*>(b)[i];
+                const float4 ca = c1 ? reinterpret_cast<const float4*>(c1)[i] : zero;
+                v[u].x = fmaf(a[u].x + ca.x, gate_of(za[u].x + ba.x), v[u].x); v[u].y = fmaf(a[u].y + ca.y, gate_of(za[u].y + ba.y), v[u].y);
+                v[u].z = fmaf(a[u].z + ca.z, gate_of(za[u].z + ba.z), v[u].z); v[u].w = fmaf(a[u].w + ca.w, gate_of(za[u].w + ba.w), v[u].w);
+                if (store_x) reinterpret_cast<float4*>(xr)[i] = v[u];
+                if (clear & 1) reinterpret_cast<float4*>(y1r)[i] = zero;
+                if (clear & 2) reinterpret_cast<float4*>(y2r)[i] = zero;
+                if constexpr (sizeof(TZ) == 4)
+                    if (clear & 4) {
+                        reinterpret_cast<float4*>(zr)[i] = zero;
+                        if (y2r) reinterpret_cast<float4*>(zr + W)[i] = zero;
+                    }
+                reinterpret_cast<float4*>(u_row)[i] = v[u];
+                ss = fmaf(v[u].x, v[u].x, ss); ss = fmaf(v[u].y, v[u].y, ss); ss = fmaf(v[u].z, v[u].z, ss); ss = fmaf(v[u].w, v[u].w, ss);
+            }
         }
         if (!h) return;
         ss = block_sum<NT>(ss, red);
@@ -350,7 +360,7 @@ TFF_API int tff_gated_join(float* x, int W, void* z, int zld, int z_is_bf16, con
                               row_index, (TO*)h);                                                                   \
     } while (0)
 #define TFF_JOIN_N(TO, TZ)                                                                                          \
-    do { if (W >= 2048) TFF_JOIN(TO, TZ, 512); if (W >= 512) TFF_JOIN(TO, TZ, 128); TFF_JOIN(TO, TZ, 64); } while (0)
+    do { if (W >= 2048 && rows <= 256) TFF_JOIN(TO, TZ, 512); if (W >= 2048) TFF_JOIN(TO, TZ, 256); if (W >= 512) TFF_JOIN(TO, TZ, 128); TFF_JOIN(TO, TZ, 64); } while (0)
     if (h_is_bf16) { if (z_is_bf16) TFF_JOIN_N(bf16, bf16); TFF_JOIN_N(bf16, float); }
     if (z_is_bf16) TFF_JOIN_N(float, bf16);
     TFF_JOIN_N(float, float);

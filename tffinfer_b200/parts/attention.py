@@ -171,8 +171,8 @@ class GatedSinkAttention(Mixer):
         self.conv_w = self.conv_wt = self.norm_w = self.bias = None
 
     def kernel_files(self):
-        return ("attention_bf16", "attention_decode", "attention_prefill", "attention_generic",
-                "qkv_finish", "short_conv", "streams")
+        files = ("attention_bf16", "attention_decode", "attention_prefill", "attention_generic", "qkv_finish", "streams")
+        return files if getattr(self, "head_finish", False) else files + ("short_conv",)
 
     def cache_need(self):
         kv = KVNeed(self.num_kv_heads, self.cache_dim, self.window, keep_first=self.keep_first)
