@@ -484,6 +484,56 @@ def test_memory_tokens_and_chunks_agree(ops, D, V):
         assert float(err.max()) < 1e-3 and float(err.median()) < 2e-5
 
 
+@pytest.mark.parametrize("H,D,V", [(2, 64, 96), (3, 20, 9), (1, 300, 36), (2, 128, 128)])
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+def test_memory_decode_steps_of_many_requests_up_to_the_gate(ops, H, D, V, dtype):
+    """One token of each of so many requests that the step kernel takes its small CTAs, on to norm and gate in the same
+    kernel, against the plain equations; the projection's rows set to zero where they were read, and the same states and
+    outputs as in steps of few requests."""
+    dev, cap, B, eps = "cuda", 4.0, 310, 1e-4
+    g = torch.Generator().manual_seed(D)
+    at = 2 * H * D + 2 * H * V
+    start = torch.randn(B, mlstm_state_size(H, D, V), generator=g)
+    bias, w = torch.randn(2 * H, generator=g), 1 + 0.3 * torch.randn(H * V, generator=g)
+    rows = torch.randn(B, at + 2 * H + 3, generator=g)
+    slots = torch.randperm(B, generator=g).tolist()
+    fresh = [5 if i % 7 else 0 for i in range(B)]                # some requests bring their first token
+    buf = ops.projection_buffer(B, at + 2 * H + 3, torch.device(dev), torch.bfloat16, use=f"memory {H} {D} {dtype}") \
+        if B <= ops.SWAP_MAX_M else torch.zeros(B, at + 2 * H + 3, device=dev)
+    ops._acc_zero[buf.data_ptr()] = False
+    buf.copy_(rows)
+    st, mixed = start.clone().to(dev), torch.full((B, H * V), float("nan"), device=dev, dtype=dtype)
+    ops.mlstm_recurrence(buf, st, fake_batch([1] * B, fresh, dev, 8, slots=slots), bias.to(dev), cap, None, H, D, V,
+                         finish=(2 * H * D + H * V, w.to(dev), eps, mixed))
+    torch.cuda.synchronize()
+    assert not buf[:, :at + 2 * H].any() and torch.equal(buf[:, at + 2 * H:].cpu(), rows[:, at + 2 * H:])
+    del ops._acc_zero[buf.data_ptr()]
+    few = start.clone().to(dev)
+    for lo in range(0, B, 100):
+        out = torch.full((min(100, B - lo), H * V), float("nan"), device=dev)
+        b = fake_batch([1] * out.shape[0], fresh[lo:lo + 100], dev, 8, slots=slots[lo:lo + 100])
+        ops.mlstm_recurrence(rows[lo:lo + 100].contiguous().to(dev), few, b, bias.to(dev), cap, out, H, D, V)
+        o = out.double().cpu().view(-1, H, V)
+        gate = torch.sigmoid(rows[lo:lo + 100, 2 * H * D + H * V:at].double())
+        want = (o / P.rms(o, eps)).reshape(-1, H * V) * w.double() * gate
+        err = (mixed[lo:lo + 100].double().cpu() - want).abs().max() / want.abs().max()
+        assert float(err) < (1e-4 if dtype == torch.float32 else 1e-2)
+    assert torch.allclose(st, few, rtol=1e-5, atol=1e-5)
+    for i in (0, 1, 7, 309):                                     # and the plain equations, request by request
+        s = start[slots[i]].double()
+        r = rows[i].double()
+        for h in range(H):
+            state = (s[h * D * V:(h + 1) * D * V].view(D, V), s[H * D * V + h * D:H * D * V + (h + 1) * D], s[H * D * V + H * D + h])
+            ig = P.capped(r[at + h] + bias[h].double(), cap)
+            fg = torch.nn.functional.logsigmoid(P.capped(r[at + H + h] + bias[H + h].double(), cap))
+            o, (S, n, m) = P.mlstm_recurrence(r[None, h * D:(h + 1) * D] * D ** -0.5, r[None, (H + h) * D:(H + h + 1) * D],
+                                              r[None, 2 * H * D + h * V:2 * H * D + (h + 1) * V], ig[None], fg[None],
+                                              None if fresh[i] == 0 else state)
+            got = st[slots[i]].double().cpu()
+            assert float((got[h * D * V:(h + 1) * D * V].view(D, V) - S).abs().max()) < 2e-5 * float(S.abs().max())
+            assert abs(float(got[H * D * V + H * D + h] - m)) < 1e-4
+
+
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 @pytest.mark.parametrize("T", [1, 9, 70, 300])
 @pytest.mark.parametrize("H,D,V,W", [(3, 16, 24, 64), (2, 40, 40, 50)])

@@ -45,11 +45,14 @@ __device__ __forceinline__ float forget_gate(float z, float cap) {      // log o
 __device__ __forceinline__ float divide(float num, float nq, float m) { return num / (fmaxf(fabsf(nq), expf(-m)) + 1e-6f); }
 
 // ------------------------------------------------------------------ token by token
-constexpr int ST = 512, ROWS = 8;      // threads of a CTA; rows of a column group that a thread has in flight
+// Threads of a CTA: small ones, four an SM, for steps of one token of many requests, which stream the states (64 requests of 16
+// heads of 128 x 128: 35 us against 43, 57 with one large CTA an SM); large ones, whose registers hold such a head, for few
+// requests and for portions.  ROWS: rows of a column group that a thread has in flight.
+constexpr int FEW = 256, MANY = 512, ROWS = 8;
 
 // VEC value columns a thread; KEEP: the head's state stays in registers (ROWS rows a thread and one column group cover it)
-template <int VEC, bool KEEP>
-__global__ void __launch_bounds__(ST)
+template <int VEC, bool KEEP, int ST>
+__global__ void __launch_bounds__(ST, ST == FEW ? 4 : 2)
 mlstm_step_kernel(MlstmParams p) {
     extern __shared__ __align__(16) float sm[];
     __shared__ float red[32];
@@ -424,13 +427,17 @@ TFF_API int tff_mlstm(const float* proj, int ld, int q_off, int k_off, int v_off
                         q_start, pos_start, slots, out, H, d, dv, rows, g_off, norm_w, eps, mixed, mixed_is_bf16, clear};
     if (chunked) return launch_chunked(p, num_requests, workspace, num_tokens, stream);
     const bool vec = dv % 4 == 0 && ((uintptr_t)state & 15) == 0 && (H * d * dv) % 4 == 0;
-    const int width = vec ? 4 : 1, groups = dv / width, lx = groups < ST ? groups : ST, ny = ST / lx;
-    const bool keep = groups <= ST && ny * ROWS >= d;
+    const bool single = num_tokens == num_requests && (long long)H * num_requests > 300;      // one token of many requests
+    const int threads = single ? FEW : MANY, width = vec ? 4 : 1, groups = dv / width, lx = groups < threads ? groups : threads;
+    const int ny = threads / lx;
+    const bool keep = !single && groups <= threads && ny * ROWS >= d;
     const size_t smem = sizeof(float) * ((size_t)3 * d + dv + (size_t)ny * groups * width);
     if (smem > 48 * 1024) return TFF_ERR_UNSUPPORTED;
     const dim3 grid(H, num_requests);
-    if (vec && keep) return tff_launch_pdl(mlstm_step_kernel<4, true>, grid, dim3(ST), smem, stream, p);
-    if (vec) return tff_launch_pdl(mlstm_step_kernel<4, false>, grid, dim3(ST), smem, stream, p);
-    if (keep) return tff_launch_pdl(mlstm_step_kernel<1, true>, grid, dim3(ST), smem, stream, p);
-    return tff_launch_pdl(mlstm_step_kernel<1, false>, grid, dim3(ST), smem, stream, p);
+#define TFF_STEP(VEC, KEEP, ST) return tff_launch_pdl(mlstm_step_kernel<VEC, KEEP, ST>, grid, dim3(ST), smem, stream, p)
+    if (single) { if (vec) TFF_STEP(4, false, FEW); TFF_STEP(1, false, FEW); }
+    if (vec) { if (keep) TFF_STEP(4, true, MANY); TFF_STEP(4, false, MANY); }
+    if (keep) TFF_STEP(1, true, MANY);
+    TFF_STEP(1, false, MANY);
+#undef TFF_STEP
 }

@@ -26,7 +26,7 @@ namespace {
 
 // Tokens a block of moe_route_kernel takes (one warp each for the choice) and its threads: steps of many tokens share the
 // reading of the router's rows, steps of few give every output a warp of its own.
-constexpr int ROUTE_MANY_TOK = 4, ROUTE_MANY_THREADS = 256, ROUTE_FEW_TOK = 1, ROUTE_FEW_THREADS = 512, ROUTE_FEW = 256;
+constexpr int ROUTE_MANY_TOK = 4, ROUTE_MANY_THREADS = 256, ROUTE_FEW_TOK = 1, ROUTE_FEW_THREADS = 1024, ROUTE_FEW = 256;
 
 template <typename TH, typename TW, int ROUTE_TOK, int ROUTE_THREADS>
 __global__ void __launch_bounds__(ROUTE_THREADS)
@@ -38,8 +38,12 @@ moe_route_kernel(const TH* __restrict__ h, const TW* __restrict__ w_router, cons
     // 2,048 times otherwise), every token keeps sums of its own, and behind the products warp i does token i's choice.
     extern __shared__ float sm[];              // per token W floats (its row) and 3 E: the scores, the choice scores, groups
     pdl_launch_dependents();
-    pdl_wait();
     const int t0 = blockIdx.x * ROUTE_TOK, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    // the weights are older than the kernels ahead: into the second-level cache while those are still at work
+    if (ROUTE_TOK == 1)
+        for (size_t e = (size_t)threadIdx.x * 128; e < (size_t)E * W * sizeof(TW); e += (size_t)ROUTE_THREADS * 128)
+            asm volatile("prefetch.global.L2 [%0];" ::"l"(reinterpret_cast<const char*>(w_router) + e));
+    pdl_wait();
     const int nt = min(ROUTE_TOK, T - t0);
     float* rows = sm;                          // [ROUTE_TOK][W]
     float* scores = sm + (size_t)ROUTE_TOK * W;   // [ROUTE_TOK][3 E]
@@ -70,7 +74,7 @@ moe_route_kernel(const TH* __restrict__ h, const TW* __restrict__ w_router, cons
     // A warp takes up to RE outputs side by side (a row's elements are read once for them), a lane eight neighbouring
     // elements a load where the rows allow it (16-byte loads, several in flight), else one.  Either way the order of a dot
     // product's additions is fixed by W alone.  (Index E is the row beside the router's, when there is one.)
-    constexpr int RE = ROUTE_TOK > 1 ? 3 : 1, RW = ROUTE_THREADS / 32;
+    constexpr int RE = ROUTE_TOK > 1 ? 3 : 1, RW = ROUTE_THREADS / 32, UNROLL = ROUTE_TOK > 1 ? 2 : 8;
     const bool wide = (W & 7) == 0 && (((size_t)w_router | (size_t)row_w) & 15) == 0;
     const int outputs = E + (row_w ? 1 : 0);
     for (int e0 = warp; e0 < outputs; e0 += RW * RE) {
@@ -84,7 +88,7 @@ moe_route_kernel(const TH* __restrict__ h, const TW* __restrict__ w_router, cons
             for (int k = 0; k < ROUTE_TOK; ++k) acc[x][k] = 0.f;
         }
         if (wide) {
-#pragma unroll 2
+#pragma unroll UNROLL
             for (int i = lane * 8; i < W; i += 256) {
                 float w8[RE][8];
 #pragma unroll
