@@ -58,7 +58,7 @@ def config(name: str) -> GumodraConfig:
     if name == "d":      # heads of 128, windows of 64 over pages of 32, more kept tokens than the window, 16 groups
         return make(vocab_size=150, hidden_size=96, norm_eps=1e-6, embed_scale=9.0, layers=(
             att(4, 4, 128, 64, 1, 128, mlp=moe(32, 16, 3, (16, 7), 40)), mem(2, 72, 24, mlp=dense(40)),
-            att(8, 2, 128, 33, 100, 32, base=3e5, mlp=moe(32, 12, 4, (2, 1), 32)), mem(8, 8, 8, mlp=moe(16, 7, 2, (7, 3), 8))))
+            att(8, 2, 128, 33, 100, 32, base=3e5, mlp=moe(32, 12, 4, (3, 2), 32)), mem(8, 8, 8, mlp=moe(16, 7, 2, (7, 3), 8))))
     raise KeyError(name)
 
 
@@ -214,7 +214,7 @@ def _attention_part(ops, dtype, W, H, G, D, window, keep, scale, rot, base, w):
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-@pytest.mark.parametrize("H,G,D,rot,window,keep", [(4, 2, 64, 32, 50, 20), (6, 2, 128, 128, 100, 7), (3, 3, 24, 10, 33, 130),
+@pytest.mark.parametrize("H,G,D,rot,window,keep", [(4, 2, 64, 24, 50, 21), (6, 2, 128, 128, 100, 7), (3, 3, 24, 10, 33, 130),
                                                    (8, 1, 64, 64, 1, 1), (2, 1, 200, 0, 64, 64), (20, 1, 64, 2, 65, 0),
                                                    (4, 4, 128, 6, 0, 0), (4, 2, 40, 40, 1, 300)])
 def test_attention_alone(ops, dtype, H, G, D, rot, window, keep):
